@@ -18,8 +18,14 @@
 // The `rep` = Hq / Hkv (<= 32) query heads sharing a kv head are rows 0..rep-1 of the 128-row MMA tile; the other
 // rows are never read.  The reference reaches paged decode attention through vLLM
 // (siirl/engine/rollout/vllm_rollout/vllm_rollout_spmd.py:261-416).
+//
+// The windowed variant (WIN) serves attention with a sliding window, kept first tokens and a linear distance bias
+// (win_params.h): an item's tiles are the cache blocks that hold a visible key (those of the kept tokens, then those of
+// the window), key and value widths may differ and be any multiple of 8 up to D (TMA fills the missing columns with
+// zeros), the bias is one multiply-add per score, and the output goes to a column range of a wider row, scaled.
 #include "common.cuh"
 #include "launchers.h"
+#include "win_params.h"
 
 namespace sb {
 
@@ -38,7 +44,23 @@ struct SplitParams {
   int q_rows_per_seq;      // rows of width D per sequence in the q tensor map (row_stride / D)
   float scale_log2;
   int* status;
+  // windowed variant
+  int window, keep_first, dv;
+  long long out_stride;    // `out` points at the branch's first column
+  float bias_exp, out_scale;
 };
+
+// cache blocks a query at position ctx - 1 visits: blocks 0 .. sinks - 1, then w0 .. ; `n` of them in all
+__host__ __device__ __forceinline__ void visible_tiles(int ctx, int window, int keep_first, int& sinks, int& w0, int& n) {
+  const int tiles = (ctx + kSBlk - 1) / kSBlk;
+  sinks = 0;
+  w0 = 0;
+  if (window > 0) {
+    sinks = min((keep_first + kSBlk - 1) / kSBlk, tiles);
+    w0 = max(sinks, max(0, ctx - window) / kSBlk);
+  }
+  n = sinks + max(0, tiles - w0);
+}
 
 template <int D>
 struct SplitSmem {
@@ -67,10 +89,10 @@ __device__ __forceinline__ void split_item(int idx, int B, int Hkv, int& c, int&
   g = r - b * Hkv;
 }
 
-template <int D>
+template <int D, bool WIN>
 __global__ void __launch_bounds__(160, 1)
-fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __grid_constant__ CUtensorMap map_q,
-                         SplitParams p) {
+fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __grid_constant__ CUtensorMap map_v,
+                         const __grid_constant__ CUtensorMap map_q, SplitParams p) {
   using L = SplitSmem<D>;
   constexpr int NS = L::kStages;
   constexpr int kDChunks = D / 64;
@@ -107,6 +129,7 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
 
   if (tid == 0) {
     tma_prefetch_desc(&map_cache);
+    if (WIN) tma_prefetch_desc(&map_v);
     tma_prefetch_desc(&map_q);
     for (int i = 0; i < L::kNumBars; ++i) mbar_init(&kv_full[i], 1);
     fence_barrier_init();
@@ -131,6 +154,10 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
       split_item(idx, p.B, p.Hkv, c, b, g);
       const int ctx = p.seq_lens[b];
       seq_tiles = (ctx + kSBlk - 1) / kSBlk;
+      if constexpr (WIN) {
+        int sinks, w0;
+        visible_tiles(ctx, p.window, p.keep_first, sinks, w0, seq_tiles);
+      }
       t0 = c * kChunkTiles;
       const int t1 = min(seq_tiles, t0 + kChunkTiles);
       if (t1 > t0) {
@@ -151,9 +178,13 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
         if (!mbar_wait(&q_empty[qb], ((item >> 1) & 1) ^ 1, p.status, kStatusTimeoutProducer)) return false;
         mbar_arrive_expect_tx(&q_full[qb], (uint32_t)(kDChunks * q_box_rows * 128));
 #pragma unroll
-        for (int cc = 0; cc < kDChunks; ++cc)
-          tma_load_2d(sQ + qb * L::kQBytes + cc * 16384, &map_q, &q_full[qb], cc * 64,
-                      b * p.q_rows_per_seq + g * rep);
+        for (int cc = 0; cc < kDChunks; ++cc) {
+          if constexpr (WIN)
+            tma_load_3d(sQ + qb * L::kQBytes + cc * 16384, &map_q, &q_full[qb], cc * 64, g * rep, b);
+          else
+            tma_load_2d(sQ + qb * L::kQBytes + cc * 16384, &map_q, &q_full[qb], cc * 64,
+                        b * p.q_rows_per_seq + g * rep);
+        }
         return true;
       };
       int idx = blockIdx.x, c, b, g, t0, n, st;
@@ -166,6 +197,8 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
         const bool have2 = find_item(idx2, c2, b2, g2, t02, n2, st2);
         const int q_at = min(n - 1, 3);
         const int* blocks = p.block_table + (size_t)b * p.max_blocks;
+        int sinks = 0, w0 = 0, vis = 0;
+        if constexpr (WIN) visible_tiles(p.seq_lens[b], p.window, p.keep_first, sinks, w0, vis);
         for (int t = 0; t < n && ok; ++t, ++tile_no) {
           const int stage = tile_no % NS;
           const uint32_t round = tile_no / NS;
@@ -173,7 +206,8 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
             ok = false;
             break;
           }
-          const int blk = blocks[t0 + t];
+          int blk = blocks[!WIN || t0 + t < sinks ? t0 + t : w0 + t0 + t - sinks];
+          if (WIN && blk < 0) blk = 0;      // never among the visible blocks of a well-formed table
           uint8_t* sk = sKV + stage * 2 * L::kKBytes;
           uint8_t* sv = sk + L::kKBytes;
           mbar_arrive_expect_tx(&kv_full[stage], 2 * L::kKBytes);
@@ -181,8 +215,13 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
           const int vrow = ((blk * 2 + 1) * p.Hkv + g) * kSBlk;
 #pragma unroll
           for (int cc = 0; cc < kDChunks; ++cc) {
-            tma_load_2d(sk + cc * 8192, &map_cache, &kv_full[stage], cc * 64, krow);
-            tma_load_2d(sv + cc * 8192, &map_cache, &kv_full[stage], cc * 64, vrow);
+            if constexpr (WIN) {
+              tma_load_3d(sk + cc * 8192, &map_cache, &kv_full[stage], cc * 64, g * kSBlk, blk);
+              tma_load_3d(sv + cc * 8192, &map_v, &kv_full[stage], cc * 64, g * kSBlk, blk);
+            } else {
+              tma_load_2d(sk + cc * 8192, &map_cache, &kv_full[stage], cc * 64, krow);
+              tma_load_2d(sv + cc * 8192, &map_cache, &kv_full[stage], cc * 64, vrow);
+            }
           }
           if (t == q_at && have2) ok = load_q(item_no + 1, b2, g2);
         }
@@ -265,6 +304,20 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
     int idx = blockIdx.x, c, b, g, t0, n, n_seq_tiles;
     for (; ok && find_item(idx, c, b, g, t0, n, n_seq_tiles); idx += gridDim.x) {
       const int ctx = p.seq_lens[b];
+      int sinks = 0, w0 = 0, vis = 0;
+      if constexpr (WIN) visible_tiles(ctx, p.window, p.keep_first, sinks, w0, vis);
+      auto first_pos = [&](int t) { return (!WIN || t0 + t < sinks ? t0 + t : w0 + t0 + t - sinks) * kSBlk; };
+      // some key of the tile at kv0 is not visible / the key at `col` is not
+      auto need_mask = [&](int kv0) {
+        return kv0 + kSBlk > ctx || (WIN && p.window > 0 && ctx - 1 - kv0 >= p.window && kv0 + kSBlk > p.keep_first);
+      };
+      auto hidden = [&](int col) {
+        return col >= ctx || (WIN && p.window > 0 && ctx - 1 - col >= p.window && col >= p.keep_first);
+      };
+      auto slope_of = [&](int row) {
+        return WIN && p.bias_exp > 0.f
+                   ? exp2f(-p.bias_exp * (float)(g * rep + row + 1) / (float)p.Hq) * 1.4426950408889634f : 0.f;
+      };
       const uint32_t tmem_oi = tmem_o + (item_no & 1) * 128;
       float m_ref = -INFINITY, l_run = 0.f;
       if (rep <= 8) {
@@ -274,6 +327,7 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
         // the 4 threads), l_run is a per-thread partial sum that is reduced at the end of the item.
         const int frow = lane >> 2, fq = lane & 3;
         const bool fvalid = frow < rep;
+        const float slope = slope_of(frow);
         for (int t = 0; t < n; ++t) {
           const uint32_t tn = tile_no + t;
           const int sb_ = tn & 1;
@@ -296,13 +350,21 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
           tc_fence_before();
           __syncwarp();
           if (lane == 0) mbar_arrive(&s_empty[sb_]);
-          const int kv0 = (t0 + t) * kSBlk;
-          if (kv0 + kSBlk > ctx) {
+          const int kv0 = first_pos(t);
+          if constexpr (WIN) {
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+              const float dist = (float)(kv0 + 8 * i + 2 * fq - (ctx - 1));
+              sv[2 * i] = fmaf(slope, dist, sv[2 * i]);
+              sv[2 * i + 1] = fmaf(slope, dist + 1.f, sv[2 * i + 1]);
+            }
+          }
+          if (need_mask(kv0)) {
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
               const int col = kv0 + 8 * i + 2 * fq;
-              if (col >= ctx) sv[2 * i] = -INFINITY;
-              if (col + 1 >= ctx) sv[2 * i + 1] = -INFINITY;
+              if (hidden(col)) sv[2 * i] = -INFINITY;
+              if (hidden(col + 1)) sv[2 * i + 1] = -INFINITY;
             }
           }
           float m_tile = -INFINITY;
@@ -366,6 +428,7 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
         l_run = __shfl_sync(0xffffffffu, l_run, (lane * 4) & 31);
         m_ref = __shfl_sync(0xffffffffu, m_ref, (lane * 4) & 31);
       } else {
+        const float slope = slope_of(lane);
         for (int t = 0; t < n; ++t) {
           const uint32_t tn = tile_no + t;
           const int sb_ = tn & 1;
@@ -389,11 +452,15 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
           tc_fence_before();
           __syncwarp();
           if (lane == 0) mbar_arrive(&s_empty[sb_]);   // the MMA warp may overwrite this S buffer
-          const int kv0 = (t0 + t) * kSBlk;
-          if (kv0 + kSBlk > ctx) {
+          const int kv0 = first_pos(t);
+          if constexpr (WIN) {
+  #pragma unroll
+            for (int i = 0; i < kSBlk; ++i) sv[i] = fmaf(slope, (float)(kv0 + i - (ctx - 1)), sv[i]);
+          }
+          if (need_mask(kv0)) {
   #pragma unroll
             for (int i = 0; i < kSBlk; ++i)
-              if (kv0 + i >= ctx) sv[i] = -INFINITY;
+              if (hidden(kv0 + i)) sv[i] = -INFINITY;
           }
           float m_tile = -INFINITY;
   #pragma unroll
@@ -491,7 +558,9 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
       const float inv_l = l_run > 0.f ? 1.f / l_run : 0.f;
       const int head = g * rep + (row_valid ? lane : 0);
       const bool single = n_seq_tiles <= kChunkTiles;
-      __nv_bfloat16* orow = p.out + (size_t)b * (p.Hq * D) + (size_t)head * D;
+      const int dv = WIN ? p.dv : D;
+      __nv_bfloat16* orow = p.out + (WIN ? (size_t)b * p.out_stride : (size_t)b * (p.Hq * D)) + (size_t)head * dv;
+      const float out_f = WIN ? inv_l * p.out_scale : inv_l;
       float* wrow = p.ws_o + (((size_t)b * p.Hq + head) * p.max_chunks + c) * D;
 #pragma unroll 1
       for (int cc = 0; cc < D / 32; ++cc) {
@@ -502,11 +571,12 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
           if (single) {
 #pragma unroll
             for (int q = 0; q < 4; ++q) {
+              if (WIN && cc * 32 + q * 8 >= dv) break;
               uint4 o;
-              o.x = pack_bf16x2(__uint_as_float(r[q * 8 + 0]) * inv_l, __uint_as_float(r[q * 8 + 1]) * inv_l);
-              o.y = pack_bf16x2(__uint_as_float(r[q * 8 + 2]) * inv_l, __uint_as_float(r[q * 8 + 3]) * inv_l);
-              o.z = pack_bf16x2(__uint_as_float(r[q * 8 + 4]) * inv_l, __uint_as_float(r[q * 8 + 5]) * inv_l);
-              o.w = pack_bf16x2(__uint_as_float(r[q * 8 + 6]) * inv_l, __uint_as_float(r[q * 8 + 7]) * inv_l);
+              o.x = pack_bf16x2(__uint_as_float(r[q * 8 + 0]) * out_f, __uint_as_float(r[q * 8 + 1]) * out_f);
+              o.y = pack_bf16x2(__uint_as_float(r[q * 8 + 2]) * out_f, __uint_as_float(r[q * 8 + 3]) * out_f);
+              o.z = pack_bf16x2(__uint_as_float(r[q * 8 + 4]) * out_f, __uint_as_float(r[q * 8 + 5]) * out_f);
+              o.w = pack_bf16x2(__uint_as_float(r[q * 8 + 6]) * out_f, __uint_as_float(r[q * 8 + 7]) * out_f);
               *reinterpret_cast<uint4*>(orow + cc * 32 + q * 8) = o;
             }
           } else {
@@ -540,13 +610,19 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
 }
 
 // merges the chunk partials of sequences longer than one chunk; zero rows for empty slots
-template <int D>
+template <int D, bool WIN>
 __global__ void fmha_decode_merge_kernel(SplitParams p) {
   const int b = blockIdx.x, h = blockIdx.y;
   const int ctx = p.seq_lens[b];
-  const int n_tiles = (ctx + kSBlk - 1) / kSBlk;
-  __nv_bfloat16* orow = p.out + (size_t)b * (p.Hq * D) + (size_t)h * D;
+  int n_tiles = (ctx + kSBlk - 1) / kSBlk;
+  if constexpr (WIN) {
+    int sinks, w0;
+    visible_tiles(ctx, p.window, p.keep_first, sinks, w0, n_tiles);
+  }
+  const int dv = WIN ? p.dv : D;
+  __nv_bfloat16* orow = p.out + (WIN ? (size_t)b * p.out_stride : (size_t)b * (p.Hq * D)) + (size_t)h * dv;
   const int d = threadIdx.x;   // blockDim.x == D
+  if (WIN && d >= dv) return;
   if (ctx <= 0) {
     orow[d] = __float2bfloat16(0.f);
     return;
@@ -563,13 +639,14 @@ __global__ void fmha_decode_merge_kernel(SplitParams p) {
     wsum += w;
     acc += w * wo[(size_t)c * D + d];
   }
-  orow[d] = __float2bfloat16(wsum > 0.f ? acc / wsum : 0.f);
+  orow[d] = __float2bfloat16(wsum > 0.f ? acc / wsum * (WIN ? p.out_scale : 1.f) : 0.f);
 }
 
-template <int D>
-static int launch_decode_split(const CUtensorMap& mc, const CUtensorMap& mq, const SplitParams& p, cudaStream_t stream) {
+template <int D, bool WIN>
+static int launch_decode_split(const CUtensorMap& mc, const CUtensorMap& mv, const CUtensorMap& mq, const SplitParams& p,
+                               cudaStream_t stream) {
   using L = SplitSmem<D>;
-  auto kernel = fmha_decode_split_kernel<D>;
+  auto kernel = fmha_decode_split_kernel<D, WIN>;
   static bool configured = false;
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, L::kTotal);
@@ -578,10 +655,10 @@ static int launch_decode_split(const CUtensorMap& mc, const CUtensorMap& mq, con
   }
   const int items = p.max_chunks * p.B * p.Hkv;
   const int grid = items < num_sms() ? items : num_sms();
-  kernel<<<grid, 160, L::kTotal, stream>>>(mc, mq, p);
+  kernel<<<grid, 160, L::kTotal, stream>>>(mc, mv, mq, p);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return (int)e;
-  fmha_decode_merge_kernel<D><<<dim3(p.B, p.Hq), D, 0, stream>>>(p);
+  fmha_decode_merge_kernel<D, WIN><<<dim3(p.B, p.Hq), D, 0, stream>>>(p);
   return (int)cudaGetLastError();
 }
 
@@ -619,5 +696,57 @@ extern "C" int sb_fmha_decode_split(const void* q, int row_stride, const void* c
   p.out = (__nv_bfloat16*)out; p.ws_o = ws_o; p.ws_lse = ws_lse;
   p.B = B; p.Hq = Hq; p.Hkv = Hkv; p.q_rows_per_seq = row_stride / D;
   p.scale_log2 = scale * 1.4426950408889634f; p.status = status;
-  return D == 128 ? launch_decode_split<128>(mc, mq, p, stream) : launch_decode_split<64>(mc, mq, p, stream);
+  p.window = 0; p.keep_first = 0; p.dv = D; p.out_stride = 0; p.bias_exp = 0.f; p.out_scale = 1.f;
+  return D == 128 ? launch_decode_split<128, false>(mc, mc, mq, p, stream)
+                  : launch_decode_split<64, false>(mc, mc, mq, p, stream);
+}
+
+// Chunks of the workspace of sb_attn_window_decode (ws_o = B * Hq * chunks * D floats with D = 64 or 128, the smallest
+// that holds both widths; ws_lse = B * Hq * chunks), or -1 when the sizes need sb_attn_window_simt.
+extern "C" int sb_attn_window_decode_chunks(const void* params) {
+  const WinParams& p = *reinterpret_cast<const WinParams*>(params);
+  if (p.dk % 8 || p.dv % 8 || p.dk > 128 || p.dv > 128 || p.Hq % p.Hkv || p.Hq / p.Hkv > 32 || p.row_stride % 8 ||
+      p.q_off % 8 || p.out_stride % 8 || p.out_off % 8 || p.block_elems % 8)
+    return -1;
+  int tiles = p.max_blocks;
+  if (p.window > 0) {
+    const int most = (p.keep_first + kSBlk - 1) / kSBlk + (p.window + kSBlk - 1) / kSBlk + 1;
+    if (most < tiles) tiles = most;
+  }
+  return (tiles + kChunkTiles - 1) / kChunkTiles;
+}
+
+// One query row per sequence (row b = cache slot b) against its cached context of seq_lens[b] tokens, the current one
+// included; 0: idle slot, its output row is zero.
+extern "C" int sb_attn_window_decode(const void* params, const int* seq_lens, float* ws_o, float* ws_lse, int* status,
+                                     cudaStream_t stream) {
+  const WinParams& w = *reinterpret_cast<const WinParams*>(params);
+  if (w.T == 0) return 0;
+  const int chunks = sb_attn_window_decode_chunks(params);
+  if (chunks < 0) return -2;
+  static thread_local bool tl_context_bound = false;
+  if (!tl_context_bound) {
+    cudaFree(0);
+    tl_context_bound = true;
+  }
+  const int rep = w.Hq / w.Hkv;
+  const __nv_bfloat16* cache = reinterpret_cast<const __nv_bfloat16*>(w.cache);
+  CUtensorMap mk, mv, mq;
+  int r = make_tensor_map_bf16_3d(&mk, cache, w.dk, (long long)w.Hkv * kSBlk, w.num_blocks, w.dk, w.block_elems, 64, kSBlk, 1);
+  if (r) return r;
+  r = make_tensor_map_bf16_3d(&mv, cache + (size_t)w.Hkv * kSBlk * w.dk, w.dv, (long long)w.Hkv * kSBlk, w.num_blocks, w.dv,
+                              w.block_elems, 64, kSBlk, 1);
+  if (r) return r;
+  r = make_tensor_map_bf16_3d(&mq, reinterpret_cast<const __nv_bfloat16*>(w.x) + w.q_off, w.dk, w.Hq, w.T, w.dk,
+                              w.row_stride, 64, (rep + 7) & ~7, 1);
+  if (r) return r;
+  SplitParams p;
+  p.seq_lens = seq_lens; p.block_table = w.block_table; p.max_blocks = w.max_blocks; p.max_chunks = chunks;
+  p.out = reinterpret_cast<__nv_bfloat16*>(w.out) + w.out_off; p.ws_o = ws_o; p.ws_lse = ws_lse;
+  p.B = w.T; p.Hq = w.Hq; p.Hkv = w.Hkv; p.q_rows_per_seq = 0;
+  p.scale_log2 = w.scale * 1.4426950408889634f; p.status = status;
+  p.window = w.window; p.keep_first = w.keep_first; p.dv = w.dv; p.out_stride = w.out_stride;
+  p.bias_exp = w.bias_exp; p.out_scale = w.out_scale;
+  return w.dk > 64 || w.dv > 64 ? launch_decode_split<128, true>(mk, mv, mq, p, stream)
+                                : launch_decode_split<64, true>(mk, mv, mq, p, stream);
 }

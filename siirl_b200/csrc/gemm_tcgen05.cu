@@ -953,6 +953,21 @@ int make_tensor_map_bf16_2d(CUtensorMap* map, const void* base, long long inner,
   return r == CUDA_SUCCESS ? 0 : (int)r;
 }
 
+// 3-D form: dims d0 (contiguous) x d1 x d2 with pitches in elements, box = b0 x b1 x b2
+int make_tensor_map_bf16_3d(CUtensorMap* map, const void* base, long long d0, long long d1, long long d2,
+                            long long pitch1, long long pitch2, int b0, int b1, int b2) {
+  EncodeTiledFn fn = get_encode_fn();
+  if (!fn) return -1;
+  cuuint64_t dims[3] = {(cuuint64_t)d0, (cuuint64_t)d1, (cuuint64_t)d2};
+  cuuint64_t strides[2] = {(cuuint64_t)pitch1 * 2, (cuuint64_t)pitch2 * 2};
+  cuuint32_t box[3] = {(cuuint32_t)b0, (cuuint32_t)b1, (cuuint32_t)b2};
+  cuuint32_t estr[3] = {1, 1, 1};
+  CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr,
+                  CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                  CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? 0 : (int)r;
+}
+
 static int g_num_sms = 0;
 int num_sms() {
   if (!g_num_sms) {

@@ -1,0 +1,269 @@
+// Row operations of decoders whose residual stream is kept in 32-bit floats, and a plain SIMT matrix product for the
+// shapes and number formats the tensor-core GEMM does not take.
+//
+//   embed_scaled       h[t] = table[id[t]] * scale                               (fp32 stream)
+//   add_norm           h += delta;  y = norm(h) * w                              (layer norm or RMS norm, one launch)
+//   gated_act          y = act(gate) * up   for a fused projection [gate | up]   (SiLU or tanh-form GELU)
+//   softcap            z = cap * tanh(z / cap) in place on fp32 logits
+//   gemm_simt          C[M, N] = A[M, K] B[N, K]^T with fp32 accumulation on the FMA pipes: fp32 models (true 32-bit
+//                      products) and bf16 operands whose row pitch TMA cannot address (not a multiple of 16 bytes)
+//
+// Templates: T is the activation / weight format (bf16 or fp32); V elements per access (4, or 1 for odd widths).
+#include "common.cuh"
+#include "launchers.h"
+#include "typed.cuh"
+
+namespace sb {
+
+template <typename T, int V>
+__global__ void embed_scaled_kernel(const long long* __restrict__ ids, const T* __restrict__ table,
+                                    float* __restrict__ h, int T_, int W, int vocab, float scale) {
+  const int nv = W / V;
+  const long long total = (long long)T_ * nv;
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const int t = (int)(i / nv), c = (int)(i % nv) * V;
+    long long id = ids[t];
+    id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
+    float x[V];
+    load_vec<T, V>(table + (size_t)id * W + c, x);
+#pragma unroll
+    for (int k = 0; k < V; ++k) x[k] *= scale;
+    store_vec<float, V>(h + (size_t)t * W + c, x);
+  }
+}
+
+constexpr int kRowThreads = 256;
+
+__device__ __forceinline__ float row_sum(float v, float* red) {
+  v = warp_sum(v);
+  const int w = threadIdx.x >> 5, l = threadIdx.x & 31;
+  __syncthreads();
+  if (l == 0) red[w] = v;
+  __syncthreads();
+  float t = red[0];
+#pragma unroll
+  for (int i = 1; i < kRowThreads / 32; ++i) t += red[i];
+  return t;
+}
+
+// CH register chunks of V elements per thread hold the row (CH = 0: the row is re-read from memory)
+template <typename T, int V, int CH>
+__global__ void __launch_bounds__(kRowThreads)
+add_norm_kernel(float* __restrict__ h, const T* __restrict__ delta, const T* __restrict__ w, T* __restrict__ y, int rows,
+                int W, float eps, int layer_norm) {
+  __shared__ float red[kRowThreads / 32];
+  const int nv = W / V;
+  for (int row = blockIdx.x; row < rows; row += gridDim.x) {
+    float* hr = h + (size_t)row * W;
+    float x[CH > 0 ? CH : 1][V];
+    float s = 0.f;
+    auto fetch = [&](int vi, float (&v)[V]) {
+      load_vec<float, V>(hr + (size_t)vi * V, v);
+      if (delta) {
+        float d[V];
+        load_vec<T, V>(delta + (size_t)row * W + (size_t)vi * V, d);
+#pragma unroll
+        for (int k = 0; k < V; ++k) v[k] += d[k];
+        store_vec<float, V>(hr + (size_t)vi * V, v);
+      }
+    };
+    auto each = [&](auto&& fn) {
+      if constexpr (CH > 0) {
+#pragma unroll
+        for (int c = 0; c < CH; ++c) {
+          const int vi = threadIdx.x + c * kRowThreads;
+          if (vi < nv) fn(vi, x[c]);
+        }
+      } else {
+        for (int vi = threadIdx.x; vi < nv; vi += kRowThreads) {
+          load_vec<float, V>(hr + (size_t)vi * V, x[0]);   // written by this same thread below
+          fn(vi, x[0]);
+        }
+      }
+    };
+    if constexpr (CH > 0) {
+      each([&](int vi, float (&v)[V]) { fetch(vi, v); });
+    } else {
+      for (int vi = threadIdx.x; vi < nv; vi += kRowThreads) fetch(vi, x[0]);
+    }
+    float mean = 0.f;
+    if (layer_norm) {
+      each([&](int, float (&v)[V]) {
+#pragma unroll
+        for (int k = 0; k < V; ++k) s += v[k];
+      });
+      mean = row_sum(s, red) / (float)W;
+    }
+    float ss = 0.f;
+    each([&](int, float (&v)[V]) {
+#pragma unroll
+      for (int k = 0; k < V; ++k) ss += (v[k] - mean) * (v[k] - mean);
+    });
+    const float rstd = 1.f / sqrtf(row_sum(ss, red) / (float)W + eps);
+    each([&](int vi, float (&v)[V]) {
+      float wv[V], o[V];
+      load_vec<T, V>(w + (size_t)vi * V, wv);
+#pragma unroll
+      for (int k = 0; k < V; ++k) o[k] = (v[k] - mean) * rstd * wv[k];
+      store_vec<T, V>(y + (size_t)row * W + (size_t)vi * V, o);
+    });
+  }
+}
+
+__device__ __forceinline__ float gelu_tanh_f(float z) {
+  const float u = 0.7978845608028654f * (z + 0.044715f * z * z * z);
+  return 0.5f * z * (1.f + tanhf(u));
+}
+
+template <typename T, int V>
+__global__ void gated_act_kernel(const T* __restrict__ gu, T* __restrict__ out, long long rows, int I, int act) {
+  const int nv = I / V;
+  const long long total = rows * nv;
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const long long t = i / nv;
+    const int c = (int)(i % nv) * V;
+    float g[V], u[V];
+    load_vec<T, V>(gu + t * 2 * I + c, g);
+    load_vec<T, V>(gu + t * 2 * I + I + c, u);
+#pragma unroll
+    for (int k = 0; k < V; ++k) g[k] = (act == 1 ? gelu_tanh_f(g[k]) : g[k] / (1.f + __expf(-g[k]))) * u[k];
+    store_vec<T, V>(out + t * I + c, g);
+  }
+}
+
+__global__ void softcap_kernel(float* __restrict__ z, long long n, float cap) {
+  const float inv = 1.f / cap;
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x)
+    z[i] = cap * tanhf(z[i] * inv);
+}
+
+// 64 x 64 output tile per 256 threads, 4 x 4 values each, contraction in steps of 16 through shared memory
+template <typename TI, typename TO>
+__global__ void __launch_bounds__(256)
+gemm_simt_kernel(const TI* __restrict__ A, const TI* __restrict__ B, TO* __restrict__ C, int M, int N, int K,
+                 long long lda, long long ldb, long long ldc) {
+  __shared__ float sa[16][68], sb_[16][68];
+  const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < K; k0 += 16) {
+    for (int i = threadIdx.x; i < 64 * 16; i += 256) {
+      const int r = i >> 4, k = i & 15;
+      sa[k][r] = (m0 + r < M && k0 + k < K) ? to_float(A[(size_t)(m0 + r) * lda + k0 + k]) : 0.f;
+      sb_[k][r] = (n0 + r < N && k0 + k < K) ? to_float(B[(size_t)(n0 + r) * ldb + k0 + k]) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < 16; ++k) {
+      float a[4], b[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) a[i] = sa[k][ty * 4 + i];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) b[j] = sb_[k][tx * 4 + j];
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
+      if (m < M && n < N) C[(size_t)m * ldc + n] = from_float<TO>(acc[i][j]);
+    }
+}
+
+static int grid_for(long long total, int threads) {
+  long long b = (total + threads - 1) / threads;
+  const long long cap = (long long)num_sms() * 8;
+  return (int)(b < 1 ? 1 : (b > cap ? cap : b));
+}
+
+template <typename T>
+static int launch_add_norm(float* h, const T* delta, const T* w, T* y, int rows, int W, float eps, int ln, cudaStream_t s) {
+  const int grid = rows < num_sms() * 8 ? rows : num_sms() * 8;
+  if (W % 4) {
+    add_norm_kernel<T, 1, 0><<<grid, kRowThreads, 0, s>>>(h, delta, w, y, rows, W, eps, ln);
+  } else if (W <= 4 * kRowThreads) {
+    add_norm_kernel<T, 4, 1><<<grid, kRowThreads, 0, s>>>(h, delta, w, y, rows, W, eps, ln);
+  } else if (W <= 4 * 4 * kRowThreads) {
+    add_norm_kernel<T, 4, 4><<<grid, kRowThreads, 0, s>>>(h, delta, w, y, rows, W, eps, ln);
+  } else {
+    add_norm_kernel<T, 4, 0><<<grid, kRowThreads, 0, s>>>(h, delta, w, y, rows, W, eps, ln);
+  }
+  return (int)cudaGetLastError();
+}
+
+}  // namespace sb
+
+using namespace sb;
+
+// f32: 1 when tables, activations and weights are fp32, 0 for bf16 (the stream `h` is always fp32)
+extern "C" int sb_embed_scaled(const long long* ids, const void* table, float* h, int T, int W, int vocab, float scale,
+                               int f32, cudaStream_t stream) {
+  if (T == 0) return 0;
+  const int grid = grid_for((long long)T * W / 4, 256);
+  if (f32) {
+    if (W % 4 == 0) embed_scaled_kernel<float, 4><<<grid, 256, 0, stream>>>(ids, (const float*)table, h, T, W, vocab, scale);
+    else embed_scaled_kernel<float, 1><<<grid, 256, 0, stream>>>(ids, (const float*)table, h, T, W, vocab, scale);
+  } else {
+    using B = __nv_bfloat16;
+    if (W % 4 == 0) embed_scaled_kernel<B, 4><<<grid, 256, 0, stream>>>(ids, (const B*)table, h, T, W, vocab, scale);
+    else embed_scaled_kernel<B, 1><<<grid, 256, 0, stream>>>(ids, (const B*)table, h, T, W, vocab, scale);
+  }
+  return (int)cudaGetLastError();
+}
+
+// h [rows, W] fp32 is updated in place (+= delta when given); y = norm(h) * w in the activation format
+extern "C" int sb_add_norm(float* h, const void* delta, const void* w, void* y, int rows, int W, float eps,
+                           int layer_norm, int f32, cudaStream_t stream) {
+  if (rows == 0) return 0;
+  if (f32)
+    return launch_add_norm<float>(h, (const float*)delta, (const float*)w, (float*)y, rows, W, eps, layer_norm, stream);
+  return launch_add_norm<__nv_bfloat16>(h, (const __nv_bfloat16*)delta, (const __nv_bfloat16*)w, (__nv_bfloat16*)y, rows,
+                                        W, eps, layer_norm, stream);
+}
+
+// act: 0 SiLU, 1 tanh-form GELU; gu [rows, 2 I] -> out [rows, I]
+extern "C" int sb_gated_act(const void* gu, void* out, long long rows, int I, int act, int f32, cudaStream_t stream) {
+  if (rows == 0) return 0;
+  const int V = f32 ? 4 : 8;
+  const int grid = grid_for(rows * I / (I % V ? 1 : V), 256);
+  if (f32) {
+    if (I % 4 == 0) gated_act_kernel<float, 4><<<grid, 256, 0, stream>>>((const float*)gu, (float*)out, rows, I, act);
+    else gated_act_kernel<float, 1><<<grid, 256, 0, stream>>>((const float*)gu, (float*)out, rows, I, act);
+  } else {
+    using B = __nv_bfloat16;
+    if (I % 8 == 0) gated_act_kernel<B, 8><<<grid, 256, 0, stream>>>((const B*)gu, (B*)out, rows, I, act);
+    else gated_act_kernel<B, 1><<<grid, 256, 0, stream>>>((const B*)gu, (B*)out, rows, I, act);
+  }
+  return (int)cudaGetLastError();
+}
+
+extern "C" int sb_softcap(float* z, long long n, float cap, cudaStream_t stream) {
+  if (n == 0) return 0;
+  if (!(cap > 0.f)) return -3;
+  softcap_kernel<<<grid_for(n, 256), 256, 0, stream>>>(z, n, cap);
+  return (int)cudaGetLastError();
+}
+
+// in_f32: operands fp32 (else bf16); out_f32: result fp32 (else bf16)
+extern "C" int sb_gemm_simt(const void* A, const void* B, void* C, int M, int N, int K, long long lda, long long ldb,
+                            long long ldc, int in_f32, int out_f32, cudaStream_t stream) {
+  if (M <= 0 || N <= 0) return 0;
+  if ((M + 63) / 64 > 65535) return -3;
+  const dim3 grid((N + 63) / 64, (M + 63) / 64);
+  using H = __nv_bfloat16;
+  if (in_f32 && out_f32)
+    gemm_simt_kernel<float, float><<<grid, 256, 0, stream>>>((const float*)A, (const float*)B, (float*)C, M, N, K, lda, ldb, ldc);
+  else if (!in_f32 && out_f32)
+    gemm_simt_kernel<H, float><<<grid, 256, 0, stream>>>((const H*)A, (const H*)B, (float*)C, M, N, K, lda, ldb, ldc);
+  else if (!in_f32)
+    gemm_simt_kernel<H, H><<<grid, 256, 0, stream>>>((const H*)A, (const H*)B, (H*)C, M, N, K, lda, ldb, ldc);
+  else
+    return -2;
+  return (int)cudaGetLastError();
+}

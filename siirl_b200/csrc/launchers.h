@@ -10,6 +10,8 @@ namespace sb {
 int num_sms();
 int make_tensor_map_bf16_2d(CUtensorMap* map, const void* base, long long inner, long long outer,
                             long long pitch_elems, int box_inner, int box_outer);
+int make_tensor_map_bf16_3d(CUtensorMap* map, const void* base, long long d0, long long d1, long long d2,
+                            long long pitch1, long long pitch2, int b0, int b1, int b2);
 }  // namespace sb
 
 extern "C" {
@@ -180,4 +182,33 @@ extern "C" {
 int sb_resize_bilinear_u8(const void* src, void* dst, int N, int H, int W, int C, int OH, int OW, float crop_y0,
                           float crop_x0, float crop_h, float crop_w, cudaStream_t stream);
 int sb_raster_synth_env(const float* state, void* out, int N, int H, int W, cudaStream_t stream);
+}
+
+extern "C" {
+// ---- hybrid_ops.cu (f32: activations and weights fp32, else bf16) ----
+int sb_embed_scaled(const long long* ids, const void* table, float* h, int T, int W, int vocab, float scale, int f32,
+                    cudaStream_t stream);
+int sb_add_norm(float* h, const void* delta, const void* w, void* y, int rows, int W, float eps, int layer_norm, int f32,
+                cudaStream_t stream);
+int sb_gated_act(const void* gu, void* out, long long rows, int I, int act, int f32, cudaStream_t stream);
+int sb_softcap(float* z, long long n, float cap, cudaStream_t stream);
+int sb_gemm_simt(const void* A, const void* B, void* C, int M, int N, int K, long long lda, long long ldb, long long ldc,
+                 int in_f32, int out_f32, cudaStream_t stream);
+// ---- recurrence.cu (params: host RecParams) ----
+int sb_recurrence_step(const void* params, const int* row0, const int* nrow, const int* slots, const int* pos0, int n_seq,
+                       int f32, cudaStream_t stream);
+int sb_recurrence_chunk();
+long long sb_recurrence_workspace(const void* params, int n_chunks, int T);
+int sb_recurrence_prefill(const void* params, const int* row0, const int* nrow, const int* slots, const int* pos0,
+                          int n_seq, const int* seq_chunk0, const int* chunk_row, const int* chunk_len, int n_chunks,
+                          int T, void* workspace, int* status, cudaStream_t stream);
+// ---- fmha_window.cu (params: host WinParams) ----
+int sb_kv_append_split(const void* params, int f32, cudaStream_t stream);
+int sb_attn_window_simt(const void* params, int f32, cudaStream_t stream);
+int sb_attn_window_prefill(const void* params, const int* tile_row, const int* tile_rows, const int* tile_pos,
+                           const int* tile_slot, int n_tiles, int* status, cudaStream_t stream);
+// ---- fmha_decode_split.cu, windowed variant ----
+int sb_attn_window_decode_chunks(const void* params);
+int sb_attn_window_decode(const void* params, const int* seq_lens, float* ws_o, float* ws_lse, int* status,
+                          cudaStream_t stream);
 }

@@ -1,0 +1,58 @@
+// Element access for kernels that exist in bf16 and fp32: conversion to fp32 registers and vector loads / stores.
+#pragma once
+#include "common.cuh"
+
+namespace sb {
+
+__device__ __forceinline__ float to_float(float x) { return x; }
+__device__ __forceinline__ float to_float(__nv_bfloat16 x) { return __bfloat162float(x); }
+
+template <typename T>
+__device__ __forceinline__ T from_float(float x);
+template <>
+__device__ __forceinline__ float from_float<float>(float x) { return x; }
+template <>
+__device__ __forceinline__ __nv_bfloat16 from_float<__nv_bfloat16>(float x) { return __float2bfloat16(x); }
+
+// V consecutive elements; the pointer is aligned to the access (V * sizeof(T) bytes, at most 16)
+template <typename T, int V>
+__device__ __forceinline__ void load_vec(const T* p, float (&x)[V]) {
+  if constexpr (V == 1) {
+    x[0] = to_float(p[0]);
+  } else if constexpr (sizeof(T) == 4) {
+    static_assert(V == 4, "fp32 vectors of four");
+    const float4 v = *reinterpret_cast<const float4*>(p);
+    x[0] = v.x; x[1] = v.y; x[2] = v.z; x[3] = v.w;
+  } else if constexpr (V == 4) {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.y));
+    x[0] = a.x; x[1] = a.y; x[2] = b.x; x[3] = b.y;
+  } else {
+    static_assert(V == 8, "bf16 vectors of four or eight");
+    const uint4 v = *reinterpret_cast<const uint4*>(p);
+    const __nv_bfloat162* q = reinterpret_cast<const __nv_bfloat162*>(&v);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 a = __bfloat1622float2(q[i]);
+      x[2 * i] = a.x;
+      x[2 * i + 1] = a.y;
+    }
+  }
+}
+
+template <typename T, int V>
+__device__ __forceinline__ void store_vec(T* p, const float (&x)[V]) {
+  if constexpr (V == 1) {
+    p[0] = from_float<T>(x[0]);
+  } else if constexpr (sizeof(T) == 4) {
+    *reinterpret_cast<float4*>(p) = make_float4(x[0], x[1], x[2], x[3]);
+  } else if constexpr (V == 4) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(x[0], x[1]), pack_bf16x2(x[2], x[3]));
+  } else {
+    *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(x[0], x[1]), pack_bf16x2(x[2], x[3]), pack_bf16x2(x[4], x[5]),
+                                              pack_bf16x2(x[6], x[7]));
+  }
+}
+
+}  // namespace sb

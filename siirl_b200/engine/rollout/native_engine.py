@@ -11,11 +11,17 @@ Scheduling model
   tokens, finished flags, the sampler's counter) lives in device tensors, so a step is replayed from a CUDA
   graph; the host looks at the finished flags only every ``sync_interval`` steps, and at that point retires
   finished sequences, admits waiting requests into the freed slots and grows block tables.
+* Hybrid decoders (``cfg.hybrid``) keep, beside the paged keys and values of their attention layers, one recurrent state
+  per slot (32-bit, ``model.new_states``).  A prompt that starts at position 0 overwrites its slot's state, samples of
+  one prompt copy it, and the prefix cache is off for them (a block of keys does not carry the state that led there).
+  When every attention layer has a sliding window, blocks that left all windows go back to the allocator while their
+  sequence is still running.
 * Slots of the running batch are fixed-size (``max_num_seqs`` rounded to the captured batch sizes); empty slots
   have context length 0 and are skipped by the kernels.
 """
 from __future__ import annotations
 
+import math
 import os
 import time
 from dataclasses import dataclass, field
@@ -27,6 +33,7 @@ from ...models.decoder import DecoderLM
 from ...ops import kv_cache as kvc
 from ...ops.attention import SeqInfo
 from ...ops.lm_head import lm_head_logits
+from ...ops.recurrence import copy_states
 from ...ops.sampling import sample
 
 BLOCK = kvc.BLOCK
@@ -66,6 +73,7 @@ class _Seq:
     slot: int = -1
     generated: int = 0
     prefilled: int = 0          # prompt tokens whose K/V are in the cache (first sample of a group)
+    hidden_until: int = 0       # blocks below this index have been checked for leaving every window
 
 
 class BlockAllocator:
@@ -160,6 +168,14 @@ class RolloutEngine:
         # the same wake period (multi-turn conversations re-send their history; n-sample groups already share blocks).
         self.enable_chunked_prefill = bool(enable_chunked_prefill)
         self.enable_prefix_caching = bool(enable_prefix_caching)
+        hybrid = model.cfg.hybrid
+        self.recurrent = hybrid is not None and any(b.kind != "attention" for x in hybrid.layers for b in x.branches)
+        self.visible_span = hybrid.visible_span() if hybrid is not None else None
+        if hybrid is not None and lockstep_group is not None:
+            raise ValueError("hybrid decoders have no expert layers: no lock-step group")
+        if self.recurrent:
+            self.enable_prefix_caching = False
+        self.states: List[Dict[str, torch.Tensor]] = []      # per recurrent branch, indexed by slot
         # Device memory the engine may use for KV blocks while it is awake (the trainer's fp32 gradient buffer, idle
         # and about to be zeroed between an optimizer step and the next backward): on a 180 GB part with the Adam
         # state resident this is what lets all sequences of a step decode in one wave.  Its contents are clobbered.
@@ -188,8 +204,17 @@ class RolloutEngine:
 
     # ---- memory hand-off with the trainer -------------------------------------------------------
     def _block_bytes(self) -> int:
-        c = self.cfg
-        return c.num_layers * 2 * c.num_kv_heads * BLOCK * c.head_dim * torch.finfo(self.dtype).bits // 8
+        return sum(self._layer_elems()) * torch.finfo(self.dtype).bits // 8
+
+    def _layer_elems(self) -> List[int]:
+        """Elements of one block, for every layer that keeps keys and values."""
+        return [g * BLOCK * (dk + dv) for g, dk, dv in self.cfg.paged_layers()]
+
+    def _state_bytes(self, slots: int) -> int:
+        if not self.recurrent:
+            return 0
+        return 4 * slots * sum(math.prod(s) for br in self.model.recurrent_branches()
+                               for s in br.spec.state_shapes().values())
 
     def wake_up(self) -> None:
         if self.cache is not None:
@@ -204,22 +229,28 @@ class RolloutEngine:
             if self.device.type == "cuda":
                 torch.cuda.empty_cache()        # cached training blocks would hide free memory from the query
                 free, _total = torch.cuda.mem_get_info(self.device)
-                nb = max(16, (int(free * self._mem_util) + lent) // self._block_bytes())
+                free = max(0, free - self._state_bytes(self.max_num_seqs))
+                nb = max(16, (int(free * self._mem_util) + lent) // max(self._block_bytes(), 1))
             else:
                 nb = max(16, self.max_num_seqs * self.max_blocks_per_seq)
             nb = min(nb, self.max_num_seqs * self.max_blocks_per_seq + 8)
-        # one tensor per layer [nb, 2, Hkv, 64, D]: the first layers live in the borrowed buffer, the rest is new
-        per_layer = nb * 2 * c.num_kv_heads * BLOCK * c.head_dim
-        n_lent = min(c.num_layers, lent // (per_layer * esize)) if lent else 0
-        shape = (nb, 2, c.num_kv_heads, BLOCK, c.head_dim)
-        layers = []
+        # one tensor per layer [nb, 2, Hkv, 64, D] (hybrid decoders: [nb, elements of a block]): the first layers live
+        # in the borrowed buffer, the rest is new
+        elems = self._layer_elems()
+        n_lent = used = 0
+        while n_lent < len(elems) and used + nb * elems[n_lent] * esize <= lent:
+            used += nb * elems[n_lent] * esize
+            n_lent += 1
+        pieces = []
         if n_lent:
-            flat = self.borrowed.reshape(-1).view(torch.uint8)[: n_lent * per_layer * esize].view(self.dtype)
+            flat = self.borrowed.reshape(-1).view(torch.uint8)[:used].view(self.dtype)
             flat.zero_()    # rows past a sequence's length are multiplied by zero weights: they must be finite
-            layers += [flat[i * per_layer:(i + 1) * per_layer].view(shape) for i in range(n_lent)]
-        if n_lent < c.num_layers:
-            own = torch.zeros(c.num_layers - n_lent, *shape, dtype=self.dtype, device=self.device)
-            layers += [own[i] for i in range(c.num_layers - n_lent)]
+            pieces += flat.split([nb * e for e in elems[:n_lent]])
+        if n_lent < len(elems):
+            own = torch.zeros(nb * sum(elems[n_lent:]), dtype=self.dtype, device=self.device)
+            pieces += own.split([nb * e for e in elems[n_lent:]])
+        shape = (nb, -1) if c.hybrid is not None else (nb, 2, c.num_kv_heads, BLOCK, c.head_dim)
+        layers = [x.view(shape) for x in pieces]
         self.cache = layers
         self.kv_layout = {"blocks": nb, "layers_in_borrowed_memory": n_lent}
         self.alloc = BlockAllocator(nb)
@@ -233,6 +264,8 @@ class RolloutEngine:
             return
         dev = self.device
         self.num_slots = S
+        self.states = []                # the old ones go before the new ones come
+        self.states = self.model.new_states(S) if self.recurrent else []
         self.block_table = torch.full((S, self.max_blocks_per_seq), -1, dtype=torch.int32, device=dev)
         self.ctx_len = torch.zeros(S, dtype=torch.int32, device=dev)       # tokens in the cache
         self.last_token = torch.zeros(S, dtype=torch.int64, device=dev)
@@ -253,6 +286,8 @@ class RolloutEngine:
         """Free the cache arena (the trainer gets the memory back)."""
         self.cache = None
         self.alloc = None
+        self.states = []
+        self.num_slots = 0
         self._graphs.clear()
         if self.device.type == "cuda":
             torch.cuda.empty_cache()
@@ -260,11 +295,11 @@ class RolloutEngine:
     # ---- prefill --------------------------------------------------------------------------------
     @torch.no_grad()
     def _prefill(self, seqs: List[_Seq], chunks: List[List[int]], starts: Optional[List[int]] = None,
-                 mm_inputs=None) -> torch.Tensor:
+                 mm_inputs=None, all_rows: bool = False) -> torch.Tensor:
         """Prefill one packed batch: ``chunks[i]`` are the next tokens of the prompt of ``seqs[i]`` (sample 0 of its
         group), ``starts[i]`` how many of its tokens the cache holds already (a prefix-cache hit or earlier chunks;
         default 0 = whole prompts).  Returns the final hidden state of the last token of each chunk
-        ``[len(seqs), H]``.  ``mm_inputs[i]`` (optional, whole prompts only) holds prompt i's ``pixel_values
+        ``[len(seqs), H]`` (``all_rows``: of every token).  ``mm_inputs[i]`` (optional, whole prompts only) holds prompt i's ``pixel_values
         [patches, D]``, ``image_grid_thw [images, 3]`` and ``rope_positions [3, len]``."""
         lens = [len(p) for p in chunks]
         starts = list(starts) if starts is not None else [0] * len(chunks)
@@ -288,12 +323,52 @@ class RolloutEngine:
             positions = torch.cat([torch.arange(st, st + n, dtype=torch.int32) for st, n in zip(starts, lens)]).to(
                 self.device)
             mm["prefix_lens"] = starts
+        if any(starts) or self.cfg.hybrid is not None:
             mm["prefill_slots"] = [s.slot for s in seqs]
         hidden = self.model.forward_cached(ids, positions, self.cache, self.block_table, seq_ids,
-                                           prefill_info=info, **mm)
-        last = torch.tensor([c - 1 for c in info.cu_seqlens_cpu[1:]], dtype=torch.int64, device=self.device)
+                                           prefill_info=info, **mm, **self._state_kw())
         self.stats["prefill_tokens"] += sum(lens)
+        if all_rows:
+            return hidden
+        last = torch.tensor([c - 1 for c in info.cu_seqlens_cpu[1:]], dtype=torch.int64, device=self.device)
         return hidden.index_select(0, last)
+
+    def _state_kw(self) -> dict:
+        return {"states": self.states} if self.cfg.hybrid is not None else {}
+
+    # ---- sequences' places -----------------------------------------------------------------------
+    def _reset_slots(self) -> None:
+        self.finished.fill_(True)
+        self.ctx_len.zero_()
+        self.remaining.zero_()
+        self.rope_delta.zero_()
+        self.block_table.fill_(-1)
+
+    def _write_block_tables(self, seqs: Sequence[_Seq]) -> None:
+        bt = self.block_table.cpu()
+        for seq in seqs:
+            bt[seq.slot, : len(seq.blocks)] = torch.tensor(seq.blocks, dtype=torch.int32)
+        self.block_table.copy_(bt)
+
+    def _release_blocks(self, seq: _Seq) -> None:
+        for b in seq.blocks:
+            if b >= 0:
+                self.alloc.release(b)
+        seq.blocks = []
+
+    def _release_hidden_blocks(self, seq: _Seq, next_pos: int) -> None:
+        """Give back the blocks of ``seq`` that no layer looks at from position ``next_pos`` on."""
+        if self.visible_span is None:
+            return
+        window, keep_first = self.visible_span
+        first, end = (keep_first + BLOCK - 1) // BLOCK, max(0, next_pos - window + 1) // BLOCK
+        dead = [j for j in range(max(first, seq.hidden_until), end) if seq.blocks[j] >= 0]
+        seq.hidden_until = max(seq.hidden_until, end)
+        if dead:
+            for j in dead:
+                self.alloc.release(seq.blocks[j])
+                seq.blocks[j] = -1
+            self.block_table[seq.slot, dead[0]:dead[-1] + 1] = -1
 
     # ---- decode ---------------------------------------------------------------------------------
     def _decode_step(self, sp: SamplingParams, tokens_out: torch.Tensor, logp_out: torch.Tensor) -> None:
@@ -302,12 +377,7 @@ class RolloutEngine:
         if self.device.type == "cuda":
             return self._decode_step_native(sp, tokens_out, logp_out)
         active = ~self.finished
-        pos = torch.where(active, self.ctx_len, torch.full_like(self.ctx_len, -1))
-        seq_ids = torch.where(active, self.slot_ids, torch.full_like(self.slot_ids, -1))
-        seq_lens = torch.where(active, self.ctx_len + 1, torch.zeros_like(self.ctx_len))
-        hidden = self.model.forward_cached(self.last_token, pos.clamp(min=0), self.cache, self.block_table, seq_ids,
-                                           seq_lens=seq_lens, rope_positions=(pos - self.rope_delta).clamp(min=0))
-        logits = lm_head_logits(hidden, self.model.head_weight)
+        logits = self._decode_logits()
         tok, lp = sample(logits, sp.temperature, sp.top_k, sp.top_p, seed=sp.seed, step_dev=self.step_counter
                          if self.device.type == "cuda" else None, step=int(self.step_counter.item())
                          if self.device.type != "cuda" else 0)
@@ -328,6 +398,31 @@ class RolloutEngine:
         self.step_counter += 1
         _ = pad
 
+    def _decode_logits(self) -> torch.Tensor:
+        """fp32 logits ``[slots, V]`` of one decode forward: every slot that is not finished consumes its
+        ``last_token`` at position ``ctx_len`` (rows of idle slots are meaningless)."""
+        if self.device.type != "cuda":
+            active = ~self.finished
+            pos = torch.where(active, self.ctx_len, torch.full_like(self.ctx_len, -1))
+            seq_ids = torch.where(active, self.slot_ids, torch.full_like(self.slot_ids, -1))
+            seq_lens = torch.where(active, self.ctx_len + 1, torch.zeros_like(self.ctx_len))
+            hidden = self.model.forward_cached(self.last_token, pos.clamp(min=0), self.cache, self.block_table, seq_ids,
+                                               seq_lens=seq_lens, rope_positions=(pos - self.rope_delta).clamp(min=0),
+                                               **self._state_kw())
+            return self._logits(hidden)
+        from ...ops import lib as _lib
+        st = self._step_bufs
+        _lib.check(_lib.get_lib().sb_decode_prepare(
+            _lib.ptr(self.finished), _lib.ptr(self.ctx_len), _lib.ptr(self.rope_delta), _lib.ptr(st["pos"]),
+            _lib.ptr(st["seq_ids"]), _lib.ptr(st["seq_lens"]), _lib.ptr(st["rope_pos"]), self.num_slots,
+            _lib.stream()), "sb_decode_prepare")
+        hidden = self.model.forward_cached(self.last_token, st["pos"], self.cache, self.block_table, st["seq_ids"],
+                                           seq_lens=st["seq_lens"], rope_positions=st["rope_pos"], **self._state_kw())
+        return self._logits(hidden)
+
+    def _logits(self, hidden: torch.Tensor) -> torch.Tensor:
+        return lm_head_logits(hidden, self.model.head_weight, self.cfg.logit_softcap)
+
     def _decode_step_native(self, sp: SamplingParams, tokens_out: torch.Tensor, logp_out: torch.Tensor) -> None:
         """The same step on CUDA: two bookkeeping kernels (``csrc/decode_state.cu``) around forward, LM head and
         sampler; no element-wise torch launches."""
@@ -336,13 +431,7 @@ class RolloutEngine:
         from ...ops import lib as _lib
         L = _lib.get_lib()
         S = self.num_slots
-        st = self._step_bufs
-        _lib.check(L.sb_decode_prepare(_lib.ptr(self.finished), _lib.ptr(self.ctx_len), _lib.ptr(self.rope_delta),
-                                       _lib.ptr(st["pos"]), _lib.ptr(st["seq_ids"]), _lib.ptr(st["seq_lens"]),
-                                       _lib.ptr(st["rope_pos"]), S, _lib.stream()), "sb_decode_prepare")
-        hidden = self.model.forward_cached(self.last_token, st["pos"], self.cache, self.block_table, st["seq_ids"],
-                                           seq_lens=st["seq_lens"], rope_positions=st["rope_pos"])
-        logits = lm_head_logits(hidden, self.model.head_weight)
+        logits = self._decode_logits()
         # the request's seed lives in the device-side step counter (see ``generate``), not in a launch argument, so
         # that one captured graph serves every seed
         tok, lp = sample(logits, sp.temperature, sp.top_k, sp.top_p, seed=_STREAM_KEY, step_dev=self.step_counter)
@@ -368,6 +457,8 @@ class RolloutEngine:
                                             self.step_counter, self.gen_index, self.hit_eos, tokens_out, logp_out)]
             s = torch.cuda.Stream()
             s.wait_stream(torch.cuda.current_stream())
+            if self.recurrent:
+                self.finished.fill_(True)       # all idle: the warm-up step must not advance the recurrent states
             with torch.cuda.stream(s):
                 self._decode_step(sp, tokens_out, logp_out)
             torch.cuda.current_stream().wait_stream(s)
@@ -419,11 +510,7 @@ class RolloutEngine:
         if dev.type == "cuda":
             # random stream of this call: counter range [seed << 24, ...) of the fixed key (16 M steps per seed)
             self.step_counter.fill_((int(sp.seed) & 0x7FFFFFFF) << 24)
-        self.finished.fill_(True)
-        self.ctx_len.zero_()
-        self.remaining.zero_()
-        self.rope_delta.zero_()
-        self.block_table.fill_(-1)
+        self._reset_slots()
 
         def blocks_needed(plen: int) -> int:
             return (plen + R + BLOCK - 1) // BLOCK
@@ -435,8 +522,7 @@ class RolloutEngine:
             self.stats["d2h_bytes"] = self.stats.get("d2h_bytes", 0) + 12 * n_gen
             results[(seq.prompt_index, seq.sample_index)] = RolloutOutput(seq.prompt_index, seq.sample_index, toks,
                                                                          lps, fin_reason)
-            for b in seq.blocks:
-                self.alloc.release(b)
+            self._release_blocks(seq)
             slots[slot] = None
             self.stats["generated_tokens"] += n_gen
 
@@ -516,16 +602,12 @@ class RolloutEngine:
                                           prefill_info=one)
             if jobs:
                 if new_groups:
-                    bt = self.block_table.cpu()
-                    for group in new_groups:
-                        for seq in group:
-                            bt[seq.slot, : len(seq.blocks)] = torch.tensor(seq.blocks, dtype=torch.int32)
-                    self.block_table.copy_(bt)
+                    self._write_block_tables([seq for group in new_groups for seq in group])
                 batch_mm = [mm_inputs[g[0].prompt_index] for g, _, _ in jobs] if mm_inputs is not None else None
                 hidden = self._prefill([g[0] for g, _, _ in jobs],
                                        [list(prompts[g[0].prompt_index])[a:b] for g, a, b in jobs],
                                        [a for _, a, _ in jobs], batch_mm)
-                done_rows, batch_seqs, forks = [], [], []
+                done_rows, batch_seqs, forks, state_forks = [], [], [], []
                 for row, (group, _a, b) in enumerate(jobs):
                     lead = group[0]
                     lead.prefilled = b
@@ -537,19 +619,26 @@ class RolloutEngine:
                     full = plen // BLOCK
                     if plen % BLOCK:
                         forks += [(lead.blocks[full], other.blocks[full]) for other in group[1:]]
+                    if self.recurrent:
+                        state_forks += [(lead.slot, other.slot) for other in group[1:]]
                     if use_cache:
                         for j, k in enumerate(_prefix_hashes(list(prompts[lead.prompt_index]), full)):
-                            self.alloc.register(k, lead.blocks[j])
+                            if lead.blocks[j] >= 0:
+                                self.alloc.register(k, lead.blocks[j])
                 pending = [g for g in pending if g[0].prefilled < g[0].prompt_len]
                 if forks:
                     src = torch.tensor([a for a, _ in forks], dtype=torch.int32, device=dev)
                     dst = torch.tensor([b for _, b in forks], dtype=torch.int32, device=dev)
-                    for li in range(self.cfg.num_layers):
-                        kvc.kv_copy_blocks(self.cache[li], src, dst)
+                    for layer in self.cache:
+                        kvc.kv_copy_blocks(layer, src, dst)
+                if state_forks:
+                    src, dst = (torch.tensor(x, dtype=torch.int64, device=dev) for x in zip(*state_forks))
+                    for state in self.states:
+                        copy_states(state, src, dst)
             if jobs and batch_seqs:
                 # first token of every sample comes from the prompt's last hidden state
                 rep_idx = torch.tensor([done_rows[i] for i, g in enumerate(batch_seqs) for _ in g], device=dev)
-                logits = lm_head_logits(hidden.index_select(0, rep_idx), self.model.head_weight)
+                logits = self._logits(hidden.index_select(0, rep_idx))
                 tok, lp = sample(logits, sp.temperature, sp.top_k, sp.top_p, seed=sp.seed ^ 0x5bd1e995,
                                  step=int(self.step_counter.item()))
                 self.step_counter += 1
@@ -591,7 +680,12 @@ class RolloutEngine:
             eos_cpu = self.hit_eos.cpu().tolist()
             self.stats["d2h_bytes"] = self.stats.get("d2h_bytes", 0) + 6 * S
             prefilling = {s.slot for g in pending for s in g}
+            if self.visible_span is not None:
+                for group in pending:
+                    self._release_hidden_blocks(group[0], group[0].prefilled)
             for slot, seq in enumerate(slots):
+                if seq is not None and not fin_cpu[slot] and slot not in prefilling:
+                    self._release_hidden_blocks(seq, seq.prompt_len + gen_cpu[slot] - 1)
                 if seq is not None and fin_cpu[slot] and slot not in prefilling:
                     retire(slot, "stop" if eos_cpu[slot] else "length", gen_cpu[slot])
                     self.ctx_len[slot] = 0

@@ -13,6 +13,7 @@ from typing import List, Optional, Sequence
 import torch
 
 from ...ops.attention import SeqInfo
+from ...ops.rows import softcap_
 from ...ops.sampling import sample
 from .native_engine import RolloutOutput, SamplingParams
 
@@ -86,6 +87,8 @@ class RecomputeEngine:
                 hidden = self.model.forward_hidden(ids, positions, info, **kw)
                 last = torch.tensor(info.cu_seqlens_cpu[1:], device=dev) - 1
                 logits = hidden.index_select(0, last).float() @ self.model.head_weight.float().t()
+                if self.model.cfg.logit_softcap:
+                    logits = softcap_(logits, self.model.cfg.logit_softcap)
                 tok, lp = sample(logits, sp.temperature, sp.top_k, sp.top_p, seed=sp.seed, step=step * 4099 + g0,
                                  generator=gen)
                 self.stats["decode_steps"] += 1

@@ -685,6 +685,8 @@ class ActorRolloutRefWorker(_ModelWorkerBase):
             if getattr(self, "_tp_train", None) is not None and tp == 1:
                 raise ValueError("a tensor-parallel trainer needs rollout.tensor_model_parallel_size equal to "
                                  "megatron.tensor_model_parallel_size (the engine runs on the trainer's slices)")
+            if tp > 1 and self.model_config.hybrid is not None:
+                raise ValueError("hybrid decoders run on whole weights: set rollout.tensor_model_parallel_size=1")
             if tp > 1:
                 self.tp_model = self._build_tp_model(tp, r.max_num_batched_tokens)
             if str(r.name).lower() == "hf" or self.model_config.is_mla:

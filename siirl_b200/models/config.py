@@ -97,6 +97,56 @@ class PrismaticConfig:
 
 
 @dataclass
+class MixerBranch:
+    """One token mixer of a hybrid layer.  ``kind``: "attention" (paged cache, sliding window with kept first tokens,
+    linear distance bias), "gated_linear" (matrix state, decay per key channel) or "matrix_memory" (stabilised mLSTM)."""
+    kind: str = "attention"
+    heads: int = 4
+    dim: int = 32                   # query / key width of a head
+    vdim: int = 32                  # value width of a head
+    out_scale: float = 1.0          # factor of this branch in the layer's sum
+    # attention
+    kv_heads: int = 0
+    scale: float = 0.0
+    window: int = 0                 # 0: no limit
+    keep_first: int = 0
+    bias_exp: float = 8.0           # slope of head h: 2^(-bias_exp (h + 1) / heads); 0: no bias
+    # gated_linear
+    tau: float = 16.0
+    rank: int = 0                   # width of the decay's low-rank bottleneck (the checkpoint's tensor shape)
+    # matrix_memory
+    gate_cap: float = 15.0
+
+
+@dataclass
+class HybridLayer:
+    branches: List[MixerBranch] = field(default_factory=list)
+    ff: int = 0                     # 0: the layer has no feed-forward
+
+
+@dataclass
+class HybridSpec:
+    """Decoders whose layers mix attention and recurrences; the residual stream is kept in 32-bit."""
+    layers: List[HybridLayer] = field(default_factory=list)
+    embed_scale: float = 1.0
+    logit_softcap: float = 0.0      # 0: none
+    norm: str = "layer_norm"        # or "rms_norm"
+    act: str = "gelu_tanh"          # or "silu"
+    hf_naming: str = "domavik"
+
+    @property
+    def attention(self) -> List[MixerBranch]:
+        return [b for layer in self.layers for b in layer.branches if b.kind == "attention"]
+
+    def visible_span(self):
+        """(window, keep_first) outside which no layer looks, or ``None`` when some layer sees everything."""
+        att = self.attention
+        if any(b.window <= 0 for b in att):
+            return None
+        return (max((b.window for b in att), default=1), max((b.keep_first for b in att), default=0))
+
+
+@dataclass
 class DecoderConfig:
     model_type: str = "qwen2"
     vocab_size: int = 1024
@@ -164,6 +214,8 @@ class DecoderConfig:
     # ``action_vocab_size`` (the tokenizer's size: the embedding matrix is padded beyond it)
     prismatic: Optional[PrismaticConfig] = None
     moonvit: Optional[MoonViTConfig] = None
+    # per-layer mixers of a hybrid decoder (models/hybrid.py); the uniform attention fields above do not apply then
+    hybrid: Optional[HybridSpec] = None
     action_vocab_size: int = 0
     n_action_bins: int = 256
     image_token_id: int = 151655
@@ -200,7 +252,19 @@ class DecoderConfig:
     def qkv_width(self) -> int:
         return self.q_width + 2 * self.kv_width
 
+    @property
+    def logit_softcap(self) -> float:
+        return self.hybrid.logit_softcap if self.hybrid is not None else 0.0
+
+    def paged_layers(self) -> List[tuple]:
+        """(kv heads, key width, value width) of every layer that keeps keys and values in the paged cache."""
+        if self.hybrid is not None:
+            return [(b.kv_heads, b.dim, b.vdim) for b in self.hybrid.attention]
+        return [(self.num_kv_heads, self.head_dim, self.head_dim)] * self.num_layers
+
     def num_parameters(self) -> int:
+        if self.hybrid is not None:
+            return self._hybrid_parameters()
         H, I, V = self.hidden_size, self.intermediate_size, self.vocab_size
         attn = H * self.qkv_width + (self.qkv_width if self.qkv_bias else 0) + self.q_width * H
         if self.qk_norm:
@@ -213,6 +277,19 @@ class DecoderConfig:
         per_layer = attn + mlp + 2 * H
         head = 0 if self.tie_word_embeddings else (H if self.value_head else V * H)
         return V * H + self.num_layers * per_layer + H + head
+
+    def _hybrid_parameters(self) -> int:
+        W, n = self.hidden_size, 2 * self.vocab_size * self.hidden_size + self.hidden_size
+        for layer in self.hybrid.layers:
+            n += W + (W + 3 * W * layer.ff if layer.ff else 0)
+            for b in layer.branches:
+                hk, hv = b.heads * b.dim, b.heads * b.vdim
+                if b.kind == "attention":
+                    n += W * (hk + b.kv_heads * (b.dim + b.vdim) + hv)
+                    continue
+                n += W * (2 * hk + 3 * hv)
+                n += (b.rank * (W + hk) + hk + b.vdim) if b.kind == "gated_linear" else 2 * b.heads * (W + 1) + hv
+        return n
 
     def to_dict(self) -> Dict[str, Any]:
         return asdict(self)
@@ -237,6 +314,11 @@ class DecoderConfig:
             pr["featurizer"] = build(ViTConfig, pr.get("featurizer"))
             pr["fused_featurizer"] = build(ViTConfig, pr.get("fused_featurizer"))
             d["prismatic"] = build(PrismaticConfig, pr)
+        if isinstance(d.get("hybrid"), dict):
+            hy = dict(d["hybrid"])
+            hy["layers"] = [build(HybridLayer, dict(x, branches=[build(MixerBranch, b) for b in x["branches"]]))
+                            for x in hy.get("layers", [])]
+            d["hybrid"] = build(HybridSpec, hy)
         for key in ("lora_targets", "mrope_section"):
             if isinstance(d.get(key), list) and key == "lora_targets":
                 d[key] = tuple(d[key])
@@ -246,6 +328,8 @@ class DecoderConfig:
     # ---- HF interchange -----------------------------------------------------------------------
     @classmethod
     def from_hf_config(cls, cfg: Dict[str, Any]) -> "DecoderConfig":
+        if cfg.get("architecture") == "Domavik":
+            return cls._from_domavik_config(cfg)
         text = cfg.get("text_config") or cfg.get("llm_config") or cfg
         mt = cfg.get("model_type", "qwen2")
         if mt in ("llama4", "llama4_text"):
@@ -405,11 +489,81 @@ class DecoderConfig:
         return out
 
     @classmethod
+    def _from_domavik_config(cls, cfg: Dict[str, Any]) -> "DecoderConfig":
+        """Domavik: every layer is either one matrix memory ("mlstm") or window attention beside gated linear attention
+        ("parallel"), with an optional gated feed-forward.  The decay's low-rank width is not in the file: it is the
+        shape of a tensor, filled in by ``from_pretrained``."""
+        def attention(m, scale):
+            mask = m["mask"]
+            return MixerBranch(kind="attention", heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]),
+                               vdim=int(m["vdim"]), scale=float(m["scale"]), window=int(mask["size"]),
+                               keep_first=int(mask["keep_first"]), bias_exp=8.0, out_scale=float(scale))
+
+        def gated(m, scale):
+            return MixerBranch(kind="gated_linear", heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
+                               tau=float(m["tau"]), out_scale=float(scale))
+        layers = []
+        for x in cfg["layers"]:
+            m, mlp = x["mixer"], x.get("mlp")
+            if x["type"] == "mlstm":
+                branches = [MixerBranch(kind="matrix_memory", heads=int(m["heads"]), dim=int(m["dim"]),
+                                        vdim=int(m["vdim"]), gate_cap=float(m["gate_cap"]))]
+            elif x["type"] == "parallel":
+                branches = [attention(m["left"], m["left_scale"]), gated(m["right"], m["right_scale"])]
+            else:
+                raise ValueError(f"unknown layer type {x['type']!r}")
+            if mlp is not None and mlp["kind"] != "dense":
+                raise ValueError(f"unknown feed-forward kind {mlp['kind']!r}")
+            layers.append(HybridLayer(branches=branches, ff=int(mlp["ff"]) if mlp is not None else 0))
+        spec = HybridSpec(layers=layers, embed_scale=float(cfg["embedding"]["scale"]),
+                          logit_softcap=float(cfg.get("logit_softcap") or 0.0))
+        return cls.for_hybrid(spec, vocab_size=int(cfg["vocab"]), hidden_size=int(cfg["width"]),
+                              rms_norm_eps=float(cfg["norm"]["eps"]), model_type="domavik",
+                              eos_token_id=int(cfg.get("eos_token_id", -1)), pad_token_id=int(cfg.get("pad_token_id", 0)))
+
+    @classmethod
+    def for_hybrid(cls, spec: HybridSpec, **kw) -> "DecoderConfig":
+        """Configuration around a hybrid spec: the uniform fields that metrics and launchers read are filled from it."""
+        att = spec.attention
+        b = att[0] if att else (spec.layers[0].branches[0] if spec.layers else MixerBranch())
+        return cls(hybrid=spec, num_layers=len(spec.layers), num_heads=b.heads, num_kv_heads=b.kv_heads or b.heads,
+                   head_dim=b.dim, intermediate_size=max((x.ff for x in spec.layers), default=0), qkv_bias=False, **kw)
+
+    def _to_domavik_config(self) -> Dict[str, Any]:
+        hy = self.hybrid
+
+        def sizes(b, *names):
+            return {n: getattr(b, n) for n in ("heads", "dim", "vdim") + names}
+        layers = []
+        for x in hy.layers:
+            b = x.branches[0]
+            if b.kind == "matrix_memory":
+                t, m = "mlstm", sizes(b, "gate_cap")
+            else:
+                r = x.branches[1]
+                t, m = "parallel", {"left": dict(sizes(b, "kv_heads", "scale"), mask={"size": b.window,
+                                                                                      "keep_first": b.keep_first}),
+                                    "right": sizes(r, "tau"), "left_scale": b.out_scale, "right_scale": r.out_scale}
+            layers.append({"type": t, "mixer": m, "mlp": {"kind": "dense", "ff": x.ff} if x.ff else None})
+        d = {"architecture": "Domavik", "vocab": self.vocab_size, "width": self.hidden_size,
+             "embedding": {"scale": hy.embed_scale}, "norm": {"eps": self.rms_norm_eps},
+             "logit_softcap": hy.logit_softcap, "layers": layers}
+        if self.eos_token_id >= 0:
+            d["eos_token_id"] = self.eos_token_id
+        return d
+
+    @classmethod
     def from_pretrained(cls, path: str) -> "DecoderConfig":
         with open(os.path.join(os.path.expanduser(path), "config.json")) as f:
-            return cls.from_hf_config(json.load(f))
+            out = cls.from_hf_config(json.load(f))
+        if out.hybrid is not None:
+            from .hf_io import fill_hybrid_ranks
+            fill_hybrid_ranks(out, path)
+        return out
 
     def to_hf_config(self) -> Dict[str, Any]:
+        if self.hybrid is not None:
+            return self._to_domavik_config()
         arch = {"qwen2": "Qwen2ForCausalLM", "qwen3": "Qwen3ForCausalLM", "qwen3_moe": "Qwen3MoeForCausalLM",
                 "llama": "LlamaForCausalLM", "qwen2_5_vl": "Qwen2_5_VLForConditionalGeneration",
                 "mixtral": "MixtralForCausalLM", "qwen2_moe": "Qwen2MoeForCausalLM",
@@ -511,7 +665,33 @@ def vit_from_timm_id(model_id: str, image_size: int = 224) -> ViTConfig:
     raise ValueError(f"unknown vision backbone {model_id}")
 
 
+def _domavik(n_layers: int, width: int, ff: int, vocab: int, att: dict, gla: dict, mem: dict, scales=(1.0, 1.0),
+             softcap: float = 30.0, embed_scale: float = 1.0, **kw) -> DecoderConfig:
+    """Alternating Domavik layers: attention beside gated linear attention, then a matrix memory."""
+    layers = []
+    for i in range(n_layers):
+        if i % 2 == 0:
+            br = [MixerBranch(kind="attention", out_scale=scales[0], scale=att["dim"] ** -0.5, **att),
+                  MixerBranch(kind="gated_linear", out_scale=scales[1], **gla)]
+        else:
+            br = [MixerBranch(kind="matrix_memory", **mem)]
+        layers.append(HybridLayer(branches=br, ff=ff))
+    spec = HybridSpec(layers=layers, embed_scale=embed_scale, logit_softcap=softcap)
+    return DecoderConfig.for_hybrid(spec, vocab_size=vocab, hidden_size=width, rms_norm_eps=1e-5, model_type="domavik",
+                                    **kw)
+
+
 PRESETS: Dict[str, DecoderConfig] = {
+    "tiny-domavik": _domavik(3, 128, 192, 1024, dict(heads=4, kv_heads=2, dim=32, vdim=24, window=70, keep_first=5),
+                             dict(heads=2, dim=16, vdim=32, tau=4.0, rank=8), dict(heads=2, dim=32, vdim=40),
+                             scales=(0.9, 0.6)),
+    # layer sizes of a 7B / 1.5B-class decoder (benchmark shapes, random weights)
+    "domavik-7b": _domavik(28, 3584, 18944, 152064, dict(heads=28, kv_heads=4, dim=128, vdim=128, window=1024,
+                                                         keep_first=64),
+                           dict(heads=16, dim=64, vdim=128, rank=16), dict(heads=16, dim=128, vdim=128)),
+    "domavik-1.5b": _domavik(28, 1536, 8960, 152064, dict(heads=12, kv_heads=2, dim=128, vdim=128, window=1024,
+                                                          keep_first=64),
+                             dict(heads=8, dim=64, vdim=128, rank=16), dict(heads=8, dim=96, vdim=128)),
     # 2-layer gate model used by the CPU/gloo end-to-end test
     "tiny": DecoderConfig(model_type="qwen2", vocab_size=1024, hidden_size=128, intermediate_size=352, num_layers=2,
                           num_heads=4, num_kv_heads=2, head_dim=32, rope_theta=1e4, eos_token_id=2),

@@ -598,5 +598,9 @@ class DecoderLM(nn.Module):
 
 
 def build_model(cfg: DecoderConfig, dtype=torch.bfloat16, device="cpu", seed: int = 0,
-                gradient_checkpointing: bool = False) -> DecoderLM:
+                gradient_checkpointing: bool = False) -> nn.Module:
+    """The model class of a configuration: :class:`DecoderLM`, or :class:`HybridLM` for hybrid decoders."""
+    if cfg.hybrid is not None:
+        from .hybrid import HybridLM
+        return HybridLM(cfg, dtype=dtype, device=device, seed=seed, gradient_checkpointing=gradient_checkpointing)
     return DecoderLM(cfg, dtype=dtype, device=device, seed=seed, gradient_checkpointing=gradient_checkpointing)

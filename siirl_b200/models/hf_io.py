@@ -276,10 +276,56 @@ def _qwen_visual_state(vision, prefix: str = "model.visual.") -> Iterator[Tuple[
     yield prefix + "merger.mlp.2.bias", vision.merger_fc2_bias.data
 
 
+def _domavik_state(model) -> Iterator[Tuple[str, torch.Tensor]]:
+    """Domavik checkpoint names and the views of the fused, padded parameters they fill (models/hybrid.py)."""
+    yield "embed", model.embed_tokens.data
+    for i, layer in enumerate(model.layers):
+        p = f"l{i}."
+        yield p + "norm1", layer.norm1.data
+        parallel = len(layer.branches) > 1
+        for j, br in enumerate(layer.branches):
+            m = p + "mix." + (("left.", "right.")[j] if parallel else "")
+            for name, (at, n) in br.cols.items():
+                yield m + name, layer.in_proj_weight.data[at:at + n]
+            n = br.b.heads * br.b.vdim
+            yield m + "o", layer.o_proj_weight.data[:, br.out_off:br.out_off + n]
+            if br.b.kind == "gated_linear":
+                yield m + "norm", br.norm.data
+                yield m + "a2", br.w2.data
+                yield m + "a2.b", br.b_e.data
+            elif br.b.kind == "matrix_memory":
+                yield m + "norm", br.norm.data
+                yield m + "i.b", br.b_e.data
+                yield m + "f.b", br.b_f.data
+        if layer.ff:
+            yield p + "norm2", layer.norm2.data
+            yield p + "mlp.gate", layer.gate_up_proj_weight.data[:layer.ff]
+            yield p + "mlp.up", layer.gate_up_proj_weight.data[layer.ffp:layer.ffp + layer.ff]
+            yield p + "mlp.down", layer.down_proj_weight.data[:, :layer.ff]
+    yield "final.norm", model.norm.data
+    yield "head", model.lm_head.data
+
+
+def fill_hybrid_ranks(cfg: DecoderConfig, path: str) -> None:
+    """Sizes that only tensor shapes give: the low-rank width of every decay projection."""
+    handles = _open_all(path)
+    where = {k: h for h in handles for k in h.keys()}
+    for i, layer in enumerate(cfg.hybrid.layers):
+        for j, b in enumerate(layer.branches):
+            if b.kind == "gated_linear" and not b.rank:
+                name = f"l{i}.mix." + (("left.", "right.")[j] if len(layer.branches) > 1 else "") + "a1"
+                if name not in where:
+                    raise KeyError(f"{name} missing in {path}")
+                b.rank = int(where[name].get_slice(name).get_shape()[0])
+
+
 def _hf_targets(model) -> Iterator[Tuple[str, object]]:
     """(checkpoint name, view into the model's parameter) for every tensor of the family's HF checkpoint; InternLM2's
     fused ``wqkv`` comes as the tuple of its three views."""
     cfg: DecoderConfig = model.cfg
+    if cfg.hybrid is not None:
+        yield from _domavik_state(model)
+        return
     prefix, head = _llm_names(cfg)
     internlm2 = cfg.vit is not None and cfg.hf_naming == "internvl_chat" and cfg.llm_type == "internlm2"
     held: Dict[str, torch.Tensor] = {}
@@ -415,4 +461,7 @@ def load_hf_weights(model, path: str, strict: bool = True) -> None:
                 for d, part in zip(dst, _split_wqkv(src, cfg)):
                     d.copy_(part.to(d.dtype))
             else:
+                if cfg.hybrid is not None and tuple(src.shape) != tuple(dst.shape):
+                    raise ValueError(f"{name}: shape {tuple(src.shape)} where the configuration needs "
+                                     f"{tuple(dst.shape)}")
                 dst.copy_(src.reshape(dst.shape).to(dst.dtype))

@@ -1,0 +1,276 @@
+"""Hybrid decoder: layers that mix window attention and matrix-state recurrences, with the residual stream in 32-bit.
+
+Every layer is a list of branches over one normed input (``DecoderConfig.hybrid``): their projections are one fused
+matrix (``in_proj``), each branch writes its (scaled) heads into its columns of one row, and one matrix (``o_proj``) adds
+the branches up.  The serving path is the one of :class:`DecoderLM`: ``forward_cached`` over the engine's paged blocks,
+plus the engine's per-slot recurrent states.  A prompt portion appends its keys and values and reads everything it sees
+back from the cache, so whole prompts, portions and single tokens use the same memory.
+
+bf16 models run the tensor-core kernels; fp32 models run true 32-bit kernels (FMA-pipe matrix products).  Weights keep
+the checkpoint's values; fused matrices are padded with zero rows / columns to multiples of eight.  Scoring
+(``logprobs``) is supported; there is no backward pass on CUDA."""
+from __future__ import annotations
+
+import ctypes
+from typing import Dict, List, Optional, Sequence, Tuple
+
+import torch
+import torch.nn as nn
+
+from .. import ops
+from ..ops import kv_cache as kvc
+from ..ops import rows as R
+from ..ops.attention import SeqInfo
+from ..ops.lm_head import lm_head_logits
+from ..ops.recurrence import PortionPlan, RecurrenceSpec, empty_state, recurrence_decode, recurrence_prefill
+from ..ops.window_attention import QueryTiles, WindowSpec, window_attention
+from .config import DecoderConfig, MixerBranch
+from .decoder import _Init, _param
+
+
+def _pad8(n: int) -> int:
+    return (n + 7) // 8 * 8
+
+
+def branch_segments(b: MixerBranch) -> List[Tuple[str, int]]:
+    """(name, rows) of a branch's projections in ``in_proj``, in order."""
+    hk, hv = b.heads * b.dim, b.heads * b.vdim
+    if b.kind == "attention":
+        return [("q", hk), ("k", b.kv_heads * b.dim), ("v", b.kv_heads * b.vdim)]
+    seg = [("q", hk), ("k", hk), ("v", hv), ("g", hv)]
+    return seg + ([("a1", b.rank)] if b.kind == "gated_linear" else [("i", b.heads), ("f", b.heads)])
+
+
+class HybridBranch(nn.Module):
+    """Small parameters of one branch and its place in the layer's fused rows."""
+
+    def __init__(self, b: MixerBranch, cfg: DecoderConfig, in_off: int, out_off: int, dtype, device, gen):
+        super().__init__()
+        self.b = b
+        self.out_off = out_off
+        self.cols: Dict[str, Tuple[int, int]] = {}
+        for name, n in branch_segments(b):
+            self.cols[name] = (in_off, n)
+            in_off += _pad8(n)
+        self.in_end = in_off
+        off = {k: v[0] for k, v in self.cols.items()}
+        if b.kind == "attention":
+            self.spec = WindowSpec(b.heads, b.kv_heads, b.dim, b.vdim, off["q"], off["k"], off["v"], b.scale, b.window,
+                                   b.keep_first, b.bias_exp, b.out_scale)
+            return
+        hk, hv = b.heads * b.dim, b.heads * b.vdim
+        common = dict(heads=b.heads, dim=b.dim, vdim=b.vdim, q_off=off["q"], k_off=off["k"], v_off=off["v"],
+                      g_off=off["g"], eps=cfg.rms_norm_eps, out_scale=b.out_scale)
+        if b.kind == "gated_linear":
+            if b.rank < 1:
+                raise ValueError("gated_linear: the decay's low-rank width is not set")
+            self.norm = _param((b.vdim,), dtype, device, -1, gen)
+            self.w2 = _param((hk, b.rank), dtype, device, b.rank ** -0.5, gen)
+            self.b_e = _param((hk,), dtype, device, 1.0, gen)
+            self.spec = RecurrenceSpec("channel", e_off=off["a1"], rank=b.rank, tau=b.tau, gate_act="silu", **common)
+        elif b.kind == "matrix_memory":
+            self.norm = _param((hv,), dtype, device, -1, gen)
+            self.b_e = _param((b.heads,), dtype, device, 0, gen)
+            self.b_f = _param((b.heads,), dtype, device, 1.0, gen)
+            self.spec = RecurrenceSpec("head", e_off=off["i"], f_off=off["f"], cap=b.gate_cap, gate_act="sigmoid",
+                                       norm_per_head=True, **common)
+        else:
+            raise ValueError(f"unknown mixer {b.kind!r}")
+
+    @property
+    def recurrent(self) -> bool:
+        return self.b.kind != "attention"
+
+    def weights(self) -> Dict[str, torch.Tensor]:
+        return {k: getattr(self, k).detach() for k in ("norm", "w2", "b_e", "b_f") if hasattr(self, k)}
+
+
+class HybridLayer(nn.Module):
+    def __init__(self, cfg: DecoderConfig, index: int, dtype, device, gen):
+        super().__init__()
+        lay, W, std = cfg.hybrid.layers[index], cfg.hidden_size, cfg.initializer_range
+        self.cfg, self.ff = cfg, lay.ff
+        in_off = out_off = 0
+        branches = []
+        for b in lay.branches:
+            br = HybridBranch(b, cfg, in_off, out_off, dtype, device, gen)
+            in_off, out_off = br.in_end, out_off + _pad8(b.heads * b.vdim)
+            branches.append(br)
+        self.branches = nn.ModuleList(branches)
+        self.padded_out = any(b.heads * b.vdim % 8 for b in lay.branches)
+        self.norm1 = _param((W,), dtype, device, -1, gen)
+        self.in_proj_weight = _param((in_off, W), dtype, device, std, gen)
+        self.o_proj_weight = _param((W, out_off), dtype, device, std, gen)
+        with torch.no_grad():
+            for br in self.branches:
+                for at, n in br.cols.values():
+                    self.in_proj_weight[at + n:at + _pad8(n)] = 0
+                n = br.b.heads * br.b.vdim
+                self.o_proj_weight[:, br.out_off + n:br.out_off + _pad8(n)] = 0
+        if self.ff:
+            self.ffp = _pad8(self.ff)
+            self.norm2 = _param((W,), dtype, device, -1, gen)
+            self.gate_up_proj_weight = _param((2 * self.ffp, W), dtype, device, std, gen)
+            self.down_proj_weight = _param((W, self.ffp), dtype, device, std, gen)
+            with torch.no_grad():
+                self.gate_up_proj_weight[self.ff:self.ffp] = 0
+                self.gate_up_proj_weight[self.ffp + self.ff:] = 0
+                self.down_proj_weight[:, self.ff:] = 0
+
+    def mix(self, x: torch.Tensor, io: "_Batch") -> torch.Tensor:
+        p = ops.linear(x, self.in_proj_weight)
+        alloc = torch.zeros if self.padded_out else torch.empty
+        out = alloc(x.shape[0], self.o_proj_weight.shape[1], dtype=x.dtype, device=x.device)
+        for br in self.branches:
+            if not br.recurrent:
+                window_attention(br.spec, p, io.seq_ids, io.positions, io.block_table, io.next_cache(), out, br.out_off,
+                                 tiles=io.tiles, seq_lens=io.seq_lens)
+            elif io.plan is not None:
+                recurrence_prefill(br.spec, p, br.weights(), io.next_state(), io.plan, out, br.out_off)
+            else:
+                recurrence_decode(br.spec, p, br.weights(), io.next_state(), io.seq_ids, io.positions, out, br.out_off)
+        return ops.linear(out, self.o_proj_weight)
+
+    def mlp(self, x: torch.Tensor) -> torch.Tensor:
+        return ops.linear(R.gated_act(ops.linear(x, self.gate_up_proj_weight), self.cfg.hybrid.act),
+                          self.down_proj_weight)
+
+
+class _Batch:
+    """What one forward pass needs besides the rows: places in the cache, prompt portions or decode lengths."""
+
+    def __init__(self, seq_ids, positions, block_table, cache, states, plan=None, tiles=None, seq_lens=None):
+        self.seq_ids, self.positions, self.block_table = seq_ids, positions, block_table
+        self.plan, self.tiles, self.seq_lens = plan, tiles, seq_lens
+        self._cache, self._states = iter(cache), iter(states)
+
+    def next_cache(self):
+        return next(self._cache)
+
+    def next_state(self):
+        return next(self._states)
+
+
+class HybridLM(nn.Module):
+    def __init__(self, cfg: DecoderConfig, dtype=torch.bfloat16, device="cpu", seed: int = 0,
+                 gradient_checkpointing: bool = False):
+        super().__init__()
+        if cfg.value_head or cfg.lora_rank > 0:
+            raise NotImplementedError("hybrid decoders have no value head and no adapters")
+        self.cfg, self.dtype = cfg, dtype
+        self.gradient_checkpointing = gradient_checkpointing
+        self.vision = None
+        gen = _Init(seed, device)
+        std = cfg.initializer_range
+        self.embed_tokens = _param((cfg.vocab_size, cfg.hidden_size), dtype, device, std, gen)
+        self.layers = nn.ModuleList([HybridLayer(cfg, i, dtype, device, gen) for i in range(cfg.num_layers)])
+        self.norm = _param((cfg.hidden_size,), dtype, device, -1, gen)
+        self.lm_head = _param((cfg.vocab_size, cfg.hidden_size), dtype, device, std, gen)
+
+    @property
+    def head_weight(self) -> torch.Tensor:
+        return self.lm_head
+
+    # ---- state description for the cache manager ---------------------------------------------------
+    def recurrent_branches(self) -> List[HybridBranch]:
+        return [br for layer in self.layers for br in layer.branches if br.recurrent]
+
+    def new_states(self, slots: int) -> List[Dict[str, torch.Tensor]]:
+        """Recurrent states of ``slots`` sequences, one dictionary per recurrent branch."""
+        return [empty_state(br.spec, slots, self.embed_tokens.device) for br in self.recurrent_branches()]
+
+    # ---- forward -----------------------------------------------------------------------------------
+    def _layers(self, ids: torch.Tensor, io: _Batch) -> torch.Tensor:
+        cfg = self.cfg
+        kind, eps = cfg.hybrid.norm, cfg.rms_norm_eps
+        h = R.embed_scaled(ids, self.embed_tokens.detach(), cfg.hybrid.embed_scale)
+        delta = None
+        for layer in self.layers:
+            delta = layer.mix(R.add_norm(h, delta, layer.norm1, eps, kind), io)
+            if layer.ff:
+                delta = layer.mlp(R.add_norm(h, delta, layer.norm2, eps, kind))
+        return R.add_norm(h, delta, self.norm, eps, kind)
+
+    @torch.no_grad()
+    def forward_cached(self, input_ids: torch.Tensor, positions: torch.Tensor, cache: Sequence[torch.Tensor],
+                       block_table: torch.Tensor, seq_ids: torch.Tensor, *, states=None,
+                       prefill_info: Optional[SeqInfo] = None, seq_lens: Optional[torch.Tensor] = None,
+                       rope_positions=None, prefix_lens=None, prefill_slots=None) -> torch.Tensor:
+        """Final-norm hidden states of new tokens (see :meth:`DecoderLM.forward_cached`).  ``states``: one dictionary
+        per recurrent branch, indexed by slot; ``prefill_slots[i]`` / ``prefix_lens[i]``: the slot of portion ``i`` and
+        the tokens it holds already."""
+        pos = positions.to(torch.int32).contiguous()
+        seq = seq_ids.to(torch.int32).contiguous()
+        if prefill_info is None:
+            return self._layers(input_ids, _Batch(seq, pos, block_table, cache, states, seq_lens=seq_lens))
+        lens = prefill_info.seqlens
+        starts = list(prefix_lens) if prefix_lens is not None else [0] * len(lens)
+        dev = input_ids.device
+        io = _Batch(seq, pos, block_table, cache, states, plan=PortionPlan(lens, starts, prefill_slots, dev),
+                    tiles=QueryTiles(lens, starts, prefill_slots, dev))
+        return self._layers(input_ids, io)
+
+    @torch.no_grad()
+    def _score_hidden(self, input_ids: torch.Tensor, info: SeqInfo) -> torch.Tensor:
+        """Packed whole sequences through the prompt path: one scratch arena serves every attention layer (each layer
+        writes before it reads), the recurrent states are dropped."""
+        cfg, dev = self.cfg, input_ids.device
+        nb = [(n + kvc.BLOCK - 1) // kvc.BLOCK for n in info.seqlens]
+        table = torch.full((max(len(nb), 1), max(max(nb, default=1), 1)), -1, dtype=torch.int32)
+        at = 0
+        for i, n in enumerate(nb):
+            table[i, :n] = torch.arange(at, at + n, dtype=torch.int32)
+            at += n
+        paged = cfg.paged_layers()
+        elems = [g * kvc.BLOCK * (dk + dv) for g, dk, dv in paged]
+        arena = torch.zeros(at * max(elems, default=0), dtype=self.embed_tokens.dtype, device=dev)
+        cache = [arena[:at * e].view(at, e) for e in elems]
+        seq_ids = torch.repeat_interleave(torch.arange(len(nb), dtype=torch.int32), torch.tensor(info.seqlens)).to(dev)
+        return self.forward_cached(input_ids, info.positions, cache, table.to(dev), seq_ids,
+                                   states=self.new_states(len(nb)), prefill_info=info,
+                                   prefill_slots=list(range(len(nb))))
+
+    def forward_hidden(self, input_ids: torch.Tensor, positions: torch.Tensor, info: SeqInfo, **mm) -> torch.Tensor:
+        if torch.is_grad_enabled() and self.lm_head.requires_grad:
+            raise NotImplementedError("hybrid decoders are served and scored; they have no backward pass")
+        if any(v is not None for v in mm.values()):
+            raise ValueError("hybrid decoders take token ids only")
+        return self._score_hidden(input_ids, info)
+
+    def token_logprobs(self, hidden: torch.Tensor, labels: torch.Tensor, temperature: float = 1.0,
+                       with_entropy: bool = True):
+        """``log p(label)`` and entropy of the capped, tempered distribution, a bounded block of rows at a time."""
+        from ..ops import lib as _lib
+        T, V = hidden.shape[0], self.cfg.vocab_size
+        labels = labels.to(torch.int64).contiguous()
+        logp = torch.empty(T, dtype=torch.float32, device=hidden.device)
+        ent = torch.empty_like(logp)
+        step = max(128, (1 << 28) // V // 128 * 128)
+        for s in range(0, T, step):
+            e = min(T, s + step)
+            z = self.logits_of(hidden[s:e])
+            if z.is_cuda:
+                ws = torch.empty_like(logp[s:e])
+                _lib.check(_lib.get_lib().sb_lmhead_stats(
+                    _lib.ptr(z), ctypes.c_longlong(V), _lib.ptr(labels[s:e]), ctypes.c_float(1.0 / temperature),
+                    _lib.ptr(logp[s:e]), _lib.ptr(ent[s:e]), _lib.ptr(ws), e - s, V, _lib.stream()), "sb_lmhead_stats")
+            else:
+                lp = torch.log_softmax(z / temperature, -1)
+                logp[s:e] = lp.gather(1, labels[s:e, None])[:, 0]
+                ent[s:e] = -(lp.exp() * lp).sum(-1)
+        return logp, (ent if with_entropy else None)
+
+    def logits_of(self, hidden: torch.Tensor) -> torch.Tensor:
+        """Capped fp32 logits of final-norm hidden states."""
+        return lm_head_logits(hidden, self.lm_head.detach(), self.cfg.logit_softcap)
+
+    def logprobs(self, input_ids, positions, info: SeqInfo, labels, temperature: float = 1.0,
+                 with_entropy: bool = True, **mm):
+        return self.token_logprobs(self.forward_hidden(input_ids, positions, info, **mm), labels, temperature,
+                                   with_entropy)
+
+    def logits(self, input_ids, positions, info: SeqInfo, **mm) -> torch.Tensor:
+        return self.logits_of(self.forward_hidden(input_ids, positions, info, **mm))
+
+    def named_flat_order(self):
+        return list(self.named_parameters())

@@ -211,6 +211,13 @@ def linear(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] =
         return F.linear(x, weight, bias)
     _lib.use_native(x)
     rows = x.numel() // x.shape[-1]
+    if x.dtype == torch.float32 or x.shape[-1] % 8 or weight.shape[0] % 8:
+        # 32-bit models, and row pitches or widths the tensor-core kernel cannot address: inference only
+        from .rows import gemm_simt
+        assert not (torch.is_grad_enabled() and (x.requires_grad or weight.requires_grad)) and bias is None, \
+            "32-bit and unaligned CUDA projections have no backward pass and no bias"
+        y = gemm_simt(x.reshape(rows, x.shape[-1]).contiguous(), weight.detach(), x.dtype)
+        return y.reshape(*x.shape[:-1], weight.shape[0])
     if rows <= 512 and not (torch.is_grad_enabled() and (x.requires_grad or weight.requires_grad)):
         y = linear_skinny(x.reshape(rows, x.shape[-1]).contiguous(), weight, bias)
         return y.reshape(*x.shape[:-1], weight.shape[0])

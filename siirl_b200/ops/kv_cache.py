@@ -68,7 +68,7 @@ def kv_copy_blocks(cache_layer: torch.Tensor, src: torch.Tensor, dst: torch.Tens
         return
     if cache_layer.is_cuda:
         L = _lib.get_lib()
-        block_elems = cache_layer[0].numel()
+        block_elems = cache_layer[0].numel() * cache_layer.element_size() // 2      # the kernel counts 16-bit units
         _lib.check(L.sb_kv_copy_blocks(_lib.ptr(cache_layer), _lib.ptr(src), _lib.ptr(dst), src.numel(),
                                        ctypes.c_longlong(block_elems), _lib.stream()), "sb_kv_copy_blocks")
         return

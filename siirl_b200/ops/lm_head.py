@@ -135,8 +135,13 @@ def lm_head_logprob_entropy(hidden: torch.Tensor, weight: torch.Tensor, labels: 
     return logp, (ent if with_entropy else None)
 
 
-def lm_head_logits(hidden: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
-    """fp32 logits ``[T, V]`` (decode path: T = number of running sequences)."""
+def lm_head_logits(hidden: torch.Tensor, weight: torch.Tensor, softcap: float = 0.0) -> torch.Tensor:
+    """fp32 logits ``[T, V]`` (decode path: T = number of running sequences); ``softcap > 0``: ``cap * tanh(z / cap)``."""
+    from .rows import gemm_simt, softcap_
     if not hidden.is_cuda:
-        return hidden.float() @ weight.float().t()
-    return dense.gemm(hidden.contiguous(), weight, epi=dense.EPI_F32)
+        z = hidden.float() @ weight.float().t()
+    elif hidden.dtype == torch.float32 or hidden.shape[-1] % 8 or weight.shape[0] % 4:
+        z = gemm_simt(hidden.contiguous(), weight.detach(), torch.float32)
+    else:
+        z = dense.gemm(hidden.contiguous(), weight, epi=dense.EPI_F32)
+    return softcap_(z, softcap) if softcap else z
