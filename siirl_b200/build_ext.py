@@ -21,6 +21,11 @@ SRC_DIR = PKG_DIR / "csrc"
 OBJ_DIR = PKG_DIR / "build"
 LIB_DIR = PKG_DIR / "lib"
 LIB_PATH = LIB_DIR / "libsiirl_b200.so"
+# the kernels that serving a decoder-only model calls, as a library of their own: what a fresh checkout compiles when it
+# only replays or serves (ops/lib.py loads it when the whole library is missing or older than its sources)
+SERVE_LIB_PATH = LIB_DIR / "libsiirl_b200_serve.so"
+SERVE_SOURCES = ("gemm_tcgen05.cu", "hybrid_ops.cu", "fmha_window.cu", "fmha_decode_split.cu", "fmha_decode.cu",
+                 "recurrence.cu", "decode_state.cu", "sampling.cu", "lm_head.cu")
 # debug-bounds variant (-DSB_DEBUG_BOUNDS: data-dependent indices report their first violation, see csrc/common.cuh)
 DBG_OBJ_DIR = PKG_DIR / "build_dbg"
 DBG_LIB_PATH = LIB_DIR / "libsiirl_b200_dbg.so"
@@ -32,6 +37,17 @@ COMMON_FLAGS = ["-O3", "-std=c++17", "-lineinfo", "-Xcompiler", "-fPIC", "-Xcomp
 
 def _sources() -> list[Path]:
     return sorted(list(SRC_DIR.rglob("*.cu")) + list(SRC_DIR.rglob("*.cpp")))
+
+
+def _fresh(lib_path: Path, srcs: list[Path]) -> bool:
+    return lib_path.exists() and lib_path.stat().st_mtime >= max([_headers_mtime()] + [x.stat().st_mtime for x in srcs])
+
+
+def build_serving() -> Path:
+    """The library serving needs: the whole one when it is up to date, else only the serving kernels are compiled."""
+    if _fresh(LIB_PATH, _sources()):
+        return LIB_PATH
+    return build(serving_only=True)
 
 
 def _headers_mtime() -> float:
@@ -58,14 +74,16 @@ def _compile(src: Path, verbose: bool, debug_bounds: bool = False) -> tuple[Path
     return obj, proc.stderr
 
 
-def build(force: bool = False, verbose: bool = False, debug_bounds: bool = False) -> Path:
+def build(force: bool = False, verbose: bool = False, debug_bounds: bool = False, serving_only: bool = False) -> Path:
     """Compile stale objects and link the shared library; returns its path."""
     obj_dir, lib_path = (DBG_OBJ_DIR, DBG_LIB_PATH) if debug_bounds else (OBJ_DIR, LIB_PATH)
+    if serving_only:
+        lib_path = SERVE_LIB_PATH
     obj_dir.mkdir(exist_ok=True)
     LIB_DIR.mkdir(exist_ok=True)
     hdr_m = _headers_mtime()
-    srcs = _sources()
-    if not force and lib_path.exists() and lib_path.stat().st_mtime >= max([hdr_m] + [x.stat().st_mtime for x in srcs]):
+    srcs = [x for x in _sources() if not serving_only or x.name in SERVE_SOURCES]
+    if not force and _fresh(lib_path, srcs):
         return lib_path         # a library newer than every source: nothing to do (object files may be absent)
     stale = []
     for s in srcs:

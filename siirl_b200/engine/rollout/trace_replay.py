@@ -115,12 +115,6 @@ class TraceReplay:
             self.free.append(seq.slot)
 
 
-def ensure_native_library() -> None:
-    """Compile the library when it is missing or older than its sources (a fresh checkout)."""
-    from ... import build_ext
-    build_ext.build()
-
-
 def load_engine(path: str, dtype: torch.dtype, max_tokens: int, slots: int = 16, device="cuda") -> RolloutEngine:
     from ...models.config import get_config
     from ...models.decoder import build_model
@@ -148,7 +142,8 @@ def main(argv=None) -> int:
     if dtype == torch.float32 and get_config(args.model).hybrid is None:
         print("trace_run: this model family runs in bfloat16 only", file=sys.stderr)
         return 3
-    ensure_native_library()
+    from ...ops import lib
+    lib.use_serving_library()       # compiled on first use in a fresh checkout
     if not torch.cuda.is_available():
         raise RuntimeError("trace_run needs a GPU")
     torch.backends.cuda.matmul.allow_tf32 = False

@@ -71,6 +71,17 @@ class KernelStatusError(RuntimeError):
         self.code = code
 
 
+def use_serving_library() -> Path:
+    """Compile (if need be) and select the library that serving needs, before any kernel is called: the whole library
+    when it is up to date, else the one with the serving kernels only."""
+    global _LIB_PATH
+    from .. import build_ext
+    path = build_ext.build_serving()
+    if _lib is None:
+        _LIB_PATH = path
+    return path
+
+
 def lib_path() -> Path:
     return _LIB_PATH
 
