@@ -56,6 +56,9 @@ def parse_args():
     ap.add_argument("--impl", default="native", choices=["native", "reference", "library"],
                     help="library: the same step through vLLM + transformers + flash-attn + torch AdamW (1 GPU), a bar "
                          "on this box that is not the reference")
+    ap.add_argument("--workload", default="grpo", choices=["grpo", "serve"],
+                    help="serve: prefill and decode throughput of a hybrid decoder (Domavik) beside the closest uniform "
+                         "decoder of equal size (1 GPU; benchmarks/hybrid_serving.py)")
     ap.add_argument("--budget-s", type=float, default=600.0,
                     help="wall-clock budget of the whole run, from process start; --steps/--warmup are upper bounds")
     ap.add_argument("--model", default="qwen2.5-7b")
@@ -192,6 +195,14 @@ def build_config(args, world: int):
 
 def main() -> int:
     args = parse_args()
+    if args.workload == "serve":
+        from siirl_b200.benchmarks.hybrid_serving import SIZES, serve
+        sampler = ClockSampler(0)
+        sampler.start()
+        res = serve(list(SIZES))
+        res["clocks"] = sampler.stop()
+        print(json.dumps(res), flush=True)
+        return 0
     if args.impl == "reference":
         return reference_arm(args)
     if args.impl == "library":

@@ -1,0 +1,254 @@
+"""Serving throughput of a hybrid decoder (Domavik) beside the closest uniform decoder of equal size, and its kernels
+beside the like kernels of that model.
+
+    python bench.py --workload serve                       # end to end, a few sizes
+    python -m siirl_b200.benchmarks.hybrid_serving --kernels
+
+End to end: random weights, the rollout engine's own prefill pass and CUDA-graph decode rounds, CUDA events on the
+launching stream.  Weights and caches are larger than L2 in every case.  Kernels: each alone, L2 flushed between
+iterations, against the measured copy bandwidth and GEMM rate (MEASURED_PEAKS.json, else the figures below)."""
+from __future__ import annotations
+
+import argparse
+import copy
+import json
+import os
+from typing import Callable, Dict, List
+
+import torch
+
+from ..engine.rollout.native_engine import RolloutEngine, SamplingParams, _Seq
+from ..models.config import DecoderConfig, get_config
+from ..models.decoder import build_model
+from ..ops import lib
+
+SIZES = {     # preset, layers, (prompts, tokens) of a prefill pass, (sequences, context) of a decode step
+    "1.5b": ("domavik-1.5b", 14, [(8, 1024), (1, 8192)], [(32, 2048), (256, 1024)]),
+    "7b": ("domavik-7b", 8, [(8, 1024), (1, 8192)], [(32, 2048), (256, 1024)]),
+}
+
+
+def peaks() -> Dict[str, float]:
+    here = os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
+    try:
+        with open(os.path.join(here, "MEASURED_PEAKS.json")) as f:
+            p = json.load(f)
+        return {"gbs": p["hbm_gbs"], "tflops": p["bf16_tflops"], "source": "measured"}
+    except (OSError, KeyError, ValueError):
+        return {"gbs": 6650.0, "tflops": 1590.0, "source": "fallback"}
+
+
+def closest(cfg: DecoderConfig) -> DecoderConfig:
+    """The uniform decoder of the same width, feed-forward, depth, vocabulary and attention heads."""
+    b = cfg.hybrid.attention[0]
+    return DecoderConfig(model_type="qwen2", vocab_size=cfg.vocab_size, hidden_size=cfg.hidden_size,
+                         intermediate_size=cfg.intermediate_size, num_layers=cfg.num_layers, num_heads=b.heads,
+                         num_kv_heads=b.kv_heads, head_dim=b.dim, rope_theta=1e6, eos_token_id=2)
+
+
+def _events(fn: Callable[[], None], warmup: int, iters: int, flush=None) -> float:
+    """Median milliseconds of ``fn`` on the current stream."""
+    times: List[float] = []
+    for i in range(warmup + iters):
+        if flush is not None:
+            flush.zero_()
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        a.record()
+        fn()
+        b.record()
+        torch.cuda.synchronize()
+        if i >= warmup:
+            times.append(a.elapsed_time(b))
+    return sorted(times)[len(times) // 2]
+
+
+def serve_one(cfg: DecoderConfig, prefill, decode, iters: int) -> dict:
+    model = build_model(cfg, dtype=torch.bfloat16, device="cuda", seed=0)
+    for p in model.parameters():
+        p.requires_grad_(False)
+    out = {"parameters": cfg.num_parameters(), "prefill": [], "decode": []}
+    g = torch.Generator().manual_seed(0)
+    for n, length in prefill:
+        eng = RolloutEngine(model, max_num_seqs=n, max_model_len=length + 64,
+                            num_blocks=n * ((length + 63) // 64 + 1), use_cuda_graph=False)
+        eng._ensure_slots(n)
+        eng._reset_slots()
+        toks = [torch.randint(3, cfg.vocab_size, (length,), generator=g).tolist() for _ in range(n)]
+        seqs = [_Seq(i, 0, length, 0, slot=i) for i in range(n)]
+        for s in seqs:
+            s.blocks = [eng.alloc.alloc() for _ in range((length + 63) // 64)]
+        eng._write_block_tables(seqs)
+        ms = _events(lambda: eng._prefill(seqs, toks), 3, iters)
+        out["prefill"].append({"prompts": n, "tokens": length, "ms": round(ms, 3),
+                               "tokens_per_s": round(n * length / ms * 1e3)})
+        eng.sleep()
+    for n, ctx in decode:
+        steps = 8
+        eng = RolloutEngine(model, max_num_seqs=n, max_model_len=ctx + 8 * steps + 64,
+                            num_blocks=n * ((ctx + 8 * steps + 127) // 64), sync_interval=steps,
+                            max_num_batched_tokens=max(ctx * n, 8192))
+        times: List[float] = []
+        run = eng._run_decode_steps
+
+        def timed(k, *a, **kw):
+            x, y = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            x.record()
+            run(k, *a, **kw)
+            y.record()
+            torch.cuda.synchronize()
+            times.append(x.elapsed_time(y) / k)
+        eng._run_decode_steps = timed
+        prompt = torch.randint(3, cfg.vocab_size, (ctx,), generator=g).tolist()
+        eng.max_num_batched_tokens = 8192
+        eng.generate([prompt[i:] + prompt[:i] for i in range(n)],
+                     SamplingParams(n=1, temperature=1.0, max_new_tokens=1 + 6 * steps, ignore_eos=True))
+        full = times[-5:-1]      # every sequence active, graph captured
+        ms = sorted(full)[len(full) // 2]
+        out["decode"].append({"sequences": n, "context": ctx, "ms_per_step": round(ms, 4),
+                              "tokens_per_s": round(n / ms * 1e3)})
+        eng.sleep()
+    lib.check_status()
+    del model
+    torch.cuda.empty_cache()
+    return out
+
+
+def serve(sizes, iters: int = 5) -> dict:
+    res = {"metric": "serving_tokens_per_second", "data": "synthetic", "dtype": "bf16", "sizes": {}}
+    for name in sizes:
+        preset, layers, prefill, decode = SIZES[name]
+        cfg = copy.deepcopy(get_config(preset))
+        cfg.hybrid.layers = cfg.hybrid.layers[:layers]
+        cfg.num_layers = layers
+        res["sizes"][name] = {"hybrid": preset, "layers": layers,
+                              "domavik": serve_one(cfg, prefill, decode, iters),
+                              "closest (uniform attention)": serve_one(closest(cfg), prefill, decode, iters)}
+    return res
+
+
+# ---- kernels ----------------------------------------------------------------------------------------------------------------
+def kernels(only: str = "", iters: int = 20) -> dict:
+    from ..ops import dense, kv_cache
+    from ..ops import rows as R
+    from ..ops.attention import SeqInfo, attention_packed
+    from ..ops.recurrence import PortionPlan, RecurrenceSpec, empty_state, recurrence_decode, recurrence_prefill
+    from ..ops.window_attention import QueryTiles, WindowSpec, window_attention
+    dev = torch.device("cuda")
+    pk = peaks()
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    rows: List[dict] = []
+
+    def add(name, fn, flops=0.0, nbytes=0.0):
+        if only and only not in name:
+            return
+        ms = _events(fn, 3, iters, flush)
+        ideal = max(flops / (pk["tflops"] * 1e9), nbytes / (pk["gbs"] * 1e6))
+        rows.append({"kernel": name, "us": round(ms * 1e3, 1), "roofline_us": round(ideal * 1e3, 1),
+                     "of_roofline": round(ideal / ms, 3)})
+
+    def rnd(*s):
+        return (torch.randn(*s, device=dev) * 0.5).bfloat16()
+
+    # attention on prompts: 28 heads, 4 kv heads, width 128
+    H, G, D = 28, 4, 128
+    for n, L in ((8, 1024), (1, 8192)):
+        T = n * L
+        x = rnd(T, (H + 2 * G) * D)
+        info = SeqInfo([L] * n, device=dev)
+        flops = n * 4 * D * H * L * (L + 1) / 2
+        add(f"uniform: fmha_fwd {n}x{L}", lambda: attention_packed(x, info, H, G, D), flops)
+        nb = L // 64
+        table = torch.randperm(n * nb, device=dev).to(torch.int32).view(n, nb)
+        cache = torch.zeros(n * nb, G * 64 * 2 * D, dtype=torch.bfloat16, device=dev)
+        out = torch.empty(T, H * D, dtype=torch.bfloat16, device=dev)
+        ids = torch.repeat_interleave(torch.arange(n, dtype=torch.int32), L).to(dev)
+        pos = torch.arange(L, dtype=torch.int32).repeat(n).to(dev)
+        tiles = QueryTiles([L] * n, [0] * n, list(range(n)), dev)
+        for w, kf in ((0, 0), (1024, 64)):
+            spec = WindowSpec(H, G, D, D, 0, H * D, (H + G) * D, D ** -0.5, w, kf, 8.0)
+            seen = sum(min(i + 1, w) + max(0, min(kf, i + 1 - w)) for i in range(L)) if w else L * (L + 1) / 2
+            add(f"domavik: window attention {n}x{L} window {w or 'none'} (with cache append)",
+                lambda: window_attention(spec, x, ids, pos, table, cache, out, 0, tiles=tiles), n * 4 * D * H * seen)
+    # attention on single tokens
+    for B, ctx in ((32, 2048), (256, 1024)):
+        nb = (ctx + 63) // 64
+        table = torch.randperm(B * nb, device=dev).to(torch.int32).view(B, nb)
+        cache = torch.zeros(B * nb, 2, G, 64, D, dtype=torch.bfloat16, device=dev)
+        x = rnd(B, (H + 2 * G) * D)
+        lens = torch.full((B,), ctx, dtype=torch.int32, device=dev)
+        add(f"uniform: decode attention {B}x{ctx}", lambda: kv_cache.decode_attention(x, cache, lens, table, H, G, D),
+            nbytes=B * ctx * 2 * G * D * 2)
+        out = torch.empty(B, H * D, dtype=torch.bfloat16, device=dev)
+        ids, pos = torch.arange(B, dtype=torch.int32, device=dev), lens - 1
+        flat = cache.view(B * nb, -1)
+        for w, kf in ((0, 0), (1024, 64)):
+            spec = WindowSpec(H, G, D, D, 0, H * D, (H + G) * D, D ** -0.5, w, kf, 8.0)
+            seen = min(ctx, w) + max(0, min(kf, ctx - w)) if w else ctx
+            add(f"domavik: window decode {B}x{ctx} window {w or 'none'} (with cache append)",
+                lambda: window_attention(spec, x, ids, pos, table, flat, out, 0, seq_lens=lens),
+                nbytes=B * seen * 2 * G * D * 2)
+    # recurrences
+    for gate, h, dk, dv in (("channel", 16, 64, 128), ("head", 16, 128, 128)):
+        up, at, off = (lambda n: (n + 7) // 8 * 8), 0, {}
+        for key, wd in (("q", h * dk), ("k", h * dk), ("v", h * dv), ("g", h * dv)) + (
+                (("e", 16),) if gate == "channel" else (("e", h), ("f", h))):
+            off[key], at = at, at + up(wd)
+        spec = RecurrenceSpec(gate, h, dk, dv, off["q"], off["k"], off["v"], off["g"], off["e"], off.get("f", 0),
+                              16 if gate == "channel" else 0, 16.0, 15.0, 1e-5, 1.0,
+                              "silu" if gate == "channel" else "sigmoid", gate == "head")
+        wts = {"norm": rnd(h * dv if gate == "head" else dv)}
+        wts.update({"w2": rnd(h * dk, 16), "b_e": rnd(h * dk)} if gate == "channel" else {"b_e": rnd(h), "b_f": rnd(h) + 3})
+        for n, L in ((8, 1024), (1, 8192)):
+            x = rnd(n * L, at)
+            out = torch.empty(n * L, h * dv, dtype=torch.bfloat16, device=dev)
+            st = empty_state(spec, n, dev)
+            plan = PortionPlan([L] * n, [0] * n, list(range(n)), dev)
+            nbytes = n * L * (at + h * dv) * 2 + n * h * spec.rows * dk * 4
+            flops = n * L * h * 2.0 * dk * dv * 2
+            add(f"domavik: {gate} recurrence {n}x{L}", lambda: recurrence_prefill(spec, x, wts, st, plan, out, 0), flops,
+                nbytes)
+        for B in (32, 256):
+            x = rnd(B, at)
+            out = torch.empty(B, h * dv, dtype=torch.bfloat16, device=dev)
+            st = empty_state(spec, B, dev)
+            slots, pos = torch.arange(B, dtype=torch.int32, device=dev), torch.full((B,), 9, dtype=torch.int32, device=dev)
+            add(f"domavik: {gate} recurrence step {B}",
+                lambda: recurrence_decode(spec, x, wts, st, slots, pos, out, 0), nbytes=B * h * spec.rows * dk * 8)
+    # row operations
+    for T in (256, 8192):
+        W, I, V = 3584, 18944, 152064
+        h32, d, w = torch.randn(T, W, device=dev), rnd(T, W), rnd(W)
+        res = rnd(T, W)
+        add(f"uniform: residual + RMS norm {T}x{W} (bf16 stream)", lambda: dense.rmsnorm(d, w, 1e-6, residual=res),
+            nbytes=T * W * 8)
+        add(f"domavik: residual + layer norm {T}x{W} (fp32 stream)", lambda: R.add_norm(h32, d, w, 1e-5),
+            nbytes=T * W * 12)
+        gu = rnd(T, 2 * I)
+        add(f"uniform: swiglu {T}x{I}", lambda: dense.swiglu(gu), nbytes=T * I * 6)
+        add(f"domavik: gelu gate {T}x{I}", lambda: R.gated_act(gu), nbytes=T * I * 6)
+        ids = torch.randint(0, V, (T,), device=dev)
+        table = torch.zeros(V, W, dtype=torch.bfloat16, device=dev)
+        add(f"uniform: embedding {T}x{W}", lambda: dense.embedding(ids, table), nbytes=T * W * 4)
+        add(f"domavik: scaled embedding {T}x{W}", lambda: R.embed_scaled(ids, table, 2.0), nbytes=T * W * 6)
+        if T == 256:
+            z = torch.randn(T, V, device=dev)
+            add(f"domavik: soft cap {T}x{V}", lambda: R.softcap_(z, 30.0), nbytes=T * V * 8)
+    torch.cuda.synchronize()
+    lib.check_status()
+    return {"peaks": pk, "kernels": rows}
+
+
+def main(argv=None) -> int:
+    ap = argparse.ArgumentParser()
+    ap.add_argument("--kernels", action="store_true")
+    ap.add_argument("--only", default="", help="kernels whose name contains this")
+    ap.add_argument("--iters", type=int, default=20)
+    ap.add_argument("--sizes", default=",".join(SIZES))
+    args = ap.parse_args(argv)
+    res = kernels(args.only, args.iters) if args.kernels else serve(args.sizes.split(","))
+    print(json.dumps(res), flush=True)
+    return 0
+
+
+if __name__ == "__main__":
+    raise SystemExit(main())

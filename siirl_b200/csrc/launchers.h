@@ -198,10 +198,10 @@ int sb_gemm_simt(const void* A, const void* B, void* C, int M, int N, int K, lon
 int sb_recurrence_step(const void* params, const int* row0, const int* nrow, const int* slots, const int* pos0, int n_seq,
                        int f32, cudaStream_t stream);
 int sb_recurrence_chunk();
-long long sb_recurrence_workspace(const void* params, int n_chunks, int T);
+long long sb_recurrence_workspace(const void* params, int n_chunks, int n_seg, int T);
 int sb_recurrence_prefill(const void* params, const int* row0, const int* nrow, const int* slots, const int* pos0,
-                          int n_seq, const int* seq_chunk0, const int* chunk_row, const int* chunk_len, int n_chunks,
-                          int T, void* workspace, int* status, cudaStream_t stream);
+                          int n_seq, const int* chunk_row, const int* chunk_len, int n_chunks, const int* segs, int n_seg,
+                          int T, void* workspace, cudaStream_t stream);
 // ---- fmha_window.cu (params: host WinParams) ----
 int sb_kv_append_split(const void* params, int f32, cudaStream_t stream);
 int sb_attn_window_simt(const void* params, int f32, cudaStream_t stream);

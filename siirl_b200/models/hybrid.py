@@ -250,10 +250,12 @@ class HybridLM(nn.Module):
             e = min(T, s + step)
             z = self.logits_of(hidden[s:e])
             if z.is_cuda:
+                if V % 4:       # the statistics kernel reads vectors of four: columns without weight
+                    z = torch.nn.functional.pad(z, (0, -V % 4), value=-1e30)
                 ws = torch.empty_like(logp[s:e])
                 _lib.check(_lib.get_lib().sb_lmhead_stats(
-                    _lib.ptr(z), ctypes.c_longlong(V), _lib.ptr(labels[s:e]), ctypes.c_float(1.0 / temperature),
-                    _lib.ptr(logp[s:e]), _lib.ptr(ent[s:e]), _lib.ptr(ws), e - s, V, _lib.stream()), "sb_lmhead_stats")
+                    _lib.ptr(z), ctypes.c_longlong(z.shape[1]), _lib.ptr(labels[s:e]), ctypes.c_float(1.0 / temperature),
+                    _lib.ptr(logp[s:e]), _lib.ptr(ent[s:e]), _lib.ptr(ws), e - s, z.shape[1], _lib.stream()), "sb_lmhead_stats")
             else:
                 lp = torch.log_softmax(z / temperature, -1)
                 logp[s:e] = lp.gather(1, labels[s:e, None])[:, 0]

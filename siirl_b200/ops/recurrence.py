@@ -15,7 +15,7 @@ from __future__ import annotations
 
 import ctypes
 from dataclasses import dataclass
-from typing import Dict, List, Optional, Sequence
+from typing import Dict, List, Optional, Sequence, Tuple
 
 import torch
 import torch.nn.functional as F
@@ -23,6 +23,7 @@ import torch.nn.functional as F
 from . import lib as _lib
 
 CHUNK = 16
+SEGMENT_CTAS = 148 * 3      # (segment, head) blocks of a long prompt's scan
 
 
 @dataclass
@@ -81,20 +82,40 @@ class PortionPlan:
 
     def __init__(self, lens: Sequence[int], starts: Sequence[int], slots: Sequence[int], device):
         self.lens, self.starts, self.slots = list(lens), list(starts), list(slots)
-        row0, chunk_row, chunk_len, seq_chunk0, at = [], [], [], [0], 0
+        row0, chunk_row, chunk_len, at = [], [], [], 0
         for n in self.lens:
             row0.append(at)
             for c in range(0, n, CHUNK):
                 chunk_row.append(at + c)
                 chunk_len.append(min(CHUNK, n - c))
-            seq_chunk0.append(len(chunk_row))
             at += n
         self.row0_cpu, self.n_seq, self.n_chunks, self.total = row0, len(row0), len(chunk_row), at
+        self.device = device
+        self._segments: Dict[int, Tuple[torch.Tensor, int]] = {}
         # one copy to the device: the pieces are views
-        parts = [row0, self.lens, self.slots, self.starts, seq_chunk0, chunk_row, chunk_len]
+        parts = [row0, self.lens, self.slots, self.starts, chunk_row, chunk_len]
         flat = torch.tensor([v for p in parts for v in p], dtype=torch.int32).to(device)
-        self.row0, self.nrow, self.slot, self.pos0, self.seq_chunk0, self.chunk_row, self.chunk_len = flat.split(
-            [len(p) for p in parts])
+        self.row0, self.nrow, self.slot, self.pos0, self.chunk_row, self.chunk_len = flat.split([len(p) for p in parts])
+
+    def segments(self, heads: int) -> Tuple[torch.Tensor, int]:
+        """Runs of chunks that work in parallel, sized so that ``heads`` heads of all of them fill the GPU about once:
+        ``[5 n + sequences + 1]`` ints (sequence, first chunk, first row, tokens, flags; first segment per sequence)."""
+        per = max(4, -(-self.n_chunks * heads // SEGMENT_CTAS))
+        if per not in self._segments:
+            seq, chunk0, row, tokens, flags, first, base = [], [], [], [], [], [0], 0
+            for i, n in enumerate(self.lens):
+                chunks = -(-n // CHUNK)
+                for c in range(0, chunks, per):
+                    seq.append(i)
+                    chunk0.append(base + c)
+                    row.append(self.row0_cpu[i] + c * CHUNK)
+                    tokens.append(min(per * CHUNK, n - c * CHUNK))
+                    flags.append((1 if c == 0 else 0) | (2 if c + per >= chunks else 0))
+                base += chunks
+                first.append(len(seq))
+            flat = torch.tensor(seq + chunk0 + row + tokens + flags + first, dtype=torch.int32)
+            self._segments[per] = (flat.to(self.device), len(seq))
+        return self._segments[per]
 
 
 def _params(spec: RecurrenceSpec, x, weights, state, out, out_off) -> _Params:
@@ -129,16 +150,16 @@ def recurrence_prefill(spec: RecurrenceSpec, x: torch.Tensor, weights: Dict[str,
     if x.dtype == torch.bfloat16 and not stepwise:
         fn = L._cdll.sb_recurrence_workspace
         fn.restype = ctypes.c_longlong
-        nbytes = int(fn(ref, plan.n_chunks, x.shape[0]))
+        segs, n_seg = plan.segments(spec.heads)
+        nbytes = int(fn(ref, plan.n_chunks, n_seg, x.shape[0]))
         if nbytes >= 0:
             ws = torch.empty(max(nbytes, 16), dtype=torch.uint8, device=x.device)
             _lib.check(L.sb_recurrence_prefill(
                 ref, _lib.ptr(plan.row0), _lib.ptr(plan.nrow), _lib.ptr(plan.slot), _lib.ptr(plan.pos0), plan.n_seq,
-                _lib.ptr(plan.seq_chunk0), _lib.ptr(plan.chunk_row), _lib.ptr(plan.chunk_len), plan.n_chunks,
-                x.shape[0], _lib.ptr(ws), _lib.ptr(_lib.status_word(x.device)), _lib.stream()),
-                "sb_recurrence_prefill")
-            if spec.gate == "channel":      # counted as three kernels (gate scan, chunk preparation, scan)
-                _lib.add_launches(-1)
+                _lib.ptr(plan.chunk_row), _lib.ptr(plan.chunk_len), plan.n_chunks, _lib.ptr(segs), n_seg, x.shape[0],
+                _lib.ptr(ws), _lib.stream()), "sb_recurrence_prefill")
+            # counted as two kernels (chunk preparation, scan): gates and segment states come on top
+            _lib.add_launches((2 if n_seg > plan.n_seq else 0) + (1 if spec.gate == "head" else 0))
             return
     _lib.check(L.sb_recurrence_step(ref, _lib.ptr(plan.row0), _lib.ptr(plan.nrow), _lib.ptr(plan.slot),
                                     _lib.ptr(plan.pos0), plan.n_seq, int(x.dtype == torch.float32), _lib.stream()),

@@ -42,8 +42,8 @@ def window_attention_fast(q, k, v, scale, size, keep_first):
     """The same by dense matrices (whole prompts of some hundred tokens)."""
     T, H, _ = q.shape
     G = k.shape[1]
-    i = torch.arange(T)[:, None]
-    j = torch.arange(T)[None, :]
+    i = torch.arange(T, dtype=q.dtype)[:, None]
+    j = torch.arange(T, dtype=q.dtype)[None, :]
     seen = (j <= i) & ((i - j < size) | (j < keep_first))
     out = torch.zeros(T, H, v.shape[-1], dtype=q.dtype)
     for h in range(H):
