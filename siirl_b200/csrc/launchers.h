@@ -198,6 +198,7 @@ int sb_gemm_simt(const void* A, const void* B, void* C, int M, int N, int K, lon
 int sb_recurrence_step(const void* params, const int* row0, const int* nrow, const int* slots, const int* pos0, int n_seq,
                        int f32, cudaStream_t stream);
 int sb_recurrence_chunk();
+int sb_recurrence_resident(const void* params);
 long long sb_recurrence_workspace(const void* params, int n_chunks, int n_seg, int T);
 int sb_recurrence_prefill(const void* params, const int* row0, const int* nrow, const int* slots, const int* pos0,
                           int n_seq, const int* chunk_row, const int* chunk_len, int n_chunks, const int* segs, int n_seg,

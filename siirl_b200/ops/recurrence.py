@@ -23,7 +23,6 @@ import torch.nn.functional as F
 from . import lib as _lib
 
 CHUNK = 16
-SEGMENT_CTAS = 148 * 3      # (segment, head) blocks of a long prompt's scan
 
 
 @dataclass
@@ -97,14 +96,15 @@ class PortionPlan:
         flat = torch.tensor([v for p in parts for v in p], dtype=torch.int32).to(device)
         self.row0, self.nrow, self.slot, self.pos0, self.chunk_row, self.chunk_len = flat.split([len(p) for p in parts])
 
-    def segments(self, heads: int) -> Tuple[torch.Tensor, int]:
-        """Runs of chunks that work in parallel, sized so that ``heads`` heads of all of them fill the GPU about once:
+    def segments(self, blocks: int) -> Tuple[torch.Tensor, int]:
+        """Runs of chunks that work in parallel, about ``blocks`` of them in all, equal within a sequence:
         ``[5 n + sequences + 1]`` ints (sequence, first chunk, first row, tokens, flags; first segment per sequence)."""
-        per = max(4, -(-self.n_chunks * heads // SEGMENT_CTAS))
-        if per not in self._segments:
+        want = max(4, -(-self.n_chunks // max(blocks, 1)))
+        if want not in self._segments:
             seq, chunk0, row, tokens, flags, first, base = [], [], [], [], [], [0], 0
             for i, n in enumerate(self.lens):
                 chunks = -(-n // CHUNK)
+                per = -(-chunks // max(1, chunks // want)) if chunks else 1
                 for c in range(0, chunks, per):
                     seq.append(i)
                     chunk0.append(base + c)
@@ -114,8 +114,8 @@ class PortionPlan:
                 base += chunks
                 first.append(len(seq))
             flat = torch.tensor(seq + chunk0 + row + tokens + flags + first, dtype=torch.int32)
-            self._segments[per] = (flat.to(self.device), len(seq))
-        return self._segments[per]
+            self._segments[want] = (flat.to(self.device), len(seq))
+        return self._segments[want]
 
 
 def _params(spec: RecurrenceSpec, x, weights, state, out, out_off) -> _Params:
@@ -150,7 +150,7 @@ def recurrence_prefill(spec: RecurrenceSpec, x: torch.Tensor, weights: Dict[str,
     if x.dtype == torch.bfloat16 and not stepwise:
         fn = L._cdll.sb_recurrence_workspace
         fn.restype = ctypes.c_longlong
-        segs, n_seg = plan.segments(spec.heads)
+        segs, n_seg = plan.segments(int(L._cdll.sb_recurrence_resident(ref)) // spec.heads)
         nbytes = int(fn(ref, plan.n_chunks, n_seg, x.shape[0]))
         if nbytes >= 0:
             ws = torch.empty(max(nbytes, 16), dtype=torch.uint8, device=x.device)
@@ -158,8 +158,8 @@ def recurrence_prefill(spec: RecurrenceSpec, x: torch.Tensor, weights: Dict[str,
                 ref, _lib.ptr(plan.row0), _lib.ptr(plan.nrow), _lib.ptr(plan.slot), _lib.ptr(plan.pos0), plan.n_seq,
                 _lib.ptr(plan.chunk_row), _lib.ptr(plan.chunk_len), plan.n_chunks, _lib.ptr(segs), n_seg, x.shape[0],
                 _lib.ptr(ws), _lib.stream()), "sb_recurrence_prefill")
-            # counted as two kernels (chunk preparation, scan): gates and segment states come on top
-            _lib.add_launches((2 if n_seg > plan.n_seq else 0) + (1 if spec.gate == "head" else 0))
+            # counted as two kernels (chunk preparation or gate scan, chunk scan): segment states come on top
+            _lib.add_launches(2 if n_seg > plan.n_seq else 0)
             return
     _lib.check(L.sb_recurrence_step(ref, _lib.ptr(plan.row0), _lib.ptr(plan.nrow), _lib.ptr(plan.slot),
                                     _lib.ptr(plan.pos0), plan.n_seq, int(x.dtype == torch.float32), _lib.stream()),
