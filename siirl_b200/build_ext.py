@@ -21,8 +21,8 @@ SRC_DIR = PKG_DIR / "csrc"
 OBJ_DIR = PKG_DIR / "build"
 LIB_DIR = PKG_DIR / "lib"
 LIB_PATH = LIB_DIR / "libsiirl_b200.so"
-# the kernels that serving a decoder-only model calls, as a library of their own: what a fresh checkout compiles when it
-# only replays or serves (ops/lib.py loads it when the whole library is missing or older than its sources)
+# the kernels that serving a decoder-only model calls, as a library of their own: all that a fresh checkout compiles when
+# it only serves (ops/lib.py::use_serving_library)
 SERVE_LIB_PATH = LIB_DIR / "libsiirl_b200_serve.so"
 SERVE_SOURCES = ("gemm_tcgen05.cu", "hybrid_ops.cu", "fmha_window.cu", "fmha_decode_split.cu", "fmha_decode.cu",
                  "recurrence.cu", "decode_state.cu", "sampling.cu", "lm_head.cu")

@@ -131,10 +131,16 @@ __global__ void gated_act_kernel(const T* __restrict__ gu, T* __restrict__ out, 
   }
 }
 
+template <int V>
 __global__ void softcap_kernel(float* __restrict__ z, long long n, float cap) {
   const float inv = 1.f / cap;
-  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x)
-    z[i] = cap * tanhf(z[i] * inv);
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n / V; i += (long long)gridDim.x * blockDim.x) {
+    float x[V];
+    load_vec<float, V>(z + i * V, x);
+#pragma unroll
+    for (int k = 0; k < V; ++k) x[k] = cap * tanhf(x[k] * inv);
+    store_vec<float, V>(z + i * V, x);
+  }
 }
 
 // 64 x 64 output tile per 256 threads, 4 x 4 values each, contraction in steps of 16 through shared memory
@@ -246,7 +252,8 @@ extern "C" int sb_gated_act(const void* gu, void* out, long long rows, int I, in
 extern "C" int sb_softcap(float* z, long long n, float cap, cudaStream_t stream) {
   if (n == 0) return 0;
   if (!(cap > 0.f)) return -3;
-  softcap_kernel<<<grid_for(n, 256), 256, 0, stream>>>(z, n, cap);
+  if (n % 4 == 0 && ((uintptr_t)z & 15) == 0) softcap_kernel<4><<<grid_for(n / 4, 256), 256, 0, stream>>>(z, n, cap);
+  else softcap_kernel<1><<<grid_for(n, 256), 256, 0, stream>>>(z, n, cap);
   return (int)cudaGetLastError();
 }
 

@@ -197,7 +197,6 @@ int sb_gemm_simt(const void* A, const void* B, void* C, int M, int N, int K, lon
 // ---- recurrence.cu (params: host RecParams) ----
 int sb_recurrence_step(const void* params, const int* row0, const int* nrow, const int* slots, const int* pos0, int n_seq,
                        int f32, cudaStream_t stream);
-int sb_recurrence_chunk();
 int sb_recurrence_resident(const void* params);
 long long sb_recurrence_workspace(const void* params, int n_chunks, int n_seg, int T);
 int sb_recurrence_prefill(const void* params, const int* row0, const int* nrow, const int* slots, const int* pos0,

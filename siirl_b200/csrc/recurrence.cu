@@ -977,8 +977,6 @@ extern "C" int sb_recurrence_step(const void* params, const int* row0, const int
   return p.dk % 4 ? run(recurrence_step_kernel<__nv_bfloat16, 1>) : run(recurrence_step_kernel<__nv_bfloat16, 4>);
 }
 
-extern "C" int sb_recurrence_chunk() { return kChunk; }
-
 // (segment, head) blocks of the chunk scan that run at a time on the whole GPU
 extern "C" int sb_recurrence_resident(const void* params) {
   const RecParams& p = *reinterpret_cast<const RecParams*>(params);

@@ -22,7 +22,7 @@ import torch.nn.functional as F
 
 from . import lib as _lib
 
-CHUNK = 16
+CHUNK = 16      # tokens per tile of the chunked kernels (kChunk in csrc/recurrence.cu)
 
 
 @dataclass
