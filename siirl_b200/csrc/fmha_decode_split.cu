@@ -706,7 +706,7 @@ extern "C" int sb_fmha_decode_split(const void* q, int row_stride, const void* c
 extern "C" int sb_attn_window_decode_chunks(const void* params) {
   const WinParams& p = *reinterpret_cast<const WinParams*>(params);
   if (p.dk % 8 || p.dv % 8 || p.dk > 128 || p.dv > 128 || p.Hq % p.Hkv || p.Hq / p.Hkv > 32 || p.row_stride % 8 ||
-      p.q_off % 8 || p.out_stride % 8 || p.out_off % 8 || p.block_elems % 8)
+      p.q_off % 8 || p.out_stride % 8 || p.out_off % 8 || p.block_elems % 8 || p.kv_mode != kPaged || p.gain || p.gate)
     return -1;
   int tiles = p.max_blocks;
   if (p.window > 0) {

@@ -3,7 +3,8 @@
 //
 // The portion's keys and values are appended to the cache first; a query tile then walks the cache blocks in which any
 // of its rows sees a key: the blocks of the kept first tokens, then those of the window.  Whole prompts, later portions
-// and reused prefixes take the same path, and blocks that left every window are never touched.
+// and reused prefixes take the same path, and blocks that left every window are never touched.  Keys and values may also
+// lie in packed rows (latent attention expands them from its cache), and the result may be gated.
 //
 //   window_prefill_kernel   bf16, dk and dv multiples of 8 up to 256: 128 query rows of one head per CTA, S = Q K^T and
 //                           O += P V on tcgen05 with accumulators in TMEM; one cache block is one K/V tile, fetched by
@@ -62,7 +63,8 @@ __global__ void __launch_bounds__(kSimtThreads) window_simt_kernel(WinParams p) 
   const int kvh = h / (p.Hq / p.Hkv);
   const float slope = p.bias_exp > 0.f ? exp2f(-p.bias_exp * (h + 1) / p.Hq) : 0.f;
   const T* q = reinterpret_cast<const T*>(p.x) + (size_t)t * p.row_stride + p.q_off + (size_t)h * p.dk;
-  for (int d = tid; d < p.dk; d += kSimtThreads) sq[d] = to_float(q[d]);
+  const float gain = p.gain ? to_float(*reinterpret_cast<const T*>(p.gain)) : 1.f;
+  for (int d = tid; d < p.dk; d += kSimtThreads) sq[d] = to_float(q[d]) * gain;
   for (int d = tid; d < p.dv; d += kSimtThreads) so[d] = 0.f;
   // the visible keys are 0 .. first - 1 and lo .. i
   int first = 0, lo = 0;
@@ -78,8 +80,9 @@ __global__ void __launch_bounds__(kSimtThreads) window_simt_kernel(WinParams p) 
     const int blk = j / kWBlk < p.max_blocks ? bt[j / kWBlk] : -1;
     if (blk < 0 || blk >= p.num_blocks) return nullptr;
     const size_t base = (size_t)blk * p.block_elems;
-    return value ? cache + base + (size_t)p.Hkv * kWBlk * p.dk + ((size_t)kvh * kWBlk + j % kWBlk) * p.dv
-                 : cache + base + ((size_t)kvh * kWBlk + j % kWBlk) * p.dk;
+    return value && p.kv_mode != kLatent
+               ? cache + base + (size_t)p.Hkv * kWBlk * p.dk + ((size_t)kvh * kWBlk + j % kWBlk) * p.dv
+               : cache + base + ((size_t)kvh * kWBlk + j % kWBlk) * p.dk;
   };
   float m = -INFINITY, l = 0.f;
   __syncthreads();
@@ -186,7 +189,8 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
   const int kvh = h / (p.Hq / p.Hkv);
   int sinks, w0, n_tiles;
   win_blocks(q0, q0 + nrows - 1, p.window, p.keep_first, sinks, w0, n_tiles);
-  const int* bt = p.block_table + (size_t)slot * p.max_blocks;
+  const bool packed = p.kv_mode == kPackedRows;
+  const int* bt = p.block_table + (size_t)(packed ? 0 : slot) * p.max_blocks;
   auto block_of = [&](int j) { return j < sinks ? j : w0 + j - sinks; };
 
   if (tid == 0) {
@@ -208,13 +212,15 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
 
   auto load_kv = [&](int j, int stage) {
     const int lb = block_of(j);
-    int blk = lb < p.max_blocks ? bt[lb] : 0;
-    if (blk < 0 || blk >= p.num_blocks) blk = 0;      // never inside the visible range of a well-formed table
+    // packed rows: head kvh, rows from `blk`; those past the sequence are hidden by causality, past the end zeros
+    int blk = packed ? slot + lb * kWBlk : (lb < p.max_blocks ? bt[lb] : 0);
+    if (!packed && (blk < 0 || blk >= p.num_blocks)) blk = 0;      // never inside the visible range of a well-formed table
+    const int mid = packed ? kvh : kvh * kWBlk;
     mbar_arrive_expect_tx(&bar_kv[stage], (uint32_t)(L.k_bytes + L.v_bytes));
     for (int c = 0; c < ck; ++c)
-      tma_load_3d(sK + stage * L.k_bytes + c * 8192, &map_k, &bar_kv[stage], c * 64, kvh * kWBlk, blk);
+      tma_load_3d(sK + stage * L.k_bytes + c * 8192, &map_k, &bar_kv[stage], c * 64, mid, blk);
     for (int c = 0; c < cv; ++c)
-      tma_load_3d(sV + stage * L.v_bytes + c * 8192, &map_v, &bar_kv[stage], c * 64, kvh * kWBlk, blk);
+      tma_load_3d(sV + stage * L.v_bytes + c * 8192, &map_v, &bar_kv[stage], c * 64, mid, blk);
   };
   if (tid == 0) {
     mbar_arrive_expect_tx(bar_q, (uint32_t)L.q_bytes);
@@ -227,7 +233,8 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
   const uint32_t idesc_o = umma_idesc_bf16(128, vn, 0, 1);
   const uint32_t lane_off = (uint32_t)(warp * 32) << 16;
   const int qpos = q0 + tid;
-  const float scale_log2 = p.scale * 1.4426950408889634f;
+  const float gain = p.gain ? __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(p.gain)) : 1.f;
+  const float scale_log2 = p.scale * gain * 1.4426950408889634f;
   const float slope_log2 =
       p.bias_exp > 0.f ? exp2f(-p.bias_exp * (float)(h + 1) / (float)p.Hq) * 1.4426950408889634f : 0.f;
   float m_run = -INFINITY, l_run = 0.f;
@@ -344,6 +351,8 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     const float inv_l = l_run > 0.f ? p.out_scale / l_run : 0.f;
     __nv_bfloat16* orow = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)(row0 + (row_valid ? tid : 0)) * p.out_stride +
                           p.out_off + (size_t)h * p.dv;
+    const __nv_bfloat16* grow = reinterpret_cast<const __nv_bfloat16*>(p.gate) +
+                                (size_t)(row0 + (row_valid ? tid : 0)) * p.gate_stride + (size_t)h * p.dv;
 #pragma unroll 1
     for (int c = 0; c < (vn + 31) / 32; ++c) {
       uint32_t r[32];
@@ -353,12 +362,16 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
 #pragma unroll
         for (int g = 0; g < 4; ++g) {
           if (c * 32 + g * 8 >= p.dv) break;
-          uint4 o;
-          o.x = pack_bf16x2(__uint_as_float(r[g * 8 + 0]) * inv_l, __uint_as_float(r[g * 8 + 1]) * inv_l);
-          o.y = pack_bf16x2(__uint_as_float(r[g * 8 + 2]) * inv_l, __uint_as_float(r[g * 8 + 3]) * inv_l);
-          o.z = pack_bf16x2(__uint_as_float(r[g * 8 + 4]) * inv_l, __uint_as_float(r[g * 8 + 5]) * inv_l);
-          o.w = pack_bf16x2(__uint_as_float(r[g * 8 + 6]) * inv_l, __uint_as_float(r[g * 8 + 7]) * inv_l);
-          *reinterpret_cast<uint4*>(orow + c * 32 + g * 8) = o;
+          float o[8];
+#pragma unroll
+          for (int i = 0; i < 8; ++i) o[i] = __uint_as_float(r[g * 8 + i]) * inv_l;
+          if (p.gate) {
+            float z[8];
+            load_vec<__nv_bfloat16, 8>(grow + c * 32 + g * 8, z);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) o[i] /= 1.f + __expf(-gain * z[i]);
+          }
+          store_vec<__nv_bfloat16, 8>(orow + c * 32 + g * 8, o);
         }
       }
     }
@@ -404,7 +417,7 @@ extern "C" int sb_kv_append_split(const void* params, int f32, cudaStream_t stre
 extern "C" int sb_attn_window_simt(const void* params, int f32, cudaStream_t stream) {
   const WinParams& p = *reinterpret_cast<const WinParams*>(params);
   if (p.T == 0) return 0;
-  if (p.Hq % p.Hkv || p.Hq > 65535) return -3;
+  if (p.Hq % p.Hkv || p.Hq > 65535 || p.kv_mode == kPackedRows || p.gate || (p.kv_mode == kLatent && p.dk != p.dv)) return -3;
   const size_t smem = (size_t)(p.dk + kSimtThreads + p.dv) * 4;
   if (smem > 48 * 1024) return -3;
   const dim3 grid(p.T, p.Hq);
@@ -420,7 +433,8 @@ extern "C" int sb_attn_window_prefill(const void* params, const int* tile_row, c
   const WinParams& p = *reinterpret_cast<const WinParams*>(params);
   if (n_tiles == 0) return 0;
   if (p.Hq % p.Hkv || p.dk % 8 || p.dv % 8 || p.dk > 256 || p.dv > 256 || p.dk < 8 || p.dv < 8 || p.row_stride % 8 ||
-      p.q_off % 8 || p.out_stride % 8 || p.out_off % 8 || p.block_elems % 8 || ((uintptr_t)p.out & 15))
+      p.q_off % 8 || p.out_stride % 8 || p.out_off % 8 || p.block_elems % 8 || ((uintptr_t)p.out & 15) ||
+      p.kv_mode == kLatent || p.gate_stride % 8 || ((uintptr_t)p.gate & 15))
     return -2;
   static thread_local bool tl_context_bound = false;
   if (!tl_context_bound) {
@@ -433,11 +447,20 @@ extern "C" int sb_attn_window_prefill(const void* params, const int* tile_row, c
   // q: columns of one head x heads x rows, so that columns past dk read as zeros
   int r = make_tensor_map_bf16_3d(&mq, x + p.q_off, p.dk, p.Hq, p.T, p.dk, p.row_stride, 64, 1, 128);
   if (r) return r;
-  r = make_tensor_map_bf16_3d(&mk, cache, p.dk, (long long)p.Hkv * kWBlk, p.num_blocks, p.dk, p.block_elems, 64, kWBlk, 1);
-  if (r) return r;
-  r = make_tensor_map_bf16_3d(&mv, cache + (size_t)p.Hkv * kWBlk * p.dk, p.dv, (long long)p.Hkv * kWBlk, p.num_blocks,
-                              p.dv, p.block_elems, 64, kWBlk, 1);
-  if (r) return r;
+  if (p.kv_mode == kPackedRows) {
+    // columns of one head x heads x key rows
+    r = make_tensor_map_bf16_3d(&mk, cache, p.dk, p.Hkv, p.num_blocks, p.dk, p.block_elems, 64, 1, kWBlk);
+    if (r) return r;
+    r = make_tensor_map_bf16_3d(&mv, cache + (size_t)p.Hkv * p.dk, p.dv, p.Hkv, p.num_blocks, p.dv, p.block_elems, 64, 1,
+                                kWBlk);
+    if (r) return r;
+  } else {
+    r = make_tensor_map_bf16_3d(&mk, cache, p.dk, (long long)p.Hkv * kWBlk, p.num_blocks, p.dk, p.block_elems, 64, kWBlk, 1);
+    if (r) return r;
+    r = make_tensor_map_bf16_3d(&mv, cache + (size_t)p.Hkv * kWBlk * p.dk, p.dv, (long long)p.Hkv * kWBlk, p.num_blocks,
+                                p.dv, p.block_elems, 64, kWBlk, 1);
+    if (r) return r;
+  }
   const WinSmem L((p.dk + 63) / 64, (p.dv + 63) / 64);
   static int configured = 0;
   if (configured < L.total) {

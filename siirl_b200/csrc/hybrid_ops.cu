@@ -3,7 +3,10 @@
 //
 //   embed_scaled       h[t] = table[id[t]] * scale                               (fp32 stream)
 //   add_norm           h += delta;  y = norm(h) * w                              (layer norm or RMS norm, one launch)
-//   gated_act          y = act(gate) * up   for a fused projection [gate | up]   (SiLU or tanh-form GELU)
+//   stream_rows        h += mult * sum of two sublayer results, each times a sigmoid gate, then h / rms(h)  (one launch);
+//                      or h = sum of partial products + vector (entry of a loop's pass), then h / rms(h); or h as two rows
+//   gated_act          y = act(gate) * up   for a fused projection [gate | up]   (SiLU, tanh-form or exact GELU)
+//   scaled_act         y = act(gain * x)    of a column range
 //   softcap            z = cap * tanh(z / cap) in place on fp32 logits
 //   gemm_simt          C[M, N] = A[M, K] B[N, K]^T with fp32 accumulation on the FMA pipes: fp32 models (true 32-bit
 //                      products) and bf16 operands whose row pitch TMA cannot address (not a multiple of 16 bytes)
@@ -115,8 +118,15 @@ __device__ __forceinline__ float gelu_tanh_f(float z) {
   return 0.5f * z * (1.f + tanhf(u));
 }
 
-template <typename T, int V>
-__global__ void gated_act_kernel(const T* __restrict__ gu, T* __restrict__ out, long long rows, int I, int act) {
+template <int ACT>      // 0 SiLU, 1 tanh-form GELU, 2 exact GELU
+__device__ __forceinline__ float activate(float z) {
+  if constexpr (ACT == 1) return gelu_tanh_f(z);
+  if constexpr (ACT == 2) return 0.5f * z * (1.f + erff(z * 0.7071067811865476f));
+  return z / (1.f + __expf(-z));
+}
+
+template <typename T, int V, int ACT>
+__global__ void gated_act_kernel(const T* __restrict__ gu, T* __restrict__ out, long long rows, int I) {
   const int nv = I / V;
   const long long total = rows * nv;
   for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
@@ -126,8 +136,151 @@ __global__ void gated_act_kernel(const T* __restrict__ gu, T* __restrict__ out, 
     load_vec<T, V>(gu + t * 2 * I + c, g);
     load_vec<T, V>(gu + t * 2 * I + I + c, u);
 #pragma unroll
-    for (int k = 0; k < V; ++k) g[k] = (act == 1 ? gelu_tanh_f(g[k]) : g[k] / (1.f + __expf(-g[k]))) * u[k];
+    for (int k = 0; k < V; ++k) g[k] = activate<ACT>(g[k]) * u[k];
     store_vec<T, V>(out + t * I + c, g);
+  }
+}
+
+template <typename T, int V, int ACT>
+__global__ void scaled_act_kernel(const T* __restrict__ x, long long stride, const T* __restrict__ gain, T* __restrict__ out,
+                                  long long rows, int I) {
+  const int nv = I / V;
+  const long long total = rows * nv;
+  const float f = gain ? to_float(*gain) : 1.f;
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const long long t = i / nv;
+    const int c = (int)(i % nv) * V;
+    float v[V];
+    load_vec<T, V>(x + t * stride + c, v);
+#pragma unroll
+    for (int k = 0; k < V; ++k) v[k] = activate<ACT>(f * v[k]);
+    store_vec<T, V>(out + t * I + c, v);
+  }
+}
+
+// mirrored by ctypes structures in ops/rows.py
+struct StreamSub {
+  const void* y;            // [slabs, T or 2 T, W] partial sums (fp32), or one tensor in the activation format
+  long long slab;
+  int slabs, y_f32;
+  const void* gate;         // pre-activations of the gate, or null
+  long long gate_stride;
+  const void* bias;         // [W], or null
+  const void* gain;         // one number, or null
+};
+struct StreamParams {
+  float* h;                 // [rows, W]
+  int rows, W;
+  float mult, eps;
+  int n_sub, enter;         // enter: h is replaced by sub[0] + sub[1] + step
+  StreamSub sub[2];
+  const void* step;         // [W]
+  int pair, split;          // pair: sub[0] has 2 rows per row of h; split: out is h as two rows of the format, [2 rows, W]
+  const void* weight;       // one number, or null
+  void* out;                // [rows, W] (or [2 rows, W]) in the activation format
+};
+static_assert(sizeof(StreamParams) == 176, "StreamParams is mirrored from Python");
+
+// CH register chunks of V elements per thread hold the row (CH = 0: the row is re-read from memory)
+template <typename T, int V, int CH>
+__global__ void __launch_bounds__(kRowThreads) stream_rows_kernel(const __grid_constant__ StreamParams p) {
+  __shared__ float red[kRowThreads / 32];
+  const int W = p.W, nv = W / V;
+  float gain[2];
+#pragma unroll
+  for (int j = 0; j < 2; ++j) gain[j] = p.sub[j].gain ? to_float(*reinterpret_cast<const T*>(p.sub[j].gain)) : 1.f;
+  for (int row = blockIdx.x; row < p.rows; row += gridDim.x) {
+    float* hr = p.h + (size_t)row * W;
+    T* o0 = reinterpret_cast<T*>(p.out) + (size_t)row * W;
+    float x[CH > 0 ? CH : 1][V];
+    // sum of the slabs of sublayer j at vector vi of row r
+    auto add_slabs = [&](const StreamSub& s, int r, int vi, float (&v)[V]) {
+      const size_t at = (size_t)r * W + (size_t)vi * V;
+      for (int k = 0; k < s.slabs; ++k) {
+        float y[V];
+        if (s.y_f32) load_vec<float, V>(reinterpret_cast<const float*>(s.y) + k * s.slab + at, y);
+        else load_vec<T, V>(reinterpret_cast<const T*>(s.y) + k * s.slab + at, y);
+#pragma unroll
+        for (int i = 0; i < V; ++i) v[i] += y[i];
+      }
+    };
+    auto fetch = [&](int vi, float (&v)[V]) {
+      const size_t c = (size_t)vi * V;
+      if (p.enter) {
+        load_vec<T, V>(reinterpret_cast<const T*>(p.step) + c, v);
+        add_slabs(p.sub[1], row, vi, v);
+        add_slabs(p.sub[0], row, vi, v);
+        if (p.pair) add_slabs(p.sub[0], row + p.rows, vi, v);
+      } else {
+        load_vec<float, V>(hr + c, v);
+        float add[V] = {};
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+          if (j >= p.n_sub) break;
+          const StreamSub& s = p.sub[j];
+          float y[V] = {};
+          add_slabs(s, row, vi, y);
+          if (s.gate) {
+            float g[V], b[V] = {};
+            load_vec<T, V>(reinterpret_cast<const T*>(s.gate) + row * s.gate_stride + c, g);
+            if (s.bias) load_vec<T, V>(reinterpret_cast<const T*>(s.bias) + c, b);
+#pragma unroll
+            for (int i = 0; i < V; ++i) y[i] /= 1.f + __expf(-fmaf(gain[j], g[i], b[i]));
+          }
+#pragma unroll
+          for (int i = 0; i < V; ++i) add[i] += y[i];
+        }
+#pragma unroll
+        for (int i = 0; i < V; ++i) v[i] = fmaf(p.mult, add[i], v[i]);
+      }
+      if (p.enter || p.n_sub) store_vec<float, V>(hr + c, v);
+      if (p.split) {
+        store_vec<T, V>(o0 + c, v);
+        if constexpr (sizeof(T) == 2) {
+          float lo[V];
+#pragma unroll
+          for (int i = 0; i < V; ++i) lo[i] = v[i] - __bfloat162float(__float2bfloat16(v[i]));
+          store_vec<T, V>(o0 + (size_t)p.rows * W + c, lo);
+        }
+      }
+    };
+    if constexpr (CH > 0) {
+#pragma unroll
+      for (int c = 0; c < CH; ++c) {
+        const int vi = threadIdx.x + c * kRowThreads;
+        if (vi < nv) fetch(vi, x[c]);
+      }
+    } else {
+      for (int vi = threadIdx.x; vi < nv; vi += kRowThreads) fetch(vi, x[0]);
+    }
+    if (p.split) continue;
+    auto each = [&](auto&& fn) {
+      if constexpr (CH > 0) {
+#pragma unroll
+        for (int c = 0; c < CH; ++c) {
+          const int vi = threadIdx.x + c * kRowThreads;
+          if (vi < nv) fn(vi, x[c]);
+        }
+      } else {
+        for (int vi = threadIdx.x; vi < nv; vi += kRowThreads) {
+          load_vec<float, V>(hr + (size_t)vi * V, x[0]);   // written by this same thread above
+          fn(vi, x[0]);
+        }
+      }
+    };
+    float ss = 0.f;
+    each([&](int, float (&v)[V]) {
+#pragma unroll
+      for (int k = 0; k < V; ++k) ss = fmaf(v[k], v[k], ss);
+    });
+    float f = 1.f / sqrtf(row_sum(ss, red) / (float)W + p.eps);
+    if (p.weight) f *= to_float(*reinterpret_cast<const T*>(p.weight));
+    each([&](int vi, float (&v)[V]) {
+      float o[V];
+#pragma unroll
+      for (int k = 0; k < V; ++k) o[k] = v[k] * f;
+      store_vec<T, V>(o0 + (size_t)vi * V, o);
+    });
   }
 }
 
@@ -203,6 +356,36 @@ static int launch_add_norm(float* h, const T* delta, const T* w, T* y, int rows,
   return (int)cudaGetLastError();
 }
 
+template <typename T>
+static int launch_stream_rows(const StreamParams& p, cudaStream_t s) {
+  const int grid = p.rows < num_sms() * 8 ? p.rows : num_sms() * 8, W = p.W;
+  bool vec = W % 4 == 0;
+  for (int j = 0; j < 2; ++j) vec = vec && p.sub[j].gate_stride % 4 == 0 && ((uintptr_t)p.sub[j].gate & 15) % (4 * sizeof(T)) == 0;
+  if (!vec) stream_rows_kernel<T, 1, 0><<<grid, kRowThreads, 0, s>>>(p);
+  else if (W <= 4 * kRowThreads) stream_rows_kernel<T, 4, 1><<<grid, kRowThreads, 0, s>>>(p);
+  else if (W <= 2 * 4 * kRowThreads) stream_rows_kernel<T, 4, 2><<<grid, kRowThreads, 0, s>>>(p);
+  else if (W <= 4 * 4 * kRowThreads) stream_rows_kernel<T, 4, 4><<<grid, kRowThreads, 0, s>>>(p);
+  else stream_rows_kernel<T, 4, 0><<<grid, kRowThreads, 0, s>>>(p);
+  return (int)cudaGetLastError();
+}
+
+template <typename T, int V>
+static int launch_gated_act(const T* gu, T* out, long long rows, int I, int act, int grid, cudaStream_t s) {
+  if (act == 0) gated_act_kernel<T, V, 0><<<grid, 256, 0, s>>>(gu, out, rows, I);
+  else if (act == 1) gated_act_kernel<T, V, 1><<<grid, 256, 0, s>>>(gu, out, rows, I);
+  else gated_act_kernel<T, V, 2><<<grid, 256, 0, s>>>(gu, out, rows, I);
+  return (int)cudaGetLastError();
+}
+
+template <typename T, int V>
+static int launch_scaled_act(const T* x, long long stride, const T* gain, T* out, long long rows, int I, int act, int grid,
+                             cudaStream_t s) {
+  if (act == 0) scaled_act_kernel<T, V, 0><<<grid, 256, 0, s>>>(x, stride, gain, out, rows, I);
+  else if (act == 1) scaled_act_kernel<T, V, 1><<<grid, 256, 0, s>>>(x, stride, gain, out, rows, I);
+  else scaled_act_kernel<T, V, 2><<<grid, 256, 0, s>>>(x, stride, gain, out, rows, I);
+  return (int)cudaGetLastError();
+}
+
 }  // namespace sb
 
 using namespace sb;
@@ -233,20 +416,42 @@ extern "C" int sb_add_norm(float* h, const void* delta, const void* w, void* y, 
                                         W, eps, layer_norm, stream);
 }
 
-// act: 0 SiLU, 1 tanh-form GELU; gu [rows, 2 I] -> out [rows, I]
+// act: 0 SiLU, 1 tanh-form GELU, 2 exact GELU; gu [rows, 2 I] -> out [rows, I]
 extern "C" int sb_gated_act(const void* gu, void* out, long long rows, int I, int act, int f32, cudaStream_t stream) {
   if (rows == 0) return 0;
+  if (act < 0 || act > 2) return -3;
   const int V = f32 ? 4 : 8;
   const int grid = grid_for(rows * I / (I % V ? 1 : V), 256);
-  if (f32) {
-    if (I % 4 == 0) gated_act_kernel<float, 4><<<grid, 256, 0, stream>>>((const float*)gu, (float*)out, rows, I, act);
-    else gated_act_kernel<float, 1><<<grid, 256, 0, stream>>>((const float*)gu, (float*)out, rows, I, act);
-  } else {
-    using B = __nv_bfloat16;
-    if (I % 8 == 0) gated_act_kernel<B, 8><<<grid, 256, 0, stream>>>((const B*)gu, (B*)out, rows, I, act);
-    else gated_act_kernel<B, 1><<<grid, 256, 0, stream>>>((const B*)gu, (B*)out, rows, I, act);
-  }
-  return (int)cudaGetLastError();
+  using B = __nv_bfloat16;
+  if (f32)
+    return I % 4 == 0 ? launch_gated_act<float, 4>((const float*)gu, (float*)out, rows, I, act, grid, stream)
+                      : launch_gated_act<float, 1>((const float*)gu, (float*)out, rows, I, act, grid, stream);
+  return I % 8 == 0 ? launch_gated_act<B, 8>((const B*)gu, (B*)out, rows, I, act, grid, stream)
+                    : launch_gated_act<B, 1>((const B*)gu, (B*)out, rows, I, act, grid, stream);
+}
+
+// x: columns of rows `stride` apart -> out [rows, I]; gain: one number or null
+extern "C" int sb_scaled_act(const void* x, long long stride, const void* gain, void* out, long long rows, int I, int act,
+                             int f32, cudaStream_t stream) {
+  if (rows == 0 || I == 0) return 0;
+  if (act < 0 || act > 2) return -3;
+  const int V = f32 ? 4 : 8;
+  const bool vec = I % V == 0 && stride % V == 0 && ((uintptr_t)x & 15) == 0 && ((uintptr_t)out & 15) == 0;
+  const int grid = grid_for(rows * I / (vec ? V : 1), 256);
+  using B = __nv_bfloat16;
+  if (f32)
+    return vec ? launch_scaled_act<float, 4>((const float*)x, stride, (const float*)gain, (float*)out, rows, I, act, grid, stream)
+               : launch_scaled_act<float, 1>((const float*)x, stride, (const float*)gain, (float*)out, rows, I, act, grid, stream);
+  return vec ? launch_scaled_act<B, 8>((const B*)x, stride, (const B*)gain, (B*)out, rows, I, act, grid, stream)
+             : launch_scaled_act<B, 1>((const B*)x, stride, (const B*)gain, (B*)out, rows, I, act, grid, stream);
+}
+
+// params: host StreamParams
+extern "C" int sb_stream_rows(const void* params, int f32, cudaStream_t stream) {
+  const StreamParams& p = *reinterpret_cast<const StreamParams*>(params);
+  if (p.rows <= 0) return 0;
+  if (p.n_sub < 0 || p.n_sub > 2 || (p.enter && p.n_sub != 2)) return -3;
+  return f32 ? launch_stream_rows<float>(p, stream) : launch_stream_rows<__nv_bfloat16>(p, stream);
 }
 
 extern "C" int sb_softcap(float* z, long long n, float cap, cudaStream_t stream) {

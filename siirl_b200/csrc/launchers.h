@@ -191,6 +191,9 @@ int sb_embed_scaled(const long long* ids, const void* table, float* h, int T, in
 int sb_add_norm(float* h, const void* delta, const void* w, void* y, int rows, int W, float eps, int layer_norm, int f32,
                 cudaStream_t stream);
 int sb_gated_act(const void* gu, void* out, long long rows, int I, int act, int f32, cudaStream_t stream);
+int sb_scaled_act(const void* x, long long stride, const void* gain, void* out, long long rows, int I, int act, int f32,
+                  cudaStream_t stream);
+int sb_stream_rows(const void* params, int f32, cudaStream_t stream);
 int sb_softcap(float* z, long long n, float cap, cudaStream_t stream);
 int sb_gemm_simt(const void* A, const void* B, void* C, int M, int N, int K, long long lda, long long ldb, long long ldc,
                  int in_f32, int out_f32, cudaStream_t stream);
@@ -211,4 +214,14 @@ int sb_attn_window_prefill(const void* params, const int* tile_row, const int* t
 int sb_attn_window_decode_chunks(const void* params);
 int sb_attn_window_decode(const void* params, const int* seq_lens, float* ws_o, float* ws_lse, int* status,
                           cudaStream_t stream);
+// ---- head_product.cu (params: host HeadProduct) ----
+int sb_head_product(const void* params, int* status, cudaStream_t stream);
+int sb_head_product_simt(const void* params, int f32, cudaStream_t stream);
+// ---- latent_decode.cu (params: host LatentParams) ----
+int sb_latent_append(const void* params, void* rows, int f32, cudaStream_t stream);
+int sb_latent_gather(const void* params, const int* key_slot, const int* key_pos, void* rows, int n, int f32,
+                     cudaStream_t stream);
+int sb_latent_decode_groups(int H, int R);
+int sb_latent_decode_grid();
+int sb_latent_decode(const void* params, float* ws_o, float* ws_stat, int* status, cudaStream_t stream);
 }

@@ -22,8 +22,16 @@ struct WinParams {
   float scale, bias_exp, out_scale;
   void* out;                // [T, out_stride], heads at column out_off
   long long out_stride;
-  int out_off, pad_;
+  int out_off;
+  int kv_mode;              // where keys and values are, see below
+  const void* gain;         // one number that multiplies the queries and the gate, or null
+  const void* gate;         // columns like out's: the result is multiplied by sigmoid(gain * gate) (prompts); null: none
+  long long gate_stride;
 };
-static_assert(sizeof(WinParams) == 144, "WinParams is mirrored from Python");
+// kPaged: as described above.  kPackedRows (prompts): `cache` is [num_blocks, block_elems], one row per KEY, keys of all
+// heads before values, and a tile's slot is the row of its sequence's first key.  kLatent (general kernel): keys and
+// values are the same dk-wide rows, [num_blocks, 64, dk].
+enum { kPaged = 0, kPackedRows = 1, kLatent = 2 };
+static_assert(sizeof(WinParams) == 168, "WinParams is mirrored from Python");
 
 }  // namespace sb

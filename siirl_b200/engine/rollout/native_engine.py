@@ -169,7 +169,7 @@ class RolloutEngine:
         self.enable_chunked_prefill = bool(enable_chunked_prefill)
         self.enable_prefix_caching = bool(enable_prefix_caching)
         hybrid = model.cfg.hybrid
-        self.recurrent = hybrid is not None and any(b.kind != "attention" for x in hybrid.layers for b in x.branches)
+        self.recurrent = hybrid is not None and any(b.recurrent for x in hybrid.layers for b in x.branches)
         self.visible_span = hybrid.visible_span() if hybrid is not None else None
         if hybrid is not None and lockstep_group is not None:
             raise ValueError("hybrid decoders have no expert layers: no lock-step group")

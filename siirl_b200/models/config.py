@@ -99,7 +99,9 @@ class PrismaticConfig:
 @dataclass
 class MixerBranch:
     """One token mixer of a hybrid layer.  ``kind``: "attention" (paged cache, sliding window with kept first tokens,
-    linear distance bias), "gated_linear" (matrix state, decay per key channel) or "matrix_memory" (stabilised mLSTM)."""
+    linear distance bias), "latent_attention" (paged cache of one compressed row per token, from which every head's keys
+    and values are expanded), "gated_linear" (matrix state, decay per key channel) or "matrix_memory" (stabilised
+    mLSTM)."""
     kind: str = "attention"
     heads: int = 4
     dim: int = 32                   # query / key width of a head
@@ -111,11 +113,24 @@ class MixerBranch:
     window: int = 0                 # 0: no limit
     keep_first: int = 0
     bias_exp: float = 8.0           # slope of head h: 2^(-bias_exp (h + 1) / heads); 0: no bias
+    # latent_attention (with ``scale``)
+    kv_rank: int = 0                # width of the cached row
+    output_gate: bool = False       # heads times the sigmoid of a projection of the mixer's input
     # gated_linear
     tau: float = 16.0
     rank: int = 0                   # width of the decay's low-rank bottleneck (the checkpoint's tensor shape)
     # matrix_memory
     gate_cap: float = 15.0
+
+    @property
+    def recurrent(self) -> bool:
+        return self.kind in ("gated_linear", "matrix_memory")
+
+    def paged(self) -> Optional[tuple]:
+        """(kv heads, key width, value width) of what the branch keeps in the paged cache, or ``None``."""
+        if self.kind == "attention":
+            return (self.kv_heads, self.dim, self.vdim)
+        return (1, self.kv_rank, 0) if self.kind == "latent_attention" else None
 
 
 @dataclass
@@ -125,18 +140,48 @@ class HybridLayer:
 
 
 @dataclass
+class LayerLoop:
+    """Layers ``start .. stop - 1`` run ``times`` times in a row with the same weights; every pass keeps its own cache."""
+    start: int = 0
+    stop: int = 0
+    times: int = 1
+
+
+@dataclass
 class HybridSpec:
-    """Decoders whose layers mix attention and recurrences; the residual stream is kept in 32-bit."""
+    """Decoders whose layers mix attention and recurrences; the residual stream is kept in 32-bit.
+
+    ``arrangement``: "sequential" (mixer, then feed-forward on the updated stream; vector norms, gated feed-forward) or
+    "parallel" (both read the same stream, ``x += residual_mult * (mixer(norm1 x) + ff(norm2 x))``; norms of one number
+    each, plain feed-forward, optionally a sigmoid gate per element on each of the two results)."""
     layers: List[HybridLayer] = field(default_factory=list)
     embed_scale: float = 1.0
     logit_softcap: float = 0.0      # 0: none
     norm: str = "layer_norm"        # or "rms_norm"
-    act: str = "gelu_tanh"          # or "silu"
+    act: str = "gelu_tanh"          # or "silu", "gelu" (exact)
+    arrangement: str = "sequential"
+    residual_mult: float = 1.0
+    residual_gate: bool = False
+    loop: Optional[LayerLoop] = None
     hf_naming: str = "domavik"
 
     @property
     def attention(self) -> List[MixerBranch]:
-        return [b for layer in self.layers for b in layer.branches if b.kind == "attention"]
+        return [b for layer in self.layers for b in layer.branches if b.paged() is not None]
+
+    def runs(self) -> List[tuple]:
+        """``(layer, pass)`` in the order of execution; ``pass`` is the number of the pass that begins right before the
+        layer, or ``None``."""
+        n, lp = len(self.layers), self.loop
+        if lp is None:
+            return [(i, None) for i in range(n)]
+        if not (0 <= lp.start < lp.stop <= n and lp.times >= 0):
+            raise ValueError(f"loop over layers {lp.start} .. {lp.stop} of {n}, {lp.times} times")
+        body = range(lp.start, lp.stop)
+        out = [(i, None) for i in range(lp.start)]
+        for t in range(lp.times):
+            out += [(i, t if i == lp.start else None) for i in body]
+        return out + [(i, None) for i in range(lp.stop, n)]
 
     def visible_span(self):
         """(window, keep_first) outside which no layer looks, or ``None`` when some layer sees everything."""
@@ -257,9 +302,10 @@ class DecoderConfig:
         return self.hybrid.logit_softcap if self.hybrid is not None else 0.0
 
     def paged_layers(self) -> List[tuple]:
-        """(kv heads, key width, value width) of every layer that keeps keys and values in the paged cache."""
+        """(kv heads, key width, value width) of every layer run that keeps something in the paged cache."""
         if self.hybrid is not None:
-            return [(b.kv_heads, b.dim, b.vdim) for b in self.hybrid.attention]
+            return [b.paged() for i, _ in self.hybrid.runs() for b in self.hybrid.layers[i].branches
+                    if b.paged() is not None]
         return [(self.num_kv_heads, self.head_dim, self.head_dim)] * self.num_layers
 
     def num_parameters(self) -> int:
@@ -279,11 +325,20 @@ class DecoderConfig:
         return V * H + self.num_layers * per_layer + H + head
 
     def _hybrid_parameters(self) -> int:
-        W, n = self.hidden_size, 2 * self.vocab_size * self.hidden_size + self.hidden_size
-        for layer in self.hybrid.layers:
-            n += W + (W + 3 * W * layer.ff if layer.ff else 0)
+        hy, W = self.hybrid, self.hidden_size
+        parallel = hy.arrangement == "parallel"
+        norm, ffs = (1, 2) if parallel else (W, 3)
+        gate = W * (W + 1) if hy.residual_gate else 0
+        n = 2 * self.vocab_size * W + norm
+        if hy.loop is not None:
+            n += 2 * W * W + hy.loop.times * W
+        for layer in hy.layers:
+            n += norm + gate + (norm + ffs * W * layer.ff + gate if layer.ff else 0)
             for b in layer.branches:
                 hk, hv = b.heads * b.dim, b.heads * b.vdim
+                if b.kind == "latent_attention":
+                    n += W * (hk + b.kv_rank + hv * (1 + int(b.output_gate))) + b.kv_rank * (1 + hk + hv)
+                    continue
                 if b.kind == "attention":
                     n += W * (hk + b.kv_heads * (b.dim + b.vdim) + hv)
                     continue
@@ -318,6 +373,7 @@ class DecoderConfig:
             hy = dict(d["hybrid"])
             hy["layers"] = [build(HybridLayer, dict(x, branches=[build(MixerBranch, b) for b in x["branches"]]))
                             for x in hy.get("layers", [])]
+            hy["loop"] = build(LayerLoop, hy.get("loop"))
             d["hybrid"] = build(HybridSpec, hy)
         for key in ("lora_targets", "mrope_section"):
             if isinstance(d.get(key), list) and key == "lora_targets":
@@ -328,8 +384,8 @@ class DecoderConfig:
     # ---- HF interchange -----------------------------------------------------------------------
     @classmethod
     def from_hf_config(cls, cfg: Dict[str, Any]) -> "DecoderConfig":
-        if cfg.get("architecture") == "Domavik":
-            return cls._from_domavik_config(cfg)
+        if cfg.get("architecture") in ("Domavik", "Poralorn"):
+            return cls._from_domavik_config(cfg) if cfg["architecture"] == "Domavik" else cls._from_poralorn_config(cfg)
         text = cfg.get("text_config") or cfg.get("llm_config") or cfg
         mt = cfg.get("model_type", "qwen2")
         if mt in ("llama4", "llama4_text"):
@@ -553,6 +609,45 @@ class DecoderConfig:
         return d
 
     @classmethod
+    def _from_poralorn_config(cls, cfg: Dict[str, Any]) -> "DecoderConfig":
+        """Poralorn: latent attention without positions beside a plain GELU feed-forward, both gated, and a run of layers
+        that is repeated."""
+        layers = []
+        for x in cfg["layers"]:
+            m, mlp = x["mixer"], x.get("mlp")
+            if x["type"] != "latent_attention":
+                raise ValueError(f"unknown layer type {x['type']!r}")
+            if mlp is not None and mlp["kind"] != "dense":
+                raise ValueError(f"unknown feed-forward kind {mlp['kind']!r}")
+            layers.append(HybridLayer([MixerBranch(
+                kind="latent_attention", heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
+                kv_rank=int(m["kv_rank"]), scale=float(m["scale"]), output_gate=True)],
+                ff=int(mlp["ff"]) if mlp is not None else 0))
+        lp = cfg.get("loop")
+        spec = HybridSpec(layers=layers, logit_softcap=float(cfg.get("logit_softcap") or 0.0), norm="rms_norm", act="gelu",
+                          arrangement="parallel", residual_mult=float(cfg["residual_mult"]), residual_gate=True,
+                          loop=LayerLoop(int(lp["start"]), int(lp["stop"]), int(lp["times"])) if lp else None,
+                          hf_naming="poralorn")
+        spec.runs()
+        return cls.for_hybrid(spec, vocab_size=int(cfg["vocab"]), hidden_size=int(cfg["width"]),
+                              rms_norm_eps=float(cfg["norm"]["eps"]), model_type="poralorn",
+                              eos_token_id=int(cfg.get("eos_token_id", -1)), pad_token_id=int(cfg.get("pad_token_id", 0)))
+
+    def _to_poralorn_config(self) -> Dict[str, Any]:
+        hy = self.hybrid
+        layers = [{"type": "latent_attention",
+                   "mixer": {n: getattr(x.branches[0], n) for n in ("heads", "dim", "vdim", "kv_rank", "scale")},
+                   "mlp": {"kind": "dense", "ff": x.ff} if x.ff else None} for x in hy.layers]
+        d = {"architecture": "Poralorn", "vocab": self.vocab_size, "width": self.hidden_size,
+             "norm": {"eps": self.rms_norm_eps}, "residual_mult": hy.residual_mult, "logit_softcap": hy.logit_softcap,
+             "layers": layers}
+        if hy.loop is not None:
+            d["loop"] = {"start": hy.loop.start, "stop": hy.loop.stop, "times": hy.loop.times}
+        if self.eos_token_id >= 0:
+            d["eos_token_id"] = self.eos_token_id
+        return d
+
+    @classmethod
     def from_pretrained(cls, path: str) -> "DecoderConfig":
         with open(os.path.join(os.path.expanduser(path), "config.json")) as f:
             out = cls.from_hf_config(json.load(f))
@@ -563,7 +658,7 @@ class DecoderConfig:
 
     def to_hf_config(self) -> Dict[str, Any]:
         if self.hybrid is not None:
-            return self._to_domavik_config()
+            return self._to_poralorn_config() if self.hybrid.hf_naming == "poralorn" else self._to_domavik_config()
         arch = {"qwen2": "Qwen2ForCausalLM", "qwen3": "Qwen3ForCausalLM", "qwen3_moe": "Qwen3MoeForCausalLM",
                 "llama": "LlamaForCausalLM", "qwen2_5_vl": "Qwen2_5_VLForConditionalGeneration",
                 "mixtral": "MixtralForCausalLM", "qwen2_moe": "Qwen2MoeForCausalLM",
@@ -681,7 +776,21 @@ def _domavik(n_layers: int, width: int, ff: int, vocab: int, att: dict, gla: dic
                                     **kw)
 
 
+def _poralorn(n_layers: int, width: int, ff: int, vocab: int, heads: int, dim: int, vdim: int, kv_rank: int,
+              loop: Optional[LayerLoop] = None, softcap: float = 30.0, mult: float = 0.5, **kw) -> DecoderConfig:
+    layers = [HybridLayer([MixerBranch(kind="latent_attention", heads=heads, dim=dim, vdim=vdim, kv_rank=kv_rank,
+                                       scale=dim ** -0.5, output_gate=True)], ff=ff) for _ in range(n_layers)]
+    spec = HybridSpec(layers=layers, logit_softcap=softcap, norm="rms_norm", act="gelu", arrangement="parallel",
+                      residual_mult=mult, residual_gate=True, loop=loop, hf_naming="poralorn")
+    return DecoderConfig.for_hybrid(spec, vocab_size=vocab, hidden_size=width, rms_norm_eps=1e-5, model_type="poralorn",
+                                    **kw)
+
+
 PRESETS: Dict[str, DecoderConfig] = {
+    "tiny-poralorn": _poralorn(3, 128, 224, 1024, heads=3, dim=24, vdim=40, kv_rank=48, loop=LayerLoop(1, 2, 3)),
+    # layer sizes of a 7B / 1.5B-class decoder (benchmark shapes, random weights)
+    "poralorn-7b": _poralorn(28, 3584, 18944, 152064, heads=28, dim=128, vdim=128, kv_rank=512, loop=LayerLoop(2, 6, 2)),
+    "poralorn-1.5b": _poralorn(28, 1536, 8960, 152064, heads=12, dim=128, vdim=128, kv_rank=512, loop=LayerLoop(2, 8, 2)),
     "tiny-domavik": _domavik(3, 128, 192, 1024, dict(heads=4, kv_heads=2, dim=32, vdim=24, window=70, keep_first=5),
                              dict(heads=2, dim=16, vdim=32, tau=4.0, rank=8), dict(heads=2, dim=32, vdim=40),
                              scales=(0.9, 0.6)),

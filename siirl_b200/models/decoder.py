@@ -37,7 +37,7 @@ class _Init:
 
 def _param(shape, dtype, device, std: float, gen: "_Init") -> nn.Parameter:
     dev = gen.device if gen.device.type == "cuda" else torch.device("cpu")
-    t = torch.empty(*shape, dtype=torch.float32 if dev.type == "cpu" else dtype, device=dev)
+    t = torch.empty(shape, dtype=torch.float32 if dev.type == "cpu" else dtype, device=dev)
     if std > 0:
         t.normal_(0.0, std, generator=gen.gen)
     elif std == 0:

@@ -306,6 +306,36 @@ def _domavik_state(model) -> Iterator[Tuple[str, torch.Tensor]]:
     yield "head", model.lm_head.data
 
 
+def _poralorn_state(model) -> Iterator[Tuple[str, torch.Tensor]]:
+    """Poralorn checkpoint names and the views of the fused, padded parameters they fill (models/hybrid.py)."""
+    yield "embed", model.embed_tokens.data
+    if model.cfg.hybrid.loop is not None:
+        yield "loop.in", model.loop_in_weight.data
+        yield "loop.step", model.loop_step.data
+    for i, layer in enumerate(model.layers):
+        p, w = f"l{i}.", layer.in_proj_weight.data
+        br, = layer.branches
+        b = br.b
+        yield p + "norm1", layer.norm1.data
+        for ours, theirs in (("q", "q"), ("c", "dkv"), ("g", "g")):
+            at, n = br.cols[ours]
+            yield p + "mix." + theirs, w[at:at + n]
+        yield p + "mix.dkv.norm", br.c_norm.data
+        yield p + "mix.uk", br.kv_up_weight.data[:b.heads * b.dim]
+        yield p + "mix.uv", br.kv_up_weight.data[b.heads * b.dim:]
+        yield p + "mix.o", layer.o_proj_weight.data[:, :b.heads * b.vdim]
+        yield p + "rg1", w[layer.rg1_off:layer.rg1_off + model.cfg.hidden_size]
+        yield p + "rg1.b", layer.rg1_bias.data
+        if layer.ff:
+            yield p + "norm2", layer.norm2.data
+            yield p + "mlp.up", w[layer.up_off:layer.up_off + layer.ff]
+            yield p + "mlp.down", layer.down_proj_weight.data[:, :layer.ff]
+            yield p + "rg2", w[layer.rg2_off:layer.rg2_off + model.cfg.hidden_size]
+            yield p + "rg2.b", layer.rg2_bias.data
+    yield "final.norm", model.norm.data
+    yield "head", model.lm_head.data
+
+
 def fill_hybrid_ranks(cfg: DecoderConfig, path: str) -> None:
     """Sizes that only tensor shapes give: the low-rank width of every decay projection."""
     handles = _open_all(path)
@@ -324,7 +354,7 @@ def _hf_targets(model) -> Iterator[Tuple[str, object]]:
     fused ``wqkv`` comes as the tuple of its three views."""
     cfg: DecoderConfig = model.cfg
     if cfg.hybrid is not None:
-        yield from _domavik_state(model)
+        yield from (_poralorn_state if cfg.hybrid.hf_naming == "poralorn" else _domavik_state)(model)
         return
     prefix, head = _llm_names(cfg)
     internlm2 = cfg.vit is not None and cfg.hf_naming == "internvl_chat" and cfg.llm_type == "internlm2"

@@ -1,10 +1,16 @@
-"""Hybrid decoder: layers that mix window attention and matrix-state recurrences, with the residual stream in 32-bit.
+"""Hybrid decoder: layers that mix window attention, latent attention and matrix-state recurrences, with the residual
+stream in 32-bit.
 
 Every layer is a list of branches over one normed input (``DecoderConfig.hybrid``): their projections are one fused
 matrix (``in_proj``), each branch writes its (scaled) heads into its columns of one row, and one matrix (``o_proj``) adds
-the branches up.  The serving path is the one of :class:`DecoderLM`: ``forward_cached`` over the engine's paged blocks,
-plus the engine's per-slot recurrent states.  A prompt portion appends its keys and values and reads everything it sees
-back from the cache, so whole prompts, portions and single tokens use the same memory.
+the branches up.  In the parallel arrangement the feed-forward reads the same stream and the residual gates read the
+sublayers' inputs, so their matrices join ``in_proj``: the norms there are one number each, which commutes with the
+projections, and one row (the stream over its root mean square) feeds them all; the numbers are applied by the kernels
+behind.  A run of layers may be repeated (``HybridSpec.loop``).
+
+The serving path is the one of :class:`DecoderLM`: ``forward_cached`` over the engine's paged blocks, plus the engine's
+per-slot recurrent states.  A prompt portion appends its keys and values and reads everything it sees back from the
+cache, so whole prompts, portions and single tokens use the same memory.
 
 bf16 models run the tensor-core kernels; fp32 models run true 32-bit kernels (FMA-pipe matrix products).  Weights keep
 the checkpoint's values; fused matrices are padded with zero rows / columns to multiples of eight.  Scoring
@@ -21,6 +27,8 @@ from .. import ops
 from ..ops import kv_cache as kvc
 from ..ops import rows as R
 from ..ops.attention import SeqInfo
+from ..ops.dense import linear_partial
+from ..ops.latent_attention import LatentPlan, LatentSpec, latent_attention
 from ..ops.lm_head import lm_head_logits
 from ..ops.recurrence import PortionPlan, RecurrenceSpec, empty_state, recurrence_decode, recurrence_prefill
 from ..ops.window_attention import QueryTiles, WindowSpec, window_attention
@@ -37,6 +45,8 @@ def branch_segments(b: MixerBranch) -> List[Tuple[str, int]]:
     hk, hv = b.heads * b.dim, b.heads * b.vdim
     if b.kind == "attention":
         return [("q", hk), ("k", b.kv_heads * b.dim), ("v", b.kv_heads * b.vdim)]
+    if b.kind == "latent_attention":
+        return [("q", hk), ("c", b.kv_rank)] + ([("g", hv)] if b.output_gate else [])
     seg = [("q", hk), ("k", hk), ("v", hv), ("g", hv)]
     return seg + ([("a1", b.rank)] if b.kind == "gated_linear" else [("i", b.heads), ("f", b.heads)])
 
@@ -59,6 +69,14 @@ class HybridBranch(nn.Module):
                                    b.keep_first, b.bias_exp, b.out_scale)
             return
         hk, hv = b.heads * b.dim, b.heads * b.vdim
+        if b.kind == "latent_attention":
+            if b.kv_rank < 1 or b.out_scale != 1.0:
+                raise ValueError("latent_attention: a latent width and no output scale")
+            self.c_norm = _param((b.kv_rank,), dtype, device, -1, gen)
+            self.kv_up_weight = _param((hk + hv, b.kv_rank), dtype, device, b.kv_rank ** -0.5, gen)
+            self.spec = LatentSpec(b.heads, b.dim, b.vdim, b.kv_rank, off["q"], off["c"], off.get("g", -1), b.scale,
+                                   cfg.rms_norm_eps)
+            return
         common = dict(heads=b.heads, dim=b.dim, vdim=b.vdim, q_off=off["q"], k_off=off["k"], v_off=off["v"],
                       g_off=off["g"], eps=cfg.rms_norm_eps, out_scale=b.out_scale)
         if b.kind == "gated_linear":
@@ -79,10 +97,25 @@ class HybridBranch(nn.Module):
 
     @property
     def recurrent(self) -> bool:
-        return self.b.kind != "attention"
+        return self.b.recurrent
 
     def weights(self) -> Dict[str, torch.Tensor]:
         return {k: getattr(self, k).detach() for k in ("norm", "w2", "b_e", "b_f") if hasattr(self, k)}
+
+    def run(self, p: torch.Tensor, io: "_Batch", out: torch.Tensor, gain: Optional[torch.Tensor] = None) -> None:
+        """The branch's heads of the projected rows ``p`` into its columns of ``out``; ``gain``: one number that the
+        projections still have to be multiplied by (latent attention only)."""
+        if self.b.kind == "latent_attention":
+            w = {"c_norm": self.c_norm.detach(), "kv_up": self.kv_up_weight.detach(), "gain": gain}
+            latent_attention(self.spec, p, w, io.seq_ids, io.positions, io.block_table, io.next_cache(), out,
+                             self.out_off, plan=io.latent)
+        elif self.b.kind == "attention":
+            window_attention(self.spec, p, io.seq_ids, io.positions, io.block_table, io.next_cache(), out, self.out_off,
+                             tiles=io.tiles, seq_lens=io.seq_lens)
+        elif io.plan is not None:
+            recurrence_prefill(self.spec, p, self.weights(), io.next_state(), io.plan, out, self.out_off)
+        else:
+            recurrence_decode(self.spec, p, self.weights(), io.next_state(), io.seq_ids, io.positions, out, self.out_off)
 
 
 class HybridLayer(nn.Module):
@@ -122,13 +155,7 @@ class HybridLayer(nn.Module):
         alloc = torch.zeros if self.padded_out else torch.empty
         out = alloc(x.shape[0], self.o_proj_weight.shape[1], dtype=x.dtype, device=x.device)
         for br in self.branches:
-            if not br.recurrent:
-                window_attention(br.spec, p, io.seq_ids, io.positions, io.block_table, io.next_cache(), out, br.out_off,
-                                 tiles=io.tiles, seq_lens=io.seq_lens)
-            elif io.plan is not None:
-                recurrence_prefill(br.spec, p, br.weights(), io.next_state(), io.plan, out, br.out_off)
-            else:
-                recurrence_decode(br.spec, p, br.weights(), io.next_state(), io.seq_ids, io.positions, out, br.out_off)
+            br.run(p, io, out)
         return ops.linear(out, self.o_proj_weight)
 
     def mlp(self, x: torch.Tensor) -> torch.Tensor:
@@ -136,13 +163,81 @@ class HybridLayer(nn.Module):
                           self.down_proj_weight)
 
 
+class ParallelLayer(nn.Module):
+    """Mixer and feed-forward side by side on one stream (see :class:`HybridSpec`)."""
+
+    def __init__(self, cfg: DecoderConfig, index: int, dtype, device, gen):
+        super().__init__()
+        hy, W, std = cfg.hybrid, cfg.hidden_size, cfg.initializer_range
+        lay = hy.layers[index]
+        if hy.norm != "rms_norm" or any(b.kind != "latent_attention" for b in lay.branches):
+            raise ValueError("parallel layers: RMS norms of one number and latent attention")
+        self.cfg, self.ff, self.ffp = cfg, lay.ff, _pad8(lay.ff)
+        at = out_off = 0
+        branches, used = [], []
+        for b in lay.branches:
+            br = HybridBranch(b, cfg, at, out_off, dtype, device, gen)
+            used += list(br.cols.values())
+            at, out_off = br.in_end, out_off + _pad8(b.heads * b.vdim)
+            branches.append(br)
+        self.branches = nn.ModuleList(branches)
+
+        def place(n: int) -> int:
+            nonlocal at
+            used.append((at, n))
+            at += _pad8(n)
+            return at - _pad8(n)
+        self.norm1 = _param((), dtype, device, -1, gen)
+        self.rg1_off = place(W) if hy.residual_gate else -1
+        if self.ff:
+            self.norm2 = _param((), dtype, device, -1, gen)
+            self.up_off = place(self.ff)
+            self.rg2_off = place(W) if hy.residual_gate else -1
+            self.down_proj_weight = _param((W, self.ffp), dtype, device, std, gen)
+        self.in_proj_weight = _param((at, W), dtype, device, std, gen)
+        self.o_proj_weight = _param((W, out_off), dtype, device, std, gen)
+        if hy.residual_gate:
+            self.rg1_bias = _param((W,), dtype, device, 0, gen)
+            self.rg2_bias = _param((W,), dtype, device, 0, gen) if self.ff else None
+        self.padded_out = any(b.heads * b.vdim % 8 for b in lay.branches)
+        with torch.no_grad():
+            for o, n in used:
+                self.in_proj_weight[o + n:o + _pad8(n)] = 0
+            if self.ff:
+                self.down_proj_weight[:, self.ff:] = 0
+            for br in self.branches:
+                n = br.b.heads * br.b.vdim
+                self.o_proj_weight[:, br.out_off + n:br.out_off + _pad8(n)] = 0
+
+    def run(self, x: torch.Tensor, io: "_Batch") -> List[R.Sublayer]:
+        """Both sublayers of rows ``x`` (the stream over its root mean square), not yet added to the stream."""
+        W = self.cfg.hidden_size
+        p = ops.linear(x, self.in_proj_weight)
+        alloc = torch.zeros if self.padded_out else torch.empty
+        heads = alloc(x.shape[0], self.o_proj_weight.shape[1], dtype=x.dtype, device=x.device)
+        g1 = self.norm1.detach()
+        for br in self.branches:
+            br.run(p, io, heads, g1)
+
+        def result(y, off, name, gain):
+            if off < 0:
+                return R.Sublayer(y)
+            return R.Sublayer(y, p[:, off:off + W], getattr(self, name).detach(), gain)
+        out = [result(linear_partial(heads, self.o_proj_weight.detach()), self.rg1_off, "rg1_bias", g1)]
+        if self.ff:
+            g2 = self.norm2.detach()
+            u = R.scaled_act(p[:, self.up_off:self.up_off + self.ffp], self.cfg.hybrid.act, g2)
+            out.append(result(linear_partial(u, self.down_proj_weight.detach()), self.rg2_off, "rg2_bias", g2))
+        return out
+
+
 class _Batch:
     """What one forward pass needs besides the rows: places in the cache, prompt portions or decode lengths."""
 
-    def __init__(self, seq_ids, positions, block_table, cache, states, plan=None, tiles=None, seq_lens=None):
+    def __init__(self, seq_ids, positions, block_table, cache, states, plan=None, tiles=None, latent=None, seq_lens=None):
         self.seq_ids, self.positions, self.block_table = seq_ids, positions, block_table
-        self.plan, self.tiles, self.seq_lens = plan, tiles, seq_lens
-        self._cache, self._states = iter(cache), iter(states)
+        self.plan, self.tiles, self.latent, self.seq_lens = plan, tiles, latent, seq_lens
+        self._cache, self._states = iter(cache), iter(states or ())
 
     def next_cache(self):
         return next(self._cache)
@@ -163,8 +258,16 @@ class HybridLM(nn.Module):
         gen = _Init(seed, device)
         std = cfg.initializer_range
         self.embed_tokens = _param((cfg.vocab_size, cfg.hidden_size), dtype, device, std, gen)
-        self.layers = nn.ModuleList([HybridLayer(cfg, i, dtype, device, gen) for i in range(cfg.num_layers)])
-        self.norm = _param((cfg.hidden_size,), dtype, device, -1, gen)
+        self.parallel = cfg.hybrid.arrangement == "parallel"
+        if cfg.hybrid.arrangement not in ("sequential", "parallel") or (cfg.hybrid.loop is not None and not self.parallel):
+            raise ValueError("layer arrangements: sequential, or parallel with an optional loop")
+        kind = ParallelLayer if self.parallel else HybridLayer
+        self.layers = nn.ModuleList([kind(cfg, i, dtype, device, gen) for i in range(cfg.num_layers)])
+        if cfg.hybrid.loop is not None:
+            W = cfg.hidden_size
+            self.loop_in_weight = _param((W, 2 * W), dtype, device, (2 * W) ** -0.5, gen)
+            self.loop_step = _param((cfg.hybrid.loop.times, W), dtype, device, std, gen)
+        self.norm = _param(() if self.parallel else (cfg.hidden_size,), dtype, device, -1, gen)
         self.lm_head = _param((cfg.vocab_size, cfg.hidden_size), dtype, device, std, gen)
 
     @property
@@ -182,6 +285,8 @@ class HybridLM(nn.Module):
     # ---- forward -----------------------------------------------------------------------------------
     def _layers(self, ids: torch.Tensor, io: _Batch) -> torch.Tensor:
         cfg = self.cfg
+        if self.parallel:
+            return self._parallel_layers(ids, io)
         kind, eps = cfg.hybrid.norm, cfg.rms_norm_eps
         h = R.embed_scaled(ids, self.embed_tokens.detach(), cfg.hybrid.embed_scale)
         delta = None
@@ -190,6 +295,26 @@ class HybridLM(nn.Module):
             if layer.ff:
                 delta = layer.mlp(R.add_norm(h, delta, layer.norm2, eps, kind))
         return R.add_norm(h, delta, self.norm, eps, kind)
+
+    def _parallel_layers(self, ids: torch.Tensor, io: _Batch) -> torch.Tensor:
+        hy, eps, dtype = self.cfg.hybrid, self.cfg.rms_norm_eps, self.embed_tokens.dtype
+        W, mult = self.cfg.hidden_size, hy.residual_mult
+        h = R.embed_scaled(ids, self.embed_tokens.detach(), hy.embed_scale)
+        if hy.loop is not None:
+            # a pass begins with W_in [h; embedding]: the embedding's half is the same in every pass, and h keeps its 32
+            # bits as a sum of two rows of the activation format
+            w_in = self.loop_in_weight.detach()
+            x0 = R.stream_update(h, [], mult, dtype, eps, split=True)[:h.shape[0]]
+            base = linear_partial(x0, w_in[:, W:], f32=True)
+        subs: List[R.Sublayer] = []
+        for i, t in hy.runs():
+            if t is None:
+                x = R.stream_update(h, subs, mult, dtype, eps)
+            else:
+                parts = R.stream_update(h, subs, mult, dtype, eps, split=True)
+                x = R.enter_pass(h, linear_partial(parts, w_in[:, :W], f32=True), base, self.loop_step.detach()[t], eps)
+            subs = self.layers[i].run(x, io)
+        return R.stream_update(h, subs, mult, dtype, eps, weight=self.norm.detach())
 
     @torch.no_grad()
     def forward_cached(self, input_ids: torch.Tensor, positions: torch.Tensor, cache: Sequence[torch.Tensor],
@@ -206,8 +331,11 @@ class HybridLM(nn.Module):
         lens = prefill_info.seqlens
         starts = list(prefix_lens) if prefix_lens is not None else [0] * len(lens)
         dev = input_ids.device
-        io = _Batch(seq, pos, block_table, cache, states, plan=PortionPlan(lens, starts, prefill_slots, dev),
-                    tiles=QueryTiles(lens, starts, prefill_slots, dev))
+        kinds = {b.kind for layer in self.cfg.hybrid.layers for b in layer.branches}
+        io = _Batch(seq, pos, block_table, cache, states,
+                    plan=PortionPlan(lens, starts, prefill_slots, dev) if kinds & {"gated_linear", "matrix_memory"} else None,
+                    tiles=QueryTiles(lens, starts, prefill_slots, dev) if "attention" in kinds else None,
+                    latent=LatentPlan(lens, starts, prefill_slots, dev) if "latent_attention" in kinds else None)
         return self._layers(input_ids, io)
 
     @torch.no_grad()

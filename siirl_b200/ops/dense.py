@@ -205,6 +205,36 @@ def linear_skinny(x2: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.T
     return out
 
 
+def linear_partial(x: torch.Tensor, weight: torch.Tensor, f32: bool = False) -> torch.Tensor:
+    """Inference-only ``x @ W^T`` as partial sums ``[S, M, N]`` for a consumer that adds them itself: few rows give the
+    fp32 slabs of a split contraction, many rows one bf16 product (fp32 when ``f32``)."""
+    M, K = x.shape
+    N = weight.shape[0]
+    if not x.is_cuda:
+        return (x.float() @ weight.float().t() if f32 else F.linear(x, weight))[None]
+    if x.dtype == torch.float32 or K % 8 or N % 8 or x.stride(0) % 8 or weight.stride(0) % 8:
+        from .rows import gemm_simt
+        return gemm_simt(x, weight.detach(), torch.float32 if f32 else x.dtype)[None]
+    if M > 512:
+        return gemm(x, weight, epi=EPI_F32 if f32 else EPI_BF16)[None]
+    nkb = (K + 63) // 64
+    swap = M > 128 and SWAP_OPERANDS_ABOVE_128_ROWS
+    splits = _best_splits((N + 127) // 128 * ((M + 255) // 256), nkb) if swap else _skinny_splits(M, N, K)
+    if splits <= 1 and not f32:
+        return linear_skinny(x, weight, None)[None]
+    per = (nkb + splits - 1) // splits
+    eff = (nkb + per - 1) // per
+    slabs = torch.empty(eff, M, N, dtype=torch.float32, device=x.device)
+    ll = ctypes.c_longlong
+    if swap:
+        _lib.check(_lib.get_lib().sb_gemm_bf16(
+            _lib.ptr(weight), _lib.ptr(x), _lib.ptr(slabs), None, N, M, K, ll(weight.stride(0)), ll(x.stride(0)), ll(N), 0,
+            0, EPI_F32_T, 256, 0, eff, ll(M * N), _lib.ptr(_lib.status_word(x.device)), _lib.stream()), "sb_gemm_bf16")
+    else:
+        gemm(x, weight, out=slabs[0], epi=EPI_F32, tile_n=128, k_splits=eff, slab_stride=M * N)
+    return slabs
+
+
 def linear(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``x @ weight^T + bias`` (nn.Linear convention, weight ``[out, in]``)."""
     if not x.is_cuda:

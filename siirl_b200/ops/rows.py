@@ -1,16 +1,18 @@
 """Row operations of decoders with a 32-bit residual stream (``csrc/hybrid_ops.cu``): scaled embedding, residual add fused
-with the following norm, gated activations, soft-capped logits.  Inference only; CPU tensors use the plain statements."""
+with the following norm, gated residual update of two sublayers, entry of a layer loop's pass, activations, soft-capped
+logits.  Inference only; CPU tensors use the plain statements."""
 from __future__ import annotations
 
 import ctypes
-from typing import Optional
+from dataclasses import dataclass
+from typing import Optional, Sequence
 
 import torch
 import torch.nn.functional as F
 
 from . import lib as _lib
 
-ACT = {"silu": 0, "gelu_tanh": 1}
+ACT = {"silu": 0, "gelu_tanh": 1, "gelu": 2}
 
 
 def _f32(t: torch.Tensor) -> int:
@@ -53,11 +55,114 @@ def gated_act(gate_up: torch.Tensor, act: str = "gelu_tanh") -> torch.Tensor:
     T, I2 = gate_up.shape
     if not gate_up.is_cuda:
         g, u = gate_up.float().chunk(2, -1)
-        return ((F.silu(g) if act == "silu" else F.gelu(g, approximate="tanh")) * u).to(gate_up.dtype)
+        return ((F.silu(g) if act == "silu" else F.gelu(g, approximate="tanh" if act == "gelu_tanh" else "none")) * u).to(gate_up.dtype)
     gate_up = gate_up.contiguous()
     out = torch.empty(T, I2 // 2, dtype=gate_up.dtype, device=gate_up.device)
     _lib.check(_lib.get_lib().sb_gated_act(_lib.ptr(gate_up), _lib.ptr(out), ctypes.c_longlong(T), I2 // 2, ACT[act],
                                            _f32(gate_up), _lib.stream()), "sb_gated_act")
+    return out
+
+
+def scaled_act(x: torch.Tensor, act: str, gain: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``act(gain * x)`` of a column range ``x [T, I]`` of wider rows; ``gain``: one number (a tensor)."""
+    if not x.is_cuda:
+        z = x.float() * (gain.float() if gain is not None else 1.0)
+        y = F.silu(z) if act == "silu" else F.gelu(z, approximate="tanh" if act == "gelu_tanh" else "none")
+        return y.to(x.dtype)
+    assert x.stride(1) == 1
+    out = torch.empty(x.shape, dtype=x.dtype, device=x.device)
+    _lib.check(_lib.get_lib().sb_scaled_act(_lib.ptr(x), ctypes.c_longlong(x.stride(0)), _lib.ptr(gain), _lib.ptr(out),
+                                            ctypes.c_longlong(x.shape[0]), x.shape[1], ACT[act], _f32(x), _lib.stream()),
+               "sb_scaled_act")
+    return out
+
+
+@dataclass
+class Sublayer:
+    """One result waiting to enter the residual stream: ``y [S, T, W]`` (partial sums, or one tensor in the activation
+    format), optionally times ``sigmoid(gain * gate + bias)`` with ``gate [T, W]`` a column range of wider rows."""
+    y: torch.Tensor
+    gate: Optional[torch.Tensor] = None
+    bias: Optional[torch.Tensor] = None
+    gain: Optional[torch.Tensor] = None
+
+
+class _Sub(ctypes.Structure):
+    _fields_ = [("y", ctypes.c_void_p), ("slab", ctypes.c_longlong), ("slabs", ctypes.c_int), ("y_f32", ctypes.c_int),
+                ("gate", ctypes.c_void_p), ("gate_stride", ctypes.c_longlong), ("bias", ctypes.c_void_p),
+                ("gain", ctypes.c_void_p)]
+
+
+class _Stream(ctypes.Structure):
+    """Mirror of ``StreamParams`` in csrc/hybrid_ops.cu."""
+    _fields_ = [("h", ctypes.c_void_p), ("rows", ctypes.c_int), ("W", ctypes.c_int), ("mult", ctypes.c_float),
+                ("eps", ctypes.c_float), ("n_sub", ctypes.c_int), ("enter", ctypes.c_int), ("sub", _Sub * 2),
+                ("step", ctypes.c_void_p), ("pair", ctypes.c_int), ("split", ctypes.c_int),
+                ("weight", ctypes.c_void_p), ("out", ctypes.c_void_p)]
+
+
+assert ctypes.sizeof(_Stream) == 176
+
+
+def _sub(s: Sublayer, W: int) -> _Sub:
+    assert s.y.is_contiguous() and s.y.dim() == 3 and s.y.shape[2] == W
+    g = s.gate
+    assert g is None or g.stride(1) == 1
+    return _Sub(y=s.y.data_ptr(), slab=s.y.stride(0), slabs=s.y.shape[0], y_f32=_f32(s.y),
+                gate=g.data_ptr() if g is not None else None, gate_stride=g.stride(0) if g is not None else 0,
+                bias=s.bias.data_ptr() if s.bias is not None else None,
+                gain=s.gain.data_ptr() if s.gain is not None else None)
+
+
+def _finish_rows(h: torch.Tensor, dtype, eps: float, weight, split: bool) -> torch.Tensor:
+    if split:
+        if dtype == torch.float32:
+            return h.clone()
+        hi = h.to(dtype)
+        return torch.cat([hi, (h - hi.float()).to(dtype)])
+    y = h * torch.rsqrt(h.pow(2).mean(-1, keepdim=True) + eps)
+    return (y * weight.float() if weight is not None else y).to(dtype)
+
+
+def stream_update(h: torch.Tensor, subs: Sequence[Sublayer], mult: float, dtype: torch.dtype, eps: float,
+                  weight: Optional[torch.Tensor] = None, split: bool = False) -> torch.Tensor:
+    """``h += mult * (sum of at most two sublayer results)`` in place (fp32 ``[T, W]``), then ``h`` over its root mean
+    square, times ``weight`` (one number) when given.  ``split``: ``h`` itself as a sum of two ``dtype`` rows instead,
+    ``[2 T, W]`` (the rounded rows, then the remainders; fp32: ``h`` alone)."""
+    assert h.dtype == torch.float32 and h.is_contiguous() and len(subs) <= 2
+    T, W = h.shape
+    if not h.is_cuda:
+        for s in subs:
+            y = s.y.float().sum(0)
+            if s.gate is not None:
+                z = s.gate.float() * (s.gain.float() if s.gain is not None else 1.0)
+                y = y * torch.sigmoid(z + (s.bias.float() if s.bias is not None else 0.0))
+            h += mult * y
+        return _finish_rows(h, dtype, eps, weight, split)
+    f32 = dtype == torch.float32
+    out = torch.empty(2 * T if split and not f32 else T, W, dtype=dtype, device=h.device)
+    p = _Stream(h=h.data_ptr(), rows=T, W=W, mult=mult, eps=eps, n_sub=len(subs), enter=0,
+                sub=(_Sub * 2)(*[_sub(s, W) for s in subs]), split=int(split),
+                weight=weight.data_ptr() if weight is not None else None, out=out.data_ptr())
+    _lib.check(_lib.get_lib().sb_stream_rows(ctypes.byref(p), int(f32), _lib.stream()), "sb_stream_rows")
+    return out
+
+
+def enter_pass(h: torch.Tensor, mixed: torch.Tensor, base: torch.Tensor, step: torch.Tensor, eps: float) -> torch.Tensor:
+    """``h = mixed + base + step`` in place, then ``h`` over its root mean square in the format of ``step [W]``.
+    ``mixed [S, T or 2 T, W]`` and ``base [S, T, W]``: fp32 partial sums; ``2 T`` rows are the products of the two rows
+    :func:`stream_update` splits ``h`` into."""
+    T, W = h.shape
+    assert mixed.dtype == base.dtype == torch.float32 and mixed.shape[1] in (T, 2 * T) and base.shape[1] == T
+    if not h.is_cuda:
+        m = mixed.sum(0)
+        h.copy_((m[:T] + m[T:] if m.shape[0] == 2 * T and T else m) + base.sum(0) + step.float())
+        return _finish_rows(h, step.dtype, eps, None, False)
+    out = torch.empty(T, W, dtype=step.dtype, device=h.device)
+    p = _Stream(h=h.data_ptr(), rows=T, W=W, mult=1.0, eps=eps, n_sub=2, enter=1,
+                sub=(_Sub * 2)(_sub(Sublayer(mixed), W), _sub(Sublayer(base), W)), step=step.data_ptr(),
+                pair=int(mixed.shape[1] == 2 * T), out=out.data_ptr())
+    _lib.check(_lib.get_lib().sb_stream_rows(ctypes.byref(p), _f32(step), _lib.stream()), "sb_stream_rows")
     return out
 
 

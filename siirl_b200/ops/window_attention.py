@@ -50,10 +50,12 @@ class _Params(ctypes.Structure):
                 ("dv", ctypes.c_int), ("window", ctypes.c_int), ("keep_first", ctypes.c_int),
                 ("scale", ctypes.c_float), ("bias_exp", ctypes.c_float), ("out_scale", ctypes.c_float),
                 ("out", ctypes.c_void_p), ("out_stride", ctypes.c_longlong),
-                ("out_off", ctypes.c_int), ("pad_", ctypes.c_int)]
+                ("out_off", ctypes.c_int), ("kv_mode", ctypes.c_int),
+                ("gain", ctypes.c_void_p), ("gate", ctypes.c_void_p), ("gate_stride", ctypes.c_longlong)]
 
 
-assert ctypes.sizeof(_Params) == 144
+assert ctypes.sizeof(_Params) == 168
+KV_PAGED, KV_PACKED, KV_LATENT = 0, 1, 2
 
 
 class QueryTiles:
@@ -71,17 +73,27 @@ class QueryTiles:
         self.row, self.rows, self.pos, self.slot = flat.split([self.n] * 4) if self.n else (flat,) * 4
 
 
-def _params(spec: WindowSpec, x, seq_ids, positions, block_table, cache, out, out_off) -> _Params:
+def window_params(spec: WindowSpec, x, seq_ids, positions, block_table, cache, out, out_off, *, kv_mode: int = KV_PAGED,
+                  gain: torch.Tensor = None, gate: torch.Tensor = None) -> _Params:
+    """``kv_mode``: where keys and values are.  ``KV_PAGED``: in ``cache`` as described above.  ``KV_PACKED`` (prompts):
+    ``cache`` is ``[rows, kv_heads * (dim + vdim)]``, one row per key, keys before values, and a tile's slot is the row of
+    its sequence's first key.  ``KV_LATENT`` (general kernel): keys and values are the same ``dim``-wide rows of a paged
+    cache.  ``gain``: one number (a tensor) that multiplies the queries and the gate.  ``gate``: columns like ``out``'s whose
+    sigmoid multiplies the result (prompts)."""
     assert x.stride(1) == 1 and out.stride(1) == 1 and cache.dtype == x.dtype == out.dtype
-    assert cache[0].numel() == spec.block_elems and cache.is_contiguous() and block_table.is_contiguous()
+    per_row = spec.kv_heads * (spec.dim + spec.vdim)
+    elems = {KV_PAGED: spec.block_elems, KV_PACKED: per_row, KV_LATENT: BLOCK * spec.dim}[kv_mode]
+    assert cache[0].numel() == elems and cache.is_contiguous() and block_table.is_contiguous()
     assert seq_ids.dtype == positions.dtype == block_table.dtype == torch.int32
     return _Params(x=x.data_ptr(), row_stride=x.stride(0), q_off=spec.q_off, k_off=spec.k_off, v_off=spec.v_off,
                    T=x.shape[0], seq_ids=seq_ids.data_ptr(), positions=positions.data_ptr(),
                    block_table=block_table.data_ptr(), cache=cache.data_ptr(), num_blocks=cache.shape[0],
-                   block_elems=spec.block_elems, max_blocks=block_table.shape[1], Hq=spec.heads, Hkv=spec.kv_heads,
+                   block_elems=elems, max_blocks=block_table.shape[1], Hq=spec.heads, Hkv=spec.kv_heads,
                    dk=spec.dim, dv=spec.vdim, window=spec.window, keep_first=spec.keep_first, scale=spec.scale,
                    bias_exp=spec.bias_exp, out_scale=spec.out_scale, out=out.data_ptr(), out_stride=out.stride(0),
-                   out_off=out_off)
+                   out_off=out_off, kv_mode=kv_mode, gain=gain.data_ptr() if gain is not None else None,
+                   gate=gate.data_ptr() if gate is not None else None,
+                   gate_stride=gate.stride(0) if gate is not None else 0)
 
 
 _workspace: Dict[tuple, Tuple[torch.Tensor, torch.Tensor]] = {}
@@ -96,7 +108,7 @@ def window_attention(spec: WindowSpec, x: torch.Tensor, seq_ids: torch.Tensor, p
     if not x.is_cuda:
         return _cpu(spec, x, seq_ids, positions, block_table, cache, out, out_off)
     L = _lib.get_lib()
-    p = _params(spec, x, seq_ids, positions, block_table, cache, out, out_off)
+    p = window_params(spec, x, seq_ids, positions, block_table, cache, out, out_off)
     ref = ctypes.byref(p)
     f32 = int(x.dtype == torch.float32)
     _lib.check(L.sb_kv_append_split(ref, f32, _lib.stream()), "sb_kv_append_split")
