@@ -57,8 +57,9 @@ def parse_args():
                     help="library: the same step through vLLM + transformers + flash-attn + torch AdamW (1 GPU), a bar "
                          "on this box that is not the reference")
     ap.add_argument("--workload", default="grpo", choices=["grpo", "serve"],
-                    help="serve: prefill and decode throughput of a hybrid decoder (Domavik) beside the closest uniform "
-                         "decoder of equal size (1 GPU; benchmarks/hybrid_serving.py)")
+                    help="serve: prefill and decode throughput of a hybrid decoder beside the closest decoder of equal size "
+                         "(1 GPU; benchmarks/hybrid_serving.py)")
+    ap.add_argument("--design", default="domavik", choices=["domavik", "poralorn"], help="hybrid decoder of --workload serve")
     ap.add_argument("--budget-s", type=float, default=600.0,
                     help="wall-clock budget of the whole run, from process start; --steps/--warmup are upper bounds")
     ap.add_argument("--model", default="qwen2.5-7b")
@@ -196,10 +197,10 @@ def build_config(args, world: int):
 def main() -> int:
     args = parse_args()
     if args.workload == "serve":
-        from siirl_b200.benchmarks.hybrid_serving import SIZES, serve
+        from siirl_b200.benchmarks.hybrid_serving import serve
         sampler = ClockSampler(0)
         sampler.start()
-        res = serve(list(SIZES))
+        res = serve(args.design)
         res["clocks"] = sampler.stop()
         print(json.dumps(res), flush=True)
         return 0

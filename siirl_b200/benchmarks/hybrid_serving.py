@@ -1,8 +1,8 @@
-"""Serving throughput of a hybrid decoder (Domavik) beside the closest uniform decoder of equal size, and its kernels
+"""Serving throughput of a hybrid decoder (Domavik, Poralorn) beside the closest decoder of equal size, and its kernels
 beside the like kernels of that model.
 
-    python bench.py --workload serve                       # end to end, a few sizes
-    python -m siirl_b200.benchmarks.hybrid_serving --kernels
+    python bench.py --workload serve [--design poralorn]                     # end to end, a few sizes
+    python -m siirl_b200.benchmarks.hybrid_serving [--design poralorn] --kernels
 
 End to end: random weights, the rollout engine's own prefill pass and CUDA-graph decode rounds, CUDA events on the
 launching stream.  Weights and caches are larger than L2 in every case.  Kernels: each alone, L2 flushed between
@@ -22,9 +22,11 @@ from ..models.config import DecoderConfig, get_config
 from ..models.decoder import build_model
 from ..ops import lib
 
-SIZES = {     # preset, layers, (prompts, tokens) of a prefill pass, (sequences, context) of a decode step
-    "1.5b": ("domavik-1.5b", 14, [(8, 1024), (1, 8192)], [(32, 2048), (256, 1024)]),
-    "7b": ("domavik-7b", 8, [(8, 1024), (1, 8192)], [(32, 2048), (256, 1024)]),
+SIZES = {     # design -> size: preset, layers, (prompts, tokens) of a prefill pass, (sequences, context) of a decode step
+    "domavik": {"1.5b": ("domavik-1.5b", 14, [(8, 1024), (1, 8192)], [(32, 2048), (256, 1024)]),
+                "7b": ("domavik-7b", 8, [(8, 1024), (1, 8192)], [(32, 2048), (256, 1024)])},
+    "poralorn": {"1.5b": ("poralorn-1.5b", 14, [(8, 1024), (1, 8192)], [(32, 2048), (256, 1024)]),
+                 "7b": ("poralorn-7b", 8, [(8, 1024), (1, 8192)], [(32, 2048), (256, 1024)])},
 }
 
 
@@ -39,11 +41,23 @@ def peaks() -> Dict[str, float]:
 
 
 def closest(cfg: DecoderConfig) -> DecoderConfig:
-    """The uniform decoder of the same width, feed-forward, depth, vocabulary and attention heads."""
+    """The uniform decoder of the same width, feed-forward, number of layer runs, vocabulary and attention heads (seven
+    query heads, or six, per key-value head where the design shares one latent between all)."""
     b = cfg.hybrid.attention[0]
+    kv = b.kv_heads or b.heads // (7 if b.heads % 7 == 0 else 6)
     return DecoderConfig(model_type="qwen2", vocab_size=cfg.vocab_size, hidden_size=cfg.hidden_size,
-                         intermediate_size=cfg.intermediate_size, num_layers=cfg.num_layers, num_heads=b.heads,
-                         num_kv_heads=b.kv_heads, head_dim=b.dim, rope_theta=1e6, eos_token_id=2)
+                         intermediate_size=cfg.intermediate_size, num_layers=len(cfg.hybrid.runs()), num_heads=b.heads,
+                         num_kv_heads=kv, head_dim=b.dim, rope_theta=1e6, eos_token_id=2)
+
+
+def closest_latent(cfg: DecoderConfig) -> DecoderConfig:
+    """The dense multi-head-latent-attention decoder of the same sizes (with a 64-wide rotary part)."""
+    b = cfg.hybrid.attention[0]
+    n = len(cfg.hybrid.runs())
+    return DecoderConfig(model_type="deepseek_v3", vocab_size=cfg.vocab_size, hidden_size=cfg.hidden_size,
+                         intermediate_size=cfg.intermediate_size, num_layers=n, num_heads=b.heads, num_kv_heads=b.heads,
+                         head_dim=b.dim + 64, qkv_bias=False, kv_lora_rank=b.kv_rank, qk_nope_head_dim=b.dim,
+                         qk_rope_head_dim=64, v_head_dim=b.vdim, first_k_dense_replace=n, eos_token_id=2)
 
 
 def _events(fn: Callable[[], None], warmup: int, iters: int, flush=None) -> float:
@@ -113,42 +127,165 @@ def serve_one(cfg: DecoderConfig, prefill, decode, iters: int) -> dict:
     return out
 
 
-def serve(sizes, iters: int = 5) -> dict:
+def serve_latent(cfg: DecoderConfig, prefill, decode, iters: int) -> dict:
+    """The same measurements through the latent-cache engine."""
+    from ..engine.rollout.latent_engine import LatentCacheEngine
+    model = build_model(cfg, dtype=torch.bfloat16, device="cuda", seed=0)
+    for p in model.parameters():
+        p.requires_grad_(False)
+    out = {"parameters": cfg.num_parameters(), "prefill": [], "decode": []}
+    g = torch.Generator().manual_seed(0)
+    for n, length in prefill:
+        eng = LatentCacheEngine(model, max_num_seqs=n, max_model_len=length + 64)
+        eng.wake_up()
+        toks = [torch.randint(3, cfg.vocab_size, (length,), generator=g).tolist() for _ in range(n)]
+        ms = _events(lambda: eng._prefill(toks, list(range(n)), None), 3, iters)
+        out["prefill"].append({"prompts": n, "tokens": length, "ms": round(ms, 3),
+                               "tokens_per_s": round(n * length / ms * 1e3)})
+        eng.sleep()
+    for n, ctx in decode:
+        eng = LatentCacheEngine(model, max_num_seqs=n, max_model_len=ctx + 64)
+        eng.wake_up()
+        tok = torch.randint(3, cfg.vocab_size, (n,), generator=g).cuda()
+        slots, lens = torch.arange(n, device="cuda"), torch.full((n,), ctx, dtype=torch.int64, device="cuda")
+        ms = _events(lambda: eng._logits(eng._decode(tok, slots, lens, ctx, True)), 3, iters)
+        out["decode"].append({"sequences": n, "context": ctx, "ms_per_step": round(ms, 4),
+                              "tokens_per_s": round(n / ms * 1e3)})
+        eng.sleep()
+    lib.check_status()
+    del model
+    torch.cuda.empty_cache()
+    return out
+
+
+def serve(design: str = "domavik", sizes=None, iters: int = 5) -> dict:
     res = {"metric": "serving_tokens_per_second", "data": "synthetic", "dtype": "bf16", "sizes": {}}
-    for name in sizes:
-        preset, layers, prefill, decode = SIZES[name]
+    for name in sizes or SIZES[design]:
+        preset, layers, prefill, decode = SIZES[design][name]
         cfg = copy.deepcopy(get_config(preset))
         cfg.hybrid.layers = cfg.hybrid.layers[:layers]
         cfg.num_layers = layers
-        res["sizes"][name] = {"hybrid": preset, "layers": layers,
-                              "domavik": serve_one(cfg, prefill, decode, iters),
+        res["sizes"][name] = {"hybrid": preset, "layers": layers, "layer_runs": len(cfg.hybrid.runs()),
+                              design: serve_one(cfg, prefill, decode, iters),
                               "closest (uniform attention)": serve_one(closest(cfg), prefill, decode, iters)}
+        if design == "poralorn":
+            res["sizes"][name]["closest (multi-head latent attention)"] = serve_latent(closest_latent(cfg), prefill, decode,
+                                                                                       iters)
     return res
 
 
 # ---- kernels ----------------------------------------------------------------------------------------------------------------
-def kernels(only: str = "", iters: int = 20) -> dict:
+class _Bench:
+    def __init__(self, only: str, iters: int):
+        self.only, self.iters, self.pk, self.rows = only, iters, peaks(), []
+        self.flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+
+    def add(self, name, fn, flops=0.0, nbytes=0.0):
+        if self.only and self.only not in name:
+            return
+        ms = _events(fn, 3, self.iters, self.flush)
+        ideal = max(flops / (self.pk["tflops"] * 1e9), nbytes / (self.pk["gbs"] * 1e6))
+        self.rows.append({"kernel": name, "us": round(ms * 1e3, 1), "roofline_us": round(ideal * 1e3, 1),
+                          "of_roofline": round(ideal / ms, 3)})
+
+    def result(self):
+        torch.cuda.synchronize()
+        lib.check_status()
+        return {"peaks": self.pk, "kernels": self.rows}
+
+
+def _rnd(*s):
+    return (torch.randn(*s, device="cuda") * 0.5).bfloat16()
+
+
+def kernels(design: str = "domavik", only: str = "", iters: int = 20) -> dict:
+    b = _Bench(only, iters)
+    (_kernels_poralorn if design == "poralorn" else _kernels_domavik)(b)
+    return b.result()
+
+
+def _kernels_poralorn(b: _Bench) -> None:
+    """Latent attention with 28 heads of width 128 over 512-wide latents, and the row operations of its layers."""
+    from ..ops import dense, kv_cache
+    from ..ops import latent_attention as LA
+    from ..ops import rows as R
+    from ..ops.attention import SeqInfo, attention_packed
+    dev, add, rnd = torch.device("cuda"), b.add, _rnd
+    H, G, D, rank = 28, 4, 128, 512
+    hd = H * D
+    spec = LA.LatentSpec(H, D, D, rank, 0, hd, hd + rank, D ** -0.5, 1e-5)
+    w = {"c_norm": rnd(rank), "kv_up": rnd(2 * hd, rank) * 0.1, "gain": torch.ones((), device=dev).bfloat16()}
+    width = 2 * hd + rank
+    for n, L in ((8, 1024), (1, 8192)):
+        T, nb = n * L, L // 64
+        x, q = rnd(T, width), rnd(T, (H + 2 * G) * D)
+        info = SeqInfo([L] * n, device=dev)
+        flops = n * 4 * D * H * L * (L + 1) / 2
+        table = torch.randperm(n * nb, device=dev).to(torch.int32).view(n, nb)
+        cache = torch.zeros(n * nb, 64 * rank, dtype=torch.bfloat16, device=dev)
+        out = torch.empty(T, hd, dtype=torch.bfloat16, device=dev)
+        ids = torch.repeat_interleave(torch.arange(n, dtype=torch.int32), L).to(dev)
+        pos = torch.arange(L, dtype=torch.int32).repeat(n).to(dev)
+        plan = LA.LatentPlan([L] * n, [0] * n, list(range(n)), dev)
+        kv = dense.linear(rnd(T, rank), w["kv_up"])
+        add(f"uniform: fmha_fwd {n}x{L}", lambda: attention_packed(q, info, H, G, D), flops)
+        add(f"poralorn: attention over expanded keys, gated {n}x{L}",
+            lambda: LA.expanded_attention(spec, x, w["gain"], kv, ids, pos, table, out, 0, plan), flops)
+        add(f"poralorn: latent append {n}x{L}", lambda: LA.latent_append(spec, x, w, ids, pos, table, cache, plan),
+            nbytes=T * rank * 6)
+        add(f"poralorn: whole latent attention {n}x{L} (append, expansion, attention)",
+            lambda: LA.latent_attention(spec, x, w, ids, pos, table, cache, out, 0, plan=plan),
+            flops + T * 4.0 * hd * rank)
+    for B, ctx in ((32, 2048), (256, 1024)):
+        nb = (ctx + 63) // 64
+        table = torch.randperm(B * nb, device=dev).to(torch.int32).view(B, nb)
+        lens = torch.full((B,), ctx, dtype=torch.int32, device=dev)
+        q, kvc = rnd(B, (H + 2 * G) * D), torch.zeros(B * nb, 2, G, 64, D, dtype=torch.bfloat16, device=dev)
+        add(f"uniform: decode attention {B}x{ctx}", lambda: kv_cache.decode_attention(q, kvc, lens, table, H, G, D),
+            nbytes=B * ctx * 2 * G * D * 2)
+        cache = (torch.randn(B * nb, 64 * rank, device=dev) * 0.1).bfloat16()
+        x, out = rnd(B, width), torch.empty(B, hd, dtype=torch.bfloat16, device=dev)
+        ids, pos = torch.arange(B, dtype=torch.int32, device=dev), lens - 1
+        qa, mixed = rnd(B, H * rank), torch.empty(B, H * rank, dtype=torch.bfloat16, device=dev)
+        act = B * H * (D + rank) * 2
+        add(f"poralorn: absorbed attention {B}x{ctx}",
+            lambda: LA.absorbed_attention(spec, x, w, qa, ids, pos, table, cache, mixed),
+            nbytes=B * ctx * rank * 2 + 2 * B * H * rank * 2, flops=B * ctx * H * rank * 4.0)
+        add(f"poralorn: query absorption {B}", lambda: LA.head_product(x, D, w["kv_up"][:hd], H, qa, by_rows=True),
+            nbytes=hd * rank * 2 + act)
+        add(f"poralorn: value expansion, gated {B}",
+            lambda: LA.head_product(mixed, rank, w["kv_up"][hd:], H, out, by_rows=False, gate=x[:, hd + rank:],
+                                    gain=w["gain"]), nbytes=hd * rank * 2 + act + B * hd * 2)
+        add(f"poralorn: whole latent attention {B}x{ctx} (append, absorption, attention, expansion)",
+            lambda: LA.latent_attention(spec, x, w, ids, pos, table, cache, out, 0),
+            nbytes=B * ctx * rank * 2 + 2 * hd * rank * 2 + 2 * act, flops=B * ctx * H * rank * 4.0)
+    for T in (256, 8192):
+        W, I = 3584, 18944
+        h, p = torch.randn(T, W, device=dev), rnd(T, 2 * W)
+        bias, one, step = rnd(W), w["gain"], rnd(W)
+        d, res, wt = rnd(T, W), rnd(T, W), rnd(W)
+        add(f"uniform: residual + RMS norm {T}x{W} (bf16 stream)", lambda: dense.rmsnorm(d, wt, 1e-6, residual=res),
+            nbytes=T * W * 8)
+        subs = [R.Sublayer(rnd(1, T, W), p[:, :W], bias, one), R.Sublayer(rnd(1, T, W), p[:, W:], bias, one)]
+        add(f"poralorn: gated residual + norm {T}x{W} (fp32 stream)",
+            lambda: R.stream_update(h, subs, 0.5, torch.bfloat16, 1e-5), nbytes=T * W * 18)
+        add(f"poralorn: gated residual, split {T}x{W}",
+            lambda: R.stream_update(h, subs, 0.5, torch.bfloat16, 1e-5, split=True), nbytes=T * W * 20)
+        mixed, base = torch.randn(1, 2 * T, W, device=dev), torch.randn(1, T, W, device=dev)
+        add(f"poralorn: entry of a pass + norm {T}x{W}", lambda: R.enter_pass(h, mixed, base, step, 1e-5),
+            nbytes=T * W * 18)
+        gu = rnd(T, 2 * I)
+        add(f"uniform: swiglu {T}x{I}", lambda: dense.swiglu(gu), nbytes=T * I * 6)
+        add(f"poralorn: exact GELU {T}x{I}", lambda: R.scaled_act(gu[:, :I], "gelu", one), nbytes=T * I * 4)
+
+
+def _kernels_domavik(b: _Bench) -> None:
     from ..ops import dense, kv_cache
     from ..ops import rows as R
     from ..ops.attention import SeqInfo, attention_packed
     from ..ops.recurrence import PortionPlan, RecurrenceSpec, empty_state, recurrence_decode, recurrence_prefill
     from ..ops.window_attention import QueryTiles, WindowSpec, window_attention
-    dev = torch.device("cuda")
-    pk = peaks()
-    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
-    rows: List[dict] = []
-
-    def add(name, fn, flops=0.0, nbytes=0.0):
-        if only and only not in name:
-            return
-        ms = _events(fn, 3, iters, flush)
-        ideal = max(flops / (pk["tflops"] * 1e9), nbytes / (pk["gbs"] * 1e6))
-        rows.append({"kernel": name, "us": round(ms * 1e3, 1), "roofline_us": round(ideal * 1e3, 1),
-                     "of_roofline": round(ideal / ms, 3)})
-
-    def rnd(*s):
-        return (torch.randn(*s, device=dev) * 0.5).bfloat16()
-
+    dev, add, rnd = torch.device("cuda"), b.add, _rnd
     # attention on prompts: 28 heads, 4 kv heads, width 128
     H, G, D = 28, 4, 128
     for n, L in ((8, 1024), (1, 8192)):
@@ -233,9 +370,6 @@ def kernels(only: str = "", iters: int = 20) -> dict:
         if T == 256:
             z = torch.randn(T, V, device=dev)
             add(f"domavik: soft cap {T}x{V}", lambda: R.softcap_(z, 30.0), nbytes=T * V * 8)
-    torch.cuda.synchronize()
-    lib.check_status()
-    return {"peaks": pk, "kernels": rows}
 
 
 def main(argv=None) -> int:
@@ -243,9 +377,11 @@ def main(argv=None) -> int:
     ap.add_argument("--kernels", action="store_true")
     ap.add_argument("--only", default="", help="kernels whose name contains this")
     ap.add_argument("--iters", type=int, default=20)
-    ap.add_argument("--sizes", default=",".join(SIZES))
+    ap.add_argument("--design", choices=list(SIZES), default="domavik")
+    ap.add_argument("--sizes", default="", help="comma separated, default all of the design")
     args = ap.parse_args(argv)
-    res = kernels(args.only, args.iters) if args.kernels else serve(args.sizes.split(","))
+    res = kernels(args.design, args.only, args.iters) if args.kernels else serve(
+        args.design, args.sizes.split(",") if args.sizes else None)
     print(json.dumps(res), flush=True)
     return 0
 

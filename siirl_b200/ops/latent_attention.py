@@ -134,6 +134,57 @@ def _latent_params(spec: LatentSpec, x, w, seq_ids, positions, block_table, cach
                    out=out.data_ptr() if out is not None else None)
 
 
+def latent_append(spec: LatentSpec, x, w, seq_ids, positions, block_table, cache, plan: Optional[LatentPlan] = None):
+    """Norm the rows' latents and append them to the cache.  With a ``plan`` returns the latents of every visible position
+    ``[plan.keys, rank]``, sequence after sequence (portions behind a prefix read theirs back from the cache)."""
+    L, f32 = _lib.get_lib(), int(x.dtype == torch.float32)
+    p = _latent_params(spec, x, w, seq_ids, positions, block_table, cache)
+    rows = torch.empty(plan.keys, spec.rank, dtype=x.dtype, device=x.device) if plan is not None else None
+    _lib.check(L.sb_latent_append(ctypes.byref(p), _lib.ptr(rows if plan is not None and not plan.prefix else None), f32,
+                                  _lib.stream()), "sb_latent_append")
+    if plan is not None and plan.prefix:
+        _lib.check(L.sb_latent_gather(ctypes.byref(p), _lib.ptr(plan.key_slot), _lib.ptr(plan.key_pos), _lib.ptr(rows),
+                                      plan.keys, f32, _lib.stream()), "sb_latent_gather")
+    return rows
+
+
+def expanded_attention(spec: LatentSpec, x, gain, kv, seq_ids, positions, block_table, out, out_off, plan: LatentPlan) -> None:
+    """Multi-head attention of prompt portions over expanded keys and values ``kv [plan.keys, heads * (dim + vdim)]``."""
+    H = spec.heads
+    ws = WindowSpec(H, H, spec.dim, spec.vdim, spec.q_off, 0, H * spec.dim, spec.scale)
+    q = window_params(ws, x, seq_ids, positions, block_table, kv, out, out_off, kv_mode=KV_PACKED, gain=gain,
+                      gate=x[:, spec.g_off:] if spec.g_off >= 0 else None)
+    t = plan.tiles
+    _lib.check(_lib.get_lib().sb_attn_window_prefill(
+        ctypes.byref(q), _lib.ptr(t.row), _lib.ptr(t.rows), _lib.ptr(t.pos), _lib.ptr(t.slot), t.n,
+        _lib.ptr(_lib.status_word(x.device)), _lib.stream()), "sb_attn_window_prefill")
+
+
+def absorbed_attention(spec: LatentSpec, x, w, qa, seq_ids, positions, block_table, cache, mixed, *,
+                       simt: bool = False) -> None:
+    """Absorbed queries ``qa [T, heads * rank]`` against the cached latents: row ``t`` sees positions up to its own;
+    ``mixed [T, heads * rank]`` receives the weighted sums (zero where ``seq_ids[t] < 0``)."""
+    L, (T, _), H, R = _lib.get_lib(), qa.shape, spec.heads, spec.rank
+    groups = 0 if simt else int(L._cdll.sb_latent_decode_groups(H, R))
+    if not groups:
+        ws = WindowSpec(H, 1, R, R, 0, 0, 0, spec.scale)
+        q = window_params(ws, qa, seq_ids, positions, block_table, cache, mixed, 0, kv_mode=KV_LATENT, gain=w.get("gain"))
+        _lib.check(L.sb_attn_window_simt(ctypes.byref(q), int(qa.dtype == torch.float32), _lib.stream()),
+                   "sb_attn_window_simt")
+        return
+    ws = _workspace.get((x.device, H, R))
+    if ws is None:      # allocated on first use, before a CUDA graph captures the launch
+        per = 2 * int(L._cdll.sb_latent_decode_grid()) * (((H + groups - 1) // groups + 15) // 16 * 16)
+        ws = _workspace[(x.device, H, R)] = (
+            torch.empty(per * R, dtype=torch.float32, device=x.device),
+            torch.empty(per + DECODE_ROWS + 1, dtype=torch.float32, device=x.device))
+    for s in range(0, T, DECODE_ROWS):
+        e = min(s + DECODE_ROWS, T)
+        d = _latent_params(spec, x[s:e], w, seq_ids[s:e], positions[s:e], block_table, cache, qa[s:e], mixed[s:e])
+        _lib.check(L.sb_latent_decode(ctypes.byref(d), _lib.ptr(ws[0]), _lib.ptr(ws[1]),
+                                      _lib.ptr(_lib.status_word(x.device)), _lib.stream()), "sb_latent_decode")
+
+
 def latent_attention(spec: LatentSpec, x: torch.Tensor, w: Dict[str, torch.Tensor], seq_ids: torch.Tensor,
                      positions: torch.Tensor, block_table: torch.Tensor, cache: torch.Tensor, out: torch.Tensor,
                      out_off: int, *, plan: Optional[LatentPlan] = None, simt: bool = False) -> None:
@@ -143,58 +194,25 @@ def latent_attention(spec: LatentSpec, x: torch.Tensor, w: Dict[str, torch.Tenso
     forces the general kernels."""
     if not x.is_cuda:
         return _cpu(spec, x, w, seq_ids, positions, block_table, cache, out, out_off)
-    T, H, R = x.shape[0], spec.heads, spec.rank
+    T, H, R, hk, hv = x.shape[0], spec.heads, spec.rank, spec.heads * spec.dim, spec.heads * spec.vdim
     assert x.stride(1) == 1 and out.stride(1) == 1 and cache.dtype == x.dtype == out.dtype == w["kv_up"].dtype
     assert cache[0].numel() == spec.block_elems and cache.is_contiguous() and block_table.is_contiguous()
     assert seq_ids.dtype == positions.dtype == block_table.dtype == torch.int32
-    L, stream, f32 = _lib.get_lib(), _lib.stream(), int(x.dtype == torch.float32)
-    status = _lib.ptr(_lib.status_word(x.device))
+    tensor = x.dtype == torch.bfloat16 and not simt and spec.aligned and x.stride(0) % 8 == 0 and \
+        out.stride(0) % 8 == 0 and out_off % 8 == 0
     gain = w.get("gain")
-    hk, hv = H * spec.dim, H * spec.vdim
-    tensor = not f32 and not simt and spec.aligned and x.stride(0) % 8 == 0 and out.stride(0) % 8 == 0 and \
-        out_off % 8 == 0
-    expand = tensor and plan is not None and not plan.short
-    p = _latent_params(spec, x, w, seq_ids, positions, block_table, cache)
-    rows = torch.empty(plan.keys, R, dtype=x.dtype, device=x.device) if expand else None
-    _lib.check(L.sb_latent_append(ctypes.byref(p), _lib.ptr(rows if expand and not plan.prefix else None), f32, stream),
-               "sb_latent_append")
-    gate = x[:, spec.g_off:] if spec.g_off >= 0 else None
-    if expand:
-        if plan.prefix:
-            _lib.check(L.sb_latent_gather(ctypes.byref(p), _lib.ptr(plan.key_slot), _lib.ptr(plan.key_pos),
-                                          _lib.ptr(rows), plan.keys, f32, stream), "sb_latent_gather")
-        kv = linear(rows, w["kv_up"])
-        ws = WindowSpec(H, H, spec.dim, spec.vdim, spec.q_off, 0, hk, spec.scale)
-        q = window_params(ws, x, seq_ids, positions, block_table, kv, out, out_off, kv_mode=KV_PACKED, gain=gain,
-                          gate=gate)
-        t = plan.tiles
-        _lib.check(L.sb_attn_window_prefill(ctypes.byref(q), _lib.ptr(t.row), _lib.ptr(t.rows), _lib.ptr(t.pos),
-                                            _lib.ptr(t.slot), t.n, status, stream), "sb_attn_window_prefill")
+    if tensor and plan is not None and not plan.short:
+        rows = latent_append(spec, x, w, seq_ids, positions, block_table, cache, plan)
+        expanded_attention(spec, x, gain, linear(rows, w["kv_up"]), seq_ids, positions, block_table, out, out_off, plan)
         return
     # absorbed: queries against the latents, the weighted latents through the value matrices
+    latent_append(spec, x, w, seq_ids, positions, block_table, cache)
     qa = torch.empty(T, H * R, dtype=x.dtype, device=x.device)
     mixed = torch.empty_like(qa)
     head_product(x[:, spec.q_off:], spec.dim, w["kv_up"][:hk], H, qa, by_rows=True, simt=not tensor)
-    groups = int(L._cdll.sb_latent_decode_groups(H, R)) if tensor else 0
-    if groups > 0:
-        grid = int(L._cdll.sb_latent_decode_grid())
-        key = (x.device, H, R)
-        ws = _workspace.get(key)
-        if ws is None:      # allocated on first use, before a CUDA graph captures the launch
-            per = 2 * grid * (((H + groups - 1) // groups + 15) // 16 * 16)
-            ws = _workspace[key] = (torch.empty(per * R, dtype=torch.float32, device=x.device),
-                                    torch.empty(per + DECODE_ROWS + 1, dtype=torch.float32, device=x.device))
-        for s in range(0, T, DECODE_ROWS):
-            e = min(s + DECODE_ROWS, T)
-            d = _latent_params(spec, x[s:e], w, seq_ids[s:e], positions[s:e], block_table, cache, qa[s:e], mixed[s:e])
-            _lib.check(L.sb_latent_decode(ctypes.byref(d), _lib.ptr(ws[0]), _lib.ptr(ws[1]), status, stream),
-                       "sb_latent_decode")
-    else:
-        ws = WindowSpec(H, 1, R, R, 0, 0, 0, spec.scale)
-        q = window_params(ws, qa, seq_ids, positions, block_table, cache, mixed, 0, kv_mode=KV_LATENT, gain=gain)
-        _lib.check(L.sb_attn_window_simt(ctypes.byref(q), f32, stream), "sb_attn_window_simt")
-    head_product(mixed, R, w["kv_up"][hk:], H, out[:, out_off:out_off + hv], by_rows=False, gate=gate, gain=gain,
-                 simt=not tensor)
+    absorbed_attention(spec, x, w, qa, seq_ids, positions, block_table, cache, mixed, simt=not tensor)
+    head_product(mixed, R, w["kv_up"][hk:], H, out[:, out_off:out_off + hv], by_rows=False, gain=gain,
+                 gate=x[:, spec.g_off:] if spec.g_off >= 0 else None, simt=not tensor)
 
 
 def _cpu(spec: LatentSpec, x, w, seq_ids, positions, block_table, cache, out, out_off) -> None:
