@@ -13,18 +13,24 @@
 
 namespace sb {
 
-constexpr int kHpStages = 3;
 constexpr int kHpBytes = 128 * 64 * 2;     // one operand tile of a stage: 128 rows or columns x 64 of the contraction
-constexpr int kHpBarOff = kHpStages * 2 * kHpBytes;
-constexpr int kHpSmem = kHpBarOff + (2 * kHpStages + 1) * 8 + 16 + 1024;
+
+// few wide tiles with a short contraction (queries) keep two CTAs on an SM; a long contraction gets a deep ring
+template <bool B_MN>
+struct HpSmem {
+  static constexpr int kStages = B_MN ? 3 : 6;
+  static constexpr int kBarOff = kStages * 2 * kHpBytes;
+  static constexpr int kTotal = kBarOff + (2 * kStages + 1) * 8 + 16 + 1024;
+};
 
 template <bool B_MN>
 __global__ void __launch_bounds__(192)
 head_product_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b, HeadProduct p,
                     int* status) {
+  constexpr int kHpStages = HpSmem<B_MN>::kStages;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  uint64_t* full = reinterpret_cast<uint64_t*>(smem + kHpBarOff);
+  uint64_t* full = reinterpret_cast<uint64_t*>(smem + HpSmem<B_MN>::kBarOff);
   uint64_t* empty = full + kHpStages;
   uint64_t* done = empty + kHpStages;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(done + 1);
@@ -97,30 +103,38 @@ head_product_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
     __syncwarp();
   } else {
     const int quarter = warp & 3, row = m0 + quarter * 32 + lane;
+    const bool valid = row < p.T;
+    const long long col0 = (long long)h * N + n0;
+    const float gain = p.gain ? __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(p.gain)) : 1.f;
+    // the gate's row is fetched while the product runs
+    uint4 g[16];
+    const __nv_bfloat16* gate = reinterpret_cast<const __nv_bfloat16*>(p.gate) + (long long)(valid ? row : 0) * p.gate_row + col0;
+#pragma unroll
+    for (int v = 0; v < 16; ++v)
+      if (p.gate && valid && n0 + v * 8 < N) g[v] = *reinterpret_cast<const uint4*>(gate + v * 8);
     if (__all_sync(0xffffffffu, mbar_wait(done, 0, status, kStatusTimeoutEpilogue))) {
       tc_fence_after();
-      const float gain = p.gain ? __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(p.gain)) : 1.f;
-      const bool valid = row < p.T;
-      const long long col0 = (long long)h * N + n0;
       __nv_bfloat16* c = reinterpret_cast<__nv_bfloat16*>(p.c) + (long long)(valid ? row : 0) * p.c_row + col0;
-      const __nv_bfloat16* g = reinterpret_cast<const __nv_bfloat16*>(p.gate) + (long long)(valid ? row : 0) * p.gate_row + col0;
-#pragma unroll 1
-      for (int q = 0; q < 4 && n0 + q * 32 < N; ++q) {
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        if (n0 + q * 32 >= N) break;
         uint32_t r[32];
         tmem_ld_32x32(tmem + ((uint32_t)(quarter * 32) << 16) + q * 32, r);
         tmem_ld_wait();
-        if (!valid) continue;
 #pragma unroll
         for (int v = 0; v < 4; ++v) {
-          if (n0 + q * 32 + v * 8 >= N) break;
+          if (!valid || n0 + q * 32 + v * 8 >= N) break;
           float o[8];
 #pragma unroll
           for (int i = 0; i < 8; ++i) o[i] = __uint_as_float(r[v * 8 + i]);
           if (p.gate) {
-            float z[8];
-            load_vec<__nv_bfloat16, 8>(g + q * 32 + v * 8, z);
+            const __nv_bfloat162* z2 = reinterpret_cast<const __nv_bfloat162*>(&g[q * 4 + v]);
 #pragma unroll
-            for (int i = 0; i < 8; ++i) o[i] /= 1.f + __expf(-gain * z[i]);
+            for (int i = 0; i < 4; ++i) {
+              const float2 z = __bfloat1622float2(z2[i]);
+              o[2 * i] /= 1.f + __expf(-gain * z.x);
+              o[2 * i + 1] /= 1.f + __expf(-gain * z.y);
+            }
           }
           store_vec<__nv_bfloat16, 8>(c + q * 32 + v * 8, o);
         }
@@ -228,14 +242,16 @@ extern "C" int sb_head_product(const void* params, int* status, cudaStream_t str
   if (r) return r;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(head_product_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kHpSmem);
+    cudaError_t e = cudaFuncSetAttribute(head_product_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                         HpSmem<true>::kTotal);
     if (e == cudaSuccess)
-      e = cudaFuncSetAttribute(head_product_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kHpSmem);
+      e = cudaFuncSetAttribute(head_product_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                               HpSmem<false>::kTotal);
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
   const dim3 grid((N + 127) / 128, p.H, (p.T + 127) / 128);
-  if (p.b_mn) head_product_kernel<true><<<grid, 192, kHpSmem, stream>>>(ma, mb, p, status);
-  else head_product_kernel<false><<<grid, 192, kHpSmem, stream>>>(ma, mb, p, status);
+  if (p.b_mn) head_product_kernel<true><<<grid, 192, HpSmem<true>::kTotal, stream>>>(ma, mb, p, status);
+  else head_product_kernel<false><<<grid, 192, HpSmem<false>::kTotal, stream>>>(ma, mb, p, status);
   return (int)cudaGetLastError();
 }

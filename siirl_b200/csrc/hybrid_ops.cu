@@ -118,11 +118,32 @@ __device__ __forceinline__ float gelu_tanh_f(float z) {
   return 0.5f * z * (1.f + tanhf(u));
 }
 
-template <int ACT>      // 0 SiLU, 1 tanh-form GELU, 2 exact GELU
+// z Phi(z) with the normal distribution function from formula 7.1.26 of Abramowitz and Stegun, Handbook of Mathematical
+// Functions (|error of erf| <= 1.5e-7), evaluated on the side where nothing cancels: for results that are rounded to 16 bits
+__device__ __forceinline__ float gelu_erf_fast(float z) {
+  const float x = fabsf(z) * 0.7071067811865476f;
+  const float t = __fdividef(1.f, fmaf(0.3275911f, x, 1.f));
+  float q = fmaf(1.061405429f, t, -1.453152027f);
+  q = fmaf(q, t, 1.421413741f);
+  q = fmaf(q, t, -0.284496736f);
+  q = fmaf(q, t, 0.254829592f);
+  q *= 0.5f * t * __expf(-x * x);       // Phi(-|z|)
+  return z * (z < 0.f ? q : 1.f - q);
+}
+
+template <int ACT, typename T>      // 0 SiLU, 1 tanh-form GELU, 2 exact GELU; T: the format of the result
 __device__ __forceinline__ float activate(float z) {
   if constexpr (ACT == 1) return gelu_tanh_f(z);
+  if constexpr (ACT == 2 && sizeof(T) == 2) return gelu_erf_fast(z);
   if constexpr (ACT == 2) return 0.5f * z * (1.f + erff(z * 0.7071067811865476f));
   return z / (1.f + __expf(-z));
+}
+
+// sigmoid of a gate whose product is added to a 32-bit stream (T = float: every step in full precision)
+template <typename T>
+__device__ __forceinline__ float gate_sigmoid(float z) {
+  if constexpr (sizeof(T) == 2) return __fdividef(1.f, 1.f + __expf(-z));
+  return 1.f / (1.f + expf(-z));
 }
 
 template <typename T, int V, int ACT>
@@ -136,7 +157,7 @@ __global__ void gated_act_kernel(const T* __restrict__ gu, T* __restrict__ out, 
     load_vec<T, V>(gu + t * 2 * I + c, g);
     load_vec<T, V>(gu + t * 2 * I + I + c, u);
 #pragma unroll
-    for (int k = 0; k < V; ++k) g[k] = activate<ACT>(g[k]) * u[k];
+    for (int k = 0; k < V; ++k) g[k] = activate<ACT, T>(g[k]) * u[k];
     store_vec<T, V>(out + t * I + c, g);
   }
 }
@@ -144,17 +165,23 @@ __global__ void gated_act_kernel(const T* __restrict__ gu, T* __restrict__ out, 
 template <typename T, int V, int ACT>
 __global__ void scaled_act_kernel(const T* __restrict__ x, long long stride, const T* __restrict__ gain, T* __restrict__ out,
                                   long long rows, int I) {
-  const int nv = I / V;
-  const long long total = rows * nv;
+  // a thread keeps its columns and walks down the rows, four loads in flight
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
+  if (c >= I) return;
   const float f = gain ? to_float(*gain) : 1.f;
-  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
-    const long long t = i / nv;
-    const int c = (int)(i % nv) * V;
-    float v[V];
-    load_vec<T, V>(x + t * stride + c, v);
+  const long long step = gridDim.y;
+  for (long long t = blockIdx.y; t < rows; t += 4 * step) {
+    float v[4][V];
 #pragma unroll
-    for (int k = 0; k < V; ++k) v[k] = activate<ACT>(f * v[k]);
-    store_vec<T, V>(out + t * I + c, v);
+    for (int u = 0; u < 4; ++u)
+      if (t + u * step < rows) load_vec<T, V>(x + (t + u * step) * stride + c, v[u]);
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      if (t + u * step >= rows) break;
+#pragma unroll
+      for (int k = 0; k < V; ++k) v[u][k] = activate<ACT, T>(f * v[u][k]);
+      store_vec<T, V>(out + (t + u * step) * I + c, v[u]);
+    }
   }
 }
 
@@ -181,8 +208,9 @@ struct StreamParams {
 };
 static_assert(sizeof(StreamParams) == 176, "StreamParams is mirrored from Python");
 
-// CH register chunks of V elements per thread hold the row (CH = 0: the row is re-read from memory)
-template <typename T, int V, int CH>
+// CH register chunks of V elements per thread hold the row (CH = 0: the row is re-read from memory).  WHOLE: the update of
+// a prompt, both results one gated tensor each in the activation format, all loads issued before the first use.
+template <typename T, int V, int CH, bool WHOLE = false>
 __global__ void __launch_bounds__(kRowThreads) stream_rows_kernel(const __grid_constant__ StreamParams p) {
   __shared__ float red[kRowThreads / 32];
   const int W = p.W, nv = W / V;
@@ -206,7 +234,22 @@ __global__ void __launch_bounds__(kRowThreads) stream_rows_kernel(const __grid_c
     };
     auto fetch = [&](int vi, float (&v)[V]) {
       const size_t c = (size_t)vi * V;
-      if (p.enter) {
+      if constexpr (WHOLE) {
+        float y[2][V], g[2][V], b[2][V];
+        load_vec<float, V>(hr + c, v);
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+          load_vec<T, V>(reinterpret_cast<const T*>(p.sub[j].y) + (size_t)row * W + c, y[j]);
+          load_vec<T, V>(reinterpret_cast<const T*>(p.sub[j].gate) + row * p.sub[j].gate_stride + c, g[j]);
+          load_vec<T, V>(reinterpret_cast<const T*>(p.sub[j].bias) + c, b[j]);
+        }
+#pragma unroll
+        for (int i = 0; i < V; ++i) {
+          const float add = y[0][i] * gate_sigmoid<T>(fmaf(gain[0], g[0][i], b[0][i])) +
+                            y[1][i] * gate_sigmoid<T>(fmaf(gain[1], g[1][i], b[1][i]));
+          v[i] = fmaf(p.mult, add, v[i]);
+        }
+      } else if (p.enter) {
         load_vec<T, V>(reinterpret_cast<const T*>(p.step) + c, v);
         add_slabs(p.sub[1], row, vi, v);
         add_slabs(p.sub[0], row, vi, v);
@@ -225,7 +268,7 @@ __global__ void __launch_bounds__(kRowThreads) stream_rows_kernel(const __grid_c
             load_vec<T, V>(reinterpret_cast<const T*>(s.gate) + row * s.gate_stride + c, g);
             if (s.bias) load_vec<T, V>(reinterpret_cast<const T*>(s.bias) + c, b);
 #pragma unroll
-            for (int i = 0; i < V; ++i) y[i] /= 1.f + __expf(-fmaf(gain[j], g[i], b[i]));
+            for (int i = 0; i < V; ++i) y[i] *= gate_sigmoid<T>(fmaf(gain[j], g[i], b[i]));
           }
 #pragma unroll
           for (int i = 0; i < V; ++i) add[i] += y[i];
@@ -359,13 +402,30 @@ static int launch_add_norm(float* h, const T* delta, const T* w, T* y, int rows,
 template <typename T>
 static int launch_stream_rows(const StreamParams& p, cudaStream_t s) {
   const int grid = p.rows < num_sms() * 8 ? p.rows : num_sms() * 8, W = p.W;
-  bool vec = W % 4 == 0;
-  for (int j = 0; j < 2; ++j) vec = vec && p.sub[j].gate_stride % 4 == 0 && ((uintptr_t)p.sub[j].gate & 15) % (4 * sizeof(T)) == 0;
-  if (!vec) stream_rows_kernel<T, 1, 0><<<grid, kRowThreads, 0, s>>>(p);
-  else if (W <= 4 * kRowThreads) stream_rows_kernel<T, 4, 1><<<grid, kRowThreads, 0, s>>>(p);
-  else if (W <= 2 * 4 * kRowThreads) stream_rows_kernel<T, 4, 2><<<grid, kRowThreads, 0, s>>>(p);
-  else if (W <= 4 * 4 * kRowThreads) stream_rows_kernel<T, 4, 4><<<grid, kRowThreads, 0, s>>>(p);
-  else stream_rows_kernel<T, 4, 0><<<grid, kRowThreads, 0, s>>>(p);
+  auto takes = [&](int v) {      // accesses of v elements of the activation format
+    bool ok = W % v == 0;
+    for (int j = 0; j < 2; ++j)
+      ok = ok && p.sub[j].gate_stride % v == 0 && (uintptr_t)p.sub[j].gate % (v * sizeof(T)) == 0;
+    return ok;
+  };
+  bool whole = !p.enter && p.n_sub == 2;
+  for (int j = 0; j < 2; ++j)
+    whole = whole && p.sub[j].gate && p.sub[j].bias && p.sub[j].slabs == 1 && (p.sub[j].y_f32 != 0) == (sizeof(T) == 4);
+  if (sizeof(T) == 2 && takes(8) && whole && W <= 2 * 8 * kRowThreads) {
+    if (W <= 8 * kRowThreads) stream_rows_kernel<T, 8, 1, true><<<grid, kRowThreads, 0, s>>>(p);
+    else stream_rows_kernel<T, 8, 2, true><<<grid, kRowThreads, 0, s>>>(p);
+  } else if (sizeof(T) == 2 && takes(8) && W <= 2 * 8 * kRowThreads) {
+    if (W <= 8 * kRowThreads) stream_rows_kernel<T, 8, 1><<<grid, kRowThreads, 0, s>>>(p);
+    else stream_rows_kernel<T, 8, 2><<<grid, kRowThreads, 0, s>>>(p);
+  } else if (!takes(4)) {
+    stream_rows_kernel<T, 1, 0><<<grid, kRowThreads, 0, s>>>(p);
+  } else if (W <= 4 * kRowThreads) {
+    stream_rows_kernel<T, 4, 1><<<grid, kRowThreads, 0, s>>>(p);
+  } else if (W <= 2 * 4 * kRowThreads) {
+    stream_rows_kernel<T, 4, 2><<<grid, kRowThreads, 0, s>>>(p);
+  } else {
+    stream_rows_kernel<T, 4, 0><<<grid, kRowThreads, 0, s>>>(p);
+  }
   return (int)cudaGetLastError();
 }
 
@@ -378,8 +438,12 @@ static int launch_gated_act(const T* gu, T* out, long long rows, int I, int act,
 }
 
 template <typename T, int V>
-static int launch_scaled_act(const T* x, long long stride, const T* gain, T* out, long long rows, int I, int act, int grid,
+static int launch_scaled_act(const T* x, long long stride, const T* gain, T* out, long long rows, int I, int act,
                              cudaStream_t s) {
+  const int cols = (I / V + 255) / 256;
+  long long y = num_sms() * 8 / cols + 1;      // about eight blocks per SM
+  if (y > rows) y = rows;
+  const dim3 grid(cols, (unsigned)(y > 65535 ? 65535 : y));
   if (act == 0) scaled_act_kernel<T, V, 0><<<grid, 256, 0, s>>>(x, stride, gain, out, rows, I);
   else if (act == 1) scaled_act_kernel<T, V, 1><<<grid, 256, 0, s>>>(x, stride, gain, out, rows, I);
   else scaled_act_kernel<T, V, 2><<<grid, 256, 0, s>>>(x, stride, gain, out, rows, I);
@@ -437,13 +501,12 @@ extern "C" int sb_scaled_act(const void* x, long long stride, const void* gain, 
   if (act < 0 || act > 2) return -3;
   const int V = f32 ? 4 : 8;
   const bool vec = I % V == 0 && stride % V == 0 && ((uintptr_t)x & 15) == 0 && ((uintptr_t)out & 15) == 0;
-  const int grid = grid_for(rows * I / (vec ? V : 1), 256);
   using B = __nv_bfloat16;
   if (f32)
-    return vec ? launch_scaled_act<float, 4>((const float*)x, stride, (const float*)gain, (float*)out, rows, I, act, grid, stream)
-               : launch_scaled_act<float, 1>((const float*)x, stride, (const float*)gain, (float*)out, rows, I, act, grid, stream);
-  return vec ? launch_scaled_act<B, 8>((const B*)x, stride, (const B*)gain, (B*)out, rows, I, act, grid, stream)
-             : launch_scaled_act<B, 1>((const B*)x, stride, (const B*)gain, (B*)out, rows, I, act, grid, stream);
+    return vec ? launch_scaled_act<float, 4>((const float*)x, stride, (const float*)gain, (float*)out, rows, I, act, stream)
+               : launch_scaled_act<float, 1>((const float*)x, stride, (const float*)gain, (float*)out, rows, I, act, stream);
+  return vec ? launch_scaled_act<B, 8>((const B*)x, stride, (const B*)gain, (B*)out, rows, I, act, stream)
+             : launch_scaled_act<B, 1>((const B*)x, stride, (const B*)gain, (B*)out, rows, I, act, stream);
 }
 
 // params: host StreamParams

@@ -19,8 +19,12 @@ template <typename T, int V>
 __device__ __forceinline__ void load_vec(const T* p, float (&x)[V]) {
   if constexpr (V == 1) {
     x[0] = to_float(p[0]);
+  } else if constexpr (sizeof(T) == 4 && V == 8) {
+    const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+    x[0] = a.x; x[1] = a.y; x[2] = a.z; x[3] = a.w;
+    x[4] = b.x; x[5] = b.y; x[6] = b.z; x[7] = b.w;
   } else if constexpr (sizeof(T) == 4) {
-    static_assert(V == 4, "fp32 vectors of four");
+    static_assert(V == 4, "fp32 vectors of four or eight");
     const float4 v = *reinterpret_cast<const float4*>(p);
     x[0] = v.x; x[1] = v.y; x[2] = v.z; x[3] = v.w;
   } else if constexpr (V == 4) {
@@ -45,6 +49,9 @@ template <typename T, int V>
 __device__ __forceinline__ void store_vec(T* p, const float (&x)[V]) {
   if constexpr (V == 1) {
     p[0] = from_float<T>(x[0]);
+  } else if constexpr (sizeof(T) == 4 && V == 8) {
+    reinterpret_cast<float4*>(p)[0] = make_float4(x[0], x[1], x[2], x[3]);
+    reinterpret_cast<float4*>(p)[1] = make_float4(x[4], x[5], x[6], x[7]);
   } else if constexpr (sizeof(T) == 4) {
     *reinterpret_cast<float4*>(p) = make_float4(x[0], x[1], x[2], x[3]);
   } else if constexpr (V == 4) {
