@@ -230,7 +230,8 @@ def _kernels_poralorn(b: _Bench) -> None:
         kv = dense.linear(rnd(T, rank), w["kv_up"])
         add(f"uniform: fmha_fwd {n}x{L}", lambda: attention_packed(q, info, H, G, D), flops)
         add(f"poralorn: attention over expanded keys, gated {n}x{L}",
-            lambda: LA.expanded_attention(spec, x, w["gain"], kv, ids, pos, table, out, 0, plan), flops)
+            lambda: LA.expanded_attention(spec, x, w["gain"], kv, ids, pos, table, out, 0, plan), flops,
+            nbytes=T * hd * 10)
         add(f"poralorn: latent append {n}x{L}", lambda: LA.latent_append(spec, x, w, ids, pos, table, cache, plan),
             nbytes=T * rank * 6)
         add(f"poralorn: whole latent attention {n}x{L} (append, expansion, attention)",

@@ -369,7 +369,7 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
             float z[8];
             load_vec<__nv_bfloat16, 8>(grow + c * 32 + g * 8, z);
 #pragma unroll
-            for (int i = 0; i < 8; ++i) o[i] /= 1.f + __expf(-gain * z[i]);
+            for (int i = 0; i < 8; ++i) o[i] = __fdividef(o[i], 1.f + __expf(-gain * z[i]));
           }
           store_vec<__nv_bfloat16, 8>(orow + c * 32 + g * 8, o);
         }

@@ -132,8 +132,8 @@ head_product_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
               const float2 z = __bfloat1622float2(z2[i]);
-              o[2 * i] /= 1.f + __expf(-gain * z.x);
-              o[2 * i + 1] /= 1.f + __expf(-gain * z.y);
+              o[2 * i] = __fdividef(o[2 * i], 1.f + __expf(-gain * z.x));
+              o[2 * i + 1] = __fdividef(o[2 * i + 1], 1.f + __expf(-gain * z.y));
             }
           }
           store_vec<__nv_bfloat16, 8>(c + q * 32 + v * 8, o);

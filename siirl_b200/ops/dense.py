@@ -114,6 +114,7 @@ class _LinearFn(torch.autograd.Function):
 
 
 _NUM_SMS = 148
+_ONE_WAVE = 100      # from this many tiles on, the partial sums of a split cost more than the SMs that stay idle without one
 SWAP_OPERANDS_ABOVE_128_ROWS = True     # benchmarks flip this to time both forms
 
 
@@ -124,7 +125,7 @@ def _skinny_splits(M: int, N: int, K: int) -> int:
     plain kernel already fills the machine."""
     n_tiles = (N + 127) // 128 * ((M + 127) // 128)
     nkb = (K + 63) // 64
-    if n_tiles >= _NUM_SMS or nkb < 8:
+    if n_tiles >= _ONE_WAVE or nkb < 8:
         return 1
     best, best_score = 1, -1.0
     for s in range(1, min(nkb // 4, 16) + 1):
@@ -139,7 +140,7 @@ def _skinny_splits(M: int, N: int, K: int) -> int:
 def _best_splits(n_tiles: int, nkb: int) -> int:
     """Split-K factor that fills whole waves of the persistent grid with ``n_tiles`` output tiles of ``nkb``
     k-blocks (1: no split)."""
-    if n_tiles >= _NUM_SMS or nkb < 8:
+    if n_tiles >= _ONE_WAVE or nkb < 8:
         return 1
     best, best_score = 1, -1.0
     for s in range(1, min(nkb // 4, 16) + 1):
