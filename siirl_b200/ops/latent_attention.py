@@ -52,7 +52,7 @@ class LatentSpec:
     def aligned(self) -> bool:
         """Sizes the tensor-core kernels take."""
         return self.dim % 8 == 0 and self.vdim % 8 == 0 and self.rank % 8 == 0 and self.q_off % 8 == 0 and \
-            self.g_off % 8 in (0, 7) and max(self.dim, self.vdim) <= 256
+            (self.g_off < 0 or self.g_off % 8 == 0) and max(self.dim, self.vdim) <= 256
 
 
 class LatentPlan:
