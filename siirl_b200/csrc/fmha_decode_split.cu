@@ -48,6 +48,10 @@ struct SplitParams {
   int window, keep_first, dv;
   long long out_stride;    // `out` points at the branch's first column
   float bias_exp, out_scale;
+  float softcap, scale;      // softcap 0: none
+  int sink, rel_n;
+  const float* rel;          // [Hq, rel_n] bias by distance, or null
+  const float* head_gate;    // [B, Hq] factors of the result, or null
 };
 
 // cache blocks a query at position ctx - 1 visits: blocks 0 .. sinks - 1, then w0 .. ; `n` of them in all
@@ -318,6 +322,13 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
         return WIN && p.bias_exp > 0.f
                    ? exp2f(-p.bias_exp * (float)(g * rep + row + 1) / (float)p.Hq) * 1.4426950408889634f : 0.f;
       };
+      // soft cap and bias table (windowed variant): `raw` product of a head at distance ctx - 1 - col
+      const ScoreCap cap(WIN && p.softcap > 0.f ? p.softcap : 1.f, p.scale);
+      auto score_of = [&](float raw) { return WIN && p.softcap > 0.f ? cap(raw) : raw * p.scale_log2; };
+      auto rel_row = [&](int row) { return p.rel + (size_t)min(g * rep + row, p.Hq - 1) * p.rel_n; };
+      auto rel_at = [&](const float* rel, int col) {
+        return __ldg(rel + min(max(ctx - 1 - col, 0), p.rel_n - 1)) * 1.4426950408889634f;
+      };
       const uint32_t tmem_oi = tmem_o + (item_no & 1) * 128;
       float m_ref = -INFINITY, l_run = 0.f;
       if (rep <= 8) {
@@ -328,9 +339,19 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
         const int frow = lane >> 2, fq = lane & 3;
         const bool fvalid = frow < rep;
         const float slope = slope_of(frow);
+        const float* rel = WIN && p.rel ? rel_row(frow) : nullptr;
         for (int t = 0; t < n; ++t) {
           const uint32_t tn = tile_no + t;
           const int sb_ = tn & 1;
+          float rb[16] = {};
+          if (WIN && rel) {      // in flight while the scores are computed
+            const int col = first_pos(t) + 2 * fq;
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+              rb[2 * i] = rel_at(rel, col + 8 * i);
+              rb[2 * i + 1] = rel_at(rel, col + 8 * i + 1);
+            }
+          }
           if (!__all_sync(0xffffffffu, mbar_wait(&s_full[sb_], (tn >> 1) & 1, p.status, kStatusTimeoutEpilogue))) {
             ok = false;
             break;
@@ -343,8 +364,8 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
             tmem_ld_wait();
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
-              sv[2 * i] = __uint_as_float(r[4 * i]) * p.scale_log2;
-              sv[2 * i + 1] = __uint_as_float(r[4 * i + 1]) * p.scale_log2;
+              sv[2 * i] = score_of(__uint_as_float(r[4 * i]));
+              sv[2 * i + 1] = score_of(__uint_as_float(r[4 * i + 1]));
             }
           }
           tc_fence_before();
@@ -355,8 +376,8 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
               const float dist = (float)(kv0 + 8 * i + 2 * fq - (ctx - 1));
-              sv[2 * i] = fmaf(slope, dist, sv[2 * i]);
-              sv[2 * i + 1] = fmaf(slope, dist + 1.f, sv[2 * i + 1]);
+              sv[2 * i] = fmaf(slope, dist, sv[2 * i]) + rb[2 * i];
+              sv[2 * i + 1] = fmaf(slope, dist + 1.f, sv[2 * i + 1]) + rb[2 * i + 1];
             }
           }
           if (need_mask(kv0)) {
@@ -429,6 +450,7 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
         m_ref = __shfl_sync(0xffffffffu, m_ref, (lane * 4) & 31);
       } else {
         const float slope = slope_of(lane);
+        const float* rel = WIN && p.rel ? rel_row(lane) : nullptr;
         for (int t = 0; t < n; ++t) {
           const uint32_t tn = tile_no + t;
           const int sb_ = tn & 1;
@@ -445,8 +467,8 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
             tmem_ld_wait();
   #pragma unroll
             for (int i = 0; i < 32; ++i) {
-              sv[i] = __uint_as_float(r0[i]) * p.scale_log2;
-              sv[32 + i] = __uint_as_float(r1[i]) * p.scale_log2;
+              sv[i] = score_of(__uint_as_float(r0[i]));
+              sv[32 + i] = score_of(__uint_as_float(r1[i]));
             }
           }
           tc_fence_before();
@@ -456,6 +478,10 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
           if constexpr (WIN) {
   #pragma unroll
             for (int i = 0; i < kSBlk; ++i) sv[i] = fmaf(slope, (float)(kv0 + i - (ctx - 1)), sv[i]);
+            if (rel) {
+  #pragma unroll
+              for (int i = 0; i < kSBlk; ++i) sv[i] += rel_at(rel, kv0 + i);
+            }
           }
           if (need_mask(kv0)) {
   #pragma unroll
@@ -558,9 +584,11 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
       const float inv_l = l_run > 0.f ? 1.f / l_run : 0.f;
       const int head = g * rep + (row_valid ? lane : 0);
       const bool single = n_seq_tiles <= kChunkTiles;
+      const float total = WIN && p.sink ? l_run + exp2f(-m_ref) : l_run;
       const int dv = WIN ? p.dv : D;
       __nv_bfloat16* orow = p.out + (WIN ? (size_t)b * p.out_stride : (size_t)b * (p.Hq * D)) + (size_t)head * dv;
-      const float out_f = WIN ? inv_l * p.out_scale : inv_l;
+      float out_f = WIN ? (total > 0.f ? p.out_scale / total : 0.f) : inv_l;
+      if (WIN && p.head_gate) out_f *= p.head_gate[(size_t)b * p.Hq + head];
       float* wrow = p.ws_o + (((size_t)b * p.Hq + head) * p.max_chunks + c) * D;
 #pragma unroll 1
       for (int cc = 0; cc < D / 32; ++cc) {
@@ -639,7 +667,10 @@ __global__ void fmha_decode_merge_kernel(SplitParams p) {
     wsum += w;
     acc += w * wo[(size_t)c * D + d];
   }
-  orow[d] = __float2bfloat16(wsum > 0.f ? acc / wsum * (WIN ? p.out_scale : 1.f) : 0.f);
+  if (WIN && p.sink) wsum += exp2f(-m);
+  float f = WIN ? p.out_scale : 1.f;
+  if (WIN && p.head_gate) f *= p.head_gate[(size_t)b * p.Hq + h];
+  orow[d] = __float2bfloat16(wsum > 0.f ? acc / wsum * f : 0.f);
 }
 
 template <int D, bool WIN>
@@ -697,6 +728,7 @@ extern "C" int sb_fmha_decode_split(const void* q, int row_stride, const void* c
   p.B = B; p.Hq = Hq; p.Hkv = Hkv; p.q_rows_per_seq = row_stride / D;
   p.scale_log2 = scale * 1.4426950408889634f; p.status = status;
   p.window = 0; p.keep_first = 0; p.dv = D; p.out_stride = 0; p.bias_exp = 0.f; p.out_scale = 1.f;
+  p.softcap = 0.f; p.scale = scale; p.sink = 0; p.rel_n = 0; p.rel = nullptr; p.head_gate = nullptr;
   return D == 128 ? launch_decode_split<128, false>(mc, mc, mq, p, stream)
                   : launch_decode_split<64, false>(mc, mc, mq, p, stream);
 }
@@ -706,7 +738,8 @@ extern "C" int sb_fmha_decode_split(const void* q, int row_stride, const void* c
 extern "C" int sb_attn_window_decode_chunks(const void* params) {
   const WinParams& p = *reinterpret_cast<const WinParams*>(params);
   if (p.dk % 8 || p.dv % 8 || p.dk > 128 || p.dv > 128 || p.Hq % p.Hkv || p.Hq / p.Hkv > 32 || p.row_stride % 8 ||
-      p.q_off % 8 || p.out_stride % 8 || p.out_off % 8 || p.block_elems % 8 || p.kv_mode != kPaged || p.gain || p.gate)
+      p.q_off % 8 || p.out_stride % 8 || p.out_off % 8 || p.block_elems % 8 || p.kv_mode != kPaged || p.gain || p.gate ||
+      (p.rel && p.rel_n < 1))
     return -1;
   int tiles = p.max_blocks;
   if (p.window > 0) {
@@ -747,6 +780,8 @@ extern "C" int sb_attn_window_decode(const void* params, const int* seq_lens, fl
   p.scale_log2 = w.scale * 1.4426950408889634f; p.status = status;
   p.window = w.window; p.keep_first = w.keep_first; p.dv = w.dv; p.out_stride = w.out_stride;
   p.bias_exp = w.bias_exp; p.out_scale = w.out_scale;
+  p.softcap = w.softcap; p.scale = w.scale; p.sink = w.sink; p.rel_n = (int)w.rel_n; p.rel = w.rel;
+  p.head_gate = w.head_gate;
   return w.dk > 64 || w.dv > 64 ? launch_decode_split<128, true>(mk, mv, mq, p, stream)
                                 : launch_decode_split<64, true>(mk, mv, mq, p, stream);
 }

@@ -9,6 +9,7 @@
 //   window_prefill_kernel   bf16, dk and dv multiples of 8 up to 256: 128 query rows of one head per CTA, S = Q K^T and
 //                           O += P V on tcgen05 with accumulators in TMEM; one cache block is one K/V tile, fetched by
 //                           TMA straight from the paged cache (columns past dk / dv are filled with zeros)
+//                           (two forms: linear bias; soft cap and a bias table by distance)
 //   window_simt_kernel      any sizes, bf16 or fp32, one CTA per (row, head): the 32-bit path, and odd widths
 #include "common.cuh"
 #include "launchers.h"
@@ -96,6 +97,8 @@ __global__ void __launch_bounds__(kSimtThreads) window_simt_kernel(WinParams p) 
         for (int d = 0; d < p.dk; ++d) acc = fmaf(sq[d], to_float(k[d]), acc);
         const int j = v < first ? v : lo + v - first;
         s = acc * p.scale - slope * (float)(i - j);
+        if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
+        if (p.rel) s += p.rel[(size_t)h * p.rel_n + min((long long)(i - j), p.rel_n - 1)];
       }
     }
     float mx = warp_max(s);
@@ -122,7 +125,9 @@ __global__ void __launch_bounds__(kSimtThreads) window_simt_kernel(WinParams p) 
     }
     __syncthreads();
   }
-  const float inv = l > 0.f ? p.out_scale / l : 0.f;
+  if (p.sink) l += expf(-m);
+  float inv = l > 0.f ? p.out_scale / l : 0.f;
+  if (p.head_gate) inv *= p.head_gate[(size_t)t * p.Hq + h];
   for (int d = tid; d < p.dv; d += kSimtThreads) out[d] = from_float<T>(so[d] * inv);
 }
 
@@ -159,6 +164,8 @@ __host__ __device__ inline void win_blocks(int q0, int q1, int window, int keep_
   n = sinks + (last + 1 > w0 ? last + 1 - w0 : 0);
 }
 
+// TABLE: soft-capped scores and / or a bias table by distance instead of the linear bias
+template <bool TABLE>
 __global__ void __launch_bounds__(128, 2)
 window_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                       const __grid_constant__ CUtensorMap map_v, WinParams p, const int* __restrict__ tile_row,
@@ -237,6 +244,10 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
   const float scale_log2 = p.scale * gain * 1.4426950408889634f;
   const float slope_log2 =
       p.bias_exp > 0.f ? exp2f(-p.bias_exp * (float)(h + 1) / (float)p.Hq) * 1.4426950408889634f : 0.f;
+  const ScoreCap cap(p.softcap > 0.f ? p.softcap : 1.f, p.scale * gain);
+  const float* rel = TABLE && p.rel ? p.rel + (size_t)h * p.rel_n : nullptr;
+  const int rel_last = (int)p.rel_n - 1;
+  const float rel_far = rel ? __ldg(rel + rel_last) * 1.4426950408889634f : 0.f;
   float m_run = -INFINITY, l_run = 0.f;
   bool ok = true;
 
@@ -271,10 +282,35 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       tmem_ld_32x32(tmem_s + lane_off, r0);
       tmem_ld_32x32(tmem_s + lane_off + 32, r1);
       tmem_ld_wait();
+      if constexpr (TABLE) {
+        if (p.softcap > 0.f) {
 #pragma unroll
-      for (int i = 0; i < 32; ++i) {
-        sv[i] = fmaf(__uint_as_float(r0[i]), scale_log2, fmaf(slope_log2, (float)i, b0));
-        sv[32 + i] = fmaf(__uint_as_float(r1[i]), scale_log2, fmaf(slope_log2, (float)(32 + i), b0));
+          for (int i = 0; i < 32; ++i) {
+            sv[i] = cap(__uint_as_float(r0[i]));
+            sv[32 + i] = cap(__uint_as_float(r1[i]));
+          }
+        } else {
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            sv[i] = __uint_as_float(r0[i]) * scale_log2;
+            sv[32 + i] = __uint_as_float(r1[i]) * scale_log2;
+          }
+        }
+        if (rel && q0 - (kv0 + kWBlk - 1) >= rel_last) {      // the whole tile is at least as far as the last entry
+#pragma unroll
+          for (int i = 0; i < kWBlk; ++i) sv[i] += rel_far;
+        } else if (rel) {
+          const int d0 = qpos - kv0;
+#pragma unroll
+          for (int i = 0; i < kWBlk; ++i)
+            sv[i] = fmaf(__ldg(rel + min(max(d0 - i, 0), rel_last)), 1.4426950408889634f, sv[i]);
+        }
+      } else {
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          sv[i] = fmaf(__uint_as_float(r0[i]), scale_log2, fmaf(slope_log2, (float)i, b0));
+          sv[32 + i] = fmaf(__uint_as_float(r1[i]), scale_log2, fmaf(slope_log2, (float)(32 + i), b0));
+        }
       }
     }
     // every row of the tile sees every key of the block when the block lies behind q0 and, with a window, inside the
@@ -348,7 +384,9 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
   ok = __all_sync(0xffffffffu, ok);
   if (ok) {
     const bool row_valid = tid < nrows;
-    const float inv_l = l_run > 0.f ? p.out_scale / l_run : 0.f;
+    if (p.sink) l_run += exp2f(-m_run);
+    float inv_l = l_run > 0.f ? p.out_scale / l_run : 0.f;
+    if (p.head_gate && row_valid) inv_l *= p.head_gate[(size_t)(row0 + tid) * p.Hq + h];
     __nv_bfloat16* orow = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)(row0 + (row_valid ? tid : 0)) * p.out_stride +
                           p.out_off + (size_t)h * p.dv;
     const __nv_bfloat16* grow = reinterpret_cast<const __nv_bfloat16*>(p.gate) +
@@ -417,7 +455,7 @@ extern "C" int sb_kv_append_split(const void* params, int f32, cudaStream_t stre
 extern "C" int sb_attn_window_simt(const void* params, int f32, cudaStream_t stream) {
   const WinParams& p = *reinterpret_cast<const WinParams*>(params);
   if (p.T == 0) return 0;
-  if (p.Hq % p.Hkv || p.Hq > 65535 || p.kv_mode == kPackedRows || p.gate || (p.kv_mode == kLatent && p.dk != p.dv)) return -3;
+  if (p.Hq % p.Hkv || p.Hq > 65535 || p.kv_mode == kPackedRows || (p.rel && p.rel_n < 1) || p.gate || (p.kv_mode == kLatent && p.dk != p.dv)) return -3;
   const size_t smem = (size_t)(p.dk + kSimtThreads + p.dv) * 4;
   if (smem > 48 * 1024) return -3;
   const dim3 grid(p.T, p.Hq);
@@ -434,7 +472,7 @@ extern "C" int sb_attn_window_prefill(const void* params, const int* tile_row, c
   if (n_tiles == 0) return 0;
   if (p.Hq % p.Hkv || p.dk % 8 || p.dv % 8 || p.dk > 256 || p.dv > 256 || p.dk < 8 || p.dv < 8 || p.row_stride % 8 ||
       p.q_off % 8 || p.out_stride % 8 || p.out_off % 8 || p.block_elems % 8 || ((uintptr_t)p.out & 15) ||
-      p.kv_mode == kLatent || p.gate_stride % 8 || ((uintptr_t)p.gate & 15))
+      p.kv_mode == kLatent || p.gate_stride % 8 || ((uintptr_t)p.gate & 15) || (p.rel && (p.rel_n < 1 || p.bias_exp > 0.f)))
     return -2;
   static thread_local bool tl_context_bound = false;
   if (!tl_context_bound) {
@@ -462,16 +500,18 @@ extern "C" int sb_attn_window_prefill(const void* params, const int* tile_row, c
     if (r) return r;
   }
   const WinSmem L((p.dk + 63) / 64, (p.dv + 63) / 64);
-  static int configured = 0;
-  if (configured < L.total) {
-    cudaError_t e = cudaFuncSetAttribute(window_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, L.total);
+  const bool table = p.softcap > 0.f || p.rel;
+  auto kernel = table ? window_prefill_kernel<true> : window_prefill_kernel<false>;
+  static int configured[2] = {0, 0};
+  if (configured[table] < L.total) {
+    cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, L.total);
     if (e != cudaSuccess) return (int)e;
-    configured = L.total;
+    configured[table] = L.total;
   }
   const int need = 64 + (p.dv + 31) / 32 * 32;
   uint32_t cols = 128;
   while ((int)cols < need) cols *= 2;
-  window_prefill_kernel<<<dim3(n_tiles, p.Hq), 128, L.total, stream>>>(mq, mk, mv, p, tile_row, tile_rows, tile_pos,
-                                                                       tile_slot, cols, status);
+  kernel<<<dim3(n_tiles, p.Hq), 128, L.total, stream>>>(mq, mk, mv, p, tile_row, tile_rows, tile_pos, tile_slot, cols,
+                                                        status);
   return (int)cudaGetLastError();
 }

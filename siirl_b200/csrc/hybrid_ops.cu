@@ -5,7 +5,7 @@
 //   add_norm           h += delta;  y = norm(h) * w                              (layer norm or RMS norm, one launch)
 //   stream_rows        h += mult * sum of two sublayer results, each times a sigmoid gate, then h / rms(h)  (one launch);
 //                      or h = sum of partial products + vector (entry of a loop's pass), then h / rms(h); or h as two rows
-//   gated_act          y = act(gate) * up   for a fused projection [gate | up]   (SiLU, tanh-form or exact GELU)
+//   gated_act          y = act(gate) * up   for a fused projection [gate | up]   (SiLU, tanh-form or exact GELU, squared relu)
 //   scaled_act         y = act(gain * x)    of a column range
 //   softcap            z = cap * tanh(z / cap) in place on fp32 logits
 //   gemm_simt          C[M, N] = A[M, K] B[N, K]^T with fp32 accumulation on the FMA pipes: fp32 models (true 32-bit
@@ -131,8 +131,13 @@ __device__ __forceinline__ float gelu_erf_fast(float z) {
   return z * (z < 0.f ? q : 1.f - q);
 }
 
-template <int ACT, typename T>      // 0 SiLU, 1 tanh-form GELU, 2 exact GELU; T: the format of the result
+template <int ACT, typename T>      // 0 SiLU, 1 tanh-form GELU, 2 exact GELU, 3 square of relu; T: the format of the result
 __device__ __forceinline__ float activate(float z) {
+  if constexpr (ACT == 3) {
+    z = fmaxf(z, 0.f);
+    return z * z;
+  }
+  if constexpr (ACT == 0 && sizeof(T) == 4) return z / (1.f + expf(-z));
   if constexpr (ACT == 1) return gelu_tanh_f(z);
   if constexpr (ACT == 2 && sizeof(T) == 2) return gelu_erf_fast(z);
   if constexpr (ACT == 2) return 0.5f * z * (1.f + erff(z * 0.7071067811865476f));
@@ -147,11 +152,13 @@ __device__ __forceinline__ float gate_sigmoid(float z) {
 }
 
 template <typename T, int V, int ACT>
-__global__ void gated_act_kernel(const T* __restrict__ gu, T* __restrict__ out, long long rows, int I) {
+__global__ void gated_act_kernel(const T* __restrict__ gu, T* __restrict__ out, long long rows, int I,
+                                 const int* __restrict__ used) {
   const int nv = I / V;
   const long long total = rows * nv;
   for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
     const long long t = i / nv;
+    if (used && used[t] < 0) continue;      // padding row of an expert's segment
     const int c = (int)(i % nv) * V;
     float g[V], u[V];
     load_vec<T, V>(gu + t * 2 * I + c, g);
@@ -339,19 +346,34 @@ __global__ void softcap_kernel(float* __restrict__ z, long long n, float cap) {
   }
 }
 
-// 64 x 64 output tile per 256 threads, 4 x 4 values each, contraction in steps of 16 through shared memory
-template <typename TI, typename TO>
+// 64 x 64 output tile per 256 threads, 4 x 4 values each, contraction in steps of 16 through shared memory.
+// GROUPED: rows are slots of experts, 128-row blocks of one expert each (tile_group, -1: unused block); a slot's row of A is
+// a_row[slot] (-1: zeros) when given, and B holds one matrix per expert, b_group elements apart.
+template <typename TI, typename TO, bool GROUPED = false>
 __global__ void __launch_bounds__(256)
 gemm_simt_kernel(const TI* __restrict__ A, const TI* __restrict__ B, TO* __restrict__ C, int M, int N, int K,
-                 long long lda, long long ldb, long long ldc) {
+                 long long lda, long long ldb, long long ldc, const int* __restrict__ tile_group = nullptr,
+                 const int* __restrict__ a_row = nullptr, long long b_group = 0) {
   __shared__ float sa[16][68], sb_[16][68];
+  __shared__ int s_row[64];
   const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
+  if constexpr (GROUPED) {
+    const int g = tile_group[m0 / 128];
+    if (g < 0) return;
+    B += (size_t)g * b_group;
+    if (threadIdx.x < 64) {
+      const int m = m0 + threadIdx.x;
+      s_row[threadIdx.x] = m < M ? (a_row ? a_row[m] : m) : -1;
+    }
+    __syncthreads();
+  }
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
   float acc[4][4] = {};
   for (int k0 = 0; k0 < K; k0 += 16) {
     for (int i = threadIdx.x; i < 64 * 16; i += 256) {
       const int r = i >> 4, k = i & 15;
-      sa[k][r] = (m0 + r < M && k0 + k < K) ? to_float(A[(size_t)(m0 + r) * lda + k0 + k]) : 0.f;
+      const int row = GROUPED ? s_row[r] : (m0 + r < M ? m0 + r : -1);
+      sa[k][r] = (row >= 0 && k0 + k < K) ? to_float(A[(size_t)row * lda + k0 + k]) : 0.f;
       sb_[k][r] = (n0 + r < N && k0 + k < K) ? to_float(B[(size_t)(n0 + r) * ldb + k0 + k]) : 0.f;
     }
     __syncthreads();
@@ -430,10 +452,11 @@ static int launch_stream_rows(const StreamParams& p, cudaStream_t s) {
 }
 
 template <typename T, int V>
-static int launch_gated_act(const T* gu, T* out, long long rows, int I, int act, int grid, cudaStream_t s) {
-  if (act == 0) gated_act_kernel<T, V, 0><<<grid, 256, 0, s>>>(gu, out, rows, I);
-  else if (act == 1) gated_act_kernel<T, V, 1><<<grid, 256, 0, s>>>(gu, out, rows, I);
-  else gated_act_kernel<T, V, 2><<<grid, 256, 0, s>>>(gu, out, rows, I);
+static int launch_gated_act(const T* gu, T* out, long long rows, int I, int act, const int* used, int grid, cudaStream_t s) {
+  if (act == 0) gated_act_kernel<T, V, 0><<<grid, 256, 0, s>>>(gu, out, rows, I, used);
+  else if (act == 1) gated_act_kernel<T, V, 1><<<grid, 256, 0, s>>>(gu, out, rows, I, used);
+  else if (act == 2) gated_act_kernel<T, V, 2><<<grid, 256, 0, s>>>(gu, out, rows, I, used);
+  else gated_act_kernel<T, V, 3><<<grid, 256, 0, s>>>(gu, out, rows, I, used);
   return (int)cudaGetLastError();
 }
 
@@ -446,7 +469,8 @@ static int launch_scaled_act(const T* x, long long stride, const T* gain, T* out
   const dim3 grid(cols, (unsigned)(y > 65535 ? 65535 : y));
   if (act == 0) scaled_act_kernel<T, V, 0><<<grid, 256, 0, s>>>(x, stride, gain, out, rows, I);
   else if (act == 1) scaled_act_kernel<T, V, 1><<<grid, 256, 0, s>>>(x, stride, gain, out, rows, I);
-  else scaled_act_kernel<T, V, 2><<<grid, 256, 0, s>>>(x, stride, gain, out, rows, I);
+  else if (act == 2) scaled_act_kernel<T, V, 2><<<grid, 256, 0, s>>>(x, stride, gain, out, rows, I);
+  else scaled_act_kernel<T, V, 3><<<grid, 256, 0, s>>>(x, stride, gain, out, rows, I);
   return (int)cudaGetLastError();
 }
 
@@ -480,25 +504,27 @@ extern "C" int sb_add_norm(float* h, const void* delta, const void* w, void* y, 
                                         W, eps, layer_norm, stream);
 }
 
-// act: 0 SiLU, 1 tanh-form GELU, 2 exact GELU; gu [rows, 2 I] -> out [rows, I]
-extern "C" int sb_gated_act(const void* gu, void* out, long long rows, int I, int act, int f32, cudaStream_t stream) {
+// act: 0 SiLU, 1 tanh-form GELU, 2 exact GELU, 3 square of relu; gu [rows, 2 I] -> out [rows, I]; used: rows with a
+// negative entry are left out (null: none)
+extern "C" int sb_gated_act(const void* gu, void* out, long long rows, int I, int act, const int* used, int f32,
+                            cudaStream_t stream) {
   if (rows == 0) return 0;
-  if (act < 0 || act > 2) return -3;
+  if (act < 0 || act > 3) return -3;
   const int V = f32 ? 4 : 8;
   const int grid = grid_for(rows * I / (I % V ? 1 : V), 256);
   using B = __nv_bfloat16;
   if (f32)
-    return I % 4 == 0 ? launch_gated_act<float, 4>((const float*)gu, (float*)out, rows, I, act, grid, stream)
-                      : launch_gated_act<float, 1>((const float*)gu, (float*)out, rows, I, act, grid, stream);
-  return I % 8 == 0 ? launch_gated_act<B, 8>((const B*)gu, (B*)out, rows, I, act, grid, stream)
-                    : launch_gated_act<B, 1>((const B*)gu, (B*)out, rows, I, act, grid, stream);
+    return I % 4 == 0 ? launch_gated_act<float, 4>((const float*)gu, (float*)out, rows, I, act, used, grid, stream)
+                      : launch_gated_act<float, 1>((const float*)gu, (float*)out, rows, I, act, used, grid, stream);
+  return I % 8 == 0 ? launch_gated_act<B, 8>((const B*)gu, (B*)out, rows, I, act, used, grid, stream)
+                    : launch_gated_act<B, 1>((const B*)gu, (B*)out, rows, I, act, used, grid, stream);
 }
 
 // x: columns of rows `stride` apart -> out [rows, I]; gain: one number or null
 extern "C" int sb_scaled_act(const void* x, long long stride, const void* gain, void* out, long long rows, int I, int act,
                              int f32, cudaStream_t stream) {
   if (rows == 0 || I == 0) return 0;
-  if (act < 0 || act > 2) return -3;
+  if (act < 0 || act > 3) return -3;
   const int V = f32 ? 4 : 8;
   const bool vec = I % V == 0 && stride % V == 0 && ((uintptr_t)x & 15) == 0 && ((uintptr_t)out & 15) == 0;
   using B = __nv_bfloat16;
@@ -540,5 +566,22 @@ extern "C" int sb_gemm_simt(const void* A, const void* B, void* C, int M, int N,
     gemm_simt_kernel<H, H><<<grid, 256, 0, stream>>>((const H*)A, (const H*)B, (H*)C, M, N, K, lda, ldb, ldc);
   else
     return -2;
+  return (int)cudaGetLastError();
+}
+
+// Products of expert slots: C[slot] = A[a_row[slot] or slot] B[expert of the slot]^T, fp32 operands and results or bf16
+extern "C" int sb_gemm_simt_grouped(const void* A, const void* B, void* C, int M, int N, int K, long long lda, long long ldb,
+                                    long long ldc, const int* tile_group, const int* a_row, long long b_group, int f32,
+                                    cudaStream_t stream) {
+  if (M <= 0 || N <= 0) return 0;
+  if (M % 128 || M / 64 > 65535 || !tile_group) return -3;
+  const dim3 grid((N + 63) / 64, M / 64);
+  using H = __nv_bfloat16;
+  if (f32)
+    gemm_simt_kernel<float, float, true><<<grid, 256, 0, stream>>>((const float*)A, (const float*)B, (float*)C, M, N, K, lda,
+                                                                   ldb, ldc, tile_group, a_row, b_group);
+  else
+    gemm_simt_kernel<H, H, true><<<grid, 256, 0, stream>>>((const H*)A, (const H*)B, (H*)C, M, N, K, lda, ldb, ldc,
+                                                           tile_group, a_row, b_group);
   return (int)cudaGetLastError();
 }

@@ -31,6 +31,9 @@ int sb_moe_pair_dot(const void* const* y_ptrs, int world, const int* pair_rank, 
                     float* dots, int T, int k, int H, cudaStream_t stream);
 int sb_moe_route_topk(const void* logits, int is_bf16, int ld, float* w, int* idx, int T, int E, int k, int norm,
                       cudaStream_t stream);
+int sb_moe_route_grouped(const float* z, long long slab, int slabs, int ld, const void* corr, int corr_f32, float* w,
+                         int* idx, float* w_id, int T, int E, int experts, int k, int n_groups, int keep, float scale,
+                         cudaStream_t stream);
 int sb_moe_route_topk_bwd(const void* logits, int is_bf16, int ld, const int* idx, const float* dw, float* dlogits,
                           int T, int E, int k, int norm, cudaStream_t stream);
 int sb_moe_build_layout(const int* idx, int P, int E, int world, int rank, int T, int k, int capacity,
@@ -190,7 +193,13 @@ int sb_embed_scaled(const long long* ids, const void* table, float* h, int T, in
                     cudaStream_t stream);
 int sb_add_norm(float* h, const void* delta, const void* w, void* y, int rows, int W, float eps, int layer_norm, int f32,
                 cudaStream_t stream);
-int sb_gated_act(const void* gu, void* out, long long rows, int I, int act, int f32, cudaStream_t stream);
+int sb_gated_act(const void* gu, void* out, long long rows, int I, int act, const int* used, int f32, cudaStream_t stream);
+int sb_gemm_simt_grouped(const void* A, const void* B, void* C, int M, int N, int K, long long lda, long long ldb,
+                         long long ldc, const int* tile_group, const int* a_row, long long b_group, int f32,
+                         cudaStream_t stream);
+// ---- qkv_prepare.cu, hyper_rows.cu ----
+int sb_qkv_prepare(const void* params, int f32, cudaStream_t stream);
+int sb_hyper_rows(const void* params, int f32, cudaStream_t stream);
 int sb_scaled_act(const void* x, long long stride, const void* gain, void* out, long long rows, int I, int act, int f32,
                   cudaStream_t stream);
 int sb_stream_rows(const void* params, int f32, cudaStream_t stream);

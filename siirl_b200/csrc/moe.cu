@@ -456,3 +456,131 @@ extern "C" int sb_moe_build_layout(const int* idx, int P, int E, int world, int 
                                                                 slot_src_rank, slot_src_row);
   return (int)cudaGetLastError();
 }
+
+// ---------------------------------------------------------------------------------------
+// router with corrected, group-limited choice and identity experts, in 32-bit from the partial sums of its logits
+// ---------------------------------------------------------------------------------------
+// One warp per token, PL outputs per lane.  s = softmax(z) over all outputs; outputs are chosen by s + correction, only
+// inside the `keep` groups (of n_groups equal ones) whose best member is largest; the weights are s of the chosen ones over
+// their sum, times scale.  A group ranks by its best member, so the largest output outside the groups taken so far names
+// the next group.  Outputs >= experts are identity experts: they get id -1 (no slot) and their weights add up in w_id.
+template <int PL>
+__global__ void __launch_bounds__(256) moe_route_grouped_kernel(const float* __restrict__ z, long long slab, int slabs, int ld,
+                                                                const void* __restrict__ corr, int corr_f32,
+                                                                float* __restrict__ w, int* __restrict__ idx,
+                                                                float* __restrict__ w_id, int Tn, int E, int experts, int k,
+                                                                int n_groups, int keep, float scale) {
+  const int lane = threadIdx.x & 31, warps = (gridDim.x * blockDim.x) >> 5, size = E / n_groups;
+  for (int t = (blockIdx.x * blockDim.x + threadIdx.x) >> 5; t < Tn; t += warps) {
+    float s[PL], c[PL];
+    float mx = -INFINITY;
+#pragma unroll
+    for (int i = 0; i < PL; ++i) {
+      const int e = lane + 32 * i;
+      s[i] = -INFINITY;
+      if (e < E) {
+        const float* zp = z + (size_t)t * ld + e;
+        float v = zp[0];
+        for (int j = 1; j < slabs; ++j) v += zp[j * slab];
+        s[i] = v;
+      }
+      mx = fmaxf(mx, s[i]);
+    }
+    mx = warp_max(mx);
+    float sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < PL; ++i) {
+      s[i] = lane + 32 * i < E ? expf(s[i] - mx) : 0.f;
+      sum += s[i];
+    }
+    sum = warp_sum(sum);
+    unsigned kept = 0;
+#pragma unroll
+    for (int i = 0; i < PL; ++i) {
+      const int e = lane + 32 * i;
+      s[i] /= sum;
+      c[i] = -INFINITY;
+      if (e < E)
+        c[i] = s[i] + (corr_f32 ? reinterpret_cast<const float*>(corr)[e]
+                                : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(corr)[e]));
+    }
+    // largest of the outputs whose bit in `open` is set; ties go to the lower output
+    auto best_of = [&](unsigned open, float& score, int& id) {
+      score = -INFINITY;
+      id = 0x7fffffff;
+#pragma unroll
+      for (int i = 0; i < PL; ++i)
+        if ((open >> i & 1) && lane + 32 * i < E && (c[i] > score || id == 0x7fffffff)) {
+          score = c[i];
+          id = lane + 32 * i;
+        }
+#pragma unroll
+      for (int o = 16; o; o >>= 1) {
+        const float os = __shfl_xor_sync(0xffffffffu, score, o);
+        const int oi = __shfl_xor_sync(0xffffffffu, id, o);
+        if (os > score || (os == score && oi < id)) {
+          score = os;
+          id = oi;
+        }
+      }
+    };
+    for (int r = 0; r < keep; ++r) {
+      float score;
+      int id;
+      best_of(~kept, score, id);
+      const int grp = id / size;
+#pragma unroll
+      for (int i = 0; i < PL; ++i) {
+        const int e = lane + 32 * i;
+        if (e < E && e / size == grp) kept |= 1u << i;
+      }
+    }
+    unsigned open = kept;
+    float my_w = 0.f, total = 0.f;
+    int my_id = -1;
+    for (int j = 0; j < k; ++j) {
+      float score, mine = 0.f;
+      int id;
+      best_of(open, score, id);
+#pragma unroll
+      for (int i = 0; i < PL; ++i)
+        if (i == id >> 5) mine = s[i];
+      const float sw = __shfl_sync(0xffffffffu, mine, id & 31);
+      if ((id & 31) == lane) open &= ~(1u << (id >> 5));
+      total += sw;
+      if (lane == j) {
+        my_w = sw;
+        my_id = id;
+      }
+    }
+    my_w = my_w / (total + 1e-20f) * scale;
+    const bool ident = lane < k && my_id >= experts;
+    const float wi = warp_sum(ident ? my_w : 0.f);
+    if (lane < k) {
+      w[(size_t)t * k + lane] = my_w;
+      idx[(size_t)t * k + lane] = ident ? -1 : my_id;
+    }
+    if (lane == 0) w_id[t] = wi;
+  }
+}
+
+// z: [slabs, T, ld] fp32 partial sums of E router outputs, the last E - experts of them identity experts
+extern "C" int sb_moe_route_grouped(const float* z, long long slab, int slabs, int ld, const void* corr, int corr_f32,
+                                    float* w, int* idx, float* w_id, int T, int E, int experts, int k, int n_groups,
+                                    int keep, float scale, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (E < 1 || E > 512 || experts < 1 || experts > E || n_groups < 1 || E % n_groups || keep < 1 || keep > n_groups ||
+      k < 1 || k > 32 || k > keep * (E / n_groups) || slabs < 1)
+    return -3;
+  const int grid = moe_grid(T);
+  auto launch = [&](auto kernel) {
+    kernel<<<grid, 256, 0, stream>>>(z, slab, slabs, ld, corr, corr_f32, w, idx, w_id, T, E, experts, k, n_groups, keep,
+                                     scale);
+  };
+  if (E <= 32) launch(moe_route_grouped_kernel<1>);
+  else if (E <= 64) launch(moe_route_grouped_kernel<2>);
+  else if (E <= 128) launch(moe_route_grouped_kernel<4>);
+  else if (E <= 256) launch(moe_route_grouped_kernel<8>);
+  else launch(moe_route_grouped_kernel<16>);
+  return (int)cudaGetLastError();
+}

@@ -4,8 +4,11 @@
 //
 // One layer's cache is [num_blocks, block_elems]; a block holds 64 tokens as K [Hkv, 64, dk] then V [Hkv, 64, dv].
 // Query position i sees key position j when j <= i and (window == 0 or i - j < window or j < keep_first);
-// score = q . k * scale - slope_h * (i - j), slope_h = 2^(-bias_exp (h + 1) / Hq) (bias_exp == 0: no bias).
+// score = q . k * scale - slope_h * (i - j), slope_h = 2^(-bias_exp (h + 1) / Hq) (bias_exp == 0: no bias), or with a
+// soft cap and / or a table of distances cap * tanh(q . k * scale / cap) + rel[h, min(i - j, rel_n - 1)].  With a sink the
+// soft-max sum has one more term, of score 0 and without a value.
 #pragma once
+#include "common.cuh"
 
 namespace sb {
 
@@ -27,11 +30,26 @@ struct WinParams {
   const void* gain;         // one number that multiplies the queries and the gate, or null
   const void* gate;         // columns like out's: the result is multiplied by sigmoid(gain * gate) (prompts); null: none
   long long gate_stride;
+  float softcap;            // 0: none
+  int sink;
+  const float* rel;         // [Hq, rel_n] bias by distance, or null (bias_exp must be 0 then)
+  long long rel_n;
+  const float* head_gate;   // [T, Hq]: the result is multiplied by it, or null
 };
 // kPaged: as described above.  kPackedRows (prompts): `cache` is [num_blocks, block_elems], one row per KEY, keys of all
 // heads before values, and a tile's slot is the row of its sequence's first key.  kLatent (general kernel): keys and
 // values are the same dk-wide rows, [num_blocks, 64, dk].
 enum { kPaged = 0, kPackedRows = 1, kLatent = 2 };
-static_assert(sizeof(WinParams) == 168, "WinParams is mirrored from Python");
+static_assert(sizeof(WinParams) == 200, "WinParams is mirrored from Python");
+
+// soft cap in units of log 2 of a raw product x: 2 * log2(e) * scale / cap * x is the exponent's argument
+struct ScoreCap {
+  float in, out;            // cap * tanh(scale * x / cap) * log2(e) = out - 2 out / (1 + 2^(in x))
+  __device__ __forceinline__ ScoreCap(float cap, float scale)
+      : in(2.f * 1.4426950408889634f * scale / cap), out(cap * 1.4426950408889634f) {}
+  __device__ __forceinline__ float operator()(float x) const {
+    return out - __fdividef(2.f * out, 1.f + fast_exp2(in * x));
+  }
+};
 
 }  // namespace sb

@@ -99,7 +99,8 @@ class PrismaticConfig:
 @dataclass
 class MixerBranch:
     """One token mixer of a hybrid layer.  ``kind``: "attention" (paged cache, sliding window with kept first tokens,
-    linear distance bias), "latent_attention" (paged cache of one compressed row per token, from which every head's keys
+    linear or learned distance bias, rotation, query / key norms, soft-capped scores, a sink without value, gated heads),
+    "latent_attention" (paged cache of one compressed row per token, from which every head's keys
     and values are expanded), "gated_linear" (matrix state, decay per key channel) or "matrix_memory" (stabilised
     mLSTM)."""
     kind: str = "attention"
@@ -113,6 +114,17 @@ class MixerBranch:
     window: int = 0                 # 0: no limit
     keep_first: int = 0
     bias_exp: float = 8.0           # slope of head h: 2^(-bias_exp (h + 1) / heads); 0: no bias
+    proj_bias: bool = False         # biases on the projections of queries, keys, values and on the output matrix
+    qk_norm: str = ""               # "rows": RMS norm with weights over a whole projection, before the rotation;
+                                    # "heads": every head over its root mean square, after the rotation
+    rot_dims: int = 0               # rotated dimensions of a head (first half against second half); 0: no rotation
+    rot_base: float = 1e4
+    rot_scaling: Optional[Dict[str, Any]] = None     # factor, low, high, original: three-band scaling of frequencies
+    softcap: float = 0.0            # score -> softcap * tanh(score / softcap); 0: none
+    sink: bool = False              # one more key with score 0 and no value
+    rel_rows: int = 0               # rows of a learned distance table (the checkpoint's tensor shape); 0: none
+    rel_max: int = 0                # distance from which its last row is used
+    head_gate: bool = False         # heads times the sigmoid of one number each, projected from the mixer's input
     # latent_attention (with ``scale``)
     kv_rank: int = 0                # width of the cached row
     output_gate: bool = False       # heads times the sigmoid of a projection of the mixer's input
@@ -134,9 +146,34 @@ class MixerBranch:
 
 
 @dataclass
+class ExpertSpec:
+    """Routed feed-forward: gated experts, of which every token takes the ``top`` best by soft-max score plus correction
+    among the ``keep`` best of ``groups`` equal groups of neighbours; weights are the scores over their sum, times
+    ``scale``.  The last ``identity`` router outputs stand for the input itself."""
+    experts: int = 8
+    ff: int = 64
+    top: int = 2
+    groups: int = 1
+    keep: int = 1
+    identity: int = 0
+    scale: float = 1.0
+    shared_ff: int = 0              # width of an expert that takes every token; 0: none
+    act: str = "silu"
+
+    @property
+    def outputs(self) -> int:
+        return self.experts + self.identity
+
+
+@dataclass
 class HybridLayer:
     branches: List[MixerBranch] = field(default_factory=list)
-    ff: int = 0                     # 0: the layer has no feed-forward
+    ff: int = 0                     # 0: no dense feed-forward
+    moe: Optional[ExpertSpec] = None
+
+    @property
+    def has_ff(self) -> bool:
+        return self.ff > 0 or self.moe is not None
 
 
 @dataclass
@@ -151,15 +188,18 @@ class LayerLoop:
 class HybridSpec:
     """Decoders whose layers mix attention and recurrences; the residual stream is kept in 32-bit.
 
-    ``arrangement``: "sequential" (mixer, then feed-forward on the updated stream; vector norms, gated feed-forward) or
+    ``arrangement``: "sequential" (mixer, then feed-forward on the updated stream; vector norms, gated feed-forward),
     "parallel" (both read the same stream, ``x += residual_mult * (mixer(norm1 x) + ff(norm2 x))``; norms of one number
-    each, plain feed-forward, optionally a sigmoid gate per element on each of the two results)."""
+    each, plain feed-forward, optionally a sigmoid gate per element on each of the two results) or "hyper" (``streams``
+    copies of the stream: a sublayer reads a learned sum of them and every copy becomes a learned sum of all copies and
+    the sublayer's result; layer norms with biases, plain or routed feed-forward)."""
     layers: List[HybridLayer] = field(default_factory=list)
     embed_scale: float = 1.0
     logit_softcap: float = 0.0      # 0: none
     norm: str = "layer_norm"        # or "rms_norm"
-    act: str = "gelu_tanh"          # or "silu", "gelu" (exact)
+    act: str = "gelu_tanh"          # or "silu", "gelu" (exact), "relu2" (square of relu)
     arrangement: str = "sequential"
+    streams: int = 1                # "hyper"
     residual_mult: float = 1.0
     residual_gate: bool = False
     loop: Optional[LayerLoop] = None
@@ -326,6 +366,8 @@ class DecoderConfig:
 
     def _hybrid_parameters(self) -> int:
         hy, W = self.hybrid, self.hidden_size
+        if hy.arrangement == "hyper":
+            return self._hyper_parameters()
         parallel = hy.arrangement == "parallel"
         norm, ffs = (1, 2) if parallel else (W, 3)
         gate = W * (W + 1) if hy.residual_gate else 0
@@ -344,6 +386,21 @@ class DecoderConfig:
                     continue
                 n += W * (2 * hk + 3 * hv)
                 n += (b.rank * (W + hk) + hk + b.vdim) if b.kind == "gated_linear" else 2 * b.heads * (W + 1) + hv
+        return n
+
+    def _hyper_parameters(self) -> int:
+        hy, W = self.hybrid, self.hidden_size
+        conn = 2 * W + hy.streams * (hy.streams + 2)
+        n = 2 * self.vocab_size * W + 2 * W
+        for layer in hy.layers:
+            n += conn * (1 + int(layer.has_ff)) + 2 * W * layer.ff
+            for b in layer.branches:
+                hk, gk, gv, hv = b.heads * b.dim, b.kv_heads * b.dim, b.kv_heads * b.vdim, b.heads * b.vdim
+                n += W * (hk + gk + gv + hv) + (hk + gk + gv + W) * int(b.proj_bias) + (hk + gk) * int(b.qk_norm == "rows")
+                n += b.rel_rows * b.heads + W * b.heads * int(b.head_gate)
+            if layer.moe is not None:
+                e = layer.moe
+                n += 3 * W * (e.experts * e.ff + e.shared_ff) + e.outputs * (W + 1)
         return n
 
     def to_dict(self) -> Dict[str, Any]:
@@ -371,8 +428,8 @@ class DecoderConfig:
             d["prismatic"] = build(PrismaticConfig, pr)
         if isinstance(d.get("hybrid"), dict):
             hy = dict(d["hybrid"])
-            hy["layers"] = [build(HybridLayer, dict(x, branches=[build(MixerBranch, b) for b in x["branches"]]))
-                            for x in hy.get("layers", [])]
+            hy["layers"] = [build(HybridLayer, dict(x, branches=[build(MixerBranch, b) for b in x["branches"]],
+                                                    moe=build(ExpertSpec, x.get("moe")))) for x in hy.get("layers", [])]
             hy["loop"] = build(LayerLoop, hy.get("loop"))
             d["hybrid"] = build(HybridSpec, hy)
         for key in ("lora_targets", "mrope_section"):
@@ -384,8 +441,10 @@ class DecoderConfig:
     # ---- HF interchange -----------------------------------------------------------------------
     @classmethod
     def from_hf_config(cls, cfg: Dict[str, Any]) -> "DecoderConfig":
-        if cfg.get("architecture") in ("Domavik", "Poralorn"):
-            return cls._from_domavik_config(cfg) if cfg["architecture"] == "Domavik" else cls._from_poralorn_config(cfg)
+        own = {"Domavik": cls._from_domavik_config, "Poralorn": cls._from_poralorn_config,
+               "Gumazen": cls._from_gumazen_config}
+        if cfg.get("architecture") in own:
+            return own[cfg["architecture"]](cfg)
         text = cfg.get("text_config") or cfg.get("llm_config") or cfg
         mt = cfg.get("model_type", "qwen2")
         if mt in ("llama4", "llama4_text"):
@@ -648,6 +707,79 @@ class DecoderConfig:
         return d
 
     @classmethod
+    def _from_gumazen_config(cls, cfg: Dict[str, Any]) -> "DecoderConfig":
+        """Gumazen: three kinds of attention in any order, dense or routed feed-forwards, hyper-connections, a run of layers
+        that is repeated.  The rows of a distance table are not in the file: they are the shape of a tensor, filled in by
+        ``from_pretrained``."""
+        kinds = {"attention": dict(qk_norm="heads", sink=True), "attention_3": dict(qk_norm="rows", proj_bias=True),
+                 "attention_2": dict(qk_norm="rows", head_gate=True)}
+        layers = []
+        for x in cfg["layers"]:
+            m, mlp = x["mixer"], x.get("mlp")
+            if x["type"] not in kinds:
+                raise ValueError(f"unknown layer type {x['type']!r}")
+            b = MixerBranch(kind="attention", heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]),
+                            vdim=int(m["vdim"]), scale=float(m["scale"]), bias_exp=0.0, **kinds[x["type"]])
+            if x["type"] == "attention_2":
+                b.softcap, b.rel_max = float(m["softcap"]), int(m["bias_max"])
+                b.window = int(m["mask"]["size"])
+            else:
+                rot = m["rot"]
+                b.rot_dims, b.rot_base = int(rot["dims"]), float(rot["base"])
+                if x["type"] == "attention_3":
+                    b.rot_scaling = dict(rot["scaling"]) if rot.get("scaling") else None
+            layer = HybridLayer(branches=[b])
+            if mlp is not None and mlp["kind"] == "dense":
+                layer.ff = int(mlp["ff"])
+            elif mlp is not None and mlp["kind"] == "moe":
+                r, g = mlp["router"], mlp["router"].get("groups") or {"count": 1, "keep": 1}
+                layer.moe = ExpertSpec(experts=int(r["experts"]), ff=int(mlp["expert"]["ff"]), top=int(r["top"]),
+                                       groups=int(g["count"]), keep=int(g["keep"]), identity=int(r.get("identity") or 0),
+                                       scale=float(r.get("scale", 1.0)),
+                                       shared_ff=int(mlp["shared"]["ff"]) if mlp.get("shared") else 0)
+            elif mlp is not None:
+                raise ValueError(f"unknown feed-forward kind {mlp['kind']!r}")
+            layers.append(layer)
+        lp = cfg.get("loop")
+        spec = HybridSpec(layers=layers, norm="layer_norm", act="relu2", arrangement="hyper", streams=int(cfg["streams"]),
+                          loop=LayerLoop(int(lp["start"]), int(lp["stop"]), int(lp["times"])) if lp else None,
+                          hf_naming="gumazen")
+        spec.runs()
+        return cls.for_hybrid(spec, vocab_size=int(cfg["vocab"]), hidden_size=int(cfg["width"]),
+                              rms_norm_eps=float(cfg["norm"]["eps"]), model_type="gumazen",
+                              eos_token_id=int(cfg.get("eos_token_id", -1)), pad_token_id=int(cfg.get("pad_token_id", 0)))
+
+    def _to_gumazen_config(self) -> Dict[str, Any]:
+        hy, layers = self.hybrid, []
+        for x in hy.layers:
+            b, = x.branches
+            m: Dict[str, Any] = {n: getattr(b, n) for n in ("heads", "kv_heads", "dim", "vdim", "scale")}
+            if b.head_gate:
+                t = "attention_2"
+                m.update(softcap=b.softcap, bias_max=b.rel_max, mask={"size": b.window})
+            else:
+                t = "attention" if b.sink else "attention_3"
+                m["rot"] = {"base": b.rot_base, "dims": b.rot_dims}
+                if b.rot_scaling:
+                    m["rot"]["scaling"] = dict(b.rot_scaling)
+            mlp: Optional[Dict[str, Any]] = {"kind": "dense", "ff": x.ff} if x.ff else None
+            if x.moe is not None:
+                e = x.moe
+                mlp = {"kind": "moe", "expert": {"ff": e.ff},
+                       "router": {"experts": e.experts, "identity": e.identity, "top": e.top, "scale": e.scale,
+                                  "groups": {"count": e.groups, "keep": e.keep}}}
+                if e.shared_ff:
+                    mlp["shared"] = {"ff": e.shared_ff}
+            layers.append({"type": t, "mixer": m, "mlp": mlp})
+        d = {"architecture": "Gumazen", "vocab": self.vocab_size, "width": self.hidden_size,
+             "norm": {"eps": self.rms_norm_eps}, "streams": hy.streams, "layers": layers}
+        if hy.loop is not None:
+            d["loop"] = {"start": hy.loop.start, "stop": hy.loop.stop, "times": hy.loop.times}
+        if self.eos_token_id >= 0:
+            d["eos_token_id"] = self.eos_token_id
+        return d
+
+    @classmethod
     def from_pretrained(cls, path: str) -> "DecoderConfig":
         with open(os.path.join(os.path.expanduser(path), "config.json")) as f:
             out = cls.from_hf_config(json.load(f))
@@ -658,7 +790,8 @@ class DecoderConfig:
 
     def to_hf_config(self) -> Dict[str, Any]:
         if self.hybrid is not None:
-            return self._to_poralorn_config() if self.hybrid.hf_naming == "poralorn" else self._to_domavik_config()
+            return {"poralorn": self._to_poralorn_config, "gumazen": self._to_gumazen_config}.get(
+                self.hybrid.hf_naming, self._to_domavik_config)()
         arch = {"qwen2": "Qwen2ForCausalLM", "qwen3": "Qwen3ForCausalLM", "qwen3_moe": "Qwen3MoeForCausalLM",
                 "llama": "LlamaForCausalLM", "qwen2_5_vl": "Qwen2_5_VLForConditionalGeneration",
                 "mixtral": "MixtralForCausalLM", "qwen2_moe": "Qwen2MoeForCausalLM",
@@ -786,7 +919,33 @@ def _poralorn(n_layers: int, width: int, ff: int, vocab: int, heads: int, dim: i
                                     **kw)
 
 
+def _gumazen(n_layers: int, width: int, ff: int, vocab: int, heads: int, kv_heads: int, dim: int, window: int,
+             moe: ExpertSpec, rot_dims: int, streams: int = 2, loop: Optional[LayerLoop] = None, vdim: int = 0,
+             **kw) -> DecoderConfig:
+    """Gumazen layers in turn: rotated with biases, rotated with a sink, windowed with a distance table; the first layer
+    has a dense feed-forward, the others are routed."""
+    base = dict(kind="attention", heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim or dim, scale=dim ** -0.5, bias_exp=0.0)
+    kinds = [dict(qk_norm="rows", proj_bias=True, rot_dims=rot_dims, rot_base=1e6,
+                  rot_scaling={"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}),
+             dict(qk_norm="heads", sink=True, rot_dims=rot_dims, rot_base=5e4),
+             dict(qk_norm="rows", head_gate=True, softcap=50.0, rel_rows=32, rel_max=window // 2, window=window)]
+    layers = [HybridLayer([MixerBranch(**base, **kinds[i % 3])], ff=0 if i else ff, moe=moe if i else None)
+              for i in range(n_layers)]
+    spec = HybridSpec(layers=layers, act="relu2", arrangement="hyper", streams=streams, loop=loop, hf_naming="gumazen")
+    return DecoderConfig.for_hybrid(spec, vocab_size=vocab, hidden_size=width, rms_norm_eps=1e-5, model_type="gumazen", **kw)
+
+
 PRESETS: Dict[str, DecoderConfig] = {
+    "tiny-gumazen": _gumazen(3, 128, 192, 1024, heads=4, kv_heads=2, dim=32, vdim=24, window=70, rot_dims=16,
+                             moe=ExpertSpec(experts=6, ff=40, top=3, groups=2, keep=1, identity=2, scale=1.5, shared_ff=56),
+                             loop=LayerLoop(1, 3, 2)),
+    # layer sizes of decoders with about 1 / 3 billion active parameters (benchmark shapes, random weights)
+    "gumazen-a1b": _gumazen(18, 1536, 8960, 152064, heads=12, kv_heads=2, dim=128, window=1024, rot_dims=64,
+                            moe=ExpertSpec(experts=56, ff=768, top=6, groups=8, keep=4, identity=8, scale=2.0,
+                                           shared_ff=1536), loop=LayerLoop(3, 9, 2)),
+    "gumazen-a3b": _gumazen(18, 2048, 11264, 152064, heads=32, kv_heads=4, dim=128, window=1024, rot_dims=64,
+                            moe=ExpertSpec(experts=120, ff=1024, top=8, groups=8, keep=4, identity=8, scale=2.0,
+                                           shared_ff=2048), loop=LayerLoop(3, 9, 2)),
     "tiny-poralorn": _poralorn(3, 128, 224, 1024, heads=3, dim=24, vdim=40, kv_rank=48, loop=LayerLoop(1, 2, 3)),
     # layer sizes of a 7B / 1.5B-class decoder (benchmark shapes, random weights)
     "poralorn-7b": _poralorn(28, 3584, 18944, 152064, heads=28, dim=128, vdim=128, kv_rank=512, loop=LayerLoop(2, 6, 2)),

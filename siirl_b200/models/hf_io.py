@@ -336,8 +336,56 @@ def _poralorn_state(model) -> Iterator[Tuple[str, torch.Tensor]]:
     yield "head", model.lm_head.data
 
 
+def _gumazen_state(model) -> Iterator[Tuple[str, torch.Tensor]]:
+    """Gumazen checkpoint names and the views of the fused, padded parameters they fill (models/hybrid.py)."""
+    yield "embed", model.embed_tokens.data
+    for i, layer in enumerate(model.layers):
+        p, m = f"l{i}.", f"l{i}.mix."
+        for q, conn in enumerate(layer.connections(), 1):
+            yield p + f"norm{q}", conn.norm.data
+            yield p + f"norm{q}.b", conn.norm_bias.data
+            for name in ("in", "out", "mix"):
+                yield p + f"hc{q}.{name}", getattr(conn, "w_" + name).data
+        br, = layer.branches
+        for name, (at, n) in br.cols.items():
+            yield m + name, layer.in_proj_weight.data[at:at + n]
+            if br.b.proj_bias and name in ("q", "k", "v"):
+                yield m + name + ".b", br.bias.data[at:at + n]
+        yield m + "o", layer.o_proj_weight.data[:, :br.b.heads * br.b.vdim]
+        if br.b.proj_bias:
+            yield m + "o.b", layer.o_proj_bias.data
+        if br.b.qk_norm == "rows":
+            yield m + "q.norm", br.q_norm.data
+            yield m + "k.norm", br.k_norm.data
+        if br.b.rel_rows:
+            yield m + "rel", br.rel.data
+        if layer.ff:
+            yield p + "mlp.up", layer.up_proj_weight.data[:layer.ff]
+            yield p + "mlp.down", layer.down_proj_weight.data[:, :layer.ff]
+        if layer.moe is not None:
+            x, e = layer.moe, layer.moe.spec
+
+            def gated(prefix, gate_up, down, ff):
+                pad = gate_up.shape[0] // 2
+                yield prefix + "gate", gate_up[:ff]
+                yield prefix + "up", gate_up[pad:pad + ff]
+                yield prefix + "down", down[:, :ff]
+            yield p + "mlp.router", x.router_weight.data[:e.outputs]
+            yield p + "mlp.correction", x.correction.data
+            for j in range(e.experts):
+                yield from gated(p + f"mlp.e{j}.", x.gate_up_weight.data[j], x.down_weight.data[j], e.ff)
+            if e.shared_ff:
+                yield from gated(p + "mlp.shared.", x.shared_gate_up_weight.data, x.shared_down_weight.data, e.shared_ff)
+    yield "final.norm", model.norm.data
+    yield "final.norm.b", model.norm_bias.data
+    yield "head", model.lm_head.data
+
+
+_HYBRID_STATE = {"domavik": _domavik_state, "poralorn": _poralorn_state, "gumazen": _gumazen_state}
+
+
 def fill_hybrid_ranks(cfg: DecoderConfig, path: str) -> None:
-    """Sizes that only tensor shapes give: the low-rank width of every decay projection."""
+    """Sizes that only tensor shapes give: the low-rank width of every decay projection, the rows of distance tables."""
     handles = _open_all(path)
     where = {k: h for h in handles for k in h.keys()}
     for i, layer in enumerate(cfg.hybrid.layers):
@@ -347,6 +395,11 @@ def fill_hybrid_ranks(cfg: DecoderConfig, path: str) -> None:
                 if name not in where:
                     raise KeyError(f"{name} missing in {path}")
                 b.rank = int(where[name].get_slice(name).get_shape()[0])
+            elif b.rel_max and not b.rel_rows:
+                name = f"l{i}.mix.rel"
+                if name not in where:
+                    raise KeyError(f"{name} missing in {path}")
+                b.rel_rows = int(where[name].get_slice(name).get_shape()[0])
 
 
 def _hf_targets(model) -> Iterator[Tuple[str, object]]:
@@ -354,7 +407,7 @@ def _hf_targets(model) -> Iterator[Tuple[str, object]]:
     fused ``wqkv`` comes as the tuple of its three views."""
     cfg: DecoderConfig = model.cfg
     if cfg.hybrid is not None:
-        yield from (_poralorn_state if cfg.hybrid.hf_naming == "poralorn" else _domavik_state)(model)
+        yield from _HYBRID_STATE[cfg.hybrid.hf_naming](model)
         return
     prefix, head = _llm_names(cfg)
     internlm2 = cfg.vit is not None and cfg.hf_naming == "internvl_chat" and cfg.llm_type == "internlm2"

@@ -6,7 +6,8 @@ matrix (``in_proj``), each branch writes its (scaled) heads into its columns of 
 the branches up.  In the parallel arrangement the feed-forward reads the same stream and the residual gates read the
 sublayers' inputs, so their matrices join ``in_proj``: the norms there are one number each, which commutes with the
 projections, and one row (the stream over its root mean square) feeds them all; the numbers are applied by the kernels
-behind.  A run of layers may be repeated (``HybridSpec.loop``).
+behind.  In the hyper arrangement several copies of the stream are mixed between sublayers, the mixers are attention of
+several kinds and a feed-forward may be routed.  A run of layers may be repeated (``HybridSpec.loop``).
 
 The serving path is the one of :class:`DecoderLM`: ``forward_cached`` over the engine's paged blocks, plus the engine's
 per-slot recurrent states.  A prompt portion appends its keys and values and reads everything it sees back from the
@@ -18,6 +19,7 @@ the checkpoint's values; fused matrices are padded with zero rows / columns to m
 from __future__ import annotations
 
 import ctypes
+from dataclasses import replace
 from typing import Dict, List, Optional, Sequence, Tuple
 
 import torch
@@ -31,8 +33,10 @@ from ..ops.dense import linear_partial
 from ..ops.latent_attention import LatentPlan, LatentSpec, latent_attention
 from ..ops.lm_head import lm_head_logits
 from ..ops.recurrence import PortionPlan, RecurrenceSpec, empty_state, recurrence_decode, recurrence_prefill
-from ..ops.window_attention import QueryTiles, WindowSpec, window_attention
-from .config import DecoderConfig, MixerBranch
+from ..ops.moe import route_grouped, routed_experts
+from ..ops.window_attention import (QkvPrepare, QueryTiles, WindowSpec, distance_buckets, rotary_frequencies,
+                                    window_attention)
+from .config import DecoderConfig, ExpertSpec, MixerBranch
 from .decoder import _Init, _param
 
 
@@ -44,7 +48,7 @@ def branch_segments(b: MixerBranch) -> List[Tuple[str, int]]:
     """(name, rows) of a branch's projections in ``in_proj``, in order."""
     hk, hv = b.heads * b.dim, b.heads * b.vdim
     if b.kind == "attention":
-        return [("q", hk), ("k", b.kv_heads * b.dim), ("v", b.kv_heads * b.vdim)]
+        return [("q", hk), ("k", b.kv_heads * b.dim), ("v", b.kv_heads * b.vdim)] + ([("g", b.heads)] if b.head_gate else [])
     if b.kind == "latent_attention":
         return [("q", hk), ("c", b.kv_rank)] + ([("g", hv)] if b.output_gate else [])
     seg = [("q", hk), ("k", hk), ("v", hv), ("g", hv)]
@@ -66,7 +70,8 @@ class HybridBranch(nn.Module):
         off = {k: v[0] for k, v in self.cols.items()}
         if b.kind == "attention":
             self.spec = WindowSpec(b.heads, b.kv_heads, b.dim, b.vdim, off["q"], off["k"], off["v"], b.scale, b.window,
-                                   b.keep_first, b.bias_exp, b.out_scale)
+                                   b.keep_first, b.bias_exp, b.out_scale, b.softcap, b.sink)
+            self.prepare = self._prepare(cfg, in_off, off, dtype, device, gen)
             return
         hk, hv = b.heads * b.dim, b.heads * b.vdim
         if b.kind == "latent_attention":
@@ -95,6 +100,31 @@ class HybridBranch(nn.Module):
         else:
             raise ValueError(f"unknown mixer {b.kind!r}")
 
+    def _prepare(self, cfg: DecoderConfig, rows: int, off: Dict[str, int], dtype, device, gen) -> Optional[QkvPrepare]:
+        """Parameters and tables of what an attention branch does to its projections; ``None``: nothing."""
+        b = self.b
+        if not (b.proj_bias or b.qk_norm or b.rot_dims or b.rel_max or b.head_gate):
+            return None
+        if b.rot_dims % 2 or b.rot_dims > b.dim or b.heads % b.kv_heads or b.qk_norm not in ("", "rows", "heads"):
+            raise ValueError("attention: rotated dimensions, head counts or query / key norm")
+        pr = QkvPrepare(norm=b.qk_norm, eps=cfg.rms_norm_eps, g_off=off.get("g", -1))
+        if b.proj_bias:
+            self.bias = _param((rows - off["q"],), dtype, device, 0, gen)
+        if b.qk_norm == "rows":
+            self.q_norm = _param((b.heads * b.dim,), dtype, device, -1, gen)
+            self.k_norm = _param((b.kv_heads * b.dim,), dtype, device, -1, gen)
+        if b.rot_dims:
+            f = torch.tensor(rotary_frequencies(b.rot_dims, b.rot_base, b.rot_scaling), dtype=torch.float64)
+            hi = f.float()
+            pr.freq = torch.stack([hi, (f - hi.double()).float()], 1).to(device)
+        if b.rel_max:
+            if b.rel_rows < 1:
+                raise ValueError("attention: the rows of the distance table are not set")
+            self.rel = _param((b.rel_rows, b.heads), dtype, device, 1.0, gen)
+            pr.bucket = torch.tensor(distance_buckets(b.rel_rows, b.rel_max, b.window), dtype=torch.int32).to(device)
+            pr.table = torch.empty(b.heads, pr.bucket.numel(), dtype=torch.float32, device=device)
+        return pr
+
     @property
     def recurrent(self) -> bool:
         return self.b.recurrent
@@ -111,7 +141,10 @@ class HybridBranch(nn.Module):
                              self.out_off, plan=io.latent)
         elif self.b.kind == "attention":
             window_attention(self.spec, p, io.seq_ids, io.positions, io.block_table, io.next_cache(), out, self.out_off,
-                             tiles=io.tiles, seq_lens=io.seq_lens)
+                             tiles=io.tiles, seq_lens=io.seq_lens,
+                             prepare=self.prepare and replace(self.prepare, **{
+                                 k: getattr(self, k).detach() for k in ("bias", "q_norm", "k_norm", "rel")
+                                 if hasattr(self, k)}))
         elif io.plan is not None:
             recurrence_prefill(self.spec, p, self.weights(), io.next_state(), io.plan, out, self.out_off)
         else:
@@ -231,6 +264,116 @@ class ParallelLayer(nn.Module):
         return out
 
 
+class Connection(nn.Module):
+    """Hyper-connection and norm of one sublayer: what it reads from the copies of the stream and how they change."""
+
+    def __init__(self, cfg: DecoderConfig, dtype, device, gen):
+        super().__init__()
+        S, W = cfg.hybrid.streams, cfg.hidden_size
+        self.norm = _param((W,), dtype, device, -1, gen)
+        self.norm_bias = _param((W,), dtype, device, 0, gen)
+        self.w_in = _param((S,), dtype, device, 0, gen)
+        self.w_out = _param((S,), dtype, device, -1, gen)
+        self.w_mix = _param((S, S), dtype, device, 0, gen)
+        with torch.no_grad():
+            self.w_in.fill_(1.0 / S)
+            self.w_mix.copy_(torch.eye(S))
+
+
+class RoutedFeedForward(nn.Module):
+    """Router, gated experts, identity experts and an expert that takes every token (:class:`ExpertSpec`)."""
+
+    def __init__(self, e: ExpertSpec, W: int, std: float, dtype, device, gen):
+        super().__init__()
+        if e.outputs % e.groups or not 1 <= e.keep <= e.groups or e.top > e.keep * (e.outputs // e.groups):
+            raise ValueError(f"{e.top} of {e.outputs} router outputs in {e.keep} of {e.groups} groups")
+        self.spec, ffp, sp = e, _pad8(e.ff), _pad8(e.shared_ff)
+        self.router_weight = _param((_pad8(e.outputs), W), dtype, device, std, gen)
+        self.correction = _param((e.outputs,), dtype, device, 0, gen)
+        self.gate_up_weight = _param((e.experts, 2 * ffp, W), dtype, device, std, gen)
+        self.down_weight = _param((e.experts, W, ffp), dtype, device, std, gen)
+        pads = [(self.gate_up_weight, self.down_weight, e.ff, ffp)]
+        if e.shared_ff:
+            self.shared_gate_up_weight = _param((2 * sp, W), dtype, device, std, gen)
+            self.shared_down_weight = _param((W, sp), dtype, device, std, gen)
+            pads.append((self.shared_gate_up_weight, self.shared_down_weight, e.shared_ff, sp))
+        with torch.no_grad():
+            self.router_weight[e.outputs:] = 0
+            for gate_up, down, ff, pad in pads:
+                gate_up[..., ff:pad, :] = 0
+                gate_up[..., pad + ff:, :] = 0
+                down[..., ff:] = 0
+
+    def run(self, x: torch.Tensor) -> R.SublayerSum:
+        e = self.spec
+        z = linear_partial(x, self.router_weight.detach(), f32=True)
+        w, ids, w_id = route_grouped(z, self.correction.detach(), e.experts, e.top, e.groups, e.keep, e.scale)
+        ys, slots = routed_experts(x, ids, self.gate_up_weight.detach(), self.down_weight.detach(), e.act)
+        out = R.SublayerSum(ys=ys, pair_slot=slots, pair_w=w)
+        if e.identity:
+            out.x_id, out.w_id = x, w_id
+        if e.shared_ff:
+            a = R.gated_act(ops.linear(x, self.shared_gate_up_weight), e.act)
+            out.y = linear_partial(a, self.shared_down_weight.detach())
+        return out
+
+
+class HyperLayer(nn.Module):
+    """Attention and a dense or routed feed-forward around copies of the stream (see :class:`HybridSpec`)."""
+
+    def __init__(self, cfg: DecoderConfig, index: int, dtype, device, gen):
+        super().__init__()
+        hy, W, std = cfg.hybrid, cfg.hidden_size, cfg.initializer_range
+        lay = hy.layers[index]
+        if len(lay.branches) != 1 or lay.branches[0].kind != "attention" or hy.norm != "layer_norm" or hy.streams < 1:
+            raise ValueError("hyper-connected layers: one attention branch and layer norms")
+        self.cfg, self.ff, self.ffp = cfg, lay.ff, _pad8(lay.ff)
+        b = lay.branches[0]
+        br = HybridBranch(b, cfg, 0, 0, dtype, device, gen)
+        self.branches = nn.ModuleList([br])
+        heads = b.heads * b.vdim
+        self.in_proj_weight = _param((br.in_end, W), dtype, device, std, gen)
+        self.o_proj_weight = _param((W, _pad8(heads)), dtype, device, std, gen)
+        self.o_proj_bias = _param((W,), dtype, device, 0, gen) if b.proj_bias else None
+        self.mixer_connection = Connection(cfg, dtype, device, gen)
+        self.ff_connection = Connection(cfg, dtype, device, gen) if lay.has_ff else None
+        self.moe = RoutedFeedForward(lay.moe, W, std, dtype, device, gen) if lay.moe is not None else None
+        if self.ff:
+            self.up_proj_weight = _param((self.ffp, W), dtype, device, std, gen)
+            self.down_proj_weight = _param((W, self.ffp), dtype, device, std, gen)
+        with torch.no_grad():
+            for at, n in br.cols.values():
+                self.in_proj_weight[at + n:at + _pad8(n)] = 0
+            self.o_proj_weight[:, heads:] = 0
+            if self.ff:
+                self.up_proj_weight[self.ff:] = 0
+                self.down_proj_weight[:, self.ff:] = 0
+
+    def connections(self) -> List[Connection]:
+        return [self.mixer_connection] + ([self.ff_connection] if self.ff_connection is not None else [])
+
+    def sublayers(self):
+        """``(connection, function of its normed rows)`` in order."""
+        yield self.mixer_connection, self.mix
+        if self.ff_connection is not None:
+            yield self.ff_connection, self.feed_forward
+
+    def mix(self, x: torch.Tensor, io: "_Batch") -> R.SublayerSum:
+        br, = self.branches
+        p = linear_partial(x, self.in_proj_weight.detach())
+        alloc = torch.zeros if br.b.heads * br.b.vdim % 8 else torch.empty
+        heads = alloc(x.shape[0], self.o_proj_weight.shape[1], dtype=x.dtype, device=x.device)
+        br.run(p, io, heads)
+        return R.SublayerSum(linear_partial(heads, self.o_proj_weight.detach()),
+                             self.o_proj_bias.detach() if self.o_proj_bias is not None else None)
+
+    def feed_forward(self, x: torch.Tensor, io: "_Batch") -> R.SublayerSum:
+        if self.moe is not None:
+            return self.moe.run(x)
+        a = R.scaled_act(ops.linear(x, self.up_proj_weight), self.cfg.hybrid.act)
+        return R.SublayerSum(linear_partial(a, self.down_proj_weight.detach()))
+
+
 class _Batch:
     """What one forward pass needs besides the rows: places in the cache, prompt portions or decode lengths."""
 
@@ -258,16 +401,19 @@ class HybridLM(nn.Module):
         gen = _Init(seed, device)
         std = cfg.initializer_range
         self.embed_tokens = _param((cfg.vocab_size, cfg.hidden_size), dtype, device, std, gen)
-        self.parallel = cfg.hybrid.arrangement == "parallel"
-        if cfg.hybrid.arrangement not in ("sequential", "parallel") or (cfg.hybrid.loop is not None and not self.parallel):
-            raise ValueError("layer arrangements: sequential, or parallel with an optional loop")
-        kind = ParallelLayer if self.parallel else HybridLayer
-        self.layers = nn.ModuleList([kind(cfg, i, dtype, device, gen) for i in range(cfg.num_layers)])
-        if cfg.hybrid.loop is not None:
+        kinds = {"sequential": HybridLayer, "parallel": ParallelLayer, "hyper": HyperLayer}
+        self.arrangement = cfg.hybrid.arrangement
+        self.parallel = self.arrangement == "parallel"
+        if self.arrangement not in kinds or (cfg.hybrid.loop is not None and self.arrangement == "sequential"):
+            raise ValueError("layer arrangements: sequential, or parallel or hyper with an optional loop")
+        self.layers = nn.ModuleList([kinds[self.arrangement](cfg, i, dtype, device, gen) for i in range(cfg.num_layers)])
+        if cfg.hybrid.loop is not None and self.parallel:
             W = cfg.hidden_size
             self.loop_in_weight = _param((W, 2 * W), dtype, device, (2 * W) ** -0.5, gen)
             self.loop_step = _param((cfg.hybrid.loop.times, W), dtype, device, std, gen)
         self.norm = _param(() if self.parallel else (cfg.hidden_size,), dtype, device, -1, gen)
+        if self.arrangement == "hyper":
+            self.norm_bias = _param((cfg.hidden_size,), dtype, device, 0, gen)
         self.lm_head = _param((cfg.vocab_size, cfg.hidden_size), dtype, device, std, gen)
 
     @property
@@ -287,6 +433,8 @@ class HybridLM(nn.Module):
         cfg = self.cfg
         if self.parallel:
             return self._parallel_layers(ids, io)
+        if self.arrangement == "hyper":
+            return self._hyper_layers(ids, io)
         kind, eps = cfg.hybrid.norm, cfg.rms_norm_eps
         h = R.embed_scaled(ids, self.embed_tokens.detach(), cfg.hybrid.embed_scale)
         delta = None
@@ -315,6 +463,16 @@ class HybridLM(nn.Module):
                 x = R.enter_pass(h, linear_partial(parts, w_in[:, :W], f32=True), base, self.loop_step.detach()[t], eps)
             subs = self.layers[i].run(x, io)
         return R.stream_update(h, subs, mult, dtype, eps, weight=self.norm.detach())
+
+    def _hyper_layers(self, ids: torch.Tensor, io: _Batch) -> torch.Tensor:
+        hy, eps, W = self.cfg.hybrid, self.cfg.rms_norm_eps, self.cfg.hidden_size
+        h = torch.empty(ids.shape[0], hy.streams, W, dtype=torch.float32, device=ids.device)
+        step = dict(ids=ids.to(torch.int64).contiguous(), table=self.embed_tokens.detach())
+        for i, _ in hy.runs():
+            for conn, fn in self.layers[i].sublayers():
+                x = R.hyper_rows(h, conn.norm.detach(), conn.norm_bias.detach(), eps, w_in=conn.w_in.detach(), **step)
+                step = dict(result=fn(x, io), w_out=conn.w_out.detach(), w_mix=conn.w_mix.detach())
+        return R.hyper_rows(h, self.norm.detach(), self.norm_bias.detach(), eps, **step)
 
     @torch.no_grad()
     def forward_cached(self, input_ids: torch.Tensor, positions: torch.Tensor, cache: Sequence[torch.Tensor],

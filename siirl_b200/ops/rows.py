@@ -12,7 +12,13 @@ import torch.nn.functional as F
 
 from . import lib as _lib
 
-ACT = {"silu": 0, "gelu_tanh": 1, "gelu": 2}
+ACT = {"silu": 0, "gelu_tanh": 1, "gelu": 2, "relu2": 3}
+
+
+def _act(z: torch.Tensor, act: str) -> torch.Tensor:
+    if act == "relu2":
+        return F.relu(z).square()
+    return F.silu(z) if act == "silu" else F.gelu(z, approximate="tanh" if act == "gelu_tanh" else "none")
 
 
 def _f32(t: torch.Tensor) -> int:
@@ -50,16 +56,17 @@ def add_norm(h: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Tenso
     return y
 
 
-def gated_act(gate_up: torch.Tensor, act: str = "gelu_tanh") -> torch.Tensor:
-    """``act(gate) * up`` for a fused projection ``[T, 2 I]`` = ``[gate | up]``."""
+def gated_act(gate_up: torch.Tensor, act: str = "gelu_tanh", used: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``act(gate) * up`` for a fused projection ``[T, 2 I]`` = ``[gate | up]``.  Rows with a negative entry in ``used``
+    (int32) may be left unwritten."""
     T, I2 = gate_up.shape
     if not gate_up.is_cuda:
         g, u = gate_up.float().chunk(2, -1)
-        return ((F.silu(g) if act == "silu" else F.gelu(g, approximate="tanh" if act == "gelu_tanh" else "none")) * u).to(gate_up.dtype)
+        return (_act(g, act) * u).to(gate_up.dtype)
     gate_up = gate_up.contiguous()
     out = torch.empty(T, I2 // 2, dtype=gate_up.dtype, device=gate_up.device)
     _lib.check(_lib.get_lib().sb_gated_act(_lib.ptr(gate_up), _lib.ptr(out), ctypes.c_longlong(T), I2 // 2, ACT[act],
-                                           _f32(gate_up), _lib.stream()), "sb_gated_act")
+                                           _lib.ptr(used), _f32(gate_up), _lib.stream()), "sb_gated_act")
     return out
 
 
@@ -67,8 +74,7 @@ def scaled_act(x: torch.Tensor, act: str, gain: Optional[torch.Tensor] = None) -
     """``act(gain * x)`` of a column range ``x [T, I]`` of wider rows; ``gain``: one number (a tensor)."""
     if not x.is_cuda:
         z = x.float() * (gain.float() if gain is not None else 1.0)
-        y = F.silu(z) if act == "silu" else F.gelu(z, approximate="tanh" if act == "gelu_tanh" else "none")
-        return y.to(x.dtype)
+        return _act(z, act).to(x.dtype)
     assert x.stride(1) == 1
     out = torch.empty(x.shape, dtype=x.dtype, device=x.device)
     _lib.check(_lib.get_lib().sb_scaled_act(_lib.ptr(x), ctypes.c_longlong(x.stride(0)), _lib.ptr(gain), _lib.ptr(out),
@@ -163,6 +169,86 @@ def enter_pass(h: torch.Tensor, mixed: torch.Tensor, base: torch.Tensor, step: t
                 sub=(_Sub * 2)(_sub(Sublayer(mixed), W), _sub(Sublayer(base), W)), step=step.data_ptr(),
                 pair=int(mixed.shape[1] == 2 * T), out=out.data_ptr())
     _lib.check(_lib.get_lib().sb_stream_rows(ctypes.byref(p), _f32(step), _lib.stream()), "sb_stream_rows")
+    return out
+
+
+@dataclass
+class SublayerSum:
+    """Result of a sublayer on its way into hyper-connected streams: ``y [S, T, W]`` (partial sums, or one tensor in the
+    activation format) plus a bias, plus routed rows ``ys[pair_slot[t, j]] * pair_w[t, j]`` (slot -1: none), plus the
+    sublayer's input ``x_id [T, W]`` times ``w_id [T]``; every part may be missing."""
+    y: Optional[torch.Tensor] = None
+    bias: Optional[torch.Tensor] = None
+    ys: Optional[torch.Tensor] = None
+    pair_slot: Optional[torch.Tensor] = None
+    pair_w: Optional[torch.Tensor] = None
+    x_id: Optional[torch.Tensor] = None
+    w_id: Optional[torch.Tensor] = None
+
+
+class _Hyper(ctypes.Structure):
+    """Mirror of ``HyperParams`` in csrc/hyper_rows.cu."""
+    _fields_ = [("h", ctypes.c_void_p), ("rows", ctypes.c_int), ("S", ctypes.c_int), ("W", ctypes.c_int),
+                ("vocab", ctypes.c_int), ("ids", ctypes.c_void_p), ("table", ctypes.c_void_p), ("y", ctypes.c_void_p),
+                ("slab", ctypes.c_longlong), ("slabs", ctypes.c_int), ("y_f32", ctypes.c_int), ("bias", ctypes.c_void_p),
+                ("ys", ctypes.c_void_p), ("pair_slot", ctypes.c_void_p), ("pair_w", ctypes.c_void_p),
+                ("w_id", ctypes.c_void_p), ("x_id", ctypes.c_void_p), ("top", ctypes.c_int), ("eps", ctypes.c_float),
+                ("w_mix", ctypes.c_void_p), ("w_out", ctypes.c_void_p), ("w_in", ctypes.c_void_p),
+                ("norm_w", ctypes.c_void_p), ("norm_b", ctypes.c_void_p), ("out", ctypes.c_void_p)]
+
+
+assert ctypes.sizeof(_Hyper) == 168
+
+
+def hyper_rows(h: torch.Tensor, norm_w: torch.Tensor, norm_b: torch.Tensor, eps: float, *,
+               w_in: Optional[torch.Tensor] = None, result: Optional[SublayerSum] = None,
+               w_out: Optional[torch.Tensor] = None, w_mix: Optional[torch.Tensor] = None,
+               ids: Optional[torch.Tensor] = None, table: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """One step between two sublayers of a decoder with hyper-connections, ``h [T, S, W]`` fp32 in place: the copies become
+    ``table[ids]`` (``ids`` given), or ``h_t <- sum_s w_mix[s, t] h_s + w_out[t] * result`` (``result`` given); returns the
+    layer norm (weight and bias) of ``sum_s w_in[s] h_s`` in the weight's format, ``w_in = None``: of the plain sum."""
+    T, S, W = h.shape
+    assert h.dtype == torch.float32 and h.is_contiguous() and not (ids is not None and result is not None)
+    r = result
+    if not h.is_cuda:
+        if ids is not None:
+            h.copy_(F.embedding(ids, table).float()[:, None].expand(T, S, W))
+        elif r is not None:
+            y = torch.zeros(T, W)
+            if r.y is not None:
+                y = y + r.y.float().sum(0)
+            if r.bias is not None:
+                y = y + r.bias.float()
+            if r.ys is not None:
+                slot, k = r.pair_slot.reshape(T, -1).long(), r.pair_w.shape[1]
+                for j in range(k):
+                    y = y + torch.where((slot[:, j] >= 0)[:, None],
+                                        r.pair_w[:, j, None] * r.ys[slot[:, j].clamp(min=0)].float(), torch.zeros(()))
+            if r.w_id is not None:
+                y = y + r.w_id[:, None] * r.x_id.float()
+            h.copy_(torch.einsum("st,nsw->ntw", w_mix.float(), h) + w_out.float()[None, :, None] * y[:, None])
+        u = h.sum(1) if w_in is None else torch.einsum("s,nsw->nw", w_in.float(), h)
+        return F.layer_norm(u, (W,), norm_w.float(), norm_b.float(), eps).to(norm_w.dtype)
+    out = torch.empty(T, W, dtype=norm_w.dtype, device=h.device)
+    ptr = lambda t: t.data_ptr() if t is not None else None  # noqa: E731
+    p = _Hyper(h=h.data_ptr(), rows=T, S=S, W=W, eps=eps, w_in=ptr(w_in), norm_w=ptr(norm_w), norm_b=ptr(norm_b),
+               out=out.data_ptr())
+    if ids is not None:
+        assert ids.dtype == torch.int64 and ids.is_contiguous() and table.dtype == out.dtype
+        p.ids, p.table, p.vocab = ids.data_ptr(), table.data_ptr(), table.shape[0]
+    if r is not None:
+        p.w_mix, p.w_out, p.bias = w_mix.data_ptr(), w_out.data_ptr(), ptr(r.bias)
+        if r.y is not None:
+            assert r.y.is_contiguous() and r.y.shape[1:] == (T, W)
+            p.y, p.slab, p.slabs, p.y_f32 = r.y.data_ptr(), T * W, r.y.shape[0], _f32(r.y)
+            assert p.y_f32 or p.slabs == 1
+        if r.ys is not None:
+            assert r.ys.is_contiguous() and r.ys.dtype == out.dtype and r.pair_w.dtype == torch.float32
+            p.ys, p.pair_slot, p.pair_w, p.top = r.ys.data_ptr(), ptr(r.pair_slot), ptr(r.pair_w), r.pair_w.shape[1]
+        if r.w_id is not None:
+            assert r.x_id.is_contiguous() and r.x_id.dtype == out.dtype
+            p.w_id, p.x_id = r.w_id.data_ptr(), r.x_id.data_ptr()
+    _lib.check(_lib.get_lib().sb_hyper_rows(ctypes.byref(p), int(out.dtype == torch.float32), _lib.stream()), "sb_hyper_rows")
     return out
 
 

@@ -1,16 +1,20 @@
-"""Attention over a paged cache with a sliding window, kept first tokens and a linear distance bias.
+"""Attention over a paged cache with a sliding window, kept first tokens and a linear distance bias, or with a soft cap, a
+learned distance table, a sink and gated heads, and what comes before it: norms and rotation of queries and keys.
 
 Position ``i`` sees ``j <= i`` with ``i - j < window`` (``window == 0``: no limit) or ``j < keep_first``; the score is
-``q . k * scale - slope_h (i - j)`` with ``slope_h = 2^(-bias_exp (h + 1) / heads)`` (``bias_exp == 0``: no bias).
+``q . k * scale - slope_h (i - j)`` with ``slope_h = 2^(-bias_exp (h + 1) / heads)`` (``bias_exp == 0``: no bias), or
+``cap * tanh(q . k * scale / cap) + table[h, i - j]``.  A sink adds one to the soft-max's sum (score 0, no value).
 
 One layer's cache is ``[blocks, block_elems]``: a block holds 64 tokens, keys ``[kv_heads, 64, dim]`` then values
 ``[kv_heads, 64, vdim]``.  CUDA: ``csrc/fmha_window.cu`` (prompt portions on the tensor cores, any size and 32-bit on a
-SIMT kernel) and the windowed variant of ``csrc/fmha_decode_split.cu`` (single tokens).  CPU: the plain loop below."""
+SIMT kernel) and the windowed variant of ``csrc/fmha_decode_split.cu`` (single tokens); ``csrc/qkv_prepare.cu`` does
+biases, norms, rotation and the append in one launch.  CPU: the plain loop below."""
 from __future__ import annotations
 
 import ctypes
-from dataclasses import dataclass
-from typing import Dict, List, Sequence, Tuple
+import math
+from dataclasses import dataclass, replace
+from typing import Any, Dict, List, Optional, Sequence, Tuple
 
 import torch
 
@@ -34,6 +38,8 @@ class WindowSpec:
     keep_first: int = 0
     bias_exp: float = 0.0
     out_scale: float = 1.0
+    softcap: float = 0.0
+    sink: bool = False
 
     @property
     def block_elems(self) -> int:
@@ -51,11 +57,131 @@ class _Params(ctypes.Structure):
                 ("scale", ctypes.c_float), ("bias_exp", ctypes.c_float), ("out_scale", ctypes.c_float),
                 ("out", ctypes.c_void_p), ("out_stride", ctypes.c_longlong),
                 ("out_off", ctypes.c_int), ("kv_mode", ctypes.c_int),
-                ("gain", ctypes.c_void_p), ("gate", ctypes.c_void_p), ("gate_stride", ctypes.c_longlong)]
+                ("gain", ctypes.c_void_p), ("gate", ctypes.c_void_p), ("gate_stride", ctypes.c_longlong),
+                ("softcap", ctypes.c_float), ("sink", ctypes.c_int), ("rel", ctypes.c_void_p),
+                ("rel_n", ctypes.c_longlong), ("head_gate", ctypes.c_void_p)]
 
 
-assert ctypes.sizeof(_Params) == 168
+assert ctypes.sizeof(_Params) == 200
 KV_PAGED, KV_PACKED, KV_LATENT = 0, 1, 2
+
+
+class _PrepareParams(ctypes.Structure):
+    """Mirror of ``PrepareParams`` in csrc/qkv_prepare.cu."""
+    _fields_ = [("x", ctypes.c_void_p), ("slab", ctypes.c_longlong), ("row_stride", ctypes.c_longlong),
+                ("slabs", ctypes.c_int), ("x_f32", ctypes.c_int), ("bias", ctypes.c_void_p),
+                ("q_off", ctypes.c_int), ("k_off", ctypes.c_int), ("v_off", ctypes.c_int), ("g_off", ctypes.c_int),
+                ("T", ctypes.c_int), ("Hq", ctypes.c_int), ("Hkv", ctypes.c_int), ("dk", ctypes.c_int), ("dv", ctypes.c_int),
+                ("norm", ctypes.c_int), ("q_norm", ctypes.c_void_p), ("k_norm", ctypes.c_void_p), ("eps", ctypes.c_float),
+                ("half", ctypes.c_int), ("freq", ctypes.c_void_p), ("seq_ids", ctypes.c_void_p),
+                ("positions", ctypes.c_void_p), ("block_table", ctypes.c_void_p), ("cache", ctypes.c_void_p),
+                ("num_blocks", ctypes.c_longlong), ("block_elems", ctypes.c_longlong), ("max_blocks", ctypes.c_int),
+                ("rel_n", ctypes.c_int), ("q_out", ctypes.c_void_p), ("q_stride", ctypes.c_longlong),
+                ("gate_out", ctypes.c_void_p), ("rel", ctypes.c_void_p), ("bucket", ctypes.c_void_p),
+                ("rel_out", ctypes.c_void_p)]
+
+
+assert ctypes.sizeof(_PrepareParams) == 216
+_NORMS = {"": 0, "rows": 1, "heads": 2}
+
+
+def rotary_frequencies(dims: int, base: float, scaling: Optional[Dict[str, Any]] = None) -> List[float]:
+    """Angular frequency ``base^(-2 i / dims)`` of every rotated pair.  ``scaling`` (factor, low, high, original): wavelengths
+    above ``original / low`` are stretched by ``factor``, those below ``original / high`` kept, the ones between blended."""
+    out = []
+    for i in range(dims // 2):
+        f = float(base) ** (-2.0 * i / dims)
+        if scaling:
+            wave, length = 2.0 * math.pi / f, float(scaling["original"])
+            lo, hi, factor = (float(scaling[k]) for k in ("low", "high", "factor"))
+            if wave > length / lo:
+                f = f / factor
+            elif wave >= length / hi:
+                s = (length / wave - lo) / (hi - lo)
+                f = (1.0 - s) * f / factor + s * f
+        out.append(f)
+    return out
+
+
+def distance_buckets(rows: int, far: int, limit: int = 0) -> List[int]:
+    """Table row of every distance from 0 on: one each for the first half of the rows, then logarithmic until ``far``.  The
+    list ends at the first distance whose row is the last one (every later distance has it too), or at ``limit``."""
+    half, out = rows // 2, []
+    while not limit or len(out) < limit:
+        n = len(out)
+        if n < half:
+            b = n
+        elif half == 0 or far <= half:
+            b = rows - 1
+        else:
+            b = min(rows - 1, half + math.floor(math.log(n / half) / math.log(far / half) * (rows - half)))
+        out.append(b)
+        if b == rows - 1:
+            break
+    return out
+
+
+@dataclass
+class QkvPrepare:
+    """What happens to the projected rows before the attention, see csrc/qkv_prepare.cu.  Rows may come as partial sums."""
+    norm: str = ""                              # "", "rows" or "heads"
+    eps: float = 1e-6
+    freq: Optional[torch.Tensor] = None         # [pairs, 2] fp32: frequency as hi + lo
+    g_off: int = -1                             # column of the per-head output gates
+    bias: Optional[torch.Tensor] = None         # like a row of the projection
+    q_norm: Optional[torch.Tensor] = None
+    k_norm: Optional[torch.Tensor] = None
+    rel: Optional[torch.Tensor] = None          # [table rows, heads]
+    bucket: Optional[torch.Tensor] = None       # [distances] int32
+    table: Optional[torch.Tensor] = None        # [heads, distances] fp32, filled from rel and bucket
+
+    def run(self, spec: "WindowSpec", x: torch.Tensor, seq_ids, positions, block_table, cache):
+        """``x [S, T, N]`` or ``[T, N]`` -> queries ``[T, heads * dim]`` (padded rows) and gates ``[T, heads]``; keys and
+        values go to the cache."""
+        x = x if x.dim() == 3 else x[None]
+        S, T, N = x.shape
+        assert x.stride(2) == 1 and (S == 1 or x.dtype == torch.float32) and cache.is_contiguous()
+        assert self.rel is None or tuple(self.table.shape) == (spec.heads, self.bucket.numel())
+        q = torch.empty(T, (spec.heads * spec.dim + 7) // 8 * 8, dtype=cache.dtype, device=x.device)
+        gate = torch.empty(T, spec.heads, dtype=torch.float32, device=x.device) if self.g_off >= 0 else None
+        ptr = lambda t: t.data_ptr() if t is not None else None  # noqa: E731
+        p = _PrepareParams(
+            x=x.data_ptr(), slab=x.stride(0), row_stride=x.stride(1), slabs=S, x_f32=int(x.dtype == torch.float32),
+            bias=ptr(self.bias), q_off=spec.q_off, k_off=spec.k_off, v_off=spec.v_off, g_off=self.g_off, T=T, Hq=spec.heads,
+            Hkv=spec.kv_heads, dk=spec.dim, dv=spec.vdim, norm=_NORMS[self.norm], q_norm=ptr(self.q_norm),
+            k_norm=ptr(self.k_norm), eps=self.eps, half=self.freq.shape[0] if self.freq is not None else 0,
+            freq=ptr(self.freq), seq_ids=seq_ids.data_ptr(), positions=positions.data_ptr(),
+            block_table=block_table.data_ptr(), cache=cache.data_ptr(), num_blocks=cache.shape[0],
+            block_elems=spec.block_elems, max_blocks=block_table.shape[1],
+            rel_n=self.bucket.numel() if self.rel is not None else 0, q_out=q.data_ptr(), q_stride=q.stride(0),
+            gate_out=ptr(gate), rel=ptr(self.rel), bucket=ptr(self.bucket), rel_out=ptr(self.table))
+        _lib.check(_lib.get_lib().sb_qkv_prepare(ctypes.byref(p), int(cache.dtype == torch.float32), _lib.stream()),
+                   "sb_qkv_prepare")
+        return q, gate
+
+    def plain(self, spec: "WindowSpec", x: torch.Tensor, positions: torch.Tensor):
+        """The same on the CPU: rows like ``x`` with queries, keys and values as the attention takes them, and the gates."""
+        x = (x.float().sum(0) if x.dim() == 3 else x.float())
+        if self.bias is not None:
+            x = x + self.bias.float()
+        T, H, G, dk = x.shape[0], spec.heads, spec.kv_heads, spec.dim
+        out = x.clone()
+        for off, n, w in ((spec.q_off, H, self.q_norm), (spec.k_off, G, self.k_norm)):
+            y = x[:, off:off + n * dk]
+            if self.norm == "rows":
+                y = y * torch.rsqrt(y.square().mean(-1, keepdim=True) + self.eps) * w.float()
+            y = y.reshape(T, n, dk)
+            if self.freq is not None:
+                half = self.freq.shape[0]
+                a = positions.double()[:, None] * self.freq.double().sum(-1)[None]
+                c, s = torch.cos(a).float()[:, None], torch.sin(a).float()[:, None]
+                u, v = y[..., :half], y[..., half:2 * half]
+                y = torch.cat([u * c - v * s, v * c + u * s, y[..., 2 * half:]], -1)
+            if self.norm == "heads":
+                y = y * torch.rsqrt(y.square().mean(-1, keepdim=True) + self.eps)
+            out[:, off:off + n * dk] = y.reshape(T, n * dk)
+        gate = torch.sigmoid(x[:, self.g_off:self.g_off + H]) if self.g_off >= 0 else None
+        return out, gate
 
 
 class QueryTiles:
@@ -74,12 +200,14 @@ class QueryTiles:
 
 
 def window_params(spec: WindowSpec, x, seq_ids, positions, block_table, cache, out, out_off, *, kv_mode: int = KV_PAGED,
-                  gain: torch.Tensor = None, gate: torch.Tensor = None) -> _Params:
+                  gain: torch.Tensor = None, gate: torch.Tensor = None, rel: torch.Tensor = None,
+                  head_gate: torch.Tensor = None) -> _Params:
     """``kv_mode``: where keys and values are.  ``KV_PAGED``: in ``cache`` as described above.  ``KV_PACKED`` (prompts):
     ``cache`` is ``[rows, kv_heads * (dim + vdim)]``, one row per key, keys before values, and a tile's slot is the row of
     its sequence's first key.  ``KV_LATENT`` (general kernel): keys and values are the same ``dim``-wide rows of a paged
     cache.  ``gain``: one number (a tensor) that multiplies the queries and the gate.  ``gate``: columns like ``out``'s whose
-    sigmoid multiplies the result (prompts)."""
+    sigmoid multiplies the result (prompts).  ``rel [heads, distances]``: bias by distance.  ``head_gate [T, heads]``: factors
+    of the result."""
     assert x.stride(1) == 1 and out.stride(1) == 1 and cache.dtype == x.dtype == out.dtype
     per_row = spec.kv_heads * (spec.dim + spec.vdim)
     elems = {KV_PAGED: spec.block_elems, KV_PACKED: per_row, KV_LATENT: BLOCK * spec.dim}[kv_mode]
@@ -93,7 +221,9 @@ def window_params(spec: WindowSpec, x, seq_ids, positions, block_table, cache, o
                    bias_exp=spec.bias_exp, out_scale=spec.out_scale, out=out.data_ptr(), out_stride=out.stride(0),
                    out_off=out_off, kv_mode=kv_mode, gain=gain.data_ptr() if gain is not None else None,
                    gate=gate.data_ptr() if gate is not None else None,
-                   gate_stride=gate.stride(0) if gate is not None else 0)
+                   gate_stride=gate.stride(0) if gate is not None else 0, softcap=spec.softcap, sink=int(spec.sink),
+                   rel=rel.data_ptr() if rel is not None else None, rel_n=rel.shape[1] if rel is not None else 0,
+                   head_gate=head_gate.data_ptr() if head_gate is not None else None)
 
 
 _workspace: Dict[tuple, Tuple[torch.Tensor, torch.Tensor]] = {}
@@ -101,17 +231,29 @@ _workspace: Dict[tuple, Tuple[torch.Tensor, torch.Tensor]] = {}
 
 def window_attention(spec: WindowSpec, x: torch.Tensor, seq_ids: torch.Tensor, positions: torch.Tensor,
                      block_table: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, out_off: int, *,
-                     tiles: QueryTiles = None, seq_lens: torch.Tensor = None, simt: bool = False) -> None:
+                     tiles: QueryTiles = None, seq_lens: torch.Tensor = None, simt: bool = False,
+                     prepare: Optional[QkvPrepare] = None) -> None:
     """Append the rows' keys and values to ``cache`` and attend.  Prompt portions: ``tiles``.  Decoding: ``seq_lens``
     (context lengths with the current token; row ``b`` is cache slot ``b``, 0 = idle).  Results go to
-    ``out[:, out_off: ...]``.  ``simt`` forces the general kernel."""
+    ``out[:, out_off: ...]``.  ``prepare``: biases, norms, rotation, gates and distance table of the branch; ``x`` may then
+    be partial sums ``[S, T, N]``.  ``simt`` forces the general kernel."""
     if not x.is_cuda:
-        return _cpu(spec, x, seq_ids, positions, block_table, cache, out, out_off)
+        gate = None
+        if prepare is not None:
+            x, gate = prepare.plain(spec, x, positions)
+        return _cpu(spec, x, seq_ids, positions, block_table, cache, out, out_off, prepare, gate)
     L = _lib.get_lib()
-    p = window_params(spec, x, seq_ids, positions, block_table, cache, out, out_off)
+    if prepare is not None:
+        x, gate = prepare.run(spec, x, seq_ids, positions, block_table, cache)
+        spec = replace(spec, q_off=0)
+        p = window_params(spec, x, seq_ids, positions, block_table, cache, out, out_off,
+                          rel=prepare.table if prepare.rel is not None else None, head_gate=gate)
+    else:
+        p = window_params(spec, x, seq_ids, positions, block_table, cache, out, out_off)
     ref = ctypes.byref(p)
     f32 = int(x.dtype == torch.float32)
-    _lib.check(L.sb_kv_append_split(ref, f32, _lib.stream()), "sb_kv_append_split")
+    if prepare is None:
+        _lib.check(L.sb_kv_append_split(ref, f32, _lib.stream()), "sb_kv_append_split")
     status = _lib.ptr(_lib.status_word(x.device))
     aligned = spec.dim % 8 == 0 and spec.vdim % 8 == 0 and x.stride(0) % 8 == 0 and out.stride(0) % 8 == 0 and \
         spec.q_off % 8 == 0 and out_off % 8 == 0
@@ -137,7 +279,7 @@ def window_attention(spec: WindowSpec, x: torch.Tensor, seq_ids: torch.Tensor, p
     _lib.check(L.sb_attn_window_simt(ref, f32, _lib.stream()), "sb_attn_window_simt")
 
 
-def _cpu(spec: WindowSpec, x, seq_ids, positions, block_table, cache, out, out_off) -> None:
+def _cpu(spec: WindowSpec, x, seq_ids, positions, block_table, cache, out, out_off, prepare=None, gate=None) -> None:
     H, G, dk, dv = spec.heads, spec.kv_heads, spec.dim, spec.vdim
     split = G * BLOCK * dk
     kc = cache[:, :split].view(-1, G, BLOCK, dk)
@@ -172,6 +314,17 @@ def _cpu(spec: WindowSpec, x, seq_ids, positions, block_table, cache, out, out_o
         tr = torch.tensor([t for t, _ in items])
         q = x[tr, spec.q_off:spec.q_off + H * dk].view(-1, H, dk).float()
         sc = torch.einsum("thd,hjd->htj", q, k) * spec.scale - slope[:, None, None] * (idx - j)[None]
-        pr = torch.softmax(sc.masked_fill(~seen[None], float("-inf")), -1)
+        if spec.softcap:
+            sc = spec.softcap * torch.tanh(sc / spec.softcap)
+        if prepare is not None and prepare.rel is not None:
+            far = prepare.bucket.numel() - 1
+            sc = sc + prepare.rel.float()[prepare.bucket[(idx - j).clamp(0, far)].long()].permute(2, 0, 1)
+        sc = sc.masked_fill(~seen[None], float("-inf"))
+        if spec.sink:
+            pr = torch.softmax(torch.cat([sc, torch.zeros(*sc.shape[:2], 1)], -1), -1)[..., :-1]
+        else:
+            pr = torch.softmax(sc, -1)
         o = torch.einsum("htj,hjd->thd", pr, v) * spec.out_scale
+        if gate is not None:
+            o = o * gate[tr][:, :, None]
         out[tr, out_off:out_off + H * dv] = o.reshape(len(items), H * dv).to(out.dtype)
