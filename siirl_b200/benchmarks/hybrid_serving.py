@@ -1,8 +1,8 @@
-"""Serving throughput of a hybrid decoder (Domavik, Poralorn) beside the closest decoder of equal size, and its kernels
+"""Serving throughput of a hybrid decoder (Domavik, Poralorn, Gumazen) beside the closest decoder of equal size, and its kernels
 beside the like kernels of that model.
 
-    python bench.py --workload serve [--design poralorn]                     # end to end, a few sizes
-    python -m siirl_b200.benchmarks.hybrid_serving [--design poralorn] --kernels
+    python bench.py --workload serve [--design poralorn|gumazen]             # end to end, a few sizes
+    python -m siirl_b200.benchmarks.hybrid_serving [--design poralorn|gumazen] --kernels
 
 End to end: random weights, the rollout engine's own prefill pass and CUDA-graph decode rounds, CUDA events on the
 launching stream.  Weights and caches are larger than L2 in every case.  Kernels: each alone, L2 flushed between
@@ -27,6 +27,8 @@ SIZES = {     # design -> size: preset, layers, (prompts, tokens) of a prefill p
                 "7b": ("domavik-7b", 8, [(8, 1024), (1, 8192)], [(32, 2048), (256, 1024)])},
     "poralorn": {"1.5b": ("poralorn-1.5b", 14, [(8, 1024), (1, 8192)], [(32, 2048), (256, 1024)]),
                  "7b": ("poralorn-7b", 8, [(8, 1024), (1, 8192)], [(32, 2048), (256, 1024)])},
+    "gumazen": {"a1b": ("gumazen-a1b", 12, [(8, 1024), (1, 8192)], [(32, 2048), (256, 1024)]),
+                "a3b": ("gumazen-a3b", 12, [(8, 1024), (1, 8192)], [(32, 2048), (256, 1024)])},
 }
 
 
@@ -42,9 +44,17 @@ def peaks() -> Dict[str, float]:
 
 def closest(cfg: DecoderConfig) -> DecoderConfig:
     """The uniform decoder of the same width, feed-forward, number of layer runs, vocabulary and attention heads (seven
-    query heads, or six, per key-value head where the design shares one latent between all)."""
+    query heads, or six, per key-value head where the design shares one latent between all); with experts where the design
+    has them: as many, as wide, as many per token, and a shared one."""
     b = cfg.hybrid.attention[0]
     kv = b.kv_heads or b.heads // (7 if b.heads % 7 == 0 else 6)
+    moe = next((x.moe for x in cfg.hybrid.layers if x.moe is not None), None)
+    if moe is not None:
+        return DecoderConfig(model_type="qwen2_moe", vocab_size=cfg.vocab_size, hidden_size=cfg.hidden_size,
+                             intermediate_size=cfg.intermediate_size * 2 // 3 // 64 * 64, num_layers=len(cfg.hybrid.runs()),
+                             num_heads=b.heads, num_kv_heads=kv, head_dim=b.dim, rope_theta=1e6, eos_token_id=2,
+                             num_experts=moe.experts, num_experts_per_tok=moe.top, moe_intermediate_size=moe.ff,
+                             shared_expert_intermediate_size=moe.shared_ff, first_k_dense_replace=1)
     return DecoderConfig(model_type="qwen2", vocab_size=cfg.vocab_size, hidden_size=cfg.hidden_size,
                          intermediate_size=cfg.intermediate_size, num_layers=len(cfg.hybrid.runs()), num_heads=b.heads,
                          num_kv_heads=kv, head_dim=b.dim, rope_theta=1e6, eos_token_id=2)
@@ -200,7 +210,7 @@ def _rnd(*s):
 
 def kernels(design: str = "domavik", only: str = "", iters: int = 20) -> dict:
     b = _Bench(only, iters)
-    (_kernels_poralorn if design == "poralorn" else _kernels_domavik)(b)
+    {"poralorn": _kernels_poralorn, "gumazen": _kernels_gumazen, "domavik": _kernels_domavik}[design](b)
     return b.result()
 
 
@@ -278,6 +288,114 @@ def _kernels_poralorn(b: _Bench) -> None:
         gu = rnd(T, 2 * I)
         add(f"uniform: swiglu {T}x{I}", lambda: dense.swiglu(gu), nbytes=T * I * 6)
         add(f"poralorn: exact GELU {T}x{I}", lambda: R.scaled_act(gu[:, :I], "gelu", one), nbytes=T * I * 4)
+
+
+def _kernels_gumazen(b: _Bench) -> None:
+    """The three kinds of attention with 32 heads of width 128 (4 key-value heads), the routed feed-forward with 120 + 8
+    router outputs, and the row operations of two streams."""
+    from ..models.decoder import _Init
+    from ..models.hybrid import HybridBranch, RoutedFeedForward
+    from ..models.moe import moe_forward
+    from ..ops import dense, kv_cache
+    from ..ops import moe as M
+    from ..ops import rows as R
+    from ..ops.attention import SeqInfo, attention_packed
+    from ..ops.window_attention import QueryTiles, window_attention
+    dev, add, rnd = torch.device("cuda"), b.add, _rnd
+    W, H, G, D = 2048, 32, 4, 128
+    base = get_config("gumazen-a3b")
+    kinds = {"sink": base.hybrid.layers[1].branches[0], "window 1024": base.hybrid.layers[2].branches[0],
+             "biases": base.hybrid.layers[0].branches[0]}
+    gen = _Init(0, "cuda")
+    branches = {k: HybridBranch(m, base, 0, 0, torch.bfloat16, "cuda", gen) for k, m in kinds.items()}
+
+    def prepared(br):
+        return copy.copy(br.prepare), {k: getattr(br, k).detach() for k in ("bias", "q_norm", "k_norm", "rel") if hasattr(br, k)}
+
+    for n, L in ((8, 1024), (1, 8192)):
+        T, nb = n * L, L // 64
+        x = rnd(T, (H + 2 * G) * D)
+        info = SeqInfo([L] * n, device=dev)
+        flops = n * 4 * D * H * L * (L + 1) / 2
+        add(f"uniform: fmha_fwd {n}x{L}", lambda: attention_packed(x, info, H, G, D), flops)
+        table = torch.randperm(n * nb, device=dev).to(torch.int32).view(n, nb)
+        cache = torch.zeros(n * nb, G * 64 * 2 * D, dtype=torch.bfloat16, device=dev)
+        out = torch.empty(T, H * D, dtype=torch.bfloat16, device=dev)
+        ids = torch.repeat_interleave(torch.arange(n, dtype=torch.int32), L).to(dev)
+        pos = torch.arange(L, dtype=torch.int32).repeat(n).to(dev)
+        tiles = QueryTiles([L] * n, [0] * n, list(range(n)), dev)
+        tabs = dense.rope_tables(D, L, 1e6, device=dev)
+        add(f"uniform: rotation + append {n}x{L}",
+            lambda: kv_cache.rope_kv_append(x, pos, *tabs, None, ids, pos, table, cache.view(n * nb, 2, G, 64, D), H, G, D),
+            nbytes=T * ((H + G) * D * 2 + (H + 2 * G) * D * 2))
+        for name, br in branches.items():
+            m, spec = br.b, br.spec
+            xp = rnd(T, br.in_end)
+            pr, w = prepared(br)
+            for k, v in w.items():
+                setattr(pr, k, v)
+            add(f"gumazen: norms, rotation, append ({name}) {n}x{L}", lambda: pr.run(spec, xp, ids, pos, table, cache),
+                nbytes=T * (H + 2 * G) * D * 4)
+            seen = sum(min(i + 1, m.window) for i in range(L)) if m.window else L * (L + 1) / 2
+            add(f"gumazen: attention ({name}) {n}x{L}, with norms, rotation, append",
+                lambda: window_attention(spec, xp, ids, pos, table, cache, out, 0, tiles=tiles, prepare=pr),
+                n * 4 * D * H * seen)
+    for B, ctx in ((32, 2048), (256, 1024)):
+        nb = (ctx + 63) // 64
+        table = torch.randperm(B * nb, device=dev).to(torch.int32).view(B, nb)
+        lens = torch.full((B,), ctx, dtype=torch.int32, device=dev)
+        q, kvc = rnd(B, (H + 2 * G) * D), torch.zeros(B * nb, 2, G, 64, D, dtype=torch.bfloat16, device=dev)
+        add(f"uniform: decode attention {B}x{ctx}", lambda: kv_cache.decode_attention(q, kvc, lens, table, H, G, D),
+            nbytes=B * ctx * 2 * G * D * 2)
+        flat, out = kvc.view(B * nb, -1), torch.empty(B, H * D, dtype=torch.bfloat16, device=dev)
+        ids, pos = torch.arange(B, dtype=torch.int32, device=dev), lens - 1
+        for name, br in branches.items():
+            m, spec = br.b, br.spec
+            xp = rnd(B, br.in_end)
+            pr, w = prepared(br)
+            for k, v in w.items():
+                setattr(pr, k, v)
+            add(f"gumazen: norms, rotation, append ({name}) {B}", lambda: pr.run(spec, xp, ids, pos, table, flat),
+                nbytes=B * (H + 2 * G) * D * 4)
+            seen = min(ctx, m.window) if m.window else ctx
+            add(f"gumazen: decode attention ({name}) {B}x{ctx}, with norms, rotation, append",
+                lambda: window_attention(spec, xp, ids, pos, table, flat, out, 0, seq_lens=lens, prepare=pr),
+                nbytes=B * seen * 2 * G * D * 2)
+    e = base.hybrid.layers[1].moe
+    ff = RoutedFeedForward(e, W, 0.02, torch.bfloat16, "cuda", gen)
+    router, local = rnd(e.experts, W), M.ExpertParallel()
+    gu, dn = ff.gate_up_weight.detach(), ff.down_weight.detach()
+    for T in (32, 256, 8192):
+        x = rnd(T, W)
+        used = e.experts * (1 - (1 - e.top / e.experts) ** T)
+        flops, nbytes = T * e.top * 6.0 * W * e.ff, used * 6 * W * e.ff + T * W * 4
+        z = torch.randn(1, T, e.outputs, device=dev)
+        add(f"uniform: router {T}", lambda: M.route_topk(z[0, :, :e.experts].contiguous(), e.top), nbytes=T * e.outputs * 4)
+        add(f"gumazen: router {T}", lambda: M.route_grouped(z, ff.correction.detach(), e.experts, e.top, e.groups, e.keep, e.scale),
+            nbytes=T * e.outputs * 4)
+        wt, ids = M.route_topk(z[0, :, :e.experts].contiguous(), e.top)
+        add(f"uniform: routed feed-forward {T} (dispatch, experts, combine)",
+            lambda: moe_forward(x, router, gu, dn, e.top, routed=(wt, ids)), flops, nbytes)
+        i32 = ids.to(torch.int32)
+        add(f"gumazen: routed feed-forward {T} (dispatch, experts)", lambda: M.routed_experts(x, i32, gu, dn, "silu"), flops, nbytes)
+        h, y = torch.randn(T, 2, W, device=dev), rnd(1, T, W)
+        conn = [torch.ones(2, device=dev).bfloat16(), torch.eye(2, device=dev).bfloat16(), rnd(W), rnd(W)]
+        d, res, nw = rnd(T, W), rnd(T, W), rnd(W)
+        add(f"uniform: residual + RMS norm {T}x{W} (bf16 stream)", lambda: dense.rmsnorm(d, nw, 1e-6, residual=res),
+            nbytes=T * W * 8)
+        kw = dict(w_in=conn[0], w_out=conn[0], w_mix=conn[1])
+        add(f"gumazen: streams + layer norm {T}x{W} (two fp32 streams)",
+            lambda: R.hyper_rows(h, conn[2], conn[3], 1e-5, result=R.SublayerSum(y), **kw), nbytes=T * W * 20)
+        ys, slots = M.routed_experts(x, i32, gu, dn, "silu")
+        w_id = torch.rand(T, device=dev)
+        add(f"uniform: combine {T}x{W}", lambda: local.combine(ys, None, slots, wt, T, e.top), nbytes=T * W * 2 * (e.top + 1))
+        add(f"gumazen: streams + layer norm + combine {T}x{W}",
+            lambda: R.hyper_rows(h, conn[2], conn[3], 1e-5, result=R.SublayerSum(y, None, ys, slots, wt, x, w_id), **kw),
+            nbytes=T * W * (22 + 2 * e.top))
+        I = 11264
+        up = rnd(T, 2 * I)
+        add(f"uniform: swiglu {T}x{I}", lambda: dense.swiglu(up), nbytes=T * I * 6)
+        add(f"gumazen: squared relu {T}x{I}", lambda: R.scaled_act(up[:, :I], "relu2"), nbytes=T * I * 4)
 
 
 def _kernels_domavik(b: _Bench) -> None:

@@ -449,6 +449,13 @@ __device__ __forceinline__ float fast_exp2(float x) {
   return y;
 }
 
+// 1 / x by the special-function unit (rcp.approx, 1 ulp)
+__device__ __forceinline__ float fast_rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -144,7 +144,7 @@ struct WinSmem {
     v_off = k_off + 2 * k_bytes;
     p_off = v_off + 2 * v_bytes;
     bar_off = p_off + 128 * kWBlk * 2;
-    total = bar_off + 64;
+    total = bar_off + 96;
   }
 };
 
@@ -164,9 +164,12 @@ __host__ __device__ inline void win_blocks(int q0, int q1, int window, int keep_
   n = sinks + (last + 1 > w0 ? last + 1 - w0 : 0);
 }
 
-// TABLE: soft-capped scores and / or a bias table by distance instead of the linear bias
+// Warp 4 fetches and issues: S(j + 1) = Q K(j + 1)^T goes ahead of O += P(j) V(j), into the other half of a double-buffered S,
+// so the scores of the next tile are computed while warps 0 - 3 (one row per thread) are in the soft-max of this one.  A key
+// tile is given back when its scores are done, a value tile one step later.  The running maximum is only raised when it grows
+// by more than 2^8.  TABLE: soft-capped scores and / or a bias table by distance instead of the linear bias.
 template <bool TABLE>
-__global__ void __launch_bounds__(128, 2)
+__global__ void __launch_bounds__(160, 2)
 window_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                       const __grid_constant__ CUtensorMap map_v, WinParams p, const int* __restrict__ tile_row,
                       const int* __restrict__ tile_rows, const int* __restrict__ tile_pos,
@@ -185,12 +188,14 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
   uint8_t* sV = smem + L.v_off;
   uint8_t* sP = smem + L.p_off;
   uint64_t* bar_q = reinterpret_cast<uint64_t*>(smem + L.bar_off);
-  uint64_t* bar_kv = bar_q + 1;
-  uint64_t* bar_s = bar_q + 3;
-  uint64_t* bar_o = bar_q + 4;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bar_q + 5);
+  uint64_t* bar_k = bar_q + 1;      // [2] key tile has arrived
+  uint64_t* bar_v = bar_q + 3;      // [2] value tile has arrived
+  uint64_t* bar_s = bar_q + 5;      // [2] scores are in TMEM
+  uint64_t* bar_p = bar_q + 7;      // weights are in shared memory (and the scores have been read)
+  uint64_t* bar_o = bar_q + 8;      // O holds this tile
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bar_q + 9);
 
-  const int tid = threadIdx.x, warp = tid >> 5;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int tile = blockIdx.x, h = blockIdx.y;
   const int row0 = tile_row[tile], nrows = tile_rows[tile], q0 = tile_pos[tile], slot = tile_slot[tile];
   const int kvh = h / (p.Hq / p.Hkv);
@@ -204,10 +209,10 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     tma_prefetch_desc(&map_q);
     tma_prefetch_desc(&map_k);
     tma_prefetch_desc(&map_v);
-    for (int i = 0; i < 5; ++i) mbar_init(&bar_q[i], 1);
+    for (int i = 0; i < 9; ++i) mbar_init(&bar_q[i], i == 7 ? 4 : 1);
     fence_barrier_init();
   }
-  if (warp == 0) {
+  if (warp == 4) {
     tmem_alloc(tmem_slot, tmem_cols);
     tmem_relinquish();
   }
@@ -215,212 +220,266 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem_base = *tmem_slot;
-  const uint32_t tmem_s = tmem_base, tmem_o = tmem_base + 64;
-
-  auto load_kv = [&](int j, int stage) {
-    const int lb = block_of(j);
-    // packed rows: head kvh, rows from `blk`; those past the sequence are hidden by causality, past the end zeros
-    int blk = packed ? slot + lb * kWBlk : (lb < p.max_blocks ? bt[lb] : 0);
-    if (!packed && (blk < 0 || blk >= p.num_blocks)) blk = 0;      // never inside the visible range of a well-formed table
-    const int mid = packed ? kvh : kvh * kWBlk;
-    mbar_arrive_expect_tx(&bar_kv[stage], (uint32_t)(L.k_bytes + L.v_bytes));
-    for (int c = 0; c < ck; ++c)
-      tma_load_3d(sK + stage * L.k_bytes + c * 8192, &map_k, &bar_kv[stage], c * 64, mid, blk);
-    for (int c = 0; c < cv; ++c)
-      tma_load_3d(sV + stage * L.v_bytes + c * 8192, &map_v, &bar_kv[stage], c * 64, mid, blk);
-  };
-  if (tid == 0) {
-    mbar_arrive_expect_tx(bar_q, (uint32_t)L.q_bytes);
-    for (int c = 0; c < ck; ++c) tma_load_3d(sQ + c * 16384, &map_q, bar_q, c * 64, h, row0);
-    load_kv(0, 0);
-    if (n_tiles > 1) load_kv(1, 1);
-  }
-
-  const uint32_t idesc_s = umma_idesc_bf16(128, kWBlk, 0, 0);
-  const uint32_t idesc_o = umma_idesc_bf16(128, vn, 0, 1);
-  const uint32_t lane_off = (uint32_t)(warp * 32) << 16;
-  const int qpos = q0 + tid;
-  const float gain = p.gain ? __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(p.gain)) : 1.f;
-  const float scale_log2 = p.scale * gain * 1.4426950408889634f;
-  const float slope_log2 =
-      p.bias_exp > 0.f ? exp2f(-p.bias_exp * (float)(h + 1) / (float)p.Hq) * 1.4426950408889634f : 0.f;
-  const ScoreCap cap(p.softcap > 0.f ? p.softcap : 1.f, p.scale * gain);
-  const float* rel = TABLE && p.rel ? p.rel + (size_t)h * p.rel_n : nullptr;
-  const int rel_last = (int)p.rel_n - 1;
-  const float rel_far = rel ? __ldg(rel + rel_last) * 1.4426950408889634f : 0.f;
-  float m_run = -INFINITY, l_run = 0.f;
+  const uint32_t tmem_s = tmem_base, tmem_o = tmem_base + 128;
   bool ok = true;
 
-  for (int j = 0; j < n_tiles && ok; ++j) {
-    const int stage = j & 1;
-    if (tid == 0) {
-      bool w = true;
-      if (j == 0) w = mbar_wait(bar_q, 0, status, kStatusTimeoutMma);
-      w = w && mbar_wait(&bar_kv[stage], (j >> 1) & 1, status, kStatusTimeoutMma);
-      if (w) {
-        tc_fence_after();
-        const uint32_t aq = smem_u32(sQ), bk = smem_u32(sK + stage * L.k_bytes);
-        for (int kk = 0; kk < k_steps; ++kk) {
-          const uint64_t da = umma_smem_desc(aq + (kk / 4) * 16384 + (kk % 4) * 32, 16, 1024);
-          const uint64_t db = umma_smem_desc(bk + (kk / 4) * 8192 + (kk % 4) * 32, 16, 1024);
-          umma_bf16_ss(tmem_s, da, db, idesc_s, kk ? 1u : 0u);
-        }
+  if (warp == 4) {
+    // ------------------------------ copies and MMAs (the warp stays converged, lane 0 issues) ------------------------------
+    const uint32_t leader = lane == 0;
+    int k_loads = 0, v_loads = 0;
+    // packed rows: head kvh, rows from the block on; those past the sequence are hidden by causality, past the end zeros
+    auto load = [&](const CUtensorMap* map, uint8_t* dst, int bytes, int chunks, uint64_t* bar, int j) {
+      const int lb = block_of(j);
+      int blk = packed ? slot + lb * kWBlk : (lb < p.max_blocks ? bt[lb] : 0);
+      if (!packed && (blk < 0 || blk >= p.num_blocks)) blk = 0;      // never inside the visible range of a well-formed table
+      const int mid = packed ? kvh : kvh * kWBlk;
+      if (leader) {
+        mbar_arrive_expect_tx(bar, (uint32_t)bytes);
+        for (int c = 0; c < chunks; ++c) tma_load_3d(dst + c * 8192, map, bar, c * 64, mid, blk);
       }
-      umma_commit(bar_s);
+    };
+    auto load_k = [&](int j) {
+      load(&map_k, sK + (j & 1) * L.k_bytes, L.k_bytes, ck, &bar_k[j & 1], j);
+      ++k_loads;
+    };
+    auto load_v = [&](int j) {
+      load(&map_v, sV + (j & 1) * L.v_bytes, L.v_bytes, cv, &bar_v[j & 1], j);
+      ++v_loads;
+    };
+    auto wait = [&](uint64_t* bar, uint32_t parity) {
+      return __all_sync(0xffffffffu, mbar_wait(bar, parity, status, kStatusTimeoutMma));
+    };
+    if (leader) {
+      mbar_arrive_expect_tx(bar_q, (uint32_t)L.q_bytes);
+      for (int c = 0; c < ck; ++c) tma_load_3d(sQ + c * 16384, &map_q, bar_q, c * 64, h, row0);
     }
-    if (!__all_sync(0xffffffffu, mbar_wait(bar_s, j & 1, status, kStatusTimeoutEpilogue))) {
-      ok = false;
-      break;
+    for (int j = 0; j < 2 && j < n_tiles; ++j) {
+      load_k(j);
+      load_v(j);
     }
-    tc_fence_after();
-    const int kv0 = block_of(j) * kWBlk;
-    float sv[kWBlk];
-    {
-      // score in units of log 2, distance bias included: s * scale - slope * (i - j)
-      const float b0 = slope_log2 * (float)(kv0 - qpos);
-      uint32_t r0[32], r1[32];
-      tmem_ld_32x32(tmem_s + lane_off, r0);
-      tmem_ld_32x32(tmem_s + lane_off + 32, r1);
-      tmem_ld_wait();
-      if constexpr (TABLE) {
-        if (p.softcap > 0.f) {
+    const uint32_t idesc_s = umma_idesc_bf16(128, kWBlk, 0, 0);
+    const uint32_t idesc_o = umma_idesc_bf16(128, vn, 0, 1);
+    const uint64_t dq = umma_smem_desc(smem_u32(sQ), 16, 1024), dk0 = umma_smem_desc(smem_u32(sK), 16, 1024);
+    const uint64_t dp = umma_smem_desc(smem_u32(sP), 16, 1024), dv0 = umma_smem_desc(smem_u32(sV), 8192, 1024);
+    const uint32_t k_step = (uint32_t)L.k_bytes >> 4, v_step = (uint32_t)L.v_bytes >> 4;
+    auto scores = [&](int j) {
+      uint64_t da = dq, db = dk0 + (j & 1) * k_step;
+      const uint32_t d = tmem_s + (j & 1) * 64;
+      int left = k_steps;
+#pragma unroll 1
+      for (int c = 0; c < ck; ++c, da += 1024, db += 512, left -= 4) {
+        umma_bf16_ss_if(leader, d, da, db, idesc_s, c ? 1u : 0u);
+        if (left > 1) umma_bf16_ss_if(leader, d, da + 2, db + 2, idesc_s, 1u);
+        if (left > 2) umma_bf16_ss_if(leader, d, da + 4, db + 4, idesc_s, 1u);
+        if (left > 3) umma_bf16_ss_if(leader, d, da + 6, db + 6, idesc_s, 1u);
+      }
+      umma_commit_if(leader, &bar_s[j & 1]);
+    };
+    ok = wait(bar_q, 0) && wait(&bar_k[0], 0);
+    if (ok) {
+      tc_fence_after();
+      scores(0);
+    }
+    for (int j = 0; j < n_tiles && ok; ++j) {
+      if (j + 1 < n_tiles) {
+        ok = wait(&bar_k[(j + 1) & 1], ((j + 1) >> 1) & 1);
+        if (!ok) break;
+        tc_fence_after();
+        scores(j + 1);
+      }
+      ok = wait(&bar_s[j & 1], (j >> 1) & 1);
+      if (!ok) break;
+      if (j + 2 < n_tiles) load_k(j + 2);
+      if (j > 0) {
+        ok = wait(bar_o, (j - 1) & 1);
+        if (!ok) break;
+        if (j + 1 < n_tiles) load_v(j + 1);
+      }
+      ok = wait(bar_p, j & 1) && wait(&bar_v[j & 1], (j >> 1) & 1);
+      if (!ok) break;
+      tc_fence_after();
+      const uint64_t db = dv0 + (j & 1) * v_step;
+      umma_bf16_ss_if(leader, tmem_o, dp, db, idesc_o, j ? 1u : 0u);
+      umma_bf16_ss_if(leader, tmem_o, dp + 2, db + 128, idesc_o, 1u);
+      umma_bf16_ss_if(leader, tmem_o, dp + 4, db + 256, idesc_o, 1u);
+      umma_bf16_ss_if(leader, tmem_o, dp + 6, db + 384, idesc_o, 1u);
+      umma_commit_if(leader, bar_o);
+    }
+    if (!ok) {      // bounded: let the copies in flight land before shared memory is given back
+      mbar_wait(bar_q, 0, nullptr, 0);
+      for (int st = 0; st < 2; ++st) {
+        const int nk = (k_loads + 1 - st) / 2, nv = (v_loads + 1 - st) / 2;
+        if (nk) mbar_wait(&bar_k[st], (nk - 1) & 1, nullptr, 0);
+        if (nv) mbar_wait(&bar_v[st], (nv - 1) & 1, nullptr, 0);
+      }
+    }
+  } else {
+    // ------------------------------ soft-max and result ------------------------------
+    const uint32_t lane_off = (uint32_t)(warp * 32) << 16;
+    const int qpos = q0 + tid;
+    const float gain = p.gain ? __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(p.gain)) : 1.f;
+    const float scale_log2 = p.scale * gain * 1.4426950408889634f;
+    const float slope_log2 =
+        p.bias_exp > 0.f ? exp2f(-p.bias_exp * (float)(h + 1) / (float)p.Hq) * 1.4426950408889634f : 0.f;
+    const ScoreCap cap(p.softcap > 0.f ? p.softcap : 1.f, p.scale * gain);
+    const float* rel = TABLE && p.rel ? p.rel + (size_t)h * p.rel_n : nullptr;
+    const int rel_last = (int)p.rel_n - 1;
+    const float rel_far = rel ? __ldg(rel + rel_last) * 1.4426950408889634f : 0.f;
+    float m_ref = -INFINITY, l_run = 0.f;
+
+    for (int j = 0; j < n_tiles; ++j) {
+      if (!__all_sync(0xffffffffu, mbar_wait(&bar_s[j & 1], (j >> 1) & 1, status, kStatusTimeoutEpilogue))) {
+        ok = false;
+        break;
+      }
+      tc_fence_after();
+      const int kv0 = block_of(j) * kWBlk;
+      float sv[kWBlk];
+      {
+        uint32_t r0[32], r1[32];
+        tmem_ld_32x32(tmem_s + (j & 1) * 64 + lane_off, r0);
+        tmem_ld_32x32(tmem_s + (j & 1) * 64 + lane_off + 32, r1);
+        tmem_ld_wait();
+        if constexpr (TABLE) {
+          if (p.softcap > 0.f) {
 #pragma unroll
-          for (int i = 0; i < 32; ++i) {
-            sv[i] = cap(__uint_as_float(r0[i]));
-            sv[32 + i] = cap(__uint_as_float(r1[i]));
+            for (int i = 0; i < 32; ++i) {
+              sv[i] = cap(__uint_as_float(r0[i]));
+              sv[32 + i] = cap(__uint_as_float(r1[i]));
+            }
+          } else {
+#pragma unroll
+            for (int i = 0; i < 32; ++i) {
+              sv[i] = __uint_as_float(r0[i]) * scale_log2;
+              sv[32 + i] = __uint_as_float(r1[i]) * scale_log2;
+            }
+          }
+          const int d0 = qpos - kv0;      // distance of the tile's first key
+          if (rel && q0 - (kv0 + kWBlk - 1) >= rel_last) {      // the whole tile is at least as far as the last entry
+#pragma unroll
+            for (int i = 0; i < kWBlk; ++i) sv[i] += rel_far;
+          } else if (rel && q0 >= kv0 + kWBlk - 1 && q0 + 127 - kv0 <= rel_last) {      // the whole tile lies inside the table
+            const float* at = rel + d0 - (kWBlk - 1);
+#pragma unroll
+            for (int i = 0; i < kWBlk; ++i) sv[i] = fmaf(__ldg(at + (kWBlk - 1 - i)), 1.4426950408889634f, sv[i]);
+          } else if (rel) {
+#pragma unroll
+            for (int i = 0; i < kWBlk; ++i)
+              sv[i] = fmaf(__ldg(rel + min(max(d0 - i, 0), rel_last)), 1.4426950408889634f, sv[i]);
           }
         } else {
+          // score in units of log 2, distance bias included: s * scale - slope * (i - j)
+          const float b0 = slope_log2 * (float)(kv0 - qpos);
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
-            sv[i] = __uint_as_float(r0[i]) * scale_log2;
-            sv[32 + i] = __uint_as_float(r1[i]) * scale_log2;
+            sv[i] = fmaf(__uint_as_float(r0[i]), scale_log2, fmaf(slope_log2, (float)i, b0));
+            sv[32 + i] = fmaf(__uint_as_float(r1[i]), scale_log2, fmaf(slope_log2, (float)(32 + i), b0));
           }
         }
-        if (rel && q0 - (kv0 + kWBlk - 1) >= rel_last) {      // the whole tile is at least as far as the last entry
+      }
+      // every row of the tile sees every key of the block when the block lies behind q0 and, with a window, inside the
+      // last row's window or among the kept tokens
+      const bool all_seen = kv0 + kWBlk - 1 <= q0 &&
+                            (p.window <= 0 || q0 + nrows - 1 - kv0 < p.window || kv0 + kWBlk <= p.keep_first);
+      if (!all_seen) {
 #pragma unroll
-          for (int i = 0; i < kWBlk; ++i) sv[i] += rel_far;
-        } else if (rel) {
-          const int d0 = qpos - kv0;
-#pragma unroll
-          for (int i = 0; i < kWBlk; ++i)
-            sv[i] = fmaf(__ldg(rel + min(max(d0 - i, 0), rel_last)), 1.4426950408889634f, sv[i]);
-        }
-      } else {
-#pragma unroll
-        for (int i = 0; i < 32; ++i) {
-          sv[i] = fmaf(__uint_as_float(r0[i]), scale_log2, fmaf(slope_log2, (float)i, b0));
-          sv[32 + i] = fmaf(__uint_as_float(r1[i]), scale_log2, fmaf(slope_log2, (float)(32 + i), b0));
+        for (int i = 0; i < kWBlk; ++i) {
+          const int kp = kv0 + i;
+          if (!(kp <= qpos && (p.window <= 0 || qpos - kp < p.window || kp < p.keep_first))) sv[i] = -INFINITY;
         }
       }
-    }
-    // every row of the tile sees every key of the block when the block lies behind q0 and, with a window, inside the
-    // last row's window or among the kept tokens
-    const bool all_seen = kv0 + kWBlk - 1 <= q0 &&
-                          (p.window <= 0 || q0 + nrows - 1 - kv0 < p.window || kv0 + kWBlk <= p.keep_first);
-    if (!all_seen) {
+      float m4[4] = {sv[0], sv[1], sv[2], sv[3]};
 #pragma unroll
-      for (int i = 0; i < kWBlk; ++i) {
-        const int kp = kv0 + i;
-        if (!(kp <= qpos && (p.window <= 0 || qpos - kp < p.window || kp < p.keep_first))) sv[i] = -INFINITY;
+      for (int i = 4; i < kWBlk; ++i) m4[i & 3] = fmaxf(m4[i & 3], sv[i]);
+      const float m_tile = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3]));
+      float alpha = 1.f;
+      const bool raise = m_tile > m_ref + 8.f;
+      if (raise) {
+        alpha = exp2f(m_ref - m_tile);      // 0 the first time
+        l_run *= alpha;
+        m_ref = m_tile;
       }
-    }
-    float m_new = m_run;
+      const bool rescale = j > 0 && __any_sync(0xffffffffu, raise);
+      const float m_safe = m_ref == -INFINITY ? 0.f : m_ref;
+      float s4[4] = {};
+      uint32_t pk[kWBlk / 2];
 #pragma unroll
-    for (int i = 0; i < kWBlk; ++i) m_new = fmaxf(m_new, sv[i]);
-    const float m_safe = (m_new == -INFINITY) ? 0.f : m_new;
-    const float alpha = exp2f(m_run - m_safe);
-    float rsum = 0.f;
-    uint32_t pk[kWBlk / 2];
+      for (int i = 0; i < kWBlk; i += 2) {
+        const float p0 = fast_exp2(sv[i] - m_safe), p1 = fast_exp2(sv[i + 1] - m_safe);
+        s4[(i >> 1) & 3] += p0 + p1;
+        pk[i / 2] = pack_bf16x2(p0, p1);
+      }
+      l_run += (s4[0] + s4[1]) + (s4[2] + s4[3]);
+      // the tile before has left the weights' buffer and is in O
+      if (j > 0 && !__all_sync(0xffffffffu, mbar_wait(bar_o, (j - 1) & 1, status, kStatusTimeoutEpilogue))) {
+        ok = false;
+        break;
+      }
+      if (rescale) {
+        tc_fence_after();
+#pragma unroll 1
+        for (int c = 0; c < (vn + 31) / 32; ++c) {
+          uint32_t r[32];
+          tmem_ld_32x32(tmem_o + lane_off + c * 32, r);
+          tmem_ld_wait();
 #pragma unroll
-    for (int i = 0; i < kWBlk; i += 2) {
-      const float p0 = exp2f(sv[i] - m_safe), p1 = exp2f(sv[i + 1] - m_safe);
-      rsum += p0 + p1;
-      pk[i / 2] = pack_bf16x2(p0, p1);
+          for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * alpha);
+          tmem_st_32x32(tmem_o + lane_off + c * 32, r);
+        }
+        tmem_st_wait();
+      }
+      {
+        uint8_t* prow = sP + tid * 128;
+#pragma unroll
+        for (int piece = 0; piece < 8; ++piece) {
+          uint4 v = make_uint4(pk[piece * 4], pk[piece * 4 + 1], pk[piece * 4 + 2], pk[piece * 4 + 3]);
+          *reinterpret_cast<uint4*>(prow + ((piece ^ (tid & 7)) << 4)) = v;
+        }
+      }
+      fence_proxy_async_smem();
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(bar_p);
     }
-    l_run = l_run * alpha + rsum;
-    m_run = m_new;
-    if (j > 0 && __any_sync(0xffffffffu, alpha != 1.f)) {
+    if (ok)
+      ok = __all_sync(0xffffffffu, mbar_wait(bar_o, (n_tiles - 1) & 1, status, kStatusTimeoutEpilogue));
+    if (ok) {
+      tc_fence_after();
+      const bool row_valid = tid < nrows;
+      if (p.sink) l_run += exp2f(-m_ref);
+      float inv_l = l_run > 0.f ? p.out_scale / l_run : 0.f;
+      if (p.head_gate && row_valid) inv_l *= p.head_gate[(size_t)(row0 + tid) * p.Hq + h];
+      __nv_bfloat16* orow = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)(row0 + (row_valid ? tid : 0)) * p.out_stride +
+                            p.out_off + (size_t)h * p.dv;
+      const __nv_bfloat16* grow = reinterpret_cast<const __nv_bfloat16*>(p.gate) +
+                                  (size_t)(row0 + (row_valid ? tid : 0)) * p.gate_stride + (size_t)h * p.dv;
 #pragma unroll 1
       for (int c = 0; c < (vn + 31) / 32; ++c) {
         uint32_t r[32];
         tmem_ld_32x32(tmem_o + lane_off + c * 32, r);
         tmem_ld_wait();
+        if (row_valid) {
 #pragma unroll
-        for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * alpha);
-        tmem_st_32x32(tmem_o + lane_off + c * 32, r);
-      }
-      tmem_st_wait();
-    }
-    {
-      uint8_t* prow = sP + tid * 128;
+          for (int g = 0; g < 4; ++g) {
+            if (c * 32 + g * 8 >= p.dv) break;
+            float o[8];
 #pragma unroll
-      for (int piece = 0; piece < 8; ++piece) {
-        uint4 v = make_uint4(pk[piece * 4], pk[piece * 4 + 1], pk[piece * 4 + 2], pk[piece * 4 + 3]);
-        *reinterpret_cast<uint4*>(prow + ((piece ^ (tid & 7)) << 4)) = v;
-      }
-    }
-    fence_proxy_async_smem();
-    tc_fence_before();
-    __syncthreads();
-    if (tid == 0) {
-      tc_fence_after();
-      const uint32_t ap = smem_u32(sP), bv = smem_u32(sV + stage * L.v_bytes);
+            for (int i = 0; i < 8; ++i) o[i] = __uint_as_float(r[g * 8 + i]) * inv_l;
+            if (p.gate) {
+              float z[8];
+              load_vec<__nv_bfloat16, 8>(grow + c * 32 + g * 8, z);
 #pragma unroll
-      for (int kk = 0; kk < kWBlk / 16; ++kk) {
-        const uint64_t da = umma_smem_desc(ap + kk * 32, 16, 1024);
-        const uint64_t db = umma_smem_desc(bv + kk * 2048, 8192, 1024);
-        umma_bf16_ss(tmem_o, da, db, idesc_o, (j | kk) ? 1u : 0u);
-      }
-      umma_commit(bar_o);
-    }
-    if (!__all_sync(0xffffffffu, mbar_wait(bar_o, j & 1, status, kStatusTimeoutEpilogue))) {
-      ok = false;
-      break;
-    }
-    tc_fence_after();
-    if (tid == 0 && j + 2 < n_tiles) load_kv(j + 2, stage);
-  }
-
-  ok = __all_sync(0xffffffffu, ok);
-  if (ok) {
-    const bool row_valid = tid < nrows;
-    if (p.sink) l_run += exp2f(-m_run);
-    float inv_l = l_run > 0.f ? p.out_scale / l_run : 0.f;
-    if (p.head_gate && row_valid) inv_l *= p.head_gate[(size_t)(row0 + tid) * p.Hq + h];
-    __nv_bfloat16* orow = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)(row0 + (row_valid ? tid : 0)) * p.out_stride +
-                          p.out_off + (size_t)h * p.dv;
-    const __nv_bfloat16* grow = reinterpret_cast<const __nv_bfloat16*>(p.gate) +
-                                (size_t)(row0 + (row_valid ? tid : 0)) * p.gate_stride + (size_t)h * p.dv;
-#pragma unroll 1
-    for (int c = 0; c < (vn + 31) / 32; ++c) {
-      uint32_t r[32];
-      tmem_ld_32x32(tmem_o + lane_off + c * 32, r);
-      tmem_ld_wait();
-      if (row_valid) {
-#pragma unroll
-        for (int g = 0; g < 4; ++g) {
-          if (c * 32 + g * 8 >= p.dv) break;
-          float o[8];
-#pragma unroll
-          for (int i = 0; i < 8; ++i) o[i] = __uint_as_float(r[g * 8 + i]) * inv_l;
-          if (p.gate) {
-            float z[8];
-            load_vec<__nv_bfloat16, 8>(grow + c * 32 + g * 8, z);
-#pragma unroll
-            for (int i = 0; i < 8; ++i) o[i] = __fdividef(o[i], 1.f + __expf(-gain * z[i]));
+              for (int i = 0; i < 8; ++i) o[i] = __fdividef(o[i], 1.f + __expf(-gain * z[i]));
+            }
+            store_vec<__nv_bfloat16, 8>(orow + c * 32 + g * 8, o);
           }
-          store_vec<__nv_bfloat16, 8>(orow + c * 32 + g * 8, o);
         }
       }
     }
   }
-  if (!ok && tid == 0) {      // bounded: let the copies in flight land before shared memory is given back
-    mbar_wait(&bar_kv[0], 0, nullptr, 0);
-    mbar_wait(&bar_kv[1], 0, nullptr, 0);
-  }
   tc_fence_before();
   __syncthreads();
-  if (warp == 0) {
+  if (warp == 4) {
     tc_fence_after();
     tmem_dealloc(tmem_base, tmem_cols);
   }
@@ -508,10 +567,10 @@ extern "C" int sb_attn_window_prefill(const void* params, const int* tile_row, c
     if (e != cudaSuccess) return (int)e;
     configured[table] = L.total;
   }
-  const int need = 64 + (p.dv + 31) / 32 * 32;
-  uint32_t cols = 128;
+  const int need = 128 + (p.dv + 31) / 32 * 32;
+  uint32_t cols = 256;
   while ((int)cols < need) cols *= 2;
-  kernel<<<dim3(n_tiles, p.Hq), 128, L.total, stream>>>(mq, mk, mv, p, tile_row, tile_rows, tile_pos, tile_slot, cols,
+  kernel<<<dim3(n_tiles, p.Hq), 160, L.total, stream>>>(mq, mk, mv, p, tile_row, tile_rows, tile_pos, tile_slot, cols,
                                                         status);
   return (int)cudaGetLastError();
 }

@@ -10,7 +10,11 @@
 // Rotation: pairs (i, i + half) of the first 2 * half dimensions of a head turn by position * f_i.  f_i comes as two
 // floats (hi + lo) and the angle keeps its remainder, so the error does not grow with the position.
 //
-// One block per row; a row's projections stay in shared memory as 32-bit floats between the sums and the stores.
+// qkv_prepare_units_kernel: a thread keeps its units of eight columns in registers as 32-bit floats and meets the other half of
+// a rotated pair in shared memory; a block walks over rows, with the next row's loads in flight, one barrier per row.
+// qkv_prepare_kernel: any sizes, one block per row, the row in shared memory.
+#include <type_traits>
+
 #include "common.cuh"
 #include "launchers.h"
 #include "typed.cuh"
@@ -48,47 +52,257 @@ static_assert(sizeof(PrepareParams) == 216, "PrepareParams is mirrored from Pyth
 constexpr int kPrepBlk = 64;        // tokens per cache block
 constexpr int kPrepThreads = 128;
 
+// V columns of row t from `col` on, summed over the partial products, with the bias
 template <typename T, int V>
-__global__ void __launch_bounds__(kPrepThreads) qkv_prepare_kernel(const __grid_constant__ PrepareParams p) {
+__device__ __forceinline__ void prepare_fetch(const PrepareParams& p, int t, int col, float (&v)[V]) {
+  const size_t at = (size_t)t * p.row_stride + col;
+  if (p.x_f32) {
+    const float* x = reinterpret_cast<const float*>(p.x) + at;
+    load_vec<float, V>(x, v);
+    for (int s = 1; s < p.slabs; ++s) {
+      float y[V];
+      load_vec<float, V>(x + s * p.slab, y);
+#pragma unroll
+      for (int i = 0; i < V; ++i) v[i] += y[i];
+    }
+  } else {
+    load_vec<T, V>(reinterpret_cast<const T*>(p.x) + at, v);
+  }
+}
+
+// this row's place in its cache block (head 0, keys), or null
+template <typename T>
+__device__ __forceinline__ T* prepare_block(const PrepareParams& p, int t, int& pos) {
+  const int slot = p.seq_ids[t];
+  pos = p.positions[t];
+  if (slot < 0 || pos < 0 || pos / kPrepBlk >= p.max_blocks) return nullptr;
+  const int blk = p.block_table[(size_t)slot * p.max_blocks + pos / kPrepBlk];
+  if (blk < 0 || blk >= p.num_blocks) return nullptr;
+  return reinterpret_cast<T*>(p.cache) + (size_t)blk * p.block_elems;
+}
+
+// output gates of row t and the angles' cosines and sines
+template <typename T>
+__device__ __forceinline__ void prepare_gates(const PrepareParams& p, int t, int pos, float* s_cos, float* s_sin) {
+  if (p.g_off >= 0) {
+    for (int h = threadIdx.x; h < p.Hq; h += blockDim.x) {
+      float z[1];
+      prepare_fetch<T, 1>(p, t, p.g_off + h, z);
+      p.gate_out[(size_t)t * p.Hq + h] = 1.f / (1.f + expf(-z[0]));
+    }
+  }
+  for (int i = threadIdx.x; i < p.half; i += blockDim.x) {
+    const float n = (float)pos, a = n * p.freq[2 * i], lo = fmaf(n, p.freq[2 * i], -a) + n * p.freq[2 * i + 1];
+    float s, c;
+    sincosf(a, &s, &c);
+    s_cos[i] = fmaf(-s, lo, c);
+    s_sin[i] = fmaf(c, lo, s);
+  }
+}
+
+// blocks behind the `row_blocks` of the rows: the table of biases by distance
+template <typename T>
+__device__ __forceinline__ void prepare_table(const PrepareParams& p, int row_blocks) {
+  const int n = p.Hq * p.rel_n, step = (gridDim.x - row_blocks) * blockDim.x;
+  for (int i = (blockIdx.x - row_blocks) * blockDim.x + threadIdx.x; i < n; i += step) {
+    const int h = i / p.rel_n, d = i - h * p.rel_n;
+    p.rel_out[i] = to_float(reinterpret_cast<const T*>(p.rel)[(size_t)p.bucket[d] * p.Hq + h]);
+  }
+}
+
+// eight elements as they lie in memory
+template <typename T>
+struct Unit {
+  uint4 r[sizeof(T) / 2];
+  __device__ __forceinline__ void load(const T* p) {
+#pragma unroll
+    for (int i = 0; i < (int)sizeof(T) / 2; ++i) r[i] = reinterpret_cast<const uint4*>(p)[i];
+  }
+  __device__ __forceinline__ void get(float (&x)[8]) const { load_vec<T, 8>(reinterpret_cast<const T*>(r), x); }
+};
+
+// dk, dv and the rotated half are multiples of eight; a thread has U units of eight columns, the same in every row.  F32: the
+// projection comes as 32-bit partial sums.
+template <typename T, int U, bool F32>
+__global__ void __launch_bounds__(512, U == 2 && !F32 ? 2 : 1) qkv_prepare_units_kernel(const __grid_constant__ PrepareParams p, int row_blocks) {
+  extern __shared__ __align__(16) float sm[];
+  if ((int)blockIdx.x >= row_blocks) return prepare_table<T>(p, row_blocks);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int nq = p.Hq * p.dk / 8, nk = p.Hkv * p.dk / 8, nv = p.Hkv * p.dv / 8, per = p.dk / 8;      // units
+  // two buffers: [nq + nk][8] weighted values (the norm's factor still to come), cosines, sines, sums of squares (norm 2)
+  const int x_len = p.half ? 8 * (nq + nk) : 0, buf_len = (x_len + 2 * p.half + (p.norm == 2 ? nq + nk : 0) + 7) / 8 * 8;
+  __shared__ float red[2][2][16];
+  // heads whose units are a power of two lie in aligned lanes of one warp: their sums need no shared memory
+  const bool in_warp = per <= 32 && (per & (per - 1)) == 0;
+  int col[U], off[U], turn[U];        // column in x; place in the query row or in the cache block; first angle, + 1 << 16 in
+                                      // the second half of a pair, -1: not rotated
+#pragma unroll
+  for (int u = 0; u < U; ++u) {
+    const int i = tid + u * blockDim.x;
+    col[u] = off[u] = 0;
+    turn[u] = -1;
+    if (i < nq + nk && i % per < p.half / 4) {
+      const int at = i % per, half = p.half / 8;
+      turn[u] = at < half ? 8 * at : 8 * (at - half) + (1 << 16);
+    }
+    if (i < nq) {
+      col[u] = p.q_off + 8 * i;
+      off[u] = 8 * i;
+    } else if (i < nq + nk) {
+      const int e = 8 * (i - nq), head = e / p.dk;
+      col[u] = p.k_off + e;
+      off[u] = head * kPrepBlk * p.dk + e - head * p.dk;
+    } else if (i < nq + nk + nv) {
+      const int e = 8 * (i - nq - nk), head = e / p.dv;
+      col[u] = p.v_off + e;
+      off[u] = p.Hkv * kPrepBlk * p.dk + head * kPrepBlk * p.dv + e - head * p.dv;
+    }
+  }
+  using X = typename std::conditional<F32, float, T>::type;
+  Unit<X> next[U];
+  auto fetch = [&](int t) {           // the first (or only) part of row t
+#pragma unroll
+    for (int u = 0; u < U; ++u) next[u].load(reinterpret_cast<const X*>(p.x) + (size_t)t * p.row_stride + col[u]);
+  };
+  // slot and position of the row after the next, block of the next
+  auto place_of = [&](int t, int& slot, int& pos) {
+    slot = pos = -1;
+    if (t < p.T) {
+      slot = p.seq_ids[t];
+      pos = p.positions[t];
+    }
+  };
+  auto block_of = [&](int slot, int pos) {
+    return slot >= 0 && pos >= 0 && pos / kPrepBlk < p.max_blocks ? p.block_table[(size_t)slot * p.max_blocks + pos / kPrepBlk] : -1;
+  };
+  int t = blockIdx.x, slot0, pos0, slot1, pos1, buf = 0;
+  fetch(t);
+  place_of(t, slot0, pos0);
+  place_of(t + row_blocks, slot1, pos1);
+  int blk = block_of(slot0, pos0);
+  for (; t < p.T; t += row_blocks, buf ^= 1) {
+    float* s_x = sm + buf * buf_len;
+    float* s_cos = s_x + x_len;
+    float* s_sin = s_cos + p.half;
+    float* s_part = s_sin + p.half;
+    float v[U][8];
+#pragma unroll
+    for (int u = 0; u < U; ++u) next[u].get(v[u]);
+    if (t + row_blocks < p.T) fetch(t + row_blocks);
+    const int pos = pos0, place = pos % kPrepBlk;
+    T* crow = blk >= 0 && blk < p.num_blocks ? reinterpret_cast<T*>(p.cache) + (size_t)blk * p.block_elems : nullptr;
+    blk = block_of(slot1, pos1);
+    pos0 = pos1;
+    place_of(t + 2 * row_blocks, slot1, pos1);
+    if constexpr (F32) {
+      for (int s = 1; s < p.slabs; ++s)
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+          float y[8];
+          load_vec<float, 8>(reinterpret_cast<const float*>(p.x) + s * p.slab + (size_t)t * p.row_stride + col[u], y);
+#pragma unroll
+          for (int k = 0; k < 8; ++k) v[u][k] += y[k];
+        }
+    }
+    prepare_gates<T>(p, t, pos, s_cos, s_sin);
+    float ssq = 0.f, ssk = 0.f;
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int i = tid + u * blockDim.x;
+      if (p.bias && i < nq + nk + nv) {
+        float b[8];
+        load_vec<T, 8>(reinterpret_cast<const T*>(p.bias) + col[u], b);
+#pragma unroll
+        for (int k = 0; k < 8; ++k) v[u][k] += b[k];
+      }
+      if (i >= nq + nk) {
+        if (i < nq + nk + nv && crow) store_vec<T, 8>(crow + off[u] + place * p.dv, v[u]);
+        continue;
+      }
+      float ss = 0.f;
+#pragma unroll
+      for (int k = 0; k < 8; ++k) ss = fmaf(v[u][k], v[u][k], ss);
+      if (i < nq) ssq += ss;
+      else ssk += ss;
+      if (p.norm == 2 && !in_warp) s_part[i] = ss;
+      if (p.norm == 1) {
+        float w[8];
+        load_vec<T, 8>((i < nq ? reinterpret_cast<const T*>(p.q_norm) : reinterpret_cast<const T*>(p.k_norm) - 8 * nq) + 8 * i, w);
+#pragma unroll
+        for (int k = 0; k < 8; ++k) v[u][k] *= w[k];
+      }
+      if (turn[u] >= 0) store_vec<float, 8>(s_x + 8 * i, v[u]);
+    }
+    if (p.norm == 1) {
+      ssq = warp_sum(ssq);
+      ssk = warp_sum(ssk);
+      if (lane == 0) {
+        red[buf][0][warp] = ssq;
+        red[buf][1][warp] = ssk;
+      }
+    }
+    __syncthreads();      // the other buffer was last read before the barrier of the row before
+    float fq = 1.f, fk = 1.f;
+    if (p.norm == 1) {
+      ssq = ssk = 0.f;
+      for (int w = 0; w < (int)blockDim.x / 32; ++w) {
+        ssq += red[buf][0][w];
+        ssk += red[buf][1][w];
+      }
+      fq = 1.f / sqrtf(ssq / (float)(8 * nq) + p.eps);
+      fk = 1.f / sqrtf(ssk / (float)(8 * nk) + p.eps);
+    }
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int i = tid + u * blockDim.x;
+      float f = i < nq ? fq : fk;
+      if (p.norm == 2) {
+        float ss = 0.f;
+        if (in_warp) {
+#pragma unroll
+          for (int k = 0; k < 8; ++k) ss = fmaf(v[u][k], v[u][k], ss);
+          for (int o = per >> 1; o; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        } else if (i < nq + nk) {
+          const int h = i / per;
+          for (int k = 0; k < per; ++k) ss += s_part[h * per + k];
+        }
+        f = 1.f / sqrtf(ss / (float)p.dk + p.eps);
+      }
+      if (i >= nq + nk) continue;
+      if (turn[u] >= 0) {
+        const bool first = turn[u] < 1 << 16;
+        const int r = turn[u] & 0xffff;
+        float y[8], c[8], sn[8];
+        load_vec<float, 8>(s_x + 8 * i + (first ? p.half : -p.half), y);
+        load_vec<float, 8>(s_cos + r, c);
+        load_vec<float, 8>(s_sin + r, sn);
+#pragma unroll
+        for (int k = 0; k < 8; ++k) v[u][k] = fmaf(v[u][k], c[k], (first ? -y[k] : y[k]) * sn[k]);
+      }
+#pragma unroll
+      for (int k = 0; k < 8; ++k) v[u][k] *= f;
+      if (i < nq) store_vec<T, 8>(reinterpret_cast<T*>(p.q_out) + (size_t)t * p.q_stride + off[u], v[u]);
+      else if (crow) store_vec<T, 8>(crow + off[u] + place * p.dk, v[u]);
+    }
+  }
+}
+
+template <typename T, int V>
+__global__ void __launch_bounds__(kPrepThreads) qkv_prepare_kernel(const __grid_constant__ PrepareParams p, int row_blocks) {
   extern __shared__ float sm[];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  if ((int)blockIdx.x >= p.T) {      // distance table
-    const int n = p.Hq * p.rel_n, step = (gridDim.x - p.T) * kPrepThreads;
-    for (int i = (blockIdx.x - p.T) * kPrepThreads + tid; i < n; i += step) {
-      const int h = i / p.rel_n, d = i - h * p.rel_n;
-      p.rel_out[i] = to_float(reinterpret_cast<const T*>(p.rel)[(size_t)p.bucket[d] * p.Hq + h]);
-    }
-    return;
-  }
+  if ((int)blockIdx.x >= row_blocks) return prepare_table<T>(p, row_blocks);
   const int t = blockIdx.x;
   const int nq = p.Hq * p.dk, nk = p.Hkv * p.dk, nv = p.Hkv * p.dv;
   float* s_x = sm;                    // [nq + nk]
   float* s_cos = s_x + nq + nk;       // [half]
   float* s_sin = s_cos + p.half;
   __shared__ float red[2][kPrepThreads / 32];
-  const int slot = p.seq_ids[t], pos = p.positions[t];
-  T* crow = nullptr;                  // this row's place in its cache block (head 0, keys)
-  if (slot >= 0 && pos >= 0 && pos / kPrepBlk < p.max_blocks) {
-    const int blk = p.block_table[(size_t)slot * p.max_blocks + pos / kPrepBlk];
-    if (blk >= 0 && blk < p.num_blocks) crow = reinterpret_cast<T*>(p.cache) + (size_t)blk * p.block_elems;
-  }
+  int pos;
+  T* crow = prepare_block<T>(p, t, pos);
   const int place = pos % kPrepBlk;
-
-  // V columns of the row from `col` on, summed over the partial products, with the bias
   auto fetch = [&](int col, float (&v)[V]) {
-    const size_t at = (size_t)t * p.row_stride + col;
-    if (p.x_f32) {
-      const float* x = reinterpret_cast<const float*>(p.x) + at;
-      load_vec<float, V>(x, v);
-      for (int s = 1; s < p.slabs; ++s) {
-        float y[V];
-        load_vec<float, V>(x + s * p.slab, y);
-#pragma unroll
-        for (int i = 0; i < V; ++i) v[i] += y[i];
-      }
-    } else {
-      load_vec<T, V>(reinterpret_cast<const T*>(p.x) + at, v);
-    }
+    prepare_fetch<T, V>(p, t, col, v);
     if (p.bias) {
       float b[V];
       load_vec<T, V>(reinterpret_cast<const T*>(p.bias) + col, b);
@@ -116,25 +330,7 @@ __global__ void __launch_bounds__(kPrepThreads) qkv_prepare_kernel(const __grid_
     if (crow)
       store_vec<T, V>(crow + (size_t)p.Hkv * kPrepBlk * p.dk + ((size_t)head * kPrepBlk + place) * p.dv + (e - head * p.dv), v);
   }
-  if (p.g_off >= 0) {
-    for (int h = tid; h < p.Hq; h += kPrepThreads) {
-      const size_t at = (size_t)t * p.row_stride + p.g_off + h;
-      float z = 0.f;
-      if (p.x_f32) {
-        for (int s = 0; s < p.slabs; ++s) z += reinterpret_cast<const float*>(p.x)[s * p.slab + at];
-      } else {
-        z = to_float(reinterpret_cast<const T*>(p.x)[at]);
-      }
-      p.gate_out[(size_t)t * p.Hq + h] = 1.f / (1.f + expf(-z));
-    }
-  }
-  for (int i = tid; i < p.half; i += kPrepThreads) {
-    const float n = (float)pos, a = n * p.freq[2 * i], lo = fmaf(n, p.freq[2 * i], -a) + n * p.freq[2 * i + 1];
-    float s, c;
-    sincosf(a, &s, &c);
-    s_cos[i] = fmaf(-s, lo, c);
-    s_sin[i] = fmaf(c, lo, s);
-  }
+  prepare_gates<T>(p, t, pos, s_cos, s_sin);
   float fq = 1.f, fk = 1.f;
   if (p.norm == 1) {
     ssq = warp_sum(ssq);
@@ -196,23 +392,58 @@ __global__ void __launch_bounds__(kPrepThreads) qkv_prepare_kernel(const __grid_
   }
 }
 
-template <typename T, int V>
-static int launch_prepare(const PrepareParams& p, cudaStream_t s) {
-  const size_t smem = ((size_t)(p.Hq + p.Hkv) * p.dk + 2 * (size_t)p.half) * 4;
-  static size_t configured = 48 * 1024;
-  if (smem > configured) {
-    if (smem > 200 * 1024) return -3;
-    cudaError_t e = cudaFuncSetAttribute(qkv_prepare_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e != cudaSuccess) return (int)e;
-    configured = smem;
-  }
+using PrepareKernel = void (*)(PrepareParams, int);
+
+static int prepare_configure(PrepareKernel kernel, size_t smem, size_t& configured) {
+  if (smem <= configured) return 0;
+  if (smem > 200 * 1024) return -3;
+  cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  if (e != cudaSuccess) return (int)e;
+  configured = smem;
+  return 0;
+}
+
+static int prepare_launch(PrepareKernel kernel, const PrepareParams& p, int row_blocks, int threads, size_t smem, cudaStream_t s) {
   int extra = 0;
   if (p.rel) {
-    extra = (p.Hq * p.rel_n + 4 * kPrepThreads - 1) / (4 * kPrepThreads);
+    extra = (p.Hq * p.rel_n + 4 * threads - 1) / (4 * threads);
     if (extra > num_sms()) extra = num_sms();
   }
-  qkv_prepare_kernel<T, V><<<p.T + extra, kPrepThreads, smem, s>>>(p);
+  kernel<<<row_blocks + extra, threads, smem, s>>>(p, row_blocks);
   return (int)cudaGetLastError();
+}
+
+template <typename T, int V>
+static int launch_prepare(const PrepareParams& p, cudaStream_t s) {
+  static size_t configured = 48 * 1024;
+  const size_t smem = ((size_t)(p.Hq + p.Hkv) * p.dk + 2 * (size_t)p.half) * 4;
+  const int r = prepare_configure(qkv_prepare_kernel<T, V>, smem, configured);
+  return r ? r : prepare_launch(qkv_prepare_kernel<T, V>, p, p.T, kPrepThreads, smem, s);
+}
+
+template <typename T, int U, bool F32>
+static int launch_prepare_units(const PrepareParams& p, cudaStream_t s) {
+  auto kernel = qkv_prepare_units_kernel<T, U, F32>;
+  const int qk = (p.Hq + p.Hkv) * p.dk, units = (qk + p.Hkv * p.dv) / 8;
+  const int threads = ((units + U - 1) / U + 31) / 32 * 32;
+  const size_t smem = 8 * (((size_t)(p.half ? qk : 0) + 2 * (size_t)p.half + (p.norm == 2 ? qk / 8 : 0) + 7) / 8 * 8);
+  static size_t configured = 48 * 1024;
+  const int r = prepare_configure(kernel, smem, configured);
+  if (r) return r;
+  int blocks = 1;
+  if (p.T > num_sms()) {
+    cudaError_t e = cudaOccupancyMaxActiveBlocksPerMultiprocessor(&blocks, kernel, threads, smem);
+    if (e != cudaSuccess) return (int)e;
+    if (blocks < 1) blocks = 1;
+  }
+  blocks *= num_sms();
+  return prepare_launch(kernel, p, p.T < blocks ? p.T : blocks, threads, smem, s);
+}
+
+template <typename T>
+static int launch_prepare_units(const PrepareParams& p, int units, cudaStream_t s) {
+  if (p.x_f32) return units <= 2 * 512 ? launch_prepare_units<T, 2, true>(p, s) : launch_prepare_units<T, 4, true>(p, s);
+  return units <= 2 * 512 ? launch_prepare_units<T, 2, false>(p, s) : launch_prepare_units<T, 4, false>(p, s);
 }
 
 }  // namespace sb
@@ -230,6 +461,10 @@ extern "C" int sb_qkv_prepare(const void* params, int f32, cudaStream_t stream) 
   const int V = f32 ? 4 : 8;
   const bool vec = p.dk % V == 0 && p.dv % V == 0 && p.row_stride % V == 0 && p.slab % V == 0 && p.q_off % V == 0 &&
                    p.k_off % V == 0 && p.v_off % V == 0 && p.q_stride % V == 0 && p.block_elems % V == 0;
+  const int units = ((p.Hq + p.Hkv) * p.dk + p.Hkv * p.dv) / 8;
+  if (vec && p.dk % 8 == 0 && p.dv % 8 == 0 && p.half % 8 == 0 && units <= 4 * 512) {
+    return f32 ? launch_prepare_units<float>(p, units, stream) : launch_prepare_units<__nv_bfloat16>(p, units, stream);
+  }
   if (f32) return vec ? launch_prepare<float, 4>(p, stream) : launch_prepare<float, 1>(p, stream);
   return vec ? launch_prepare<__nv_bfloat16, 8>(p, stream) : launch_prepare<__nv_bfloat16, 1>(p, stream);
 }

@@ -48,7 +48,7 @@ struct ScoreCap {
   __device__ __forceinline__ ScoreCap(float cap, float scale)
       : in(2.f * 1.4426950408889634f * scale / cap), out(cap * 1.4426950408889634f) {}
   __device__ __forceinline__ float operator()(float x) const {
-    return out - __fdividef(2.f * out, 1.f + fast_exp2(in * x));
+    return fmaf(-2.f * out, fast_rcp(1.f + fast_exp2(in * x)), out);
   }
 };
 

@@ -78,6 +78,8 @@ ATT = {
                  rot=dict(dims=24, base=1e4, scaling={"factor": 4.0, "low": 1.0, "high": 4.0, "original": 60})),
     "bias_whole": dict(size=(4, 1, 128, 128), norm="rows", bias=True, rot=dict(dims=128, base=1e6)),
     "very_wide": dict(size=(2, 1, 192, 256), norm="rows", bias=True, rot=dict(dims=96, base=1e4)),
+    "many_columns": dict(size=(33, 11, 192, 16), norm="heads", rot=dict(dims=16, base=1e4), sink=True),
+    "odd_units": dict(size=(5, 5, 24, 8), norm="heads", rot=dict(dims=16, base=1e4), sink=True),
     "odd": dict(size=(3, 3, 21, 13), norm="rows", window=50, cap=15.0, rel=(10, 33), gate=True),
     "odd_sink": dict(size=(3, 1, 18, 11), norm="heads", rot=dict(dims=6, base=1e3), sink=True),
     "odd_bias": dict(size=(5, 5, 10, 7), norm="rows", bias=True, rot=dict(dims=10, base=1e3)),
