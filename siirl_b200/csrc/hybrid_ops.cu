@@ -192,6 +192,34 @@ __global__ void scaled_act_kernel(const T* __restrict__ x, long long stride, con
   }
 }
 
+// act of the sum of fp32 partial products [slabs, rows, I or 2 I] (GATED: act(first half) * second half), bf16 result
+template <int V, int ACT, bool GATED>
+__global__ void partial_act_kernel(const float* __restrict__ x, long long slab, int slabs, __nv_bfloat16* __restrict__ out,
+                                   long long rows, int I) {
+  const int nv = I / V, pitch = GATED ? 2 * I : I;
+  const long long total = rows * nv;
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const long long t = i / nv;
+    const int c = (int)(i % nv) * V;
+    float g[V] = {}, u[V] = {};
+    const float* p = x + t * pitch + c;
+    for (int s = 0; s < slabs; ++s, p += slab) {
+      float a[V];
+      load_vec<float, V>(p, a);
+#pragma unroll
+      for (int k = 0; k < V; ++k) g[k] += a[k];
+      if constexpr (GATED) {
+        load_vec<float, V>(p + I, a);
+#pragma unroll
+        for (int k = 0; k < V; ++k) u[k] += a[k];
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < V; ++k) g[k] = activate<ACT, __nv_bfloat16>(g[k]) * (GATED ? u[k] : 1.f);
+    store_vec<__nv_bfloat16, V>(out + t * I + c, g);
+  }
+}
+
 // mirrored by ctypes structures in ops/rows.py
 struct StreamSub {
   const void* y;            // [slabs, T or 2 T, W] partial sums (fp32), or one tensor in the activation format
@@ -583,5 +611,26 @@ extern "C" int sb_gemm_simt_grouped(const void* A, const void* B, void* C, int M
   else
     gemm_simt_kernel<H, H, true><<<grid, 256, 0, stream>>>((const H*)A, (const H*)B, (H*)C, M, N, K, lda, ldb, ldc,
                                                            tile_group, a_row, b_group);
+  return (int)cudaGetLastError();
+}
+
+// act of the sum of partial products; I a multiple of 4.  gated: x [slabs, rows, 2 I], else [slabs, rows, I]
+extern "C" int sb_partial_act(const float* x, long long slab, int slabs, void* out, long long rows, int I, int act, int gated,
+                              cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  if (I % 4 || slab % 4 || slabs < 1 || act < 0 || act > 3) return -3;
+  const int grid = grid_for(rows * I / 4, 256);
+  auto launch = [&](auto kernel) { kernel<<<grid, 256, 0, stream>>>(x, slab, slabs, (__nv_bfloat16*)out, rows, I); };
+  if (gated) {
+    if (act == 0) launch(partial_act_kernel<4, 0, true>);
+    else if (act == 1) launch(partial_act_kernel<4, 1, true>);
+    else if (act == 2) launch(partial_act_kernel<4, 2, true>);
+    else launch(partial_act_kernel<4, 3, true>);
+  } else {
+    if (act == 0) launch(partial_act_kernel<4, 0, false>);
+    else if (act == 1) launch(partial_act_kernel<4, 1, false>);
+    else if (act == 2) launch(partial_act_kernel<4, 2, false>);
+    else launch(partial_act_kernel<4, 3, false>);
+  }
   return (int)cudaGetLastError();
 }

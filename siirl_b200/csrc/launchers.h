@@ -24,7 +24,7 @@ int sb_gemm_ar_bf16(const void* A, const void* B, const void* bias, int M, int N
                     const void* ar_params, void* c_local, int tile_n, int k_splits, long long slab_stride,
                     int max_tiles, int* status, cudaStream_t stream);
 int sb_moe_gather_rows(const void* const* src_ptrs, int world, const int* src_rank, const int* src_row,
-                       const float* scale, void* out, int M, int H, cudaStream_t stream);
+                       const float* scale, void* out, int M, int H, int skip_empty, cudaStream_t stream);
 int sb_moe_combine(const void* const* y_ptrs, int world, const int* pair_rank, const int* pair_slot, const float* w,
                    void* out, int T, int k, int H, cudaStream_t stream);
 int sb_moe_pair_dot(const void* const* y_ptrs, int world, const int* pair_rank, const int* pair_slot, const void* dout,
@@ -194,6 +194,8 @@ int sb_embed_scaled(const long long* ids, const void* table, float* h, int T, in
 int sb_add_norm(float* h, const void* delta, const void* w, void* y, int rows, int W, float eps, int layer_norm, int f32,
                 cudaStream_t stream);
 int sb_gated_act(const void* gu, void* out, long long rows, int I, int act, const int* used, int f32, cudaStream_t stream);
+int sb_partial_act(const float* x, long long slab, int slabs, void* out, long long rows, int I, int act, int gated,
+                   cudaStream_t stream);
 int sb_gemm_simt_grouped(const void* A, const void* B, void* C, int M, int N, int K, long long lda, long long ldb,
                          long long ldc, const int* tile_group, const int* a_row, long long b_group, int f32,
                          cudaStream_t stream);

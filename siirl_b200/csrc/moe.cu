@@ -25,7 +25,8 @@ struct MoePeers {
 };
 
 __global__ void moe_gather_rows_kernel(MoePeers src, const int* __restrict__ src_rank, const int* __restrict__ src_row,
-                                       const float* __restrict__ scale, __nv_bfloat16* __restrict__ out, int M, int H) {
+                                       const float* __restrict__ scale, __nv_bfloat16* __restrict__ out, int M, int H,
+                                       int skip_empty) {
   const int warps_per_block = blockDim.x >> 5;
   const int lane = threadIdx.x & 31;
   const int nvec = H / 8;
@@ -33,7 +34,8 @@ __global__ void moe_gather_rows_kernel(MoePeers src, const int* __restrict__ src
     const int sr = src_row[row];
     uint4* dst = reinterpret_cast<uint4*>(out + (long long)row * H);
     if (sr < 0) {
-      for (int v = lane; v < nvec; v += 32) dst[v] = make_uint4(0u, 0u, 0u, 0u);
+      if (!skip_empty)
+        for (int v = lane; v < nvec; v += 32) dst[v] = make_uint4(0u, 0u, 0u, 0u);
       continue;
     }
     const uint4* s = reinterpret_cast<const uint4*>(src.p[src_rank ? src_rank[row] : 0] + (long long)sr * H);
@@ -132,12 +134,14 @@ static bool fill_peers(MoePeers& mp, const void* const* ptrs, int world) {
 
 using namespace sb;
 
+// skip_empty: rows without a source stay unwritten (inference: nothing reads their products)
 extern "C" int sb_moe_gather_rows(const void* const* src_ptrs, int world, const int* src_rank, const int* src_row,
-                                  const float* scale, void* out, int M, int H, cudaStream_t stream) {
+                                  const float* scale, void* out, int M, int H, int skip_empty, cudaStream_t stream) {
   if (M <= 0) return 0;
   MoePeers mp;
   if (H % 8 || !fill_peers(mp, src_ptrs, world)) return -3;
-  moe_gather_rows_kernel<<<moe_grid(M), 256, 0, stream>>>(mp, src_rank, src_row, scale, (__nv_bfloat16*)out, M, H);
+  moe_gather_rows_kernel<<<moe_grid(M), 256, 0, stream>>>(mp, src_rank, src_row, scale, (__nv_bfloat16*)out, M, H,
+                                                          skip_empty);
   return (int)cudaGetLastError();
 }
 
@@ -324,6 +328,7 @@ extern "C" int sb_moe_route_topk_bwd(const void* logits, int is_bf16, int ld, co
 //   count:  per-chunk histograms (chunk = 1024 consecutive pairs) + initial values of the slot arrays
 //   scan:   per-expert exclusive scan over chunks, padded expert starts, per-rank bases, block -> expert table
 //   place:  stable rank inside the chunk (warp match + per-warp counts), slot of every pair, owner's slot arrays
+// Up to kLayoutSmall pairs (a decoding step): all of it in one block, one launch.
 constexpr int kLayoutChunk = 1024;
 constexpr int kLayoutMaxE = 256;   // real experts; one dummy expert for padding tokens is appended
 
@@ -348,6 +353,42 @@ __global__ void __launch_bounds__(kLayoutChunk) moe_layout_count_kernel(
   }
 }
 
+constexpr int kLayoutSmall = 4096;
+
+// counts[0 .. E] -> padded starts s_starts[0 .. E + 1], by warp 0 (each lane sums a run of experts)
+__device__ __forceinline__ void layout_starts(const int* counts, int E, int* s_starts) {
+  const int lane = threadIdx.x & 31, run = (E + 1 + 31) / 32, e0 = lane * run;
+  int sum = 0;
+  for (int e = e0; e < e0 + run && e <= E; ++e) sum += (counts[e] + 127) / 128 * 128;
+  int acc = sum;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const int v = __shfl_up_sync(0xffffffffu, acc, o);
+    if (lane >= o) acc += v;
+  }
+  int at = acc - sum;
+  for (int e = e0; e < e0 + run && e <= E; ++e) {
+    s_starts[e] = at;
+    at += (counts[e] + 127) / 128 * 128;
+    if (e == E) s_starts[E + 1] = at;
+  }
+}
+
+// tables of my experts from the padded starts: row ranges, expert of every 128-row block (-1 beyond the last)
+__device__ __forceinline__ void layout_tables(const int* s_starts, int El, int rank, int capacity, int* tile_group,
+                                              int* group_rows) {
+  const int base = s_starts[rank * El];
+  for (int i = threadIdx.x; i <= El; i += blockDim.x) {
+    const int v = i == 0 ? 0 : s_starts[rank * El + i] - base;
+    group_rows[i] = v < capacity ? v : capacity;
+  }
+  const int used = (s_starts[rank * El + El] - base) / 128, blocks = capacity / 128;
+  for (int b = used + threadIdx.x; b < blocks; b += blockDim.x) tile_group[b] = -1;
+  for (int g = threadIdx.x; g < El; g += blockDim.x)
+    for (int b = (s_starts[rank * El + g] - base) / 128; b < (s_starts[rank * El + g + 1] - base) / 128 && b < blocks; ++b)
+      tile_group[b] = g;
+}
+
 __global__ void __launch_bounds__(1024) moe_layout_scan_kernel(int* __restrict__ chunk_counts, int n_chunks, int E,
                                                                int world, int rank, int capacity,
                                                                int* __restrict__ starts, int* __restrict__ rank_base,
@@ -355,39 +396,101 @@ __global__ void __launch_bounds__(1024) moe_layout_scan_kernel(int* __restrict__
                                                                int* __restrict__ group_rows) {
   __shared__ int counts[kLayoutMaxE + 1];
   __shared__ int s_starts[kLayoutMaxE + 2];
-  const int El = E / world;
-  for (int e = threadIdx.x; e <= E; e += blockDim.x) {
+  const int El = E / world, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int e = warp; e <= E; e += 32) {      // exclusive sums over the chunks, 32 at a time
     int running = 0;
-    for (int c = 0; c < n_chunks; ++c) {
-      const int v = chunk_counts[(size_t)c * (E + 1) + e];
-      chunk_counts[(size_t)c * (E + 1) + e] = running;
-      running += v;
+    for (int c0 = 0; c0 < n_chunks; c0 += 32) {
+      const int c = c0 + lane;
+      const int v = c < n_chunks ? chunk_counts[(size_t)c * (E + 1) + e] : 0;
+      int acc = v;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int u = __shfl_up_sync(0xffffffffu, acc, o);
+        if (lane >= o) acc += u;
+      }
+      if (c < n_chunks) chunk_counts[(size_t)c * (E + 1) + e] = running + acc - v;
+      running += __shfl_sync(0xffffffffu, acc, 31);
     }
-    counts[e] = running;
+    if (lane == 0) counts[e] = running;
   }
   __syncthreads();
-  if (threadIdx.x == 0) {
-    int acc = 0;
-    for (int e = 0; e <= E; ++e) {
-      s_starts[e] = acc;
-      acc += (counts[e] + 127) / 128 * 128;
-    }
-    s_starts[E + 1] = acc;
-  }
+  if (warp == 0) layout_starts(counts, E, s_starts);
   __syncthreads();
   for (int e = threadIdx.x; e <= E + 1; e += blockDim.x) starts[e] = s_starts[e];
   for (int r = threadIdx.x; r <= world; r += blockDim.x) rank_base[r] = s_starts[r * El];
-  const int base = s_starts[rank * El];
-  // padded end of my local experts in local coordinates: s_starts[rank*El + i + 1] - base
-  for (int i = threadIdx.x; i <= El; i += blockDim.x) {
-    const int v = i == 0 ? 0 : s_starts[rank * El + i] - base;
-    group_rows[i] = v < capacity ? v : capacity;
+  layout_tables(s_starts, El, rank, capacity, tile_group, group_rows);
+}
+
+__global__ void __launch_bounds__(kLayoutChunk) moe_layout_small_kernel(
+    const int* __restrict__ idx, int P, int E, int world, int rank, int T, int k, int capacity,
+    int* __restrict__ pair_rank, int* __restrict__ pair_slot, long long* __restrict__ slot_pair,
+    int* __restrict__ slot_src_rank, int* __restrict__ slot_src_row, int* __restrict__ tile_group,
+    int* __restrict__ group_rows) {
+  __shared__ int wc[kLayoutChunk / 32][kLayoutMaxE + 2];
+  __shared__ int counts[kLayoutMaxE + 1];
+  __shared__ int s_starts[kLayoutMaxE + 2];
+  constexpr int kRounds = kLayoutSmall / kLayoutChunk;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, El = E / world;
+  int ex[kRounds], at[kRounds];
+#pragma unroll
+  for (int c = 0; c < kRounds; ++c) {
+    const int p = c * kLayoutChunk + threadIdx.x;
+    ex[c] = E + 1;                                  // lanes past the end: a key of their own, never placed
+    if (p < P) {
+      ex[c] = idx[p];
+      if (ex[c] < 0 || ex[c] >= E) ex[c] = E;
+    }
   }
-  for (int b = threadIdx.x; b < capacity / 128; b += blockDim.x) {
-    const int row = b * 128;
-    int g = 0;   // number of local experts whose padded end is <= row
-    while (g < El && s_starts[rank * El + g + 1] - base <= row) ++g;
-    tile_group[b] = g < El ? g : -1;
+  for (int s = threadIdx.x; s < capacity; s += blockDim.x) {
+    slot_pair[s] = -1;
+    slot_src_rank[s] = 0;
+    slot_src_row[s] = -1;
+  }
+  for (int e = threadIdx.x; e <= E; e += blockDim.x) counts[e] = 0;
+#pragma unroll
+  for (int c = 0; c < kRounds; ++c) {
+    if (c * kLayoutChunk >= P) break;
+    for (int e = lane; e <= E + 1; e += 32) wc[warp][e] = 0;
+    __syncwarp();
+    const unsigned peers = __match_any_sync(0xffffffffu, ex[c]);
+    at[c] = __popc(peers & ((1u << lane) - 1u));
+    if (at[c] == 0) wc[warp][ex[c]] = __popc(peers);
+    __syncthreads();
+    for (int e = threadIdx.x; e <= E; e += blockDim.x) {
+      int running = counts[e];
+#pragma unroll 8
+      for (int w = 0; w < kLayoutChunk / 32; ++w) {
+        const int v = wc[w][e];
+        wc[w][e] = running;
+        running += v;
+      }
+      counts[e] = running;
+    }
+    __syncthreads();
+    at[c] += wc[warp][ex[c]];
+    __syncwarp();
+  }
+  if (warp == 0) layout_starts(counts, E, s_starts);
+  __syncthreads();
+  layout_tables(s_starts, El, rank, capacity, tile_group, group_rows);
+#pragma unroll
+  for (int c = 0; c < kRounds; ++c) {
+    const int p = c * kLayoutChunk + threadIdx.x;
+    if (p >= P) break;
+    const int host = ex[c] / El;                    // == world for padding pairs
+    if (ex[c] >= E || host >= world) {
+      pair_rank[p] = world - 1;
+      pair_slot[p] = -1;
+      continue;
+    }
+    const int lslot = s_starts[ex[c]] + at[c] - s_starts[host * El];
+    pair_rank[p] = host;
+    pair_slot[p] = lslot < capacity ? lslot : -1;
+    if (host == rank && lslot < capacity) {
+      slot_pair[lslot] = p;
+      slot_src_rank[lslot] = p / (T * k);
+      slot_src_row[lslot] = (p / k) % T;
+    }
   }
 }
 
@@ -446,6 +549,11 @@ extern "C" int sb_moe_build_layout(const int* idx, int P, int E, int world, int 
   if (P <= 0 || E < 1 || E > kLayoutMaxE || world < 1 || E % world || rank < 0 || rank >= world || capacity % 128 ||
       capacity <= 0 || T <= 0 || k <= 0)
     return -3;
+  if (P <= kLayoutSmall) {
+    moe_layout_small_kernel<<<1, kLayoutChunk, 0, stream>>>(idx, P, E, world, rank, T, k, capacity, pair_rank, pair_slot,
+                                                           slot_pair, slot_src_rank, slot_src_row, tile_group, group_rows);
+    return (int)cudaGetLastError();
+  }
   const int n_chunks = (P + kLayoutChunk - 1) / kLayoutChunk;
   moe_layout_count_kernel<<<n_chunks, kLayoutChunk, 0, stream>>>(idx, P, E, chunk_counts, slot_pair, slot_src_rank,
                                                                 slot_src_row, capacity);

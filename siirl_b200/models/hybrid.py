@@ -306,14 +306,14 @@ class RoutedFeedForward(nn.Module):
 
     def run(self, x: torch.Tensor) -> R.SublayerSum:
         e = self.spec
-        z = linear_partial(x, self.router_weight.detach(), f32=True)
+        z = linear_partial(x, self.router_weight.detach(), f32=True, max_splits=12)
         w, ids, w_id = route_grouped(z, self.correction.detach(), e.experts, e.top, e.groups, e.keep, e.scale)
         ys, slots = routed_experts(x, ids, self.gate_up_weight.detach(), self.down_weight.detach(), e.act)
         out = R.SublayerSum(ys=ys, pair_slot=slots, pair_w=w)
         if e.identity:
             out.x_id, out.w_id = x, w_id
         if e.shared_ff:
-            a = R.gated_act(ops.linear(x, self.shared_gate_up_weight), e.act)
+            a = R.partial_act(linear_partial(x, self.shared_gate_up_weight.detach()), e.act, gated=True)
             out.y = linear_partial(a, self.shared_down_weight.detach())
         return out
 
@@ -370,7 +370,7 @@ class HyperLayer(nn.Module):
     def feed_forward(self, x: torch.Tensor, io: "_Batch") -> R.SublayerSum:
         if self.moe is not None:
             return self.moe.run(x)
-        a = R.scaled_act(ops.linear(x, self.up_proj_weight), self.cfg.hybrid.act)
+        a = R.partial_act(linear_partial(x, self.up_proj_weight.detach()), self.cfg.hybrid.act)
         return R.SublayerSum(linear_partial(a, self.down_proj_weight.detach()))
 
 

@@ -206,9 +206,10 @@ def linear_skinny(x2: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.T
     return out
 
 
-def linear_partial(x: torch.Tensor, weight: torch.Tensor, f32: bool = False) -> torch.Tensor:
+def linear_partial(x: torch.Tensor, weight: torch.Tensor, f32: bool = False, max_splits: int = 0) -> torch.Tensor:
     """Inference-only ``x @ W^T`` as partial sums ``[S, M, N]`` for a consumer that adds them itself: few rows give the
-    fp32 slabs of a split contraction, many rows one bf16 product (fp32 when ``f32``)."""
+    fp32 slabs of a split contraction, many rows one bf16 product (fp32 when ``f32``).  ``max_splits``: a product of few
+    output tiles, whose partial sums cost next to nothing, may be split that often to use more SMs."""
     M, K = x.shape
     N = weight.shape[0]
     if not x.is_cuda:
@@ -221,6 +222,8 @@ def linear_partial(x: torch.Tensor, weight: torch.Tensor, f32: bool = False) -> 
     nkb = (K + 63) // 64
     swap = M > 128 and SWAP_OPERANDS_ABOVE_128_ROWS
     splits = _best_splits((N + 127) // 128 * ((M + 255) // 256), nkb) if swap else _skinny_splits(M, N, K)
+    if max_splits:
+        splits = max(splits, min(max_splits, nkb // 2))
     if splits <= 1 and not f32:
         return linear_skinny(x, weight, None)[None]
     per = (nkb + splits - 1) // splits

@@ -56,8 +56,8 @@ _FUSED_LAYOUT = True        # tests flip this to compare the kernels with the de
 
 def _build_layout_fused(all_idx: torch.Tensor, num_experts: int, world: int, rank: int,
                         capacity: Optional[int]) -> "MoeLayout":
-    """The same layout from three launches (histogram per 1024-pair chunk, scan, stable placement) instead of the
-    ~70 small device ops and the sort of the construction in ``build_layout``."""
+    """The same layout from three launches (histogram per 1024-pair chunk, scan, stable placement; one launch up to 4096
+    pairs) instead of the ~70 small device ops and the sort of the construction in ``build_layout``."""
     W, T, k = all_idx.shape
     dev = all_idx.device
     El = num_experts // world
@@ -207,7 +207,7 @@ class ExpertParallel:
         out = torch.empty(M, H, dtype=src.dtype, device=src.device)
         L = _lib.get_lib()
         _lib.check(L.sb_moe_gather_rows(ptrs, world, _lib.ptr(src_rank if world > 1 else None), _lib.ptr(src_row),
-                                        _lib.ptr(scale), _lib.ptr(out), M, H, _lib.stream()), "sb_moe_gather_rows")
+                                        _lib.ptr(scale), _lib.ptr(out), M, H, 0, _lib.stream()), "sb_moe_gather_rows")
         self.barrier()          # peers have finished reading my staging buffer
         return out
 
@@ -473,7 +473,8 @@ def routed_experts(x: torch.Tensor, ids: torch.Tensor, gate_up: torch.Tensor, do
     if x.dtype == torch.bfloat16 and W % 8 == 0 and I % 8 == 0:
         rows = torch.empty(capacity, W, dtype=x.dtype, device=x.device)
         _lib.check(_lib.get_lib().sb_moe_gather_rows((ctypes.c_void_p * 1)(x.data_ptr()), 1, None, _lib.ptr(lay.slot_src_row),
-                                                     None, _lib.ptr(rows), capacity, W, _lib.stream()), "sb_moe_gather_rows")
+                                                     None, _lib.ptr(rows), capacity, W, 1, _lib.stream()),
+                   "sb_moe_gather_rows")
         a = gated_act(grouped_linear(rows, gate_up, lay), act, lay.slot_src_row)
         return grouped_linear(a, down, lay), lay.pair_slot
 

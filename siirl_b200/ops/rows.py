@@ -83,6 +83,22 @@ def scaled_act(x: torch.Tensor, act: str, gain: Optional[torch.Tensor] = None) -
     return out
 
 
+def partial_act(x: torch.Tensor, act: str, gated: bool = False) -> torch.Tensor:
+    """Activation of partial products ``x [S, T, I]`` (what :func:`siirl_b200.ops.dense.linear_partial` returns for a bf16
+    model): the sum and ``act`` in one launch; ``gated``: ``act(first half) * second half`` of ``[S, T, 2 I]``."""
+    S, T, N = x.shape
+    I = N // 2 if gated else N
+    if x.is_cuda and S > 1 and x.dtype == torch.float32:
+        assert x.is_contiguous() and I % 4 == 0
+        out = torch.empty(T, I, dtype=torch.bfloat16, device=x.device)
+        _lib.check(_lib.get_lib().sb_partial_act(_lib.ptr(x), ctypes.c_longlong(T * N), S, _lib.ptr(out),
+                                                 ctypes.c_longlong(T), I, ACT[act], int(gated), _lib.stream()),
+                   "sb_partial_act")
+        return out
+    assert S == 1
+    return gated_act(x[0], act) if gated else scaled_act(x[0], act)
+
+
 @dataclass
 class Sublayer:
     """One result waiting to enter the residual stream: ``y [S, T, W]`` (partial sums, or one tensor in the activation

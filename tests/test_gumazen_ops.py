@@ -434,6 +434,23 @@ def test_activations(device, dtype):
     finish(device)
 
 
+@pytest.mark.gpu
+def test_activation_of_partial_products():
+    """Few rows split the contraction; the activation adds the parts up itself."""
+    from siirl_b200.ops.dense import linear_partial
+    g = torch.Generator().manual_seed(1)
+    for T, W, I in ((5, 2048, 96), (200, 1024, 72), (700, 512, 40)):
+        x, w = rounded(torch.randn(T, W, generator=g)), rounded(torch.randn(2 * I, W, generator=g) * W ** -0.5)
+        y = x @ w.T
+        parts = linear_partial(x.bfloat16().cuda(), w.bfloat16().cuda())
+        assert (parts.shape[0] > 1) == (T < 512)
+        close(R.partial_act(parts, "silu", gated=True), y[:, :I] * O.sigmoid(y[:, :I]) * y[:, I:], torch.bfloat16)
+        close(R.partial_act(parts, "relu2"), torch.relu(y) ** 2, torch.bfloat16)
+        z = linear_partial(x.bfloat16().cuda(), w.bfloat16().cuda(), f32=True, max_splits=12)
+        close(z.sum(0), y, torch.float32, f32=1e-5)
+    finish("cuda")
+
+
 def test_angles_keep_their_remainder():
     """Far positions: the two-float frequency gives the double-precision angle where one float is off."""
     f = torch.tensor(rotary_frequencies(64, 1e6), dtype=torch.float64)
