@@ -93,11 +93,13 @@ __device__ __forceinline__ void split_item(int idx, int B, int Hkv, int& c, int&
   g = r - b * Hkv;
 }
 
-template <int D, bool WIN>
+// MODE 0: the plain kernel; 1: windowed; 2: windowed with soft-capped scores and / or a bias table by distance
+template <int D, int MODE>
 __global__ void __launch_bounds__(160, 1)
 fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __grid_constant__ CUtensorMap map_v,
                          const __grid_constant__ CUtensorMap map_q, SplitParams p) {
   using L = SplitSmem<D>;
+  constexpr bool WIN = MODE > 0, TABLE = MODE == 2;
   constexpr int NS = L::kStages;
   constexpr int kDChunks = D / 64;
   constexpr uint32_t kTmemCols = 512;   // S: 2 x 64 columns, O: 2 x 128 columns
@@ -323,8 +325,13 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
                    ? exp2f(-p.bias_exp * (float)(g * rep + row + 1) / (float)p.Hq) * 1.4426950408889634f : 0.f;
       };
       // soft cap and bias table (windowed variant): `raw` product of a head at distance ctx - 1 - col
-      const ScoreCap cap(WIN && p.softcap > 0.f ? p.softcap : 1.f, p.scale);
-      auto score_of = [&](float raw) { return WIN && p.softcap > 0.f ? cap(raw) : raw * p.scale_log2; };
+      const ScoreCap cap(TABLE && p.softcap > 0.f ? p.softcap : 1.f, p.scale);
+      auto score_of = [&](float raw) {
+        if constexpr (TABLE) {
+          if (p.softcap > 0.f) return cap(raw);
+        }
+        return raw * p.scale_log2;
+      };
       auto rel_row = [&](int row) { return p.rel + (size_t)min(g * rep + row, p.Hq - 1) * p.rel_n; };
       auto rel_at = [&](const float* rel, int col) {
         return __ldg(rel + min(max(ctx - 1 - col, 0), p.rel_n - 1)) * 1.4426950408889634f;
@@ -339,12 +346,12 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
         const int frow = lane >> 2, fq = lane & 3;
         const bool fvalid = frow < rep;
         const float slope = slope_of(frow);
-        const float* rel = WIN && p.rel ? rel_row(frow) : nullptr;
+        const float* rel = TABLE && p.rel ? rel_row(frow) : nullptr;
         for (int t = 0; t < n; ++t) {
           const uint32_t tn = tile_no + t;
           const int sb_ = tn & 1;
           float rb[16] = {};
-          if (WIN && rel) {      // in flight while the scores are computed
+          if (TABLE && rel) {      // in flight while the scores are computed
             const int col = first_pos(t) + 2 * fq;
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
@@ -376,8 +383,8 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
               const float dist = (float)(kv0 + 8 * i + 2 * fq - (ctx - 1));
-              sv[2 * i] = fmaf(slope, dist, sv[2 * i]) + rb[2 * i];
-              sv[2 * i + 1] = fmaf(slope, dist + 1.f, sv[2 * i + 1]) + rb[2 * i + 1];
+              sv[2 * i] = TABLE ? sv[2 * i] + rb[2 * i] : fmaf(slope, dist, sv[2 * i]);
+              sv[2 * i + 1] = TABLE ? sv[2 * i + 1] + rb[2 * i + 1] : fmaf(slope, dist + 1.f, sv[2 * i + 1]);
             }
           }
           if (need_mask(kv0)) {
@@ -450,7 +457,7 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
         m_ref = __shfl_sync(0xffffffffu, m_ref, (lane * 4) & 31);
       } else {
         const float slope = slope_of(lane);
-        const float* rel = WIN && p.rel ? rel_row(lane) : nullptr;
+        const float* rel = TABLE && p.rel ? rel_row(lane) : nullptr;
         for (int t = 0; t < n; ++t) {
           const uint32_t tn = tile_no + t;
           const int sb_ = tn & 1;
@@ -477,8 +484,9 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
           const int kv0 = first_pos(t);
           if constexpr (WIN) {
   #pragma unroll
-            for (int i = 0; i < kSBlk; ++i) sv[i] = fmaf(slope, (float)(kv0 + i - (ctx - 1)), sv[i]);
-            if (rel) {
+            for (int i = 0; i < kSBlk; ++i)
+              if (!TABLE) sv[i] = fmaf(slope, (float)(kv0 + i - (ctx - 1)), sv[i]);
+            if (TABLE && rel) {
   #pragma unroll
               for (int i = 0; i < kSBlk; ++i) sv[i] += rel_at(rel, kv0 + i);
             }
@@ -673,11 +681,11 @@ __global__ void fmha_decode_merge_kernel(SplitParams p) {
   orow[d] = __float2bfloat16(wsum > 0.f ? acc / wsum * f : 0.f);
 }
 
-template <int D, bool WIN>
+template <int D, int MODE>
 static int launch_decode_split(const CUtensorMap& mc, const CUtensorMap& mv, const CUtensorMap& mq, const SplitParams& p,
                                cudaStream_t stream) {
   using L = SplitSmem<D>;
-  auto kernel = fmha_decode_split_kernel<D, WIN>;
+  auto kernel = fmha_decode_split_kernel<D, MODE>;
   static bool configured = false;
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, L::kTotal);
@@ -689,7 +697,7 @@ static int launch_decode_split(const CUtensorMap& mc, const CUtensorMap& mv, con
   kernel<<<grid, 160, L::kTotal, stream>>>(mc, mv, mq, p);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return (int)e;
-  fmha_decode_merge_kernel<D, WIN><<<dim3(p.B, p.Hq), D, 0, stream>>>(p);
+  fmha_decode_merge_kernel<D, (MODE > 0)><<<dim3(p.B, p.Hq), D, 0, stream>>>(p);
   return (int)cudaGetLastError();
 }
 
@@ -729,8 +737,8 @@ extern "C" int sb_fmha_decode_split(const void* q, int row_stride, const void* c
   p.scale_log2 = scale * 1.4426950408889634f; p.status = status;
   p.window = 0; p.keep_first = 0; p.dv = D; p.out_stride = 0; p.bias_exp = 0.f; p.out_scale = 1.f;
   p.softcap = 0.f; p.scale = scale; p.sink = 0; p.rel_n = 0; p.rel = nullptr; p.head_gate = nullptr;
-  return D == 128 ? launch_decode_split<128, false>(mc, mc, mq, p, stream)
-                  : launch_decode_split<64, false>(mc, mc, mq, p, stream);
+  return D == 128 ? launch_decode_split<128, 0>(mc, mc, mq, p, stream)
+                  : launch_decode_split<64, 0>(mc, mc, mq, p, stream);
 }
 
 // Chunks of the workspace of sb_attn_window_decode (ws_o = B * Hq * chunks * D floats with D = 64 or 128, the smallest
@@ -739,7 +747,7 @@ extern "C" int sb_attn_window_decode_chunks(const void* params) {
   const WinParams& p = *reinterpret_cast<const WinParams*>(params);
   if (p.dk % 8 || p.dv % 8 || p.dk > 128 || p.dv > 128 || p.Hq % p.Hkv || p.Hq / p.Hkv > 32 || p.row_stride % 8 ||
       p.q_off % 8 || p.out_stride % 8 || p.out_off % 8 || p.block_elems % 8 || p.kv_mode != kPaged || p.gain || p.gate ||
-      (p.rel && p.rel_n < 1))
+      (p.rel && (p.rel_n < 1 || p.bias_exp > 0.f)))
     return -1;
   int tiles = p.max_blocks;
   if (p.window > 0) {
@@ -782,6 +790,8 @@ extern "C" int sb_attn_window_decode(const void* params, const int* seq_lens, fl
   p.bias_exp = w.bias_exp; p.out_scale = w.out_scale;
   p.softcap = w.softcap; p.scale = w.scale; p.sink = w.sink; p.rel_n = (int)w.rel_n; p.rel = w.rel;
   p.head_gate = w.head_gate;
-  return w.dk > 64 || w.dv > 64 ? launch_decode_split<128, true>(mk, mv, mq, p, stream)
-                                : launch_decode_split<64, true>(mk, mv, mq, p, stream);
+  const bool wide = w.dk > 64 || w.dv > 64;
+  if (w.softcap > 0.f || w.rel)
+    return wide ? launch_decode_split<128, 2>(mk, mv, mq, p, stream) : launch_decode_split<64, 2>(mk, mv, mq, p, stream);
+  return wide ? launch_decode_split<128, 1>(mk, mv, mq, p, stream) : launch_decode_split<64, 1>(mk, mv, mq, p, stream);
 }
