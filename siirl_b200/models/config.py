@@ -721,8 +721,8 @@ class DecoderConfig:
             b = MixerBranch(kind="attention", heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]),
                             vdim=int(m["vdim"]), scale=float(m["scale"]), bias_exp=0.0, **kinds[x["type"]])
             if x["type"] == "attention_2":
-                b.softcap, b.rel_max = float(m["softcap"]), int(m["bias_max"])
-                b.window = int(m["mask"]["size"])
+                b.softcap, b.rel_max = float(m.get("softcap") or 0.0), int(m["bias_max"])
+                b.window = int((m.get("mask") or {}).get("size") or 0)
             else:
                 rot = m["rot"]
                 b.rot_dims, b.rot_base = int(rot["dims"]), float(rot["base"])
