@@ -26,7 +26,7 @@ LIB_PATH = LIB_DIR / "libsiirl_b200.so"
 SERVE_LIB_PATH = LIB_DIR / "libsiirl_b200_serve.so"
 SERVE_SOURCES = ("gemm_tcgen05.cu", "hybrid_ops.cu", "fmha_window.cu", "fmha_decode_split.cu", "fmha_decode.cu",
                  "recurrence.cu", "head_product.cu", "latent_decode.cu", "decode_state.cu", "sampling.cu", "lm_head.cu",
-                 "qkv_prepare.cu", "hyper_rows.cu", "moe.cu")
+                 "qkv_prepare.cu", "hyper_rows.cu", "moe.cu", "delta_rule.cu", "post_norm_rows.cu")
 # debug-bounds variant (-DSB_DEBUG_BOUNDS: data-dependent indices report their first violation, see csrc/common.cuh)
 DBG_OBJ_DIR = PKG_DIR / "build_dbg"
 DBG_LIB_PATH = LIB_DIR / "libsiirl_b200_dbg.so"

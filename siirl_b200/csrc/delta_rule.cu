@@ -1,0 +1,848 @@
+// Generalized delta rule with a matrix state, for prefill and for decode (arguments and state layout of recurrence.cuh):
+//
+//   S_t = diag(w_t) S_(t-1) - b_t (u_t^T S_(t-1)) + k_t v_t^T          o_t = S_t^T r_t
+//
+// per sequence and head, state in 32-bit floats, with the unit key u = k / sqrt(|k|^2 + 1e-6), b = sigmoid(a + bias) * u, the
+// decay w = exp(-e^(-1/2) sigmoid(W2 tanh(low-rank row) + bias)) per key channel; then an RMS norm of every head, a weight
+// per channel and an output gate.  State: S [slots, heads, dv, dk], value-major; a portion whose first position is 0 starts from
+// zero and does not read its slot.
+//
+// A chunk of 16 tokens.  With the decay G_t from the chunk's start through token t, r~ = G_t r_t, u~ = G_(t-1) u_t,
+// k~ = k_t / G_t, b~ = b_t / G_t and p_t = u_t^T S_(t-1):
+//
+//   p_t = u~_t S_0 + sum_(s<t) (u~_t . k~_s) v_s - (u~_t . b~_s) p_s
+//   o_t = r~_t S_0 + sum_(s<=t) (r~_t . k~_s) v_s - (r~_t . b~_s) p_s
+//   S_16 = G (S_0 + sum_s k~_s v_s^T - b~_s p_s^T)
+//
+// The first line is a unit lower triangular system in p.  Solving it for the parts that multiply S_0 and v gives tiles that do
+// not depend on the state, U = (I + ub)^-1 u~ and M = (I + ub)^-1 uk, and with them Q = r~ - rb U, A = rk - rb M,
+// K = G (k~ - M^T b~), B = G b~:
+//
+//   o = Q S_0 + A v        p' = U S_0        S_16 = G S_0 + K^T v - B^T p'
+//
+// 1 / G_t is at most 2^14 inside a chunk (w > 0.54); the tiles are formed relative to the chunk's middle.
+//
+// Kernels:
+//   delta_step_regs_kernel   one CTA per (sequence, head), the state in registers, token by token: decode, 32-bit prompts
+//   delta_step_kernel        the same for any sizes, state in shared or global memory
+//   delta_prepare_kernel     prefill: the tiles of a chunk, in parallel over chunks and heads
+//   delta_scan_kernel        prefill: walks the chunks of a (sequence, head) with the state in registers as tensor-core
+//                            fragments; tiles arrive through a ring of asynchronous copies
+// Tensor-core operands that stand for 32-bit quantities are split into two bf16 terms (16 mantissa bits), v is bf16 as projected;
+// accumulation is fp32.
+#include "recurrence.cuh"
+
+namespace sb {
+
+constexpr float kDecayRate = 0.6065306597126334f;      // e^(-1/2)
+
+// decays, unit keys and removal rates of one token of head h, for all threads of a CTA of kStepThreads: sq (r), sk, su, sb, sd [dk].
+// `se` holds rank values, `red` eight.  Ends with a barrier.
+template <typename T>
+__device__ __forceinline__ void delta_token(const RecParams& p, const T* xr, int h, float* sq, float* sk, float* su, float* sb_,
+                                            float* sd, float* se, float* red) {
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  for (int r = tid; r < p.rank; r += kStepThreads) se[r] = tanhf(to_float(xr[p.e_off + r]));
+  float ss = 0.f;
+  for (int d = tid; d < p.dk; d += kStepThreads) {
+    const float k = to_float(xr[p.k_off + h * p.dk + d]);
+    sk[d] = k;
+    sq[d] = to_float(xr[p.q_off + h * p.dk + d]);
+    ss = fmaf(k, k, ss);
+  }
+  ss = warp_sum(ss);
+  if (lane == 0) red[warp] = ss;
+  __syncthreads();
+  float tot = 0.f;
+#pragma unroll
+  for (int i = 0; i < kStepThreads / 32; ++i) tot += red[i];
+  const float inv = 1.f / sqrtf(tot + 1e-6f);
+  const bool vec = sizeof(T) == 2 && p.rank % 8 == 0 && ((uintptr_t)p.w2 & 15) == 0;
+  const int part = tid & 3;      // four lanes share a channel's product with the low-rank row
+  for (int i = tid; i < (p.dk * 4 + 31) / 32 * 32; i += kStepThreads) {
+    const int d = i >> 2;
+    float z = 0.f;
+    if (d < p.dk) {
+      const T* w = reinterpret_cast<const T*>(p.w2) + (size_t)(h * p.dk + d) * p.rank;
+      if constexpr (sizeof(T) == 2) {
+        if (vec) {
+          for (int r = part * 8; r < p.rank; r += 32) {
+            float x[8];
+            load_vec<T, 8>(w + r, x);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) z = fmaf(x[j], se[r + j], z);
+          }
+        }
+      }
+      if (!vec)
+        for (int r = part; r < p.rank; r += 4) z = fmaf(to_float(w[r]), se[r], z);
+    }
+    z += __shfl_xor_sync(0xffffffffu, z, 1);
+    z += __shfl_xor_sync(0xffffffffu, z, 2);
+    if (d < p.dk && part == 0) {
+      z += to_float(reinterpret_cast<const T*>(p.b_e)[h * p.dk + d]);
+      const float a = to_float(xr[p.f_off + h * p.dk + d]) + to_float(reinterpret_cast<const T*>(p.b_f)[h * p.dk + d]);
+      sd[d] = expf(-kDecayRate / (1.f + expf(-z)));
+      const float u = sk[d] * inv;
+      su[d] = u;
+      sb_[d] = u / (1.f + expf(-a));
+    }
+  }
+  __syncthreads();
+}
+
+// norm, weight and gate of one token's head `so` [dv]; begins with a barrier (so is complete), red: eight values
+template <typename T>
+__device__ __forceinline__ void delta_finish(const RecParams& p, const T* xr, T* out, int h, const float* so, float* red) {
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  __syncthreads();
+  float ss = 0.f;
+  for (int i = tid; i < p.dv; i += kStepThreads) ss = fmaf(so[i], so[i], ss);
+  ss = warp_sum(ss);
+  if (lane == 0) red[warp] = ss;
+  __syncthreads();
+  float tot = 0.f;
+#pragma unroll
+  for (int i = 0; i < kStepThreads / 32; ++i) tot += red[i];
+  const float rstd = 1.f / sqrtf(tot / (float)p.dv + p.eps);
+  for (int i = tid; i < p.dv; i += kStepThreads) {
+    const float w = to_float(reinterpret_cast<const T*>(p.norm_w)[p.norm_per_head ? h * p.dv + i : i]);
+    const float g = gate_value(to_float(xr[p.g_off + h * p.dv + i]), p.gate_act);
+    out[i] = from_float<T>(so[i] * rstd * w * g * p.out_scale);
+  }
+}
+
+// rows of shared memory of the step kernels: five vectors of dk, so [dv], se [rank], two reductions
+__host__ __device__ inline int delta_step_floats(int dk, int dv, int rank) {
+  return 5 * ((dk + 3) & ~3) + ((dv + 3) & ~3) + ((rank + 3) & ~3) + 16;
+}
+
+// dk = dv <= 32 N, a multiple of four.  Eight lanes hold a state row (a value column's key channels), four rows per warp and pass.
+template <typename T, int N>
+__global__ void __launch_bounds__(kStepThreads)
+delta_step_regs_kernel(RecParams p, const int* __restrict__ row0, const int* __restrict__ nrow,
+                       const int* __restrict__ slots, const int* __restrict__ pos0) {
+  extern __shared__ __align__(16) float sm[];
+  const int dkp = (p.dk + 3) & ~3;
+  float *sq = sm, *sk = sq + dkp, *su = sk + dkp, *sb_ = su + dkp, *sd = sb_ + dkp, *so = sd + dkp;
+  float *se = so + ((p.dv + 3) & ~3), *red = se + ((p.rank + 3) & ~3);
+  const int h = blockIdx.x, s = blockIdx.y, tid = threadIdx.x;
+  const int r0 = row0 ? row0[s] : s, n = nrow ? nrow[s] : 1, slot = slots[s];
+  T* out = reinterpret_cast<T*>(p.out) + p.out_off + (size_t)h * p.dv;
+  if (slot < 0) {
+    for (int t = 0; t < n; ++t)
+      for (int i = tid; i < p.dv; i += kStepThreads) out[(size_t)(r0 + t) * p.out_stride + i] = from_float<T>(0.f);
+    return;
+  }
+  if (n <= 0) return;
+  const bool fresh = pos0[s] == 0;
+  float* gs = p.S + ((size_t)slot * p.H + h) * p.dv * p.dk;
+  const int warp = tid >> 5, lane = tid & 31, row = warp * 4 + (lane >> 3), d0 = (lane & 7) * 4;
+  float st[N][N][4];      // [row row + 32 i][channels d0 + 32 c ..]
+#pragma unroll
+  for (int i = 0; i < N; ++i)
+#pragma unroll
+    for (int c = 0; c < N; ++c) {
+#pragma unroll
+      for (int j = 0; j < 4; ++j) st[i][c][j] = 0.f;
+      if (!fresh && row + 32 * i < p.dv && d0 + 32 * c < p.dk)
+        load_vec<float, 4>(gs + (size_t)(row + 32 * i) * p.dk + d0 + 32 * c, st[i][c]);
+    }
+  for (int t = 0; t < n; ++t) {
+    const T* xr = reinterpret_cast<const T*>(p.x) + (size_t)(r0 + t) * p.row_stride;
+    delta_token<T>(p, xr, h, sq, sk, su, sb_, sd, se, red);
+    float seen[N];
+#pragma unroll
+    for (int i = 0; i < N; ++i) seen[i] = 0.f;
+#pragma unroll
+    for (int c = 0; c < N; ++c) {
+      if (d0 + 32 * c >= p.dk) break;
+      float u[4];
+      load_vec<float, 4>(su + d0 + 32 * c, u);
+#pragma unroll
+      for (int i = 0; i < N; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) seen[i] = fmaf(u[j], st[i][c][j], seen[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      seen[i] += __shfl_xor_sync(0xffffffffu, seen[i], 4);
+      seen[i] += __shfl_xor_sync(0xffffffffu, seen[i], 2);
+      seen[i] += __shfl_xor_sync(0xffffffffu, seen[i], 1);
+    }
+    float v[N], o[N];
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      v[i] = row + 32 * i < p.dv ? to_float(xr[p.v_off + h * p.dv + row + 32 * i]) : 0.f;
+      o[i] = 0.f;
+    }
+#pragma unroll
+    for (int c = 0; c < N; ++c) {
+      if (d0 + 32 * c >= p.dk) break;
+      float w[4], b[4], k[4], q[4];
+      load_vec<float, 4>(sd + d0 + 32 * c, w);
+      load_vec<float, 4>(sb_ + d0 + 32 * c, b);
+      load_vec<float, 4>(sk + d0 + 32 * c, k);
+      load_vec<float, 4>(sq + d0 + 32 * c, q);
+#pragma unroll
+      for (int i = 0; i < N; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const float x = fmaf(st[i][c][j], w[j], fmaf(k[j], v[i], -b[j] * seen[i]));
+          st[i][c][j] = x;
+          o[i] = fmaf(x, q[j], o[i]);
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      o[i] += __shfl_xor_sync(0xffffffffu, o[i], 4);
+      o[i] += __shfl_xor_sync(0xffffffffu, o[i], 2);
+      o[i] += __shfl_xor_sync(0xffffffffu, o[i], 1);
+      if ((lane & 7) == 0 && row + 32 * i < p.dv) so[row + 32 * i] = o[i] * p.q_scale;
+    }
+    delta_finish<T>(p, xr, out + (size_t)(r0 + t) * p.out_stride, h, so, red + 8);
+  }
+#pragma unroll
+  for (int i = 0; i < N; ++i)
+#pragma unroll
+    for (int c = 0; c < N; ++c)
+      if (row + 32 * i < p.dv && d0 + 32 * c < p.dk)
+        store_vec<float, 4>(gs + (size_t)(row + 32 * i) * p.dk + d0 + 32 * c, st[i][c]);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kStepThreads)
+delta_step_kernel(RecParams p, const int* __restrict__ row0, const int* __restrict__ nrow, const int* __restrict__ slots,
+                  const int* __restrict__ pos0, int smem_state) {
+  extern __shared__ __align__(16) float sm[];
+  const int dkp = (p.dk + 3) & ~3;
+  float *sq = sm, *sk = sq + dkp, *su = sk + dkp, *sb_ = su + dkp, *sd = sb_ + dkp, *so = sd + dkp;
+  float *se = so + ((p.dv + 3) & ~3), *red = se + ((p.rank + 3) & ~3);
+  const int h = blockIdx.x, s = blockIdx.y, tid = threadIdx.x;
+  const int r0 = row0 ? row0[s] : s, n = nrow ? nrow[s] : 1, slot = slots[s];
+  T* out = reinterpret_cast<T*>(p.out) + p.out_off + (size_t)h * p.dv;
+  if (slot < 0) {
+    for (int t = 0; t < n; ++t)
+      for (int i = tid; i < p.dv; i += kStepThreads) out[(size_t)(r0 + t) * p.out_stride + i] = from_float<T>(0.f);
+    return;
+  }
+  if (n <= 0) return;
+  const bool fresh = pos0[s] == 0;
+  float* gs = p.S + ((size_t)slot * p.H + h) * p.dv * p.dk;
+  float* st = smem_state ? red + 16 : gs;
+  if (smem_state || fresh)
+    for (int i = tid; i < p.dv * p.dk; i += kStepThreads) st[i] = fresh ? 0.f : gs[i];
+  const int warp = tid >> 5, lane = tid & 31, grp = lane >> 3, l8 = lane & 7;
+  for (int t = 0; t < n; ++t) {
+    const T* xr = reinterpret_cast<const T*>(p.x) + (size_t)(r0 + t) * p.row_stride;
+    delta_token<T>(p, xr, h, sq, sk, su, sb_, sd, se, red);
+    for (int rb = warp * 4; rb < p.dv; rb += kStepThreads / 8) {
+      const int r = rb + grp;
+      float* sr = st + (size_t)(r < p.dv ? r : 0) * p.dk;
+      float seen = 0.f, o = 0.f;
+      if (r < p.dv)
+        for (int d = l8; d < p.dk; d += 8) seen = fmaf(su[d], sr[d], seen);
+      for (int w = 4; w; w >>= 1) seen += __shfl_xor_sync(0xffffffffu, seen, w);
+      if (r < p.dv) {
+        const float v = to_float(xr[p.v_off + h * p.dv + r]);
+        for (int d = l8; d < p.dk; d += 8) {
+          const float x = fmaf(sr[d], sd[d], fmaf(sk[d], v, -sb_[d] * seen));
+          sr[d] = x;
+          o = fmaf(x, sq[d], o);
+        }
+      }
+      for (int w = 4; w; w >>= 1) o += __shfl_xor_sync(0xffffffffu, o, w);
+      if (l8 == 0 && r < p.dv) so[r] = o * p.q_scale;
+    }
+    delta_finish<T>(p, xr, out + (size_t)(r0 + t) * p.out_stride, h, so, red + 8);
+  }
+  if (smem_state) {
+    __syncthreads();
+    for (int i = tid; i < p.dv * p.dk; i += kStepThreads) gs[i] = st[i];
+  }
+}
+
+// ---------------------------------------------------------------------------------------
+// chunk tiles: Q, U, K, B [16][dkp + 8], each as hi and lo, then A hi, lo [16][24], then the chunk's decay [dkp] fp32
+// ---------------------------------------------------------------------------------------
+__host__ __device__ inline int delta_tile_bytes(int dkp) {
+  return 8 * kChunk * tile_row(dkp) * 2 + 2 * kChunk * kARow * 2 + dkp * 4;
+}
+
+constexpr int kDeltaThreads = 128;
+
+struct DeltaPrepSmem {      // byte offsets
+  int cum, mats, ehi, elo, inv, total;
+  __host__ __device__ DeltaPrepSmem(int dkp, int rankp) {
+    cum = delta_tile_bytes(dkp);                         // [16][dkp + 1] running log2 decay
+    mats = (cum + kChunk * (dkp + 1) * 4 + 15) / 16 * 16;      // rk, rb, uk, ub, M [16][16] fp32
+    ehi = mats + 5 * kChunk * kChunk * 4;                // tanh of the low-rank rows [16][rankp + 8]
+    elo = ehi + kChunk * (rankp + 8) * 2;
+    inv = elo + kChunk * (rankp + 8) * 2;                // [16] 1 / |k|
+    total = inv + kChunk * 4;
+  }
+};
+
+// 16 log2 of the decay is fetched from here by everything that follows: -e^(-1/2) log2(e) sigmoid(z)
+__device__ __forceinline__ float delta_log2_decay(float z) { return __fdividef(-kDecayRate * kLog2e, 1.f + __expf(-z)); }
+
+template <int NK>
+__global__ void __launch_bounds__(kDeltaThreads)
+delta_prepare_kernel(RecParams p, const int* __restrict__ chunk_row, const int* __restrict__ chunk_len,
+                     uint8_t* __restrict__ tiles) {
+  using B16 = __nv_bfloat16;
+  constexpr int dkp = NK * 16, rs = dkp + 8, ld = dkp + 1;
+  const int rankp = (p.rank + 15) / 16 * 16;
+  const DeltaPrepSmem L(dkp, rankp);
+  extern __shared__ __align__(16) uint8_t smem[];
+  B16* t_q = reinterpret_cast<B16*>(smem);      // every tile: hi, then lo `part` elements later
+  constexpr int part = kChunk * rs;
+  B16 *t_u = t_q + 2 * part, *t_k = t_q + 4 * part, *t_b = t_q + 6 * part, *t_a = t_q + 8 * part;
+  float* t_d = reinterpret_cast<float*>(t_a + 2 * kChunk * kARow);
+  float* cum = reinterpret_cast<float*>(smem + L.cum);
+  float* mats = reinterpret_cast<float*>(smem + L.mats);
+  float *m_rk = mats, *m_rb = mats + 256, *m_uk = mats + 512, *m_ub = mats + 768, *m_m = mats + 1024;
+  B16 *ehi = reinterpret_cast<B16*>(smem + L.ehi), *elo = reinterpret_cast<B16*>(smem + L.elo);
+  float* s_inv = reinterpret_cast<float*>(smem + L.inv);
+  const int h = blockIdx.x, c = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int row = chunk_row[c], len = chunk_len[c];
+  const B16* x = reinterpret_cast<const B16*>(p.x) + (size_t)row * p.row_stride;
+  const B16* w2 = reinterpret_cast<const B16*>(p.w2) + (size_t)h * p.dk * p.rank;
+  const B16* w0 = reinterpret_cast<const B16*>(p.b_e) + h * p.dk;
+  const B16* ab = reinterpret_cast<const B16*>(p.b_f) + h * p.dk;
+
+  // low-rank rows, two terms each; lengths of the keys
+  for (int i = tid; i < kChunk * rankp; i += kDeltaThreads) {
+    const int t = i / rankp, r = i - t * rankp;
+    const float e = t < len && r < p.rank ? tanhf(to_float(x[(size_t)t * p.row_stride + p.e_off + r])) : 0.f;
+    const B16 hi = __float2bfloat16(e);
+    ehi[t * (rankp + 8) + r] = hi;
+    elo[t * (rankp + 8) + r] = __float2bfloat16(e - __bfloat162float(hi));
+  }
+  {
+    const int t = tid >> 3;
+    float ss = 0.f;
+    if (t < len) {
+      const B16* k = x + (size_t)t * p.row_stride + p.k_off + h * p.dk;
+      for (int d = (tid & 7) * 8; d < p.dk; d += 64) {
+        float v[8];
+        load_vec<B16, 8>(k + d, v);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) ss = fmaf(v[j], v[j], ss);
+      }
+    }
+    ss += __shfl_xor_sync(0xffffffffu, ss, 4);
+    ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+    ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+    if ((tid & 7) == 0) s_inv[t] = 1.f / sqrtf(ss + 1e-6f);
+  }
+  __syncthreads();
+  // log2 decays: rows t = g, g + 8, channels 8 j + 2 (lane % 4) + {0, 1} of a warp's column groups
+  const int g = lane >> 2, q2 = (lane & 3) * 2;
+  const int nrm_row = (lane & 7) + ((lane >> 4) << 3), nrm_col = ((lane >> 3) & 1) * 8;
+  const int trn_row = (lane & 7) + (((lane >> 3) & 1) << 3), trn_col = (lane >> 4) * 8;
+  const bool pairs = p.rank % 2 == 0 && ((uintptr_t)w2 & 3) == 0;
+  for (int j = warp; j < dkp / 8; j += kDeltaThreads / 32) {
+    float z[4] = {};
+    const int ch = 8 * j + g;      // the channel whose weights this lane brings
+    for (int k0 = 0; k0 < rankp; k0 += 16) {
+      uint32_t a[4], b[2] = {0, 0};
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int r = k0 + q2 + 8 * half;
+        if (ch < p.dk && r < p.rank) {
+          const B16* w = w2 + (size_t)ch * p.rank + r;
+          if (pairs) b[half] = *reinterpret_cast<const uint32_t*>(w);
+          else b[half] = pack_bf16x2(to_float(w[0]), r + 1 < p.rank ? to_float(w[1]) : 0.f);
+        }
+      }
+      const uint32_t off = (uint32_t)(trn_row * (rankp + 8) + k0 + trn_col) * 2;
+      ldsm_x4(a, smem_u32(ehi) + off);
+      mma_16816(z, a, b[0], b[1]);
+      ldsm_x4(a, smem_u32(elo) + off);
+      mma_16816(z, a, b[0], b[1]);
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int t = g + (i >> 1) * 8, d = 8 * j + q2 + (i & 1);
+      cum[t * ld + d] = t < len && d < p.dk ? delta_log2_decay(z[i] + to_float(w0[d])) : 0.f;
+    }
+  }
+  __syncthreads();
+  for (int d = tid; d < dkp; d += kDeltaThreads) {
+    float acc = 0.f;
+#pragma unroll
+    for (int t = 0; t < kChunk; ++t) {
+      acc += cum[t * ld + d];
+      cum[t * ld + d] = acc;
+    }
+    t_d[d] = ex2(acc);
+  }
+  __syncthreads();
+  // r~, u~, k~, b~ relative to the decay through token 7
+  for (int i = tid; i < kChunk * (dkp / 8); i += kDeltaThreads) {
+    const int t = i / (dkp / 8), d = i % (dkp / 8) * 8;
+    float r[8] = {}, k[8] = {}, a[8] = {}, bias[8] = {};
+    if (t < len && d < p.dk) {
+      const B16* xr = x + (size_t)t * p.row_stride + h * p.dk + d;
+      load_vec<B16, 8>(xr + p.q_off, r);
+      load_vec<B16, 8>(xr + p.k_off, k);
+      load_vec<B16, 8>(xr + p.f_off, a);
+      load_vec<B16, 8>(ab + d, bias);
+    }
+    const float inv = s_inv[t];
+    uint32_t out[8][4];
+#pragma unroll
+    for (int j = 0; j < 8; j += 2) {
+      float v[4][2];
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const float mid = cum[7 * ld + d + j + e], now = cum[t * ld + d + j + e];
+        const float before = t ? cum[(t - 1) * ld + d + j + e] : 0.f;
+        const float up = ex2(mid - now), u = k[j + e] * inv;
+        v[0][e] = r[j + e] * p.q_scale * ex2(now - mid);
+        v[1][e] = u * ex2(before - mid);
+        v[2][e] = k[j + e] * up;
+        v[3][e] = u * up * __fdividef(1.f, 1.f + __expf(-(a[j + e] + bias[j + e])));
+      }
+#pragma unroll
+      for (int m = 0; m < 4; ++m) split_pair(v[m][0], v[m][1], out[2 * m][j / 2], out[2 * m + 1][j / 2]);
+    }
+#pragma unroll
+    for (int m = 0; m < 8; ++m)
+      *reinterpret_cast<uint4*>(t_q + m * part + t * rs + d) = make_uint4(out[m][0], out[m][1], out[m][2], out[m][3]);
+  }
+  __syncthreads();
+  // the four 16 x 16 products: warp w takes r~ or u~ (w / 2) with k~ or b~ (w % 2)
+  {
+    const B16 *X = warp >> 1 ? t_u : t_q, *Y = warp & 1 ? t_b : t_k;
+    float pr[2][4] = {};
+#pragma unroll
+    for (int kk = 0; kk < NK; ++kk) {
+      uint32_t xh[4], xl[4], yh[4], yl[4];
+      const uint32_t ax = smem_u32(X) + (uint32_t)(trn_row * rs + kk * 16 + trn_col) * 2;
+      const uint32_t ay = smem_u32(Y) + (uint32_t)(nrm_row * rs + kk * 16 + nrm_col) * 2;
+      ldsm_x4(xh, ax);
+      ldsm_x4(xl, ax + part * 2);
+      ldsm_x4(yh, ay);
+      ldsm_x4(yl, ay + part * 2);
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt) {
+        mma_16816(pr[nt], xh, yh[2 * nt], yh[2 * nt + 1]);
+        mma_16816(pr[nt], xh, yl[2 * nt], yl[2 * nt + 1]);
+        mma_16816(pr[nt], xl, yh[2 * nt], yh[2 * nt + 1]);
+      }
+    }
+    float* m = mats + warp * 256;
+#pragma unroll
+    for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int t = g + (i >> 1) * 8, s = nt * 8 + q2 + (i & 1);
+        m[t * kChunk + s] = s < t + (warp >> 1 ? 0 : 1) ? pr[nt][i] : 0.f;
+      }
+  }
+  __syncthreads();
+  // the triangular system, one right-hand side per thread: channels of u~, then columns of uk
+  for (int i = tid; i < dkp + kChunk; i += kDeltaThreads) {
+    const bool channel = i < dkp;
+    const int col = channel ? i : i - dkp;
+    float sol[kChunk];
+#pragma unroll
+    for (int t = 0; t < kChunk; ++t) {
+      float v = channel ? to_float(t_u[t * rs + col]) + to_float(t_u[part + t * rs + col]) : m_uk[t * kChunk + col];
+#pragma unroll
+      for (int s4 = 0; s4 < t; s4 += 4) {
+        const float4 l = *reinterpret_cast<const float4*>(m_ub + t * kChunk + s4);
+        v = fmaf(-l.x, sol[s4], v);
+        if (s4 + 1 < t) v = fmaf(-l.y, sol[s4 + 1], v);
+        if (s4 + 2 < t) v = fmaf(-l.z, sol[s4 + 2], v);
+        if (s4 + 3 < t) v = fmaf(-l.w, sol[s4 + 3], v);
+      }
+      sol[t] = v;
+    }
+    const float f = channel ? ex2(cum[7 * ld + col]) : 1.f;      // from the middle back to the chunk's start
+#pragma unroll
+    for (int t = 0; t < kChunk; ++t) {
+      float v = channel ? to_float(t_q[t * rs + col]) + to_float(t_q[part + t * rs + col]) : m_rk[t * kChunk + col];
+#pragma unroll
+      for (int s4 = 0; s4 <= t; s4 += 4) {
+        const float4 l = *reinterpret_cast<const float4*>(m_rb + t * kChunk + s4);
+        v = fmaf(-l.x, sol[s4], v);
+        if (s4 + 1 <= t) v = fmaf(-l.y, sol[s4 + 1], v);
+        if (s4 + 2 <= t) v = fmaf(-l.z, sol[s4 + 2], v);
+        if (s4 + 3 <= t) v = fmaf(-l.w, sol[s4 + 3], v);
+      }
+      if (channel) {
+        const float q = v * f, u = sol[t] * f;
+        const B16 qh = __float2bfloat16(q), uh = __float2bfloat16(u);
+        t_q[t * rs + col] = qh;
+        t_q[part + t * rs + col] = __float2bfloat16(q - __bfloat162float(qh));
+        t_u[t * rs + col] = uh;
+        t_u[part + t * rs + col] = __float2bfloat16(u - __bfloat162float(uh));
+      } else {
+        const B16 vh = __float2bfloat16(v);
+        t_a[t * kARow + col] = vh;
+        t_a[kChunk * kARow + t * kARow + col] = __float2bfloat16(v - __bfloat162float(vh));
+        m_m[t * kChunk + col] = sol[t];
+      }
+    }
+  }
+  __syncthreads();
+  // K = G (k~ - M^T b~) and B = G b~, relative to the chunk's end
+  for (int d = tid; d < dkp; d += kDeltaThreads) {
+    float b[kChunk], k[kChunk];
+#pragma unroll
+    for (int t = 0; t < kChunk; ++t) {
+      b[t] = to_float(t_b[t * rs + d]) + to_float(t_b[part + t * rs + d]);
+      k[t] = to_float(t_k[t * rs + d]) + to_float(t_k[part + t * rs + d]);
+    }
+#pragma unroll
+    for (int t = 1; t < kChunk; ++t)
+#pragma unroll
+      for (int s4 = 0; s4 < t; s4 += 4) {
+        const float4 l = *reinterpret_cast<const float4*>(m_m + t * kChunk + s4);
+        k[s4] = fmaf(-l.x, b[t], k[s4]);
+        if (s4 + 1 < t) k[s4 + 1] = fmaf(-l.y, b[t], k[s4 + 1]);
+        if (s4 + 2 < t) k[s4 + 2] = fmaf(-l.z, b[t], k[s4 + 2]);
+        if (s4 + 3 < t) k[s4 + 3] = fmaf(-l.w, b[t], k[s4 + 3]);
+      }
+    const float f = ex2(cum[15 * ld + d] - cum[7 * ld + d]);
+#pragma unroll
+    for (int t = 0; t < kChunk; ++t) {
+      const float kv = k[t] * f, bv = b[t] * f;
+      const B16 kh = __float2bfloat16(kv), bh = __float2bfloat16(bv);
+      t_k[t * rs + d] = kh;
+      t_k[part + t * rs + d] = __float2bfloat16(kv - __bfloat162float(kh));
+      t_b[t * rs + d] = bh;
+      t_b[part + t * rs + d] = __float2bfloat16(bv - __bfloat162float(bh));
+    }
+  }
+  __syncthreads();
+  uint8_t* tile = tiles + ((size_t)c * p.H + h) * delta_tile_bytes(dkp);
+  for (int i = tid * 16; i < delta_tile_bytes(dkp); i += kDeltaThreads * 16)
+    *reinterpret_cast<uint4*>(tile + i) = *reinterpret_cast<const uint4*>(smem + i);
+}
+
+// ---------------------------------------------------------------------------------------
+// scan
+// ---------------------------------------------------------------------------------------
+constexpr int kDeltaStages = 3;
+
+struct DeltaScanSmem {
+  int tile, v_row, v_off, stage, obuf_off, obuf_row, obuf, norm_off, total;
+  __host__ __device__ DeltaScanSmem(int dkp, int dvp) {
+    tile = delta_tile_bytes(dkp);
+    v_row = dvp + 8;
+    v_off = tile;
+    stage = (v_off + kChunk * v_row * 2 + 127) / 128 * 128;
+    obuf_off = kDeltaStages * stage;
+    obuf_row = dvp + 4;
+    obuf = kChunk * obuf_row;
+    norm_off = obuf_off + 2 * obuf * 4;
+    total = norm_off + dvp * 4;
+  }
+};
+
+// Warp w owns value columns 16 w .. 16 w + 15 and all key channels.  Iteration c multiplies chunk c and finishes (norm, gate,
+// store) chunk c - 1: one block barrier per chunk.
+template <int NK>
+__global__ void __launch_bounds__(NK * 32, NK > 4 ? 1 : 2)
+delta_scan_kernel(RecParams p, const int* __restrict__ row0s, const int* __restrict__ nrow, const int* __restrict__ slots,
+                  const int* __restrict__ pos0, const int* __restrict__ chunk0, const uint8_t* __restrict__ tiles) {
+  constexpr int dkp = NK * 16, rs = dkp + 8, KD = (dkp + 63) / 64, part = kChunk * rs * 2;      // part: bytes of one tile half
+  extern __shared__ __align__(128) uint8_t smem[];
+  const int dvp = (p.dv + 15) / 16 * 16;
+  const DeltaScanSmem L(dkp, dvp);
+  float* obuf = reinterpret_cast<float*>(smem + L.obuf_off);
+  float* nw = reinterpret_cast<float*>(smem + L.norm_off);
+  const int h = blockIdx.x, s = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int n_warps = blockDim.x >> 5;
+  const int slot = slots[s], tokens = nrow[s], n = (tokens + kChunk - 1) / kChunk, row0 = row0s[s];
+  const __nv_bfloat16* x = reinterpret_cast<const __nv_bfloat16*>(p.x) + (size_t)row0 * p.row_stride;
+  __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)row0 * p.out_stride + p.out_off + (size_t)h * p.dv;
+  if (slot < 0) {
+    for (int i = tid; i < tokens * p.dv; i += blockDim.x)
+      out[(size_t)(i / p.dv) * p.out_stride + i % p.dv] = __float2bfloat16(0.f);
+    return;
+  }
+  if (n <= 0) return;
+  const uint8_t* my_tiles = tiles + ((size_t)chunk0[s] * p.H + h) * L.tile;
+  const size_t tile_step = (size_t)p.H * L.tile;
+  for (int st = 0; st < kDeltaStages; ++st) {      // value columns past dv: no copy writes them
+    __nv_bfloat16* v = reinterpret_cast<__nv_bfloat16*>(smem + st * L.stage + L.v_off);
+    const int extra = L.v_row - p.dv;
+    for (int i = tid; i < kChunk * extra; i += blockDim.x) v[i / extra * L.v_row + p.dv + i % extra] = __float2bfloat16(0.f);
+  }
+  const int v_vecs = p.dv / 8;
+  auto issue = [&](int c) {      // copies of chunk c into its stage (an empty group past the end)
+    if (c < n) {
+      uint8_t* st = smem + (c % kDeltaStages) * L.stage;
+      const int len = min(kChunk, tokens - c * kChunk);
+      const uint8_t* src = my_tiles + (size_t)c * tile_step;
+      for (int i = tid * 16; i < L.tile; i += blockDim.x * 16) copy16(st + i, src + i);
+      for (int i = tid; i < kChunk * v_vecs; i += blockDim.x) {
+        const int t = i / v_vecs, e = (i - t * v_vecs) * 8;
+        uint8_t* dst = st + L.v_off + (t * L.v_row + e) * 2;
+        if (t < len) copy16(dst, x + (size_t)(c * kChunk + t) * p.row_stride + p.v_off + h * p.dv + e);
+        else *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
+      }
+    }
+    copy_commit();
+  };
+#pragma unroll
+  for (int i = 0; i < kDeltaStages - 1; ++i) issue(i);
+
+  // state fragments: acc[j] holds key channels 8 j + 2 (lane % 4) + {0, 1} of value columns r and r + 8
+  const int g = lane >> 2, q2 = (lane & 3) * 2, r = warp * 16 + g;
+  float* slot_S = p.S + ((size_t)slot * p.H + h) * p.dv * p.dk;
+  const bool zero = pos0[s] == 0;
+  float acc[2 * NK][4];
+#pragma unroll
+  for (int j = 0; j < 2 * NK; ++j)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int rr = r + (i >> 1) * 8, d = 8 * j + q2 + (i & 1);
+      acc[j][i] = (!zero && rr < p.dv && d < p.dk) ? slot_S[(size_t)rr * p.dk + d] : 0.f;
+    }
+  for (int i = tid; i < p.dv; i += blockDim.x)
+    nw[i] = to_float(reinterpret_cast<const __nv_bfloat16*>(p.norm_w)[(p.norm_per_head ? h * p.dv : 0) + i]);
+  const float inv_dv = 1.f / (float)p.dv;
+  const int nrm_row = (lane & 7) + ((lane >> 4) << 3), nrm_col = ((lane >> 3) & 1) * 8;   // rows 0-7: columns 0-7, 8-15
+  const int trn_row = (lane & 7) + (((lane >> 3) & 1) << 3), trn_col = (lane >> 4) * 8;   // columns 0-7: rows 0-7, 8-15
+
+  for (int c = 0; c <= n; ++c) {
+    if (c < n) copy_wait<kDeltaStages - 2>();
+    __syncthreads();            // chunk c has landed, chunk c - 1 is multiplied, chunk c - 2 is out
+    issue(c + kDeltaStages - 1);
+    // each half warp finishes one token: four values per lane and 64 columns
+    const int et = (c - 1) * kChunk + warp * 2 + (lane >> 4);
+    uint2 gpre[KD];             // output-gate values of chunk c - 1, fetched ahead of their use
+#pragma unroll
+    for (int k = 0; k < KD; ++k) {
+      const int i = (lane & 15) * 4 + k * 64;
+      gpre[k] = make_uint2(0, 0);
+      if (c > 0 && warp * 2 < kChunk && et < tokens && i < p.dv)
+        gpre[k] = *reinterpret_cast<const uint2*>(x + (size_t)et * p.row_stride + p.g_off + h * p.dv + i);
+    }
+    if (c < n) {
+      const uint8_t* st = smem + (c % kDeltaStages) * L.stage;
+      const uint32_t a_q = smem_u32(st), a_u = a_q + 2 * part, a_k = a_q + 4 * part, a_b = a_q + 6 * part, a_a = a_q + 8 * part;
+      const float* D = reinterpret_cast<const float*>(st + 8 * part + 2 * kChunk * kARow * 2);
+      float* ob = obuf + (c & 1) * L.obuf;
+      uint32_t va[4];             // v^T: value columns x tokens
+      ldsm_x4_t(va, smem_u32(st + L.v_off) + (uint32_t)(nrm_row * L.v_row + warp * 16 + nrm_col) * 2);
+      float p0[2][4] = {}, p1[2][4] = {}, p2[2][4] = {}, o0[2][4] = {}, o1[2][4] = {}, o2[2][4] = {};
+#pragma unroll
+      for (int kk = 0; kk < NK; ++kk) {
+        uint32_t hi[4], lo[4], uh[4], ul[4], qh[4], ql[4];
+        const uint32_t off = (uint32_t)(nrm_row * rs + kk * 16 + nrm_col) * 2;
+        ldsm_x4(uh, a_u + off);
+        ldsm_x4(ul, a_u + part + off);
+        ldsm_x4(qh, a_q + off);
+        ldsm_x4(ql, a_q + part + off);
+        split_pair(acc[2 * kk][0], acc[2 * kk][1], hi[0], lo[0]);
+        split_pair(acc[2 * kk][2], acc[2 * kk][3], hi[1], lo[1]);
+        split_pair(acc[2 * kk + 1][0], acc[2 * kk + 1][1], hi[2], lo[2]);
+        split_pair(acc[2 * kk + 1][2], acc[2 * kk + 1][3], hi[3], lo[3]);
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt) {
+          mma_16816(p0[nt], hi, uh[2 * nt], uh[2 * nt + 1]);
+          mma_16816(p1[nt], hi, ul[2 * nt], ul[2 * nt + 1]);
+          mma_16816(p2[nt], lo, uh[2 * nt], uh[2 * nt + 1]);
+          mma_16816(o0[nt], hi, qh[2 * nt], qh[2 * nt + 1]);
+          mma_16816(o1[nt], hi, ql[2 * nt], ql[2 * nt + 1]);
+          mma_16816(o2[nt], lo, qh[2 * nt], qh[2 * nt + 1]);
+        }
+      }
+      // -p'^T as the left operand of the state update: the accumulator's places are those of a 16 x 16 operand
+      uint32_t ph[4], pl[4];
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+        for (int e = 0; e < 2; ++e)
+          split_pair(-(p0[nt][2 * e] + p1[nt][2 * e] + p2[nt][2 * e]),
+                     -(p0[nt][2 * e + 1] + p1[nt][2 * e + 1] + p2[nt][2 * e + 1]), ph[2 * nt + e], pl[2 * nt + e]);
+#pragma unroll
+      for (int kk = 0; kk < NK; ++kk) {
+        uint32_t kh[4], kl[4], bh[4], bl[4];
+        const uint32_t off = (uint32_t)(trn_row * rs + kk * 16 + trn_col) * 2;
+        ldsm_x4_t(kh, a_k + off);
+        ldsm_x4_t(kl, a_k + part + off);
+        ldsm_x4_t(bh, a_b + off);
+        ldsm_x4_t(bl, a_b + part + off);
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int j = 2 * kk + e;
+          const float2 dd = *reinterpret_cast<const float2*>(D + 8 * j + q2);
+          acc[j][0] *= dd.x;
+          acc[j][1] *= dd.y;
+          acc[j][2] *= dd.x;
+          acc[j][3] *= dd.y;
+          mma_16816(acc[j], va, kh[2 * e], kh[2 * e + 1]);
+          mma_16816(acc[j], va, kl[2 * e], kl[2 * e + 1]);
+          mma_16816(acc[j], ph, bh[2 * e], bh[2 * e + 1]);
+          mma_16816(acc[j], ph, bl[2 * e], bl[2 * e + 1]);
+          mma_16816(acc[j], pl, bh[2 * e], bh[2 * e + 1]);
+        }
+      }
+      uint32_t ah[4], al[4];
+      const uint32_t off = (uint32_t)(nrm_row * kARow + nrm_col) * 2;
+      ldsm_x4(ah, a_a + off);
+      ldsm_x4(al, a_a + kChunk * kARow * 2 + off);
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt) {
+        mma_16816(o1[nt], va, ah[2 * nt], ah[2 * nt + 1]);
+        mma_16816(o2[nt], va, al[2 * nt], al[2 * nt + 1]);
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+          ob[(nt * 8 + q2 + (i & 1)) * L.obuf_row + r + (i >> 1) * 8] = o0[nt][i] + o1[nt][i] + o2[nt][i];
+      }
+    }
+    if (c == 0) continue;
+    const float* ob = obuf + ((c - 1) & 1) * L.obuf;
+    const int t0 = (c - 1) * kChunk, len = min(kChunk, tokens - t0);
+    for (int tb = warp * 2; tb < len; tb += n_warps * 2) {
+      const int t = tb + (lane >> 4);                    // below 16; rows past `len` are computed and not stored
+      const float* orow = ob + t * L.obuf_row;
+      float4 o[KD];
+      float ss = 0.f;
+#pragma unroll
+      for (int k = 0; k < KD; ++k) {
+        const int i = (lane & 15) * 4 + k * 64;
+        o[k] = i < p.dv ? *reinterpret_cast<const float4*>(orow + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        ss += o[k].x * o[k].x + o[k].y * o[k].y + o[k].z * o[k].z + o[k].w * o[k].w;
+      }
+#pragma unroll
+      for (int w = 8; w > 0; w >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, w);
+      const float f = p.out_scale * rsqrtf(ss * inv_dv + p.eps);
+      if (t < len) {
+        __nv_bfloat16* dst = out + (size_t)(t0 + t) * p.out_stride;
+#pragma unroll
+        for (int k = 0; k < KD; ++k) {
+          const int i = (lane & 15) * 4 + k * 64;
+          if (i < p.dv) {
+            const uint2 graw = tb == warp * 2 ? gpre[k] : *reinterpret_cast<const uint2*>(
+                                   x + (size_t)(t0 + t) * p.row_stride + p.g_off + h * p.dv + i);
+            const float4 w = *reinterpret_cast<const float4*>(nw + i);
+            const float2 ga = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&graw.x));
+            const float2 gb = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&graw.y));
+            uint2 y;
+            y.x = pack_bf16x2(o[k].x * f * w.x * fast_gate(ga.x, p.gate_act), o[k].y * f * w.y * fast_gate(ga.y, p.gate_act));
+            y.y = pack_bf16x2(o[k].z * f * w.z * fast_gate(gb.x, p.gate_act), o[k].w * f * w.w * fast_gate(gb.y, p.gate_act));
+            *reinterpret_cast<uint2*>(dst + i) = y;
+          }
+        }
+      }
+    }
+  }
+  copy_wait<0>();
+#pragma unroll
+  for (int j = 0; j < 2 * NK; ++j)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int rr = r + (i >> 1) * 8, d = 8 * j + q2 + (i & 1);
+      if (rr < p.dv && d < p.dk) slot_S[(size_t)rr * p.dk + d] = acc[j][i];
+    }
+}
+
+template <typename K>
+static int delta_configure(K kernel, int smem, int& configured) {
+  if (smem <= 48 * 1024 || smem <= configured) return 0;
+  const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  if (e != cudaSuccess) return (int)e;
+  configured = smem;
+  return 0;
+}
+
+template <int NK>
+static int launch_delta(const RecParams& p, const int* row0, const int* nrow, const int* slots, const int* pos0, int n_seq,
+                        const int* chunk_row, const int* chunk_len, const int* chunk0, int n_chunks, uint8_t* tiles,
+                        cudaStream_t stream) {
+  static int prep_smem = 0, scan_smem = 0;
+  const int psm = DeltaPrepSmem(NK * 16, (p.rank + 15) / 16 * 16).total;
+  const int dvp = (p.dv + 15) / 16 * 16, ssm = DeltaScanSmem(NK * 16, dvp).total;
+  int r = delta_configure(delta_prepare_kernel<NK>, psm, prep_smem);
+  if (r || (r = delta_configure(delta_scan_kernel<NK>, ssm, scan_smem))) return r;
+  // heads before chunks: the tiles of one chunk are neighbours in memory.  The grid's second dimension ends at 65535.
+  for (int c = 0; c < n_chunks; c += 65535) {
+    const int m = n_chunks - c < 65535 ? n_chunks - c : 65535;
+    delta_prepare_kernel<NK><<<dim3(p.H, m), kDeltaThreads, psm, stream>>>(
+        p, chunk_row + c, chunk_len + c, tiles + (size_t)c * p.H * delta_tile_bytes(NK * 16));
+    const cudaError_t e = cudaGetLastError();
+    if (e != cudaSuccess) return (int)e;
+  }
+  delta_scan_kernel<NK><<<dim3(p.H, n_seq), dvp * 2, ssm, stream>>>(p, row0, nrow, slots, pos0, chunk0, tiles);
+  return (int)cudaGetLastError();
+}
+
+}  // namespace sb
+
+using namespace sb;
+
+// Arguments of sb_recurrence_step: one token per sequence (row0 / nrow null) or a packed portion each, any sizes.
+extern "C" int sb_delta_step(const void* params, const int* row0, const int* nrow, const int* slots, const int* pos0, int n_seq,
+                             int f32, cudaStream_t stream) {
+  if (n_seq == 0) return 0;
+  const RecParams& p = *reinterpret_cast<const RecParams*>(params);
+  if (n_seq > 65535 || p.kind != kGateDelta || p.dk != p.dv || p.rank < 1 || !p.w2 || !p.b_e || !p.b_f) return -3;
+  const size_t base = (size_t)delta_step_floats(p.dk, p.dv, p.rank) * 4;
+  if (base > 100 * 1024) return -3;
+  const dim3 grid(p.H, n_seq);
+  if (p.dk % 4 == 0 && p.dk <= 128 && base <= 48 * 1024) {
+    const int n = (p.dk + 31) / 32;
+    auto run = [&](auto kernel) -> int {
+      kernel<<<grid, kStepThreads, base, stream>>>(p, row0, nrow, slots, pos0);
+      return (int)cudaGetLastError();
+    };
+    if (f32)
+      return n == 1 ? run(delta_step_regs_kernel<float, 1>) : n == 2 ? run(delta_step_regs_kernel<float, 2>)
+           : n == 3 ? run(delta_step_regs_kernel<float, 3>) : run(delta_step_regs_kernel<float, 4>);
+    using H = __nv_bfloat16;
+    return n == 1 ? run(delta_step_regs_kernel<H, 1>) : n == 2 ? run(delta_step_regs_kernel<H, 2>)
+         : n == 3 ? run(delta_step_regs_kernel<H, 3>) : run(delta_step_regs_kernel<H, 4>);
+  }
+  const size_t state = (size_t)p.dv * p.dk * 4;
+  const int in_smem = nrow != nullptr && base + state <= 200 * 1024;
+  const size_t smem = base + (in_smem ? state : 0);
+  auto run = [&](auto kernel) -> int {
+    if (smem > 48 * 1024) {
+      const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+      if (e != cudaSuccess) return (int)e;
+    }
+    kernel<<<grid, kStepThreads, smem, stream>>>(p, row0, nrow, slots, pos0, in_smem);
+    return (int)cudaGetLastError();
+  };
+  return f32 ? run(delta_step_kernel<float>) : run(delta_step_kernel<__nv_bfloat16>);
+}
+
+// Bytes of workspace of sb_delta_prefill for `n_chunks` chunks, or -1 when the sizes need sb_delta_step (head width a multiple of
+// eight up to 128, 16-byte aligned rows).
+extern "C" long long sb_delta_workspace(const void* params, int n_chunks) {
+  const RecParams& p = *reinterpret_cast<const RecParams*>(params);
+  if (p.kind != kGateDelta || p.dk != p.dv || p.dk % 8 || p.dk > 128 || p.row_stride % 8 || p.q_off % 8 || p.k_off % 8 ||
+      p.v_off % 8 || p.f_off % 8 || p.g_off % 4 || p.out_stride % 4 || p.out_off % 4 || p.rank < 1 || p.rank > 512 ||
+      ((uintptr_t)p.x & 15) || ((uintptr_t)p.out & 7) || ((uintptr_t)p.b_f & 15))
+    return -1;
+  return (long long)n_chunks * p.H * delta_tile_bytes(pad_dk(p.dk));
+}
+
+// bf16 prefill of packed portions in 16-token chunks: chunk c covers rows chunk_row[c] .. + chunk_len[c]; those of sequence s
+// begin with chunk chunk0[s].
+extern "C" int sb_delta_prefill(const void* params, const int* row0, const int* nrow, const int* slots, const int* pos0, int n_seq,
+                                const int* chunk_row, const int* chunk_len, const int* chunk0, int n_chunks, void* workspace,
+                                cudaStream_t stream) {
+  if (n_seq == 0 || n_chunks == 0) return 0;
+  if (n_seq > 65535 || ((uintptr_t)workspace & 15)) return -3;
+  const RecParams& p = *reinterpret_cast<const RecParams*>(params);
+  if (sb_delta_workspace(params, n_chunks) < 0) return -2;
+  uint8_t* tiles = reinterpret_cast<uint8_t*>(workspace);
+  switch (pad_dk(p.dk) / 16) {
+#define SB_DELTA(NK) \
+  case NK:           \
+    return launch_delta<NK>(p, row0, nrow, slots, pos0, n_seq, chunk_row, chunk_len, chunk0, n_chunks, tiles, stream);
+    SB_DELTA(1) SB_DELTA(2) SB_DELTA(3) SB_DELTA(4) SB_DELTA(6) SB_DELTA(8)
+#undef SB_DELTA
+  }
+  return -2;
+}

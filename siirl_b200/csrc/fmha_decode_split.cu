@@ -21,7 +21,7 @@
 //
 // The windowed variant (WIN) serves attention with a sliding window, kept first tokens and a linear distance bias
 // (win_params.h): an item's tiles are the cache blocks that hold a visible key (those of the kept tokens, then those of
-// the window), key and value widths may differ and be any multiple of 8 up to D (TMA fills the missing columns with
+// the window; with pooled runs the blocks of their entries, then those of the window), key and value widths may differ and be any multiple of 8 up to D (TMA fills the missing columns with
 // zeros), the bias is one multiply-add per score, and the output goes to a column range of a wider row, scaled.
 #include "common.cuh"
 #include "launchers.h"
@@ -52,18 +52,31 @@ struct SplitParams {
   int sink, rel_n;
   const float* rel;          // [Hq, rel_n] bias by distance, or null
   const float* head_gate;    // [B, Hq] factors of the result, or null
+  int pool, pool_blocks;     // pooled runs before the window, their entries' blocks in pool_table [B, pool_blocks]
+  const int* pool_table;
+  const __nv_bfloat16* sink_w;      // [Hq] scores of the sink, or null
 };
 
-// cache blocks a query at position ctx - 1 visits: blocks 0 .. sinks - 1, then w0 .. ; `n` of them in all
-__host__ __device__ __forceinline__ void visible_tiles(int ctx, int window, int keep_first, int& sinks, int& w0, int& n) {
+// cache blocks a query at position ctx - 1 visits: blocks 0 .. sinks - 1 (of the tokens, or of the pooled entries), then
+// w0 .. ; `n` of them in all
+__host__ __device__ __forceinline__ void visible_tiles(int ctx, int window, int keep_first, int pool, int& sinks, int& w0, int& n) {
   const int tiles = (ctx + kSBlk - 1) / kSBlk;
   sinks = 0;
   w0 = 0;
-  if (window > 0) {
+  if (pool > 0) {
+    sinks = (pooled_entries(ctx - 1, window, pool) + kSBlk - 1) / kSBlk;
+    w0 = max(0, ctx - window) / kSBlk;
+  } else if (window > 0) {
     sinks = min((keep_first + kSBlk - 1) / kSBlk, tiles);
     w0 = max(sinks, max(0, ctx - window) / kSBlk);
   }
   n = sinks + max(0, tiles - w0);
+}
+
+// the sink's part of a soft-max sum whose terms are relative to 2^m
+__device__ __forceinline__ float sink_term(const SplitParams& p, int head, float m) {
+  if (p.sink_w) return exp2f(fmaf(__bfloat162float(p.sink_w[head]), 1.4426950408889634f, -m));
+  return p.sink ? exp2f(-m) : 0.f;
 }
 
 template <int D>
@@ -162,7 +175,7 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
       seq_tiles = (ctx + kSBlk - 1) / kSBlk;
       if constexpr (WIN) {
         int sinks, w0;
-        visible_tiles(ctx, p.window, p.keep_first, sinks, w0, seq_tiles);
+        visible_tiles(ctx, p.window, p.keep_first, p.pool, sinks, w0, seq_tiles);
       }
       t0 = c * kChunkTiles;
       const int t1 = min(seq_tiles, t0 + kChunkTiles);
@@ -204,7 +217,7 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
         const int q_at = min(n - 1, 3);
         const int* blocks = p.block_table + (size_t)b * p.max_blocks;
         int sinks = 0, w0 = 0, vis = 0;
-        if constexpr (WIN) visible_tiles(p.seq_lens[b], p.window, p.keep_first, sinks, w0, vis);
+        if constexpr (WIN) visible_tiles(p.seq_lens[b], p.window, p.keep_first, p.pool, sinks, w0, vis);
         for (int t = 0; t < n && ok; ++t, ++tile_no) {
           const int stage = tile_no % NS;
           const uint32_t round = tile_no / NS;
@@ -212,7 +225,9 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
             ok = false;
             break;
           }
-          int blk = blocks[!WIN || t0 + t < sinks ? t0 + t : w0 + t0 + t - sinks];
+          int blk;
+          if (WIN && p.pool > 0 && t0 + t < sinks) blk = t0 + t < p.pool_blocks ? p.pool_table[(size_t)b * p.pool_blocks + t0 + t] : -1;
+          else blk = blocks[!WIN || t0 + t < sinks ? t0 + t : w0 + t0 + t - sinks];
           if (WIN && blk < 0) blk = 0;      // never among the visible blocks of a well-formed table
           uint8_t* sk = sKV + stage * 2 * L::kKBytes;
           uint8_t* sv = sk + L::kKBytes;
@@ -311,13 +326,18 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
     for (; ok && find_item(idx, c, b, g, t0, n, n_seq_tiles); idx += gridDim.x) {
       const int ctx = p.seq_lens[b];
       int sinks = 0, w0 = 0, vis = 0;
-      if constexpr (WIN) visible_tiles(ctx, p.window, p.keep_first, sinks, w0, vis);
+      if constexpr (WIN) visible_tiles(ctx, p.window, p.keep_first, p.pool, sinks, w0, vis);
+      // tile t holds pooled entries (numbers first_pos(t) ..) of which the first `pool_n` are visible
+      const int pool_n = WIN ? pooled_entries(ctx - 1, p.window, p.pool) : 0;
+      auto pooled = [&](int t) { return WIN && p.pool > 0 && t0 + t < sinks; };
       auto first_pos = [&](int t) { return (!WIN || t0 + t < sinks ? t0 + t : w0 + t0 + t - sinks) * kSBlk; };
       // some key of the tile at kv0 is not visible / the key at `col` is not
-      auto need_mask = [&](int kv0) {
+      auto need_mask = [&](int t, int kv0) {
+        if (pooled(t)) return kv0 + kSBlk > pool_n;
         return kv0 + kSBlk > ctx || (WIN && p.window > 0 && ctx - 1 - kv0 >= p.window && kv0 + kSBlk > p.keep_first);
       };
-      auto hidden = [&](int col) {
+      auto hidden = [&](int t, int col) {
+        if (pooled(t)) return col >= pool_n;
         return col >= ctx || (WIN && p.window > 0 && ctx - 1 - col >= p.window && col >= p.keep_first);
       };
       auto slope_of = [&](int row) {
@@ -387,12 +407,12 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
               sv[2 * i + 1] = TABLE ? sv[2 * i + 1] + rb[2 * i + 1] : fmaf(slope, dist + 1.f, sv[2 * i + 1]);
             }
           }
-          if (need_mask(kv0)) {
+          if (need_mask(t, kv0)) {
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
               const int col = kv0 + 8 * i + 2 * fq;
-              if (hidden(col)) sv[2 * i] = -INFINITY;
-              if (hidden(col + 1)) sv[2 * i + 1] = -INFINITY;
+              if (hidden(t, col)) sv[2 * i] = -INFINITY;
+              if (hidden(t, col + 1)) sv[2 * i + 1] = -INFINITY;
             }
           }
           float m_tile = -INFINITY;
@@ -491,10 +511,10 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
               for (int i = 0; i < kSBlk; ++i) sv[i] += rel_at(rel, kv0 + i);
             }
           }
-          if (need_mask(kv0)) {
+          if (need_mask(t, kv0)) {
   #pragma unroll
             for (int i = 0; i < kSBlk; ++i)
-              if (hidden(kv0 + i)) sv[i] = -INFINITY;
+              if (hidden(t, kv0 + i)) sv[i] = -INFINITY;
           }
           float m_tile = -INFINITY;
   #pragma unroll
@@ -592,7 +612,7 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
       const float inv_l = l_run > 0.f ? 1.f / l_run : 0.f;
       const int head = g * rep + (row_valid ? lane : 0);
       const bool single = n_seq_tiles <= kChunkTiles;
-      const float total = WIN && p.sink ? l_run + exp2f(-m_ref) : l_run;
+      const float total = WIN ? l_run + sink_term(p, head, m_ref) : l_run;
       const int dv = WIN ? p.dv : D;
       __nv_bfloat16* orow = p.out + (WIN ? (size_t)b * p.out_stride : (size_t)b * (p.Hq * D)) + (size_t)head * dv;
       float out_f = WIN ? (total > 0.f ? p.out_scale / total : 0.f) : inv_l;
@@ -653,7 +673,7 @@ __global__ void fmha_decode_merge_kernel(SplitParams p) {
   int n_tiles = (ctx + kSBlk - 1) / kSBlk;
   if constexpr (WIN) {
     int sinks, w0;
-    visible_tiles(ctx, p.window, p.keep_first, sinks, w0, n_tiles);
+    visible_tiles(ctx, p.window, p.keep_first, p.pool, sinks, w0, n_tiles);
   }
   const int dv = WIN ? p.dv : D;
   __nv_bfloat16* orow = p.out + (WIN ? (size_t)b * p.out_stride : (size_t)b * (p.Hq * D)) + (size_t)h * dv;
@@ -675,7 +695,7 @@ __global__ void fmha_decode_merge_kernel(SplitParams p) {
     wsum += w;
     acc += w * wo[(size_t)c * D + d];
   }
-  if (WIN && p.sink) wsum += exp2f(-m);
+  if (WIN) wsum += sink_term(p, h, m);
   float f = WIN ? p.out_scale : 1.f;
   if (WIN && p.head_gate) f *= p.head_gate[(size_t)b * p.Hq + h];
   orow[d] = __float2bfloat16(wsum > 0.f ? acc / wsum * f : 0.f);
@@ -737,6 +757,7 @@ extern "C" int sb_fmha_decode_split(const void* q, int row_stride, const void* c
   p.scale_log2 = scale * 1.4426950408889634f; p.status = status;
   p.window = 0; p.keep_first = 0; p.dv = D; p.out_stride = 0; p.bias_exp = 0.f; p.out_scale = 1.f;
   p.softcap = 0.f; p.scale = scale; p.sink = 0; p.rel_n = 0; p.rel = nullptr; p.head_gate = nullptr;
+  p.pool = 0; p.pool_blocks = 0; p.pool_table = nullptr; p.sink_w = nullptr;
   return D == 128 ? launch_decode_split<128, 0>(mc, mc, mq, p, stream)
                   : launch_decode_split<64, 0>(mc, mc, mq, p, stream);
 }
@@ -747,10 +768,16 @@ extern "C" int sb_attn_window_decode_chunks(const void* params) {
   const WinParams& p = *reinterpret_cast<const WinParams*>(params);
   if (p.dk % 8 || p.dv % 8 || p.dk > 128 || p.dv > 128 || p.Hq % p.Hkv || p.Hq / p.Hkv > 32 || p.row_stride % 8 ||
       p.q_off % 8 || p.out_stride % 8 || p.out_off % 8 || p.block_elems % 8 || p.kv_mode != kPaged || p.gain || p.gate ||
-      (p.rel && (p.rel_n < 1 || p.bias_exp > 0.f)))
+      (p.rel && (p.rel_n < 1 || p.bias_exp > 0.f)) ||
+      (p.pool > 0 && (p.window <= 0 || !p.pool_table || p.pool_blocks < 1 || p.keep_first || p.rel || p.bias_exp > 0.f)))
     return -1;
   int tiles = p.max_blocks;
-  if (p.window > 0) {
+  if (p.pool > 0) {
+    const int most = (p.window + kSBlk - 1) / kSBlk + 1;
+    const long long entries = (long long)tiles * kSBlk / p.pool;
+    const int pooled = (int)((entries + kSBlk - 1) / kSBlk);
+    tiles = (most < tiles ? most : tiles) + (pooled < p.pool_blocks ? pooled : p.pool_blocks);
+  } else if (p.window > 0) {
     const int most = (p.keep_first + kSBlk - 1) / kSBlk + (p.window + kSBlk - 1) / kSBlk + 1;
     if (most < tiles) tiles = most;
   }
@@ -790,6 +817,8 @@ extern "C" int sb_attn_window_decode(const void* params, const int* seq_lens, fl
   p.bias_exp = w.bias_exp; p.out_scale = w.out_scale;
   p.softcap = w.softcap; p.scale = w.scale; p.sink = w.sink; p.rel_n = (int)w.rel_n; p.rel = w.rel;
   p.head_gate = w.head_gate;
+  p.pool = w.pool; p.pool_blocks = w.pool_blocks; p.pool_table = w.pool_table;
+  p.sink_w = reinterpret_cast<const __nv_bfloat16*>(w.sink_w);
   const bool wide = w.dk > 64 || w.dv > 64;
   if (w.softcap > 0.f || w.rel)
     return wide ? launch_decode_split<128, 2>(mk, mv, mq, p, stream) : launch_decode_split<64, 2>(mk, mv, mq, p, stream);

@@ -1,8 +1,8 @@
-// Attention of prompt portions against the paged cache with a sliding window, kept first tokens and a linear distance
-// bias (see win_params.h), and the cache append for heads whose key and value widths differ.
+// Attention of prompt portions against the paged cache with a sliding window, kept first tokens or pooled runs before it, and
+// a linear distance bias (see win_params.h), and the cache append for heads whose key and value widths differ.
 //
 // The portion's keys and values are appended to the cache first; a query tile then walks the cache blocks in which any
-// of its rows sees a key: the blocks of the kept first tokens, then those of the window.  Whole prompts, later portions
+// of its rows sees a key: the blocks of the kept first tokens or of the pooled entries, then those of the window.  Whole prompts, later portions
 // and reused prefixes take the same path, and blocks that left every window are never touched.  Keys and values may also
 // lie in packed rows (latent attention expands them from its cache), and the result may be gated.
 //
@@ -67,18 +67,23 @@ __global__ void __launch_bounds__(kSimtThreads) window_simt_kernel(WinParams p) 
   const float gain = p.gain ? to_float(*reinterpret_cast<const T*>(p.gain)) : 1.f;
   for (int d = tid; d < p.dk; d += kSimtThreads) sq[d] = to_float(q[d]) * gain;
   for (int d = tid; d < p.dv; d += kSimtThreads) so[d] = 0.f;
-  // the visible keys are 0 .. first - 1 and lo .. i
+  // the visible keys are 0 .. first - 1 (tokens, or pooled entries) and lo .. i
   int first = 0, lo = 0;
-  if (p.window > 0) {
+  if (p.pool > 0) {
+    first = pooled_entries(i, p.window, p.pool);
+    lo = max(0, i - p.window + 1);
+  } else if (p.window > 0) {
     first = min(p.keep_first, i + 1);
     lo = max(first, i - p.window + 1);
   }
   const int n = first + (i + 1 - lo);
   const int* bt = p.block_table + (size_t)slot * p.max_blocks;
+  const int* pt = p.pool > 0 ? p.pool_table + (size_t)slot * p.pool_blocks : bt;
+  const int pt_blocks = p.pool > 0 ? p.pool_blocks : p.max_blocks;
   const T* cache = reinterpret_cast<const T*>(p.cache);
   auto row_of = [&](int v, bool value) -> const T* {
     const int j = v < first ? v : lo + v - first;
-    const int blk = j / kWBlk < p.max_blocks ? bt[j / kWBlk] : -1;
+    const int blk = v < first ? (j / kWBlk < pt_blocks ? pt[j / kWBlk] : -1) : (j / kWBlk < p.max_blocks ? bt[j / kWBlk] : -1);
     if (blk < 0 || blk >= p.num_blocks) return nullptr;
     const size_t base = (size_t)blk * p.block_elems;
     return value && p.kv_mode != kLatent
@@ -125,7 +130,8 @@ __global__ void __launch_bounds__(kSimtThreads) window_simt_kernel(WinParams p) 
     }
     __syncthreads();
   }
-  if (p.sink) l += expf(-m);
+  if (p.sink_w) l += expf(to_float(reinterpret_cast<const T*>(p.sink_w)[h]) - m);
+  else if (p.sink) l += expf(-m);
   float inv = l > 0.f ? p.out_scale / l : 0.f;
   if (p.head_gate) inv *= p.head_gate[(size_t)t * p.Hq + h];
   for (int d = tid; d < p.dv; d += kSimtThreads) out[d] = from_float<T>(so[d] * inv);
@@ -148,10 +154,14 @@ struct WinSmem {
   }
 };
 
-// cache blocks a query tile at positions q0 .. q1 visits: `sinks` blocks from 0, then blocks w0 .. of the window
-__host__ __device__ inline void win_blocks(int q0, int q1, int window, int keep_first, int& sinks, int& w0, int& n) {
+// cache blocks a query tile at positions q0 .. q1 visits: `sinks` blocks from 0 (of the tokens, or of the pooled entries), then
+// blocks w0 .. of the window
+__host__ __device__ inline void win_blocks(int q0, int q1, int window, int keep_first, int pool, int& sinks, int& w0, int& n) {
   const int last = q1 / kWBlk;
-  if (window <= 0) {
+  if (pool > 0) {
+    sinks = (pooled_entries(q1, window, pool) + kWBlk - 1) / kWBlk;
+    w0 = q0 - window + 1 > 0 ? (q0 - window + 1) / kWBlk : 0;
+  } else if (window <= 0) {
     sinks = 0;
     w0 = 0;
   } else {
@@ -200,9 +210,10 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
   const int row0 = tile_row[tile], nrows = tile_rows[tile], q0 = tile_pos[tile], slot = tile_slot[tile];
   const int kvh = h / (p.Hq / p.Hkv);
   int sinks, w0, n_tiles;
-  win_blocks(q0, q0 + nrows - 1, p.window, p.keep_first, sinks, w0, n_tiles);
+  win_blocks(q0, q0 + nrows - 1, p.window, p.keep_first, p.pool, sinks, w0, n_tiles);
   const bool packed = p.kv_mode == kPackedRows;
   const int* bt = p.block_table + (size_t)(packed ? 0 : slot) * p.max_blocks;
+  const int* pt = p.pool > 0 ? p.pool_table + (size_t)slot * p.pool_blocks : nullptr;
   auto block_of = [&](int j) { return j < sinks ? j : w0 + j - sinks; };
 
   if (tid == 0) {
@@ -230,7 +241,9 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     // packed rows: head kvh, rows from the block on; those past the sequence are hidden by causality, past the end zeros
     auto load = [&](const CUtensorMap* map, uint8_t* dst, int bytes, int chunks, uint64_t* bar, int j) {
       const int lb = block_of(j);
-      int blk = packed ? slot + lb * kWBlk : (lb < p.max_blocks ? bt[lb] : 0);
+      int blk;
+      if (pt && j < sinks) blk = lb < p.pool_blocks ? pt[lb] : 0;
+      else blk = packed ? slot + lb * kWBlk : (lb < p.max_blocks ? bt[lb] : 0);
       if (!packed && (blk < 0 || blk >= p.num_blocks)) blk = 0;      // never inside the visible range of a well-formed table
       const int mid = packed ? kvh : kvh * kWBlk;
       if (leader) {
@@ -325,6 +338,7 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     const float* rel = TABLE && p.rel ? p.rel + (size_t)h * p.rel_n : nullptr;
     const int rel_last = (int)p.rel_n - 1;
     const float rel_far = rel ? __ldg(rel + rel_last) * 1.4426950408889634f : 0.f;
+    const int pool_q0 = pooled_entries(q0, p.window, p.pool), pool_n = pooled_entries(qpos, p.window, p.pool);
     float m_ref = -INFINITY, l_run = 0.f;
 
     for (int j = 0; j < n_tiles; ++j) {
@@ -379,9 +393,14 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       }
       // every row of the tile sees every key of the block when the block lies behind q0 and, with a window, inside the
       // last row's window or among the kept tokens
-      const bool all_seen = kv0 + kWBlk - 1 <= q0 &&
-                            (p.window <= 0 || q0 + nrows - 1 - kv0 < p.window || kv0 + kWBlk <= p.keep_first);
-      if (!all_seen) {
+      if (p.pool > 0 && j < sinks) {      // entries kv0 .. of the pooled runs
+        if (kv0 + kWBlk > pool_q0) {
+#pragma unroll
+          for (int i = 0; i < kWBlk; ++i)
+            if (kv0 + i >= pool_n) sv[i] = -INFINITY;
+        }
+      } else if (!(kv0 + kWBlk - 1 <= q0 &&
+                   (p.window <= 0 || q0 + nrows - 1 - kv0 < p.window || kv0 + kWBlk <= p.keep_first))) {
 #pragma unroll
         for (int i = 0; i < kWBlk; ++i) {
           const int kp = kv0 + i;
@@ -446,7 +465,8 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     if (ok) {
       tc_fence_after();
       const bool row_valid = tid < nrows;
-      if (p.sink) l_run += exp2f(-m_ref);
+      if (p.sink_w) l_run += exp2f(fmaf(__bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p.sink_w)[h]), 1.4426950408889634f, -m_ref));
+      else if (p.sink) l_run += exp2f(-m_ref);
       float inv_l = l_run > 0.f ? p.out_scale / l_run : 0.f;
       if (p.head_gate && row_valid) inv_l *= p.head_gate[(size_t)(row0 + tid) * p.Hq + h];
       __nv_bfloat16* orow = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)(row0 + (row_valid ? tid : 0)) * p.out_stride +
@@ -489,6 +509,11 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
 
 using namespace sb;
 
+// pooled runs: a window to be before, blocks to lie in, nothing that is defined by the distance of a key
+static bool pool_valid(const WinParams& p) {
+  return p.pool <= 0 || (p.window > 0 && p.pool_table && p.pool_blocks > 0 && p.kv_mode == kPaged && p.keep_first == 0 && !p.rel && !(p.bias_exp > 0.f));
+}
+
 static int win_grid(long long total) {
   long long b = (total + 255) / 256;
   const long long cap = (long long)num_sms() * 8;
@@ -514,7 +539,7 @@ extern "C" int sb_kv_append_split(const void* params, int f32, cudaStream_t stre
 extern "C" int sb_attn_window_simt(const void* params, int f32, cudaStream_t stream) {
   const WinParams& p = *reinterpret_cast<const WinParams*>(params);
   if (p.T == 0) return 0;
-  if (p.Hq % p.Hkv || p.Hq > 65535 || p.kv_mode == kPackedRows || (p.rel && p.rel_n < 1) || p.gate || (p.kv_mode == kLatent && p.dk != p.dv)) return -3;
+  if (p.Hq % p.Hkv || p.Hq > 65535 || p.kv_mode == kPackedRows || (p.rel && p.rel_n < 1) || p.gate || (p.kv_mode == kLatent && p.dk != p.dv) || !pool_valid(p)) return -3;
   const size_t smem = (size_t)(p.dk + kSimtThreads + p.dv) * 4;
   if (smem > 48 * 1024) return -3;
   const dim3 grid(p.T, p.Hq);
@@ -531,7 +556,7 @@ extern "C" int sb_attn_window_prefill(const void* params, const int* tile_row, c
   if (n_tiles == 0) return 0;
   if (p.Hq % p.Hkv || p.dk % 8 || p.dv % 8 || p.dk > 256 || p.dv > 256 || p.dk < 8 || p.dv < 8 || p.row_stride % 8 ||
       p.q_off % 8 || p.out_stride % 8 || p.out_off % 8 || p.block_elems % 8 || ((uintptr_t)p.out & 15) ||
-      p.kv_mode == kLatent || p.gate_stride % 8 || ((uintptr_t)p.gate & 15) || (p.rel && (p.rel_n < 1 || p.bias_exp > 0.f)))
+      p.kv_mode == kLatent || p.gate_stride % 8 || ((uintptr_t)p.gate & 15) || (p.rel && (p.rel_n < 1 || p.bias_exp > 0.f)) || !pool_valid(p))
     return -2;
   static thread_local bool tl_context_bound = false;
   if (!tl_context_bound) {

@@ -7,11 +7,15 @@
 //                      or h = sum of partial products + vector (entry of a loop's pass), then h / rms(h); or h as two rows
 //   gated_act          y = act(gate) * up   for a fused projection [gate | up]   (SiLU, tanh-form or exact GELU, squared relu)
 //   scaled_act         y = act(gain * x)    of a column range
+//   bias_act           y = act(sum of partial products + bias), xIELU with its two learned numbers among the activations
+//   token_gate         y = gelu_tanh(sum of partial products) * columns of an embedding table's row
 //   softcap            z = cap * tanh(z / cap) in place on fp32 logits
 //   gemm_simt          C[M, N] = A[M, K] B[N, K]^T with fp32 accumulation on the FMA pipes: fp32 models (true 32-bit
 //                      products) and bf16 operands whose row pitch TMA cannot address (not a multiple of 16 bytes)
 //
 // Templates: T is the activation / weight format (bf16 or fp32); V elements per access (4, or 1 for odd widths).
+#include <type_traits>
+
 #include "common.cuh"
 #include "launchers.h"
 #include "typed.cuh"
@@ -217,6 +221,101 @@ __global__ void partial_act_kernel(const float* __restrict__ x, long long slab, 
 #pragma unroll
     for (int k = 0; k < V; ++k) g[k] = activate<ACT, __nv_bfloat16>(g[k]) * (GATED ? u[k] : 1.f);
     store_vec<__nv_bfloat16, V>(out + t * I + c, g);
+  }
+}
+
+// Two learned numbers: softplus(p) z^2 + z / 2 on the right of zero, (1/2 + softplus(q)) (e^z - 1 - z) + z / 2 on the left
+struct Xielu {
+  float right = 0.f, left = 0.f;
+  Xielu() = default;
+  template <typename T>
+  __device__ __forceinline__ explicit Xielu(const T* n)
+      : right(softplus(to_float(n[0]))), left(0.5f + softplus(to_float(n[1]))) {}
+  static __device__ __forceinline__ float softplus(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+  // the result is rounded to T: next to zero (where e^z - 1 - z cancels) its first terms, z^2 (1/2 + z/6 + z^2/24 + z^3/120)
+  template <typename T>
+  __device__ __forceinline__ float operator()(float z) const {
+    if constexpr (sizeof(T) == 4) {
+      return z > 0.f ? fmaf(right * z, z, 0.5f * z) : fmaf(left, expm1f(z) - z, 0.5f * z);
+    } else {
+      const float zz = z * z;
+      const float near = zz * fmaf(z, fmaf(z, fmaf(z, 1.f / 120.f, 1.f / 24.f), 1.f / 6.f), 0.5f);
+      const float far = __expf(z) - 1.f - z;
+      return fmaf(z > 0.f ? right : left, z > 0.f ? zz : (z > -0.25f ? near : far), 0.5f * z);
+    }
+  }
+};
+
+// ACT 4: xIELU.  XT: format of x (partial sums: fp32); T: of bias, numbers and result
+template <typename XT, typename T, int V, int ACT>
+__global__ void bias_act_kernel(const XT* __restrict__ x, long long slab, int slabs, const T* __restrict__ bias,
+                                const T* __restrict__ numbers, T* __restrict__ out, long long rows, int I,
+                                const int* __restrict__ used) {
+  // a thread keeps its columns and walks down the rows, four loads in flight
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
+  if (c >= I) return;
+  float b[V] = {};
+  if (bias) load_vec<T, V>(bias + c, b);
+  Xielu xi;
+  if constexpr (ACT == 4) xi = Xielu(numbers);
+  const long long step = gridDim.y;
+  for (long long t = blockIdx.y; t < rows; t += 4 * step) {
+    float v[4][V];
+    bool on[4];
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      const long long r = t + u * step;
+      on[u] = r < rows && !(used && used[r] < 0);
+      if (on[u]) load_vec<XT, V>(x + r * I + c, v[u]);
+    }
+    for (int s = 1; s < slabs; ++s) {
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        if (!on[u]) continue;
+        float a[V];
+        load_vec<XT, V>(x + s * slab + (t + u * step) * I + c, a);
+#pragma unroll
+        for (int k = 0; k < V; ++k) v[u][k] += a[k];
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      if (!on[u]) continue;
+#pragma unroll
+      for (int k = 0; k < V; ++k) {
+        const float z = v[u][k] + b[k];
+        if constexpr (ACT == 4) v[u][k] = xi.template operator()<T>(z);
+        else v[u][k] = activate<ACT, T>(z);
+      }
+      store_vec<T, V>(out + (t + u * step) * I + c, v[u]);
+    }
+  }
+}
+
+template <typename XT, typename T, int V>
+__global__ void token_gate_kernel(const XT* __restrict__ z, long long slab, int slabs, const long long* __restrict__ ids,
+                                  const T* __restrict__ table, long long pitch, int vocab, int column, int width,
+                                  T* __restrict__ out, int rows, int I) {
+  const int nv = I / V;
+  const long long total = (long long)rows * nv;
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const int t = (int)(i / nv), c = (int)(i % nv) * V;
+    long long id = ids[t];
+    id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
+    float g[V], e[V];
+    load_vec<XT, V>(z + (size_t)t * I + c, g);
+    const T* row = table + id * pitch + column + c;
+    if constexpr (V == 1) e[0] = c < width ? to_float(*row) : 0.f;
+    else load_vec<T, V>(row, e);      // width is a multiple of V
+    for (int s = 1; s < slabs; ++s) {
+      float a[V];
+      load_vec<XT, V>(z + s * slab + (size_t)t * I + c, a);
+#pragma unroll
+      for (int k = 0; k < V; ++k) g[k] += a[k];
+    }
+#pragma unroll
+    for (int k = 0; k < V; ++k) g[k] = gelu_tanh_f(g[k]) * e[k];
+    store_vec<T, V>(out + (size_t)t * I + c, g);
   }
 }
 
@@ -488,6 +587,24 @@ static int launch_gated_act(const T* gu, T* out, long long rows, int I, int act,
   return (int)cudaGetLastError();
 }
 
+template <typename XT, typename T, int V>
+static int launch_bias_act(const XT* x, long long slab, int slabs, const T* bias, const T* numbers, T* out, long long rows,
+                           int I, int act, const int* used, cudaStream_t s) {
+  const int threads = I / V >= 256 ? 256 : 64, cols = (I / V + threads - 1) / threads;
+  long long y = (long long)num_sms() * (2048 / threads) / cols + 1;
+  if (y > rows) y = rows;
+  const dim3 grid(cols, (unsigned)(y > 65535 ? 65535 : y));
+  auto launch = [&](auto kernel) { kernel<<<grid, threads, 0, s>>>(x, slab, slabs, bias, numbers, out, rows, I, used); };
+  switch (act) {
+    case 0: launch(bias_act_kernel<XT, T, V, 0>); break;
+    case 1: launch(bias_act_kernel<XT, T, V, 1>); break;
+    case 2: launch(bias_act_kernel<XT, T, V, 2>); break;
+    case 3: launch(bias_act_kernel<XT, T, V, 3>); break;
+    default: launch(bias_act_kernel<XT, T, V, 4>); break;
+  }
+  return (int)cudaGetLastError();
+}
+
 template <typename T, int V>
 static int launch_scaled_act(const T* x, long long stride, const T* gain, T* out, long long rows, int I, int act,
                              cudaStream_t s) {
@@ -632,5 +749,60 @@ extern "C" int sb_partial_act(const float* x, long long slab, int slabs, void* o
     else if (act == 2) launch(partial_act_kernel<4, 2, false>);
     else launch(partial_act_kernel<4, 3, false>);
   }
+  return (int)cudaGetLastError();
+}
+
+// act (4: xIELU with two numbers) of the sum of x [slabs, rows, I] (fp32, or one slab in the activation format) plus bias;
+// rows with a negative entry in `used` are left out
+extern "C" int sb_bias_act(const void* x, long long slab, int slabs, int x_f32, const void* bias, const void* numbers, void* out,
+                           long long rows, int I, int act, const int* used, int f32, cudaStream_t stream) {
+  if (rows <= 0 || I <= 0) return 0;
+  if (act < 0 || act > 4 || (act == 4 && !numbers) || slabs < 1 || (f32 && !x_f32) || (slabs > 1 && !x_f32)) return -3;
+  const bool aligned = (((uintptr_t)x | (uintptr_t)out | (uintptr_t)bias) & 15) == 0;
+  using B = __nv_bfloat16;
+  auto run = [&](auto* xp, auto* op, auto vec) -> int {
+    using T = std::remove_pointer_t<decltype(op)>;
+    using XT = std::remove_const_t<std::remove_pointer_t<decltype(xp)>>;
+    constexpr int V = decltype(vec)::value;
+    return launch_bias_act<XT, T, V>(xp, slab, slabs, (const T*)bias, (const T*)numbers, op, rows, I, act, used, stream);
+  };
+  if (f32) {
+    if (I % 4 == 0 && aligned) return run((const float*)x, (float*)out, std::integral_constant<int, 4>());
+    return run((const float*)x, (float*)out, std::integral_constant<int, 1>());
+  }
+  if (x_f32) {
+    if (I % 4 == 0 && aligned) return run((const float*)x, (B*)out, std::integral_constant<int, 4>());
+    return run((const float*)x, (B*)out, std::integral_constant<int, 1>());
+  }
+  if (I % 8 == 0 && aligned) return run((const B*)x, (B*)out, std::integral_constant<int, 8>());
+  return run((const B*)x, (B*)out, std::integral_constant<int, 1>());
+}
+
+// gelu_tanh of the sum of z [slabs, rows, I] times table[ids, column .. + width] (rows `pitch` apart); columns past `width`
+// become zero
+extern "C" int sb_token_gate(const void* z, long long slab, int slabs, int z_f32, const long long* ids, const void* table,
+                             long long pitch, int vocab, int column, int width, void* out, int rows, int I, int f32,
+                             cudaStream_t stream) {
+  if (rows <= 0 || I <= 0) return 0;
+  if (slabs < 1 || (f32 && !z_f32) || (slabs > 1 && !z_f32) || width < 1 || width > I || column < 0 || column + width > pitch)
+    return -3;
+  using B = __nv_bfloat16;
+  const int V = f32 || z_f32 ? 4 : 8;
+  const bool vec = width == I && I % V == 0 && column % V == 0 && pitch % V == 0 &&
+                   (((uintptr_t)z | (uintptr_t)table | (uintptr_t)out) & 15) == 0;
+  const int grid = grid_for((long long)rows * I / (vec ? V : 1), 128);
+#define SB_GATE(XT, T, VV) \
+  token_gate_kernel<XT, T, VV><<<grid, 128, 0, stream>>>((const XT*)z, slab, slabs, ids, (const T*)table, pitch, vocab, column, width, (T*)out, rows, I)
+  if (f32) {
+    if (vec) SB_GATE(float, float, 4);
+    else SB_GATE(float, float, 1);
+  } else if (z_f32) {
+    if (vec) SB_GATE(float, B, 4);
+    else SB_GATE(float, B, 1);
+  } else {
+    if (vec) SB_GATE(B, B, 8);
+    else SB_GATE(B, B, 1);
+  }
+#undef SB_GATE
   return (int)cudaGetLastError();
 }

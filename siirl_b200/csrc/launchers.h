@@ -33,7 +33,7 @@ int sb_moe_route_topk(const void* logits, int is_bf16, int ld, float* w, int* id
                       cudaStream_t stream);
 int sb_moe_route_grouped(const float* z, long long slab, int slabs, int ld, const void* corr, int corr_f32, float* w,
                          int* idx, float* w_id, int T, int E, int experts, int k, int n_groups, int keep, float scale,
-                         cudaStream_t stream);
+                         int renorm, cudaStream_t stream);
 int sb_moe_route_topk_bwd(const void* logits, int is_bf16, int ld, const int* idx, const float* dw, float* dlogits,
                           int T, int E, int k, int norm, cudaStream_t stream);
 int sb_moe_build_layout(const int* idx, int P, int E, int world, int rank, int T, int k, int capacity,

@@ -577,7 +577,7 @@ __global__ void __launch_bounds__(256) moe_route_grouped_kernel(const float* __r
                                                                 const void* __restrict__ corr, int corr_f32,
                                                                 float* __restrict__ w, int* __restrict__ idx,
                                                                 float* __restrict__ w_id, int Tn, int E, int experts, int k,
-                                                                int n_groups, int keep, float scale) {
+                                                                int n_groups, int keep, float scale, int renorm) {
   const int lane = threadIdx.x & 31, warps = (gridDim.x * blockDim.x) >> 5, size = E / n_groups;
   for (int t = (blockIdx.x * blockDim.x + threadIdx.x) >> 5; t < Tn; t += warps) {
     float s[PL], c[PL];
@@ -609,7 +609,7 @@ __global__ void __launch_bounds__(256) moe_route_grouped_kernel(const float* __r
       s[i] /= sum;
       c[i] = -INFINITY;
       if (e < E)
-        c[i] = s[i] + (corr_f32 ? reinterpret_cast<const float*>(corr)[e]
+        c[i] = !corr ? s[i] : s[i] + (corr_f32 ? reinterpret_cast<const float*>(corr)[e]
                                 : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(corr)[e]));
     }
     // largest of the outputs whose bit in `open` is set; ties go to the lower output
@@ -661,7 +661,7 @@ __global__ void __launch_bounds__(256) moe_route_grouped_kernel(const float* __r
         my_id = id;
       }
     }
-    my_w = my_w / (total + 1e-20f) * scale;
+    my_w = (renorm ? my_w / (total + 1e-20f) : my_w) * scale;
     const bool ident = lane < k && my_id >= experts;
     const float wi = warp_sum(ident ? my_w : 0.f);
     if (lane < k) {
@@ -675,7 +675,7 @@ __global__ void __launch_bounds__(256) moe_route_grouped_kernel(const float* __r
 // z: [slabs, T, ld] fp32 partial sums of E router outputs, the last E - experts of them identity experts
 extern "C" int sb_moe_route_grouped(const float* z, long long slab, int slabs, int ld, const void* corr, int corr_f32,
                                     float* w, int* idx, float* w_id, int T, int E, int experts, int k, int n_groups,
-                                    int keep, float scale, cudaStream_t stream) {
+                                    int keep, float scale, int renorm, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (E < 1 || E > 512 || experts < 1 || experts > E || n_groups < 1 || E % n_groups || keep < 1 || keep > n_groups ||
       k < 1 || k > 32 || k > keep * (E / n_groups) || slabs < 1)
@@ -683,7 +683,7 @@ extern "C" int sb_moe_route_grouped(const float* z, long long slab, int slabs, i
   const int grid = moe_grid(T);
   auto launch = [&](auto kernel) {
     kernel<<<grid, 256, 0, stream>>>(z, slab, slabs, ld, corr, corr_f32, w, idx, w_id, T, E, experts, k, n_groups, keep,
-                                     scale);
+                                     scale, renorm);
   };
   if (E <= 32) launch(moe_route_grouped_kernel<1>);
   else if (E <= 64) launch(moe_route_grouped_kernel<2>);

@@ -1,11 +1,14 @@
 // What stands between the fused projection of an attention branch and its scores, one launch: sum of the projection's
 // partial products, biases, RMS norms of queries and keys, rotation, append of keys and values to the paged cache
 // (layout in win_params.h), queries in the activation format for the attention kernels, per-head output gates.  The
-// branch's table of biases by distance is expanded from its buckets by blocks of its own.
+// branch's table of biases by distance is expanded from its buckets by blocks of its own.  Pooled runs of tokens (win_params.h):
+// the block that appends the last token of a run writes the means of its keys and values (single tokens: pool_inline); the
+// rows of a prompt portion meet in kv_pool_kernel, one launch later.
 //
 //   norm 0  none
 //   norm 1  a whole projection (all heads at once) over its root mean square times a weight vector, before the rotation
 //   norm 2  every head over its root mean square, no weight, after the rotation
+//   norm 3  every head over its root mean square times one weight vector for all heads, before the rotation
 //
 // Rotation: pairs (i, i + half) of the first 2 * half dimensions of a head turn by position * f_i.  f_i comes as two
 // floats (hi + lo) and the angle keeps its remainder, so the error does not grow with the position.
@@ -46,8 +49,12 @@ struct PrepareParams {
   const void* rel;          // [buckets, Hq] distance table of the checkpoint, or null
   const int* bucket;        // [rel_n] its row for every distance
   float* rel_out;           // [Hq, rel_n]
+  float rot_mag;            // factor of cosines and sines
+  int pool;                 // tokens per pooled run; 0: none
+  const int* pool_table;    // [slots, pool_blocks] blocks of the pooled entries
+  int pool_blocks, pool_inline;      // pool_inline: no two rows belong to one sequence
 };
-static_assert(sizeof(PrepareParams) == 216, "PrepareParams is mirrored from Python");
+static_assert(sizeof(PrepareParams) == 240, "PrepareParams is mirrored from Python");
 
 constexpr int kPrepBlk = 64;        // tokens per cache block
 constexpr int kPrepThreads = 128;
@@ -95,8 +102,57 @@ __device__ __forceinline__ void prepare_gates(const PrepareParams& p, int t, int
     const float n = (float)pos, a = n * p.freq[2 * i], lo = fmaf(n, p.freq[2 * i], -a) + n * p.freq[2 * i + 1];
     float s, c;
     sincosf(a, &s, &c);
-    s_cos[i] = fmaf(-s, lo, c);
-    s_sin[i] = fmaf(c, lo, s);
+    s_cos[i] = fmaf(-s, lo, c) * p.rot_mag;
+    s_sin[i] = fmaf(c, lo, s) * p.rot_mag;
+  }
+}
+
+// the run that ends at `pos` of the sequence in `slot`: means of its keys and values as the cache holds them, by all threads
+// of a block.  V elements per access.
+template <typename T, int V>
+__device__ __forceinline__ void pool_run(const PrepareParams& p, int slot, int pos) {
+  const int e = pos / p.pool, first = pos + 1 - p.pool;
+  if (e / kPrepBlk >= p.pool_blocks || pos / kPrepBlk >= p.max_blocks) return;
+  const int to = p.pool_table[(size_t)slot * p.pool_blocks + e / kPrepBlk];
+  if (to < 0 || to >= p.num_blocks) return;
+  const int* bt = p.block_table + (size_t)slot * p.max_blocks;
+  T* cache = reinterpret_cast<T*>(p.cache);
+  const int nk = p.Hkv * p.dk / V, n = p.Hkv * (p.dk + p.dv) / V;
+  const float inv = 1.f / (float)p.pool;
+  for (int i = threadIdx.x; i < n; i += blockDim.x) {
+    const bool key = i < nk;
+    const int d = key ? p.dk : p.dv, at = (key ? i : i - nk) * V, head = at / d;
+    const size_t base = (key ? 0 : (size_t)p.Hkv * kPrepBlk * p.dk) + (size_t)head * kPrepBlk * d + (at - head * d);
+    float sum[V] = {};
+    // the blocks of a run are fetched one after the other, eight tokens of a block in flight
+    for (int j = first; j <= pos;) {
+      const int blk = bt[j / kPrepBlk], stop = min(pos + 1, (j / kPrepBlk + 1) * kPrepBlk);
+      if (blk < 0 || blk >= p.num_blocks) {
+        j = stop;
+        continue;
+      }
+      const T* src = cache + (size_t)blk * p.block_elems + base;
+#pragma unroll 8
+      for (; j < stop; ++j) {
+        float x[V];
+        load_vec<T, V>(src + (size_t)(j % kPrepBlk) * d, x);
+#pragma unroll
+        for (int k = 0; k < V; ++k) sum[k] += x[k];
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < V; ++k) sum[k] *= inv;
+    store_vec<T, V>(cache + (size_t)to * p.block_elems + base + (size_t)(e % kPrepBlk) * d, sum);
+  }
+}
+
+constexpr int kPoolThreads = 128;
+
+template <typename T, int V>
+__global__ void __launch_bounds__(kPoolThreads) kv_pool_kernel(const __grid_constant__ PrepareParams p) {
+  for (int t = blockIdx.x; t < p.T; t += gridDim.x) {
+    const int slot = p.seq_ids[t], pos = p.positions[t];
+    if (slot >= 0 && pos >= 0 && (pos + 1) % p.pool == 0) pool_run<T, V>(p, slot, pos);
   }
 }
 
@@ -130,7 +186,7 @@ __global__ void __launch_bounds__(512, U == 2 && !F32 ? 2 : 1) qkv_prepare_units
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int nq = p.Hq * p.dk / 8, nk = p.Hkv * p.dk / 8, nv = p.Hkv * p.dv / 8, per = p.dk / 8;      // units
   // two buffers: [nq + nk][8] weighted values (the norm's factor still to come), cosines, sines, sums of squares (norm 2)
-  const int x_len = p.half ? 8 * (nq + nk) : 0, buf_len = (x_len + 2 * p.half + (p.norm == 2 ? nq + nk : 0) + 7) / 8 * 8;
+  const int x_len = p.half ? 8 * (nq + nk) : 0, buf_len = (x_len + 2 * p.half + (p.norm >= 2 ? nq + nk : 0) + 7) / 8 * 8;
   __shared__ float red[2][2][16];
   // heads whose units are a power of two lie in aligned lanes of one warp: their sums need no shared memory
   const bool in_warp = per <= 32 && (per & (per - 1)) == 0;
@@ -205,10 +261,11 @@ __global__ void __launch_bounds__(512, U == 2 && !F32 ? 2 : 1) qkv_prepare_units
         }
     }
     prepare_gates<T>(p, t, pos, s_cos, s_sin);
-    float ssq = 0.f, ssk = 0.f;
+    float ssq = 0.f, ssk = 0.f, own[U];      // own: squares of a unit's values before weights
 #pragma unroll
     for (int u = 0; u < U; ++u) {
       const int i = tid + u * blockDim.x;
+      own[u] = 0.f;
       if (p.bias && i < nq + nk + nv) {
         float b[8];
         load_vec<T, 8>(reinterpret_cast<const T*>(p.bias) + col[u], b);
@@ -224,10 +281,12 @@ __global__ void __launch_bounds__(512, U == 2 && !F32 ? 2 : 1) qkv_prepare_units
       for (int k = 0; k < 8; ++k) ss = fmaf(v[u][k], v[u][k], ss);
       if (i < nq) ssq += ss;
       else ssk += ss;
-      if (p.norm == 2 && !in_warp) s_part[i] = ss;
-      if (p.norm == 1) {
+      own[u] = ss;
+      if (p.norm >= 2 && !in_warp) s_part[i] = ss;
+      if (p.norm == 1 || p.norm == 3) {
         float w[8];
-        load_vec<T, 8>((i < nq ? reinterpret_cast<const T*>(p.q_norm) : reinterpret_cast<const T*>(p.k_norm) - 8 * nq) + 8 * i, w);
+        const T* wp = reinterpret_cast<const T*>(i < nq ? p.q_norm : p.k_norm);
+        load_vec<T, 8>(wp + (p.norm == 3 ? 8 * (i % per) : 8 * (i < nq ? i : i - nq)), w);
 #pragma unroll
         for (int k = 0; k < 8; ++k) v[u][k] *= w[k];
       }
@@ -256,11 +315,10 @@ __global__ void __launch_bounds__(512, U == 2 && !F32 ? 2 : 1) qkv_prepare_units
     for (int u = 0; u < U; ++u) {
       const int i = tid + u * blockDim.x;
       float f = i < nq ? fq : fk;
-      if (p.norm == 2) {
+      if (p.norm >= 2) {
         float ss = 0.f;
         if (in_warp) {
-#pragma unroll
-          for (int k = 0; k < 8; ++k) ss = fmaf(v[u][k], v[u][k], ss);
+          ss = own[u];
           for (int o = per >> 1; o; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
         } else if (i < nq + nk) {
           const int h = i / per;
@@ -283,6 +341,10 @@ __global__ void __launch_bounds__(512, U == 2 && !F32 ? 2 : 1) qkv_prepare_units
       for (int k = 0; k < 8; ++k) v[u][k] *= f;
       if (i < nq) store_vec<T, 8>(reinterpret_cast<T*>(p.q_out) + (size_t)t * p.q_stride + off[u], v[u]);
       else if (crow) store_vec<T, 8>(crow + off[u] + place * p.dk, v[u]);
+    }
+    if (p.pool_inline && crow && (pos + 1) % p.pool == 0) {      // the same for the whole block
+      __syncthreads();
+      pool_run<T, 8>(p, p.seq_ids[t], pos);
     }
   }
 }
@@ -354,14 +416,14 @@ __global__ void __launch_bounds__(kPrepThreads) qkv_prepare_kernel(const __grid_
     const int kh = h - p.Hq;
     const float* x = s_x + h * p.dk;
     float f = is_q ? fq : fk;
-    if (p.norm == 2) {
+    if (p.norm >= 2) {
       float ss = 0.f;
       for (int d = lane; d < p.dk; d += 32) ss = fmaf(x[d], x[d], ss);
       f = 1.f / sqrtf(warp_sum(ss) / (float)p.dk + p.eps);
     }
     const T* w = p.norm == 1 ? (is_q ? reinterpret_cast<const T*>(p.q_norm) + h * p.dk
                                      : reinterpret_cast<const T*>(p.k_norm) + kh * p.dk)
-                             : nullptr;
+                             : (p.norm == 3 ? reinterpret_cast<const T*>(is_q ? p.q_norm : p.k_norm) : nullptr);
     T* dst = is_q ? reinterpret_cast<T*>(p.q_out) + (size_t)t * p.q_stride + (size_t)h * p.dk
                   : (crow ? crow + ((size_t)kh * kPrepBlk + place) * p.dk : nullptr);
     if (!dst) continue;
@@ -389,6 +451,10 @@ __global__ void __launch_bounds__(kPrepThreads) qkv_prepare_kernel(const __grid_
         *reinterpret_cast<float2*>(dst + d0) = make_float2(o[0], o[1]);
       }
     }
+  }
+  if (p.pool_inline && crow && (pos + 1) % p.pool == 0) {
+    __syncthreads();
+    pool_run<T, V>(p, p.seq_ids[t], pos);
   }
 }
 
@@ -426,7 +492,7 @@ static int launch_prepare_units(const PrepareParams& p, cudaStream_t s) {
   auto kernel = qkv_prepare_units_kernel<T, U, F32>;
   const int qk = (p.Hq + p.Hkv) * p.dk, units = (qk + p.Hkv * p.dv) / 8;
   const int threads = ((units + U - 1) / U + 31) / 32 * 32;
-  const size_t smem = 8 * (((size_t)(p.half ? qk : 0) + 2 * (size_t)p.half + (p.norm == 2 ? qk / 8 : 0) + 7) / 8 * 8);
+  const size_t smem = 8 * (((size_t)(p.half ? qk : 0) + 2 * (size_t)p.half + (p.norm >= 2 ? qk / 8 : 0) + 7) / 8 * 8);
   static size_t configured = 48 * 1024;
   const int r = prepare_configure(kernel, smem, configured);
   if (r) return r;
@@ -455,8 +521,8 @@ extern "C" int sb_qkv_prepare(const void* params, int f32, cudaStream_t stream) 
   const PrepareParams& p = *reinterpret_cast<const PrepareParams*>(params);
   if (p.T <= 0) return 0;
   if (p.Hkv < 1 || p.Hq % p.Hkv || p.dk < 1 || p.dv < 1 || 2 * p.half > p.dk || p.slabs < 1 || (p.slabs > 1 && !p.x_f32) ||
-      (p.norm == 1 && !(p.q_norm && p.k_norm)) || (p.half && !p.freq) || (p.g_off >= 0 && !p.gate_out) ||
-      (p.rel && !(p.bucket && p.rel_out)))
+      ((p.norm == 1 || p.norm == 3) && !(p.q_norm && p.k_norm)) || (p.half && !p.freq) || (p.g_off >= 0 && !p.gate_out) ||
+      (p.rel && !(p.bucket && p.rel_out)) || p.norm < 0 || p.norm > 3 || p.pool < 0 || (p.pool && !(p.pool_table && p.pool_blocks > 0)))
     return -3;
   const int V = f32 ? 4 : 8;
   const bool vec = p.dk % V == 0 && p.dv % V == 0 && p.row_stride % V == 0 && p.slab % V == 0 && p.q_off % V == 0 &&
@@ -467,4 +533,22 @@ extern "C" int sb_qkv_prepare(const void* params, int f32, cudaStream_t stream) 
   }
   if (f32) return vec ? launch_prepare<float, 4>(p, stream) : launch_prepare<float, 1>(p, stream);
   return vec ? launch_prepare<__nv_bfloat16, 8>(p, stream) : launch_prepare<__nv_bfloat16, 1>(p, stream);
+}
+
+// The pooled runs that end among the rows of prompt portions (their keys and values are in the cache): same arguments
+extern "C" int sb_kv_pool(const void* params, int f32, cudaStream_t stream) {
+  const PrepareParams& p = *reinterpret_cast<const PrepareParams*>(params);
+  if (p.T <= 0) return 0;
+  if (p.pool < 1 || !p.pool_table || p.pool_blocks < 1 || p.Hkv < 1 || p.dk < 1 || p.dv < 1) return -3;
+  const int V = f32 ? 4 : 8;
+  const bool vec = p.dk % V == 0 && p.dv % V == 0 && p.block_elems % V == 0;
+  const int most = num_sms() * 16, grid = p.T < most ? p.T : most;
+  if (f32) {
+    if (vec) kv_pool_kernel<float, 4><<<grid, kPoolThreads, 0, stream>>>(p);
+    else kv_pool_kernel<float, 1><<<grid, kPoolThreads, 0, stream>>>(p);
+  } else {
+    if (vec) kv_pool_kernel<__nv_bfloat16, 8><<<grid, kPoolThreads, 0, stream>>>(p);
+    else kv_pool_kernel<__nv_bfloat16, 1><<<grid, kPoolThreads, 0, stream>>>(p);
+  }
+  return (int)cudaGetLastError();
 }

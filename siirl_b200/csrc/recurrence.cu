@@ -31,31 +31,9 @@
 // bf16 as projected; accumulation is fp32.
 #include "common.cuh"
 #include "launchers.h"
-#include "typed.cuh"
+#include "recurrence.cuh"
 
 namespace sb {
-
-enum { kGateChannel = 0, kGateHead = 1 };
-constexpr int kChunk = 16;
-constexpr float kLog2e = 1.4426950408889634f;
-
-struct RecParams {
-  const void* x;               // projected rows [T, row_stride]
-  long long row_stride;
-  int q_off, k_off, v_off, g_off;
-  int e_off, f_off;            // kGateChannel: low-rank row at e_off; kGateHead: i_pre at e_off, f_pre at f_off (per head)
-  int kind, rank, norm_per_head, gate_act;   // gate_act: 0 SiLU, 1 sigmoid
-  const void* w2;              // [H * dk, rank]
-  const void* b_e;             // kGateChannel: [H * dk]; kGateHead: input-gate bias [H]
-  const void* b_f;             // kGateHead: forget-gate bias [H]
-  const void* norm_w;
-  float inv_tau, cap, q_scale, eps, out_scale;
-  float* S;
-  float* m;
-  void* out;                   // [T, out_stride], this branch at column out_off
-  long long out_stride;
-  int out_off, H, dk, dv;
-};
 
 __device__ __forceinline__ float log_sigmoid(float x) {
   return x >= 0.f ? -log1pf(expf(-x)) : x - log1pf(expf(x));
@@ -64,19 +42,6 @@ __device__ __forceinline__ float log_sigmoid(float x) {
 __device__ __forceinline__ float log2_sigmoid(float x) {
   return fminf(x, 0.f) * 1.4426950408889634f - log2f(1.f + __expf(-fabsf(x)));
 }
-__device__ __forceinline__ float ex2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-__device__ __forceinline__ float gate_value(float g, int act) {
-  const float s = 1.f / (1.f + expf(-g));
-  return act == 0 ? g * s : s;
-}
-__device__ __forceinline__ float fast_gate(float g, int act) {
-  const float s = __fdividef(1.f, 1.f + __expf(-g));
-  return act == 0 ? g * s : s;
-}
 template <typename T>
 __device__ __forceinline__ void head_gates(const RecParams& p, const T* xr, int h, float& i, float& f) {
   const float zi = to_float(xr[p.e_off + h]) + to_float(reinterpret_cast<const T*>(p.b_e)[h]);
@@ -84,8 +49,6 @@ __device__ __forceinline__ void head_gates(const RecParams& p, const T* xr, int 
   i = p.cap * tanhf(zi / p.cap);
   f = log_sigmoid(p.cap * tanhf(zf / p.cap));
 }
-
-constexpr int kStepThreads = 256;
 
 // V: key channels per access (4 when dk is a multiple of 4)
 template <typename T, int V>
@@ -269,20 +232,8 @@ gate_scan_kernel(RecParams p, const int* __restrict__ row0, const int* __restric
 // ---------------------------------------------------------------------------------------
 // chunk tiles
 // ---------------------------------------------------------------------------------------
-// key channels padded to a width the scan is compiled for: 16, 32, 48, 64, 96 or 128
-__host__ __device__ inline int pad_dk(int dk) { return dk <= 64 ? (dk + 15) / 16 * 16 : (dk + 31) / 32 * 32; }
-__host__ __device__ inline int tile_row(int dkp) { return dkp + 8; }        // bf16 elements per row of a q / k tile
-constexpr int kARow = 24;                                                    // and of the score matrix
 __host__ __device__ inline int tile_bytes(int dkp) {
   return 4 * kChunk * tile_row(dkp) * 2 + 2 * kChunk * kARow * 2 + dkp * 4;
-}
-
-// x and y as two bf16 terms each: x = hi + lo to 16 mantissa bits
-__device__ __forceinline__ void split_pair(float x, float y, uint32_t& hi, uint32_t& lo) {
-  const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
-  const float2 f = __bfloat1622float2(h);
-  hi = *reinterpret_cast<const uint32_t*>(&h);
-  lo = pack_bf16x2(x - f.x, y - f.y);
 }
 
 constexpr int kPrepThreads = 128;
@@ -468,26 +419,6 @@ chunk_prepare_kernel(RecParams p, const int* __restrict__ chunk_row, const int* 
 //   segment_states_kernel  the start state of every segment, element by element along the segments
 //   pass 1  every segment from its start state: outputs; the last one leaves the state in the slot
 // ---------------------------------------------------------------------------------------
-__device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void ldsm_x4_t(uint32_t (&r)[4], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void mma_16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void copy16(void* dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
-}
-__device__ __forceinline__ void copy_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void copy_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
-
 constexpr int kScanMaxWarps = 12;
 constexpr int kScanStages = 3;
 
@@ -948,8 +879,6 @@ static int launch_chunks(const RecParams& p, const Segments& sg, int n_seg, cons
 }  // namespace sb
 
 using namespace sb;
-
-static_assert(sizeof(RecParams) == 160, "RecParams is mirrored by a ctypes structure in ops/recurrence.py");
 
 // One token (row0 / nrow null: row s of sequence s) or a packed portion per sequence, any sizes.  `params` is a host
 // RecParams.  slots[s] < 0: idle, its output rows are zero.

@@ -6,7 +6,9 @@
 // Query position i sees key position j when j <= i and (window == 0 or i - j < window or j < keep_first);
 // score = q . k * scale - slope_h * (i - j), slope_h = 2^(-bias_exp (h + 1) / Hq) (bias_exp == 0: no bias), or with a
 // soft cap and / or a table of distances cap * tanh(q . k * scale / cap) + rel[h, min(i - j, rel_n - 1)].  With a sink the
-// soft-max sum has one more term, of score 0 and without a value.
+// soft-max sum has one more term, of score 0 (or sink_w[h]) and without a value.
+// pool = P > 0 (with a window): i also sees the whole runs of P tokens before its window, run b when (b + 1) P - 1 <= i -
+// window, as one key and one value each, entry b at row b % 64 of cache block pool_table[slot, b / 64].
 #pragma once
 #include "common.cuh"
 
@@ -35,12 +37,21 @@ struct WinParams {
   const float* rel;         // [Hq, rel_n] bias by distance, or null (bias_exp must be 0 then)
   long long rel_n;
   const float* head_gate;   // [T, Hq]: the result is multiplied by it, or null
+  int pool, pool_blocks;    // 0: none; columns of pool_table
+  const int* pool_table;    // [slots, pool_blocks]
+  const void* sink_w;       // [Hq] scores of the sink in the activation format, or null
 };
 // kPaged: as described above.  kPackedRows (prompts): `cache` is [num_blocks, block_elems], one row per KEY, keys of all
 // heads before values, and a tile's slot is the row of its sequence's first key.  kLatent (general kernel): keys and
 // values are the same dk-wide rows, [num_blocks, 64, dk].
 enum { kPaged = 0, kPackedRows = 1, kLatent = 2 };
-static_assert(sizeof(WinParams) == 200, "WinParams is mirrored from Python");
+static_assert(sizeof(WinParams) == 224, "WinParams is mirrored from Python");
+
+// pooled entries a query at position i sees
+__host__ __device__ __forceinline__ int pooled_entries(int i, int window, int pool) {
+  const int n = i - window + 1;      // tokens before the window
+  return pool > 0 && n > 0 ? n / pool : 0;
+}
 
 // soft cap in units of log 2 of a raw product x: 2 * log2(e) * scale / cap * x is the exponent's argument
 struct ScoreCap {

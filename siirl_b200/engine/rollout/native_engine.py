@@ -15,7 +15,9 @@ Scheduling model
   per slot (32-bit, ``model.new_states``).  A prompt that starts at position 0 overwrites its slot's state, samples of
   one prompt copy it, and the prefix cache is off for them (a block of keys does not carry the state that led there).
   When every attention layer has a sliding window, blocks that left all windows go back to the allocator while their
-  sequence is still running.
+  sequence is still running.  Layers that pool tokens before their window keep the pooled entries in blocks of the same
+  allocator under a second table (``pool_table``, wide enough for the smallest pool); a block that is full when a prompt
+  ends is shared by its samples, the others are copied, and the prefix cache is off.
 * Slots of the running batch are fixed-size (``max_num_seqs`` rounded to the captured batch sizes); empty slots
   have context length 0 and are skipped by the kernels.
 """
@@ -74,6 +76,7 @@ class _Seq:
     generated: int = 0
     prefilled: int = 0          # prompt tokens whose K/V are in the cache (first sample of a group)
     hidden_until: int = 0       # blocks below this index have been checked for leaving every window
+    pool_blocks: List[int] = field(default_factory=list)        # blocks of pooled entries
 
 
 class BlockAllocator:
@@ -173,7 +176,8 @@ class RolloutEngine:
         self.visible_span = hybrid.visible_span() if hybrid is not None else None
         if hybrid is not None and lockstep_group is not None:
             raise ValueError("hybrid decoders have no expert layers: no lock-step group")
-        if self.recurrent:
+        self.pools = hybrid.pools() if hybrid is not None else []
+        if self.recurrent or self.pools:
             self.enable_prefix_caching = False
         self.states: List[Dict[str, torch.Tensor]] = []      # per recurrent branch, indexed by slot
         # Device memory the engine may use for KV blocks while it is awake (the trainer's fp32 gradient buffer, idle
@@ -187,6 +191,7 @@ class RolloutEngine:
         self.max_num_seqs = max_num_seqs
         self.max_model_len = max_model_len
         self.max_blocks_per_seq = (max_model_len + BLOCK - 1) // BLOCK
+        self.max_pool_blocks = kvc.pool_blocks(max_model_len, self.pools[0]) if self.pools else 0
         self.sync_interval = max(1, sync_interval)
         self.use_cuda_graph = use_cuda_graph and self.device.type == "cuda"
         self.max_num_batched_tokens = max_num_batched_tokens
@@ -232,8 +237,8 @@ class RolloutEngine:
                 free = max(0, free - self._state_bytes(self.max_num_seqs))
                 nb = max(16, (int(free * self._mem_util) + lent) // max(self._block_bytes(), 1))
             else:
-                nb = max(16, self.max_num_seqs * self.max_blocks_per_seq)
-            nb = min(nb, self.max_num_seqs * self.max_blocks_per_seq + 8)
+                nb = max(16, self.max_num_seqs * (self.max_blocks_per_seq + self.max_pool_blocks))
+            nb = min(nb, self.max_num_seqs * (self.max_blocks_per_seq + self.max_pool_blocks) + 8)
         # one tensor per layer [nb, 2, Hkv, 64, D] (hybrid decoders: [nb, elements of a block]): the first layers live
         # in the borrowed buffer, the rest is new
         elems = self._layer_elems()
@@ -267,6 +272,8 @@ class RolloutEngine:
         self.states = []                # the old ones go before the new ones come
         self.states = self.model.new_states(S) if self.recurrent else []
         self.block_table = torch.full((S, self.max_blocks_per_seq), -1, dtype=torch.int32, device=dev)
+        # a table of one column at least: kernels get its address
+        self.pool_table = torch.full((S, max(1, self.max_pool_blocks)), -1, dtype=torch.int32, device=dev)
         self.ctx_len = torch.zeros(S, dtype=torch.int32, device=dev)       # tokens in the cache
         self.last_token = torch.zeros(S, dtype=torch.int64, device=dev)
         self.finished = torch.ones(S, dtype=torch.bool, device=dev)
@@ -334,7 +341,9 @@ class RolloutEngine:
         return hidden.index_select(0, last)
 
     def _state_kw(self) -> dict:
-        return {"states": self.states} if self.cfg.hybrid is not None else {}
+        if self.cfg.hybrid is None:
+            return {}
+        return {"states": self.states, **({"pool_table": self.pool_table} if self.pools else {})}
 
     # ---- sequences' places -----------------------------------------------------------------------
     def _reset_slots(self) -> None:
@@ -343,18 +352,32 @@ class RolloutEngine:
         self.remaining.zero_()
         self.rope_delta.zero_()
         self.block_table.fill_(-1)
+        self.pool_table.fill_(-1)
 
     def _write_block_tables(self, seqs: Sequence[_Seq]) -> None:
         bt = self.block_table.cpu()
         for seq in seqs:
             bt[seq.slot, : len(seq.blocks)] = torch.tensor(seq.blocks, dtype=torch.int32)
         self.block_table.copy_(bt)
+        if self.pools:
+            pt = self.pool_table.cpu()
+            for seq in seqs:
+                pt[seq.slot, : len(seq.pool_blocks)] = torch.tensor(seq.pool_blocks, dtype=torch.int32)
+            self.pool_table.copy_(pt)
+
+    def _clear_tables(self, slot: int) -> None:
+        self.block_table[slot].fill_(-1)
+        self.pool_table[slot].fill_(-1)
+
+    def _pool_blocks_needed(self, tokens: int) -> int:
+        """Blocks of pooled entries of a sequence of ``tokens`` tokens."""
+        return kvc.pool_blocks(tokens, self.pools[0]) if self.pools else 0
 
     def _release_blocks(self, seq: _Seq) -> None:
-        for b in seq.blocks:
+        for b in seq.blocks + seq.pool_blocks:
             if b >= 0:
                 self.alloc.release(b)
-        seq.blocks = []
+        seq.blocks, seq.pool_blocks = [], []
 
     def _release_hidden_blocks(self, seq: _Seq, next_pos: int) -> None:
         """Give back the blocks of ``seq`` that no layer looks at from position ``next_pos`` on."""
@@ -565,7 +588,11 @@ class RolloutEngine:
                         if b is None:
                             break
                         hit.append(b)
+                # blocks of pooled entries that are full, for every layer's pool, when the prompt ends are shared too
+                pooled = self._pool_blocks_needed(len(p) + R)
+                pool_full = len(p) // (self.pools[-1] * BLOCK) if self.pools else 0
                 need = blocks_needed(len(p)) - len(hit) + (sp.n - 1) * (blocks_needed(len(p)) - full)
+                need += pooled + (sp.n - 1) * (pooled - pool_full)
                 todo = len(p) - len(hit) * BLOCK
                 if len(free_slots) < sp.n or self.alloc.num_free < need or (
                         not chunked and jobs and todo > budget):
@@ -582,7 +609,10 @@ class RolloutEngine:
                 first.blocks = hit + [self.alloc.alloc() for _ in range(blocks_needed(len(p)) - len(hit))]
                 first.prefilled = len(hit) * BLOCK
                 self.stats["prefix_cache_hit_tokens"] = self.stats.get("prefix_cache_hit_tokens", 0) + first.prefilled
+                first.pool_blocks = [self.alloc.alloc() for _ in range(pooled)]
                 for other in group[1:]:
+                    other.pool_blocks = [self.alloc.share(b) for b in first.pool_blocks[:pool_full]] + \
+                        [self.alloc.alloc() for _ in range(pooled - pool_full)]
                     other.blocks = [self.alloc.share(b) for b in first.blocks[:full]]
                     for j in range(full, len(first.blocks)):
                         other.blocks.append(self.alloc.alloc())
@@ -619,6 +649,9 @@ class RolloutEngine:
                     full = plen // BLOCK
                     if plen % BLOCK:
                         forks += [(lead.blocks[full], other.blocks[full]) for other in group[1:]]
+                    if self.pools:
+                        held = range(plen // (self.pools[-1] * BLOCK), self._pool_blocks_needed(plen))
+                        forks += [(lead.pool_blocks[j], other.pool_blocks[j]) for other in group[1:] for j in held]
                     if self.recurrent:
                         state_forks += [(lead.slot, other.slot) for other in group[1:]]
                     if use_cache:
@@ -690,7 +723,7 @@ class RolloutEngine:
                     retire(slot, "stop" if eos_cpu[slot] else "length", gen_cpu[slot])
                     self.ctx_len[slot] = 0
                     self.gen_index[slot] = 0
-                    self.block_table[slot].fill_(-1)
+                    self._clear_tables(slot)
         return [results[k] for k in sorted(results)]
 
     def cache_utilization(self) -> float:

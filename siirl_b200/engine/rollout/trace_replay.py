@@ -47,10 +47,12 @@ class TraceReplay:
         need = (tokens + BLOCK - 1) // BLOCK
         if need > self.engine.max_blocks_per_seq:
             raise ValueError(f"{tokens} tokens exceed the engine's max_model_len {self.engine.max_model_len}")
-        before = len(seq.blocks)
+        before = len(seq.blocks), len(seq.pool_blocks)
         while len(seq.blocks) < need:
             seq.blocks.append(self.engine.alloc.alloc())
-        return len(seq.blocks) != before
+        while len(seq.pool_blocks) < self.engine._pool_blocks_needed(tokens):
+            seq.pool_blocks.append(self.engine.alloc.alloc())
+        return (len(seq.blocks), len(seq.pool_blocks)) != before
 
     @torch.no_grad()
     def step(self, entries: Sequence[Tuple[str, Sequence[int], Sequence[int]]]) -> torch.Tensor:
@@ -111,7 +113,7 @@ class TraceReplay:
         for rid in rids:
             seq = self.live.pop(rid)
             self.engine._release_blocks(seq)
-            self.engine.block_table[seq.slot].fill_(-1)
+            self.engine._clear_tables(seq.slot)
             self.free.append(seq.slot)
 
 
@@ -126,6 +128,9 @@ def load_engine(path: str, dtype: torch.dtype, max_tokens: int, slots: int = 16,
         p.requires_grad_(False)
     # every live request may end in a partly filled block
     blocks = (max_tokens + BLOCK - 1) // BLOCK + 64 + slots
+    pools = cfg.hybrid.pools() if cfg.hybrid is not None else []
+    if pools:       # one more entry per run of tokens, in blocks that may be partly filled too
+        blocks += max_tokens // (pools[0] * BLOCK) + 1 + slots
     return RolloutEngine(model, max_num_seqs=slots, max_model_len=max_tokens + BLOCK, num_blocks=blocks)
 
 

@@ -98,11 +98,11 @@ class PrismaticConfig:
 
 @dataclass
 class MixerBranch:
-    """One token mixer of a hybrid layer.  ``kind``: "attention" (paged cache, sliding window with kept first tokens,
-    linear or learned distance bias, rotation, query / key norms, soft-capped scores, a sink without value, gated heads),
-    "latent_attention" (paged cache of one compressed row per token, from which every head's keys
-    and values are expanded), "gated_linear" (matrix state, decay per key channel) or "matrix_memory" (stabilised
-    mLSTM)."""
+    """One token mixer of a hybrid layer.  ``kind``: "attention" (paged cache, sliding window with kept first tokens or with
+    pooled blocks before it, linear or learned distance bias, rotation, query / key norms, soft-capped scores, a sink
+    without value, gated heads), "latent_attention" (paged cache of one compressed row per token, from which every head's
+    keys and values are expanded), "gated_linear" (matrix state, decay per key channel), "matrix_memory" (stabilised mLSTM)
+    or "general_delta" (matrix state, decay and removal rate per key channel)."""
     kind: str = "attention"
     heads: int = 4
     dim: int = 32                   # query / key width of a head
@@ -113,30 +113,35 @@ class MixerBranch:
     scale: float = 0.0
     window: int = 0                 # 0: no limit
     keep_first: int = 0
+    pool: int = 0                   # tokens per pooled block: whole blocks before the window are seen as their mean; 0: none
     bias_exp: float = 8.0           # slope of head h: 2^(-bias_exp (h + 1) / heads); 0: no bias
     proj_bias: bool = False         # biases on the projections of queries, keys, values and on the output matrix
     qk_norm: str = ""               # "rows": RMS norm with weights over a whole projection, before the rotation;
-                                    # "heads": every head over its root mean square, after the rotation
+                                    # "heads": every head over its root mean square, after the rotation;
+                                    # "head_weights": every head, with one weight vector for all, before the rotation
     rot_dims: int = 0               # rotated dimensions of a head (first half against second half); 0: no rotation
     rot_base: float = 1e4
-    rot_scaling: Optional[Dict[str, Any]] = None     # factor, low, high, original: three-band scaling of frequencies
+    rot_scaling: Optional[Dict[str, Any]] = None     # factor, low, high, original: three-band scaling of frequencies;
+                                                     # factor, original, fast, slow: YaRN
     softcap: float = 0.0            # score -> softcap * tanh(score / softcap); 0: none
     sink: bool = False              # one more key with score 0 and no value
+    sink_weight: bool = False       # likewise with a learned score per head
+    key_values: bool = False        # the values are the keys as projected
     rel_rows: int = 0               # rows of a learned distance table (the checkpoint's tensor shape); 0: none
     rel_max: int = 0                # distance from which its last row is used
     head_gate: bool = False         # heads times the sigmoid of one number each, projected from the mixer's input
     # latent_attention (with ``scale``)
     kv_rank: int = 0                # width of the cached row
     output_gate: bool = False       # heads times the sigmoid of a projection of the mixer's input
-    # gated_linear
-    tau: float = 16.0
+    # gated_linear, general_delta
+    tau: float = 16.0               # "gated_linear" only
     rank: int = 0                   # width of the decay's low-rank bottleneck (the checkpoint's tensor shape)
     # matrix_memory
     gate_cap: float = 15.0
 
     @property
     def recurrent(self) -> bool:
-        return self.kind in ("gated_linear", "matrix_memory")
+        return self.kind in ("gated_linear", "matrix_memory", "general_delta")
 
     def paged(self) -> Optional[tuple]:
         """(kv heads, key width, value width) of what the branch keeps in the paged cache, or ``None``."""
@@ -147,9 +152,9 @@ class MixerBranch:
 
 @dataclass
 class ExpertSpec:
-    """Routed feed-forward: gated experts, of which every token takes the ``top`` best by soft-max score plus correction
-    among the ``keep`` best of ``groups`` equal groups of neighbours; weights are the scores over their sum, times
-    ``scale``.  The last ``identity`` router outputs stand for the input itself."""
+    """Routed feed-forward: experts, of which every token takes the ``top`` best by soft-max score (plus a learned
+    correction) among the ``keep`` best of ``groups`` equal groups of neighbours; weights are the scores (over their sum),
+    times ``scale``.  The last ``identity`` router outputs stand for the input itself."""
     experts: int = 8
     ff: int = 64
     top: int = 2
@@ -159,6 +164,9 @@ class ExpertSpec:
     scale: float = 1.0
     shared_ff: int = 0              # width of an expert that takes every token; 0: none
     act: str = "silu"
+    gated: bool = True              # act(gate x) * (up x), or act(up x)
+    corrected: bool = True          # the choice adds a learned number per output
+    renormalize: bool = True        # weights over their sum
 
     @property
     def outputs(self) -> int:
@@ -190,16 +198,20 @@ class HybridSpec:
 
     ``arrangement``: "sequential" (mixer, then feed-forward on the updated stream; vector norms, gated feed-forward),
     "parallel" (both read the same stream, ``x += residual_mult * (mixer(norm1 x) + ff(norm2 x))``; norms of one number
-    each, plain feed-forward, optionally a sigmoid gate per element on each of the two results) or "hyper" (``streams``
+    each, plain feed-forward, optionally a sigmoid gate per element on each of the two results), "hyper" (``streams``
     copies of the stream: a sublayer reads a learned sum of them and every copy becomes a learned sum of all copies and
-    the sublayer's result; layer norms with biases, plain or routed feed-forward)."""
+    the sublayer's result; layer norms with biases, plain or routed feed-forward) or "sandwich" (like "sequential" with a
+    second norm on every sublayer's result, plain or routed feed-forward, and ``token_side`` columns of a second embedding
+    table per layer that enter the stream through a gate after the feed-forward)."""
     layers: List[HybridLayer] = field(default_factory=list)
     embed_scale: float = 1.0
     logit_softcap: float = 0.0      # 0: none
     norm: str = "layer_norm"        # or "rms_norm"
-    act: str = "gelu_tanh"          # or "silu", "gelu" (exact), "relu2" (square of relu)
+    act: str = "gelu_tanh"          # or "silu", "gelu" (exact), "relu2" (square of relu), "xielu" (two learned numbers)
     arrangement: str = "sequential"
     streams: int = 1                # "hyper"
+    token_side: int = 0             # "sandwich": columns per layer of the second embedding table; 0: none
+    ff_bias: bool = False           # "sandwich": biases on both matrices of the dense feed-forward
     residual_mult: float = 1.0
     residual_gate: bool = False
     loop: Optional[LayerLoop] = None
@@ -228,7 +240,12 @@ class HybridSpec:
         att = self.attention
         if any(b.window <= 0 for b in att):
             return None
-        return (max((b.window for b in att), default=1), max((b.keep_first for b in att), default=0))
+        # a pooled block is made when its last token arrives: its tokens stay until then
+        return (max((max(b.window, b.pool) for b in att), default=1), max((b.keep_first for b in att), default=0))
+
+    def pools(self) -> List[int]:
+        """Block sizes of the attention layers that keep pooled blocks."""
+        return sorted({b.pool for b in self.attention if b.pool > 0})
 
 
 @dataclass
@@ -368,6 +385,8 @@ class DecoderConfig:
         hy, W = self.hybrid, self.hidden_size
         if hy.arrangement == "hyper":
             return self._hyper_parameters()
+        if hy.arrangement == "sandwich":
+            return self._sandwich_parameters()
         parallel = hy.arrangement == "parallel"
         norm, ffs = (1, 2) if parallel else (W, 3)
         gate = W * (W + 1) if hy.residual_gate else 0
@@ -401,6 +420,26 @@ class DecoderConfig:
             if layer.moe is not None:
                 e = layer.moe
                 n += 3 * W * (e.experts * e.ff + e.shared_ff) + e.outputs * (W + 1)
+        return n
+
+    def _sandwich_parameters(self) -> int:
+        hy, W, V = self.hybrid, self.hidden_size, self.vocab_size
+        side = hy.token_side
+        n = V * W * (1 if self.tie_word_embeddings else 2) + W + V * side * len(hy.layers)
+        for layer in hy.layers:
+            n += 2 * W * (1 + int(layer.has_ff)) + (2 * W * side + W if side else 0)
+            n += 2 * W * layer.ff + (layer.ff * int(hy.ff_bias) + W * int(hy.ff_bias) + 2 * int(hy.act == "xielu")
+                                     if layer.ff else 0)
+            for b in layer.branches:
+                hk, gk, hv = b.heads * b.dim, b.kv_heads * b.dim, b.heads * b.vdim
+                if b.kind == "attention":
+                    n += W * (hk + gk + hv) + (0 if b.key_values else W * b.kv_heads * b.vdim)
+                    n += 2 * b.dim * int(b.qk_norm == "head_weights") + b.heads * int(b.sink_weight)
+                else:
+                    n += 6 * W * hk + b.rank * (W + hk) + 3 * hk
+            if layer.moe is not None:
+                e = layer.moe
+                n += (2 + int(e.gated)) * W * e.experts * e.ff + e.outputs * (W + int(e.corrected))
         return n
 
     def to_dict(self) -> Dict[str, Any]:
@@ -442,7 +481,7 @@ class DecoderConfig:
     @classmethod
     def from_hf_config(cls, cfg: Dict[str, Any]) -> "DecoderConfig":
         own = {"Domavik": cls._from_domavik_config, "Poralorn": cls._from_poralorn_config,
-               "Gumazen": cls._from_gumazen_config}
+               "Gumazen": cls._from_gumazen_config, "Rizitar": cls._from_rizitar_config}
         if cfg.get("architecture") in own:
             return own[cfg["architecture"]](cfg)
         text = cfg.get("text_config") or cfg.get("llm_config") or cfg
@@ -780,6 +819,74 @@ class DecoderConfig:
         return d
 
     @classmethod
+    def _from_rizitar_config(cls, cfg: Dict[str, Any]) -> "DecoderConfig":
+        """Rizitar: generalized delta rule or windowed attention with pooled blocks in any order, dense or routed
+        feed-forwards, norms around every sublayer, a second embedding table per layer.  The low-rank width of the decay is
+        not in the file: it is the shape of a tensor, filled in by ``from_pretrained``."""
+        layers = []
+        for x in cfg["layers"]:
+            m, mlp = x["mixer"], x.get("mlp")
+            if x["type"] == "general_delta":
+                b = MixerBranch(kind="general_delta", heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["dim"]))
+            elif x["type"] == "attention":
+                if int(m.get("vdim", m["dim"])) != int(m["dim"]):
+                    raise ValueError("attention: values that are the keys have their width")
+                mask, rot = m.get("mask") or {}, m.get("rot")
+                b = MixerBranch(kind="attention", heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]),
+                                vdim=int(m["dim"]), scale=float(m["scale"]), window=int(mask.get("size") or 0),
+                                pool=int(mask.get("pool") or 0), bias_exp=0.0, qk_norm="head_weights", sink_weight=True,
+                                key_values=True)
+                if b.pool and not b.window:
+                    raise ValueError("attention: pooled blocks need a window")
+                if rot:
+                    b.rot_dims, b.rot_base = int(rot["dims"]), float(rot["base"])
+                    b.rot_scaling = dict(rot["scaling"]) if rot.get("scaling") else None
+            else:
+                raise ValueError(f"unknown layer type {x['type']!r}")
+            layer = HybridLayer(branches=[b])
+            if mlp is not None and mlp["kind"] == "dense":
+                layer.ff = int(mlp["ff"])
+            elif mlp is not None and mlp["kind"] == "moe":
+                r = mlp["router"]
+                layer.moe = ExpertSpec(experts=int(r["experts"]), ff=int(mlp["expert"]["ff"]), top=int(r["top"]), act="relu2",
+                                       gated=False, corrected=False, renormalize=False)
+            elif mlp is not None:
+                raise ValueError(f"unknown feed-forward kind {mlp['kind']!r}")
+            layers.append(layer)
+        spec = HybridSpec(layers=layers, embed_scale=float(cfg["embedding"]["scale"]), norm="rms_norm", act="xielu",
+                          arrangement="sandwich", token_side=int((cfg.get("token_side") or {}).get("dim") or 0),
+                          ff_bias=True, hf_naming="rizitar")
+        return cls.for_hybrid(spec, vocab_size=int(cfg["vocab"]), hidden_size=int(cfg["width"]), tie_word_embeddings=True,
+                              rms_norm_eps=float(cfg["norm"]["eps"]), model_type="rizitar",
+                              eos_token_id=int(cfg.get("eos_token_id", -1)), pad_token_id=int(cfg.get("pad_token_id", 0)))
+
+    def _to_rizitar_config(self) -> Dict[str, Any]:
+        hy, layers = self.hybrid, []
+        for x in hy.layers:
+            b, = x.branches
+            if b.kind == "general_delta":
+                m: Dict[str, Any] = {"heads": b.heads, "dim": b.dim}
+            else:
+                m = {n: getattr(b, n) for n in ("heads", "kv_heads", "dim", "vdim", "scale")}
+                if b.window:
+                    m["mask"] = {"size": b.window, **({"pool": b.pool} if b.pool else {})}
+                if b.rot_dims:
+                    m["rot"] = {"base": b.rot_base, "dims": b.rot_dims}
+                    if b.rot_scaling:
+                        m["rot"]["scaling"] = dict(b.rot_scaling)
+            mlp: Optional[Dict[str, Any]] = {"kind": "dense", "ff": x.ff} if x.ff else None
+            if x.moe is not None:
+                mlp = {"kind": "moe", "expert": {"ff": x.moe.ff}, "router": {"experts": x.moe.experts, "top": x.moe.top}}
+            layers.append({"type": b.kind, "mixer": m, "mlp": mlp})
+        d = {"architecture": "Rizitar", "vocab": self.vocab_size, "width": self.hidden_size,
+             "embedding": {"scale": hy.embed_scale}, "norm": {"eps": self.rms_norm_eps}, "layers": layers}
+        if hy.token_side:
+            d["token_side"] = {"dim": hy.token_side}
+        if self.eos_token_id >= 0:
+            d["eos_token_id"] = self.eos_token_id
+        return d
+
+    @classmethod
     def from_pretrained(cls, path: str) -> "DecoderConfig":
         with open(os.path.join(os.path.expanduser(path), "config.json")) as f:
             out = cls.from_hf_config(json.load(f))
@@ -790,7 +897,8 @@ class DecoderConfig:
 
     def to_hf_config(self) -> Dict[str, Any]:
         if self.hybrid is not None:
-            return {"poralorn": self._to_poralorn_config, "gumazen": self._to_gumazen_config}.get(
+            return {"poralorn": self._to_poralorn_config, "gumazen": self._to_gumazen_config,
+                    "rizitar": self._to_rizitar_config}.get(
                 self.hybrid.hf_naming, self._to_domavik_config)()
         arch = {"qwen2": "Qwen2ForCausalLM", "qwen3": "Qwen3ForCausalLM", "qwen3_moe": "Qwen3MoeForCausalLM",
                 "llama": "LlamaForCausalLM", "qwen2_5_vl": "Qwen2_5_VLForConditionalGeneration",
@@ -935,7 +1043,34 @@ def _gumazen(n_layers: int, width: int, ff: int, vocab: int, heads: int, kv_head
     return DecoderConfig.for_hybrid(spec, vocab_size=vocab, hidden_size=width, rms_norm_eps=1e-5, model_type="gumazen", **kw)
 
 
+def _rizitar(n_layers: int, width: int, ff: int, vocab: int, att: dict, delta: dict, moe: ExpertSpec, side: int,
+             rot_base: float = 1e6, **kw) -> DecoderConfig:
+    """Rizitar layers in turn: two delta rules, then attention; the feed-forwards alternate between dense and routed."""
+    dim = att["dim"]
+    base = dict(kind="attention", vdim=dim, scale=dim ** -0.5, bias_exp=0.0, qk_norm="head_weights", sink_weight=True,
+                key_values=True, rot_dims=dim, rot_base=rot_base,
+                rot_scaling={"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0})
+    layers = [HybridLayer([MixerBranch(**base, **att) if i % 3 == 2 else
+                           MixerBranch(kind="general_delta", vdim=delta["dim"], **delta)],
+                          ff=0 if i % 2 else ff, moe=moe if i % 2 else None) for i in range(n_layers)]
+    spec = HybridSpec(layers=layers, embed_scale=width ** 0.5, norm="rms_norm", act="xielu", arrangement="sandwich",
+                      token_side=side, ff_bias=True, hf_naming="rizitar")
+    return DecoderConfig.for_hybrid(spec, vocab_size=vocab, hidden_size=width, rms_norm_eps=1e-5, model_type="rizitar",
+                                    tie_word_embeddings=True, **kw)
+
+
+def _plain_experts(experts: int, ff: int, top: int) -> ExpertSpec:
+    return ExpertSpec(experts=experts, ff=ff, top=top, act="relu2", gated=False, corrected=False, renormalize=False)
+
+
 PRESETS: Dict[str, DecoderConfig] = {
+    "tiny-rizitar": _rizitar(3, 128, 192, 1024, dict(heads=4, kv_heads=2, dim=32, window=50, pool=12),
+                             dict(heads=3, dim=24, rank=8), _plain_experts(6, 40, 2), side=16),
+    # layer sizes of decoders with about 1 / 3 billion active parameters (benchmark shapes, random weights)
+    "rizitar-a1b": _rizitar(18, 1536, 8960, 152064, dict(heads=12, kv_heads=2, dim=128, window=1024, pool=16),
+                            dict(heads=24, dim=64, rank=64), _plain_experts(64, 1024, 6), side=128),
+    "rizitar-a3b": _rizitar(18, 2048, 11264, 152064, dict(heads=32, kv_heads=4, dim=128, window=1024, pool=16),
+                            dict(heads=32, dim=64, rank=64), _plain_experts(128, 1536, 8), side=256),
     "tiny-gumazen": _gumazen(3, 128, 192, 1024, heads=4, kv_heads=2, dim=32, vdim=24, window=70, rot_dims=16,
                              moe=ExpertSpec(experts=6, ff=40, top=3, groups=2, keep=1, identity=2, scale=1.5, shared_ff=56),
                              loop=LayerLoop(1, 3, 2)),

@@ -381,7 +381,48 @@ def _gumazen_state(model) -> Iterator[Tuple[str, torch.Tensor]]:
     yield "head", model.lm_head.data
 
 
-_HYBRID_STATE = {"domavik": _domavik_state, "poralorn": _poralorn_state, "gumazen": _gumazen_state}
+def _rizitar_state(model) -> Iterator[Tuple[str, torch.Tensor]]:
+    """Rizitar checkpoint names and the views of the fused, padded parameters they fill (models/hybrid.py)."""
+    side = model.cfg.hybrid.token_side
+    yield "embed", model.embed_tokens.data
+    if side:
+        yield "side.embed", model.side_embed.data
+    for i, layer in enumerate(model.layers):
+        p, m = f"l{i}.", f"l{i}.mix."
+        for name in ("norm1", "norm1b") + (("norm2", "norm2b") if layer.has_ff else ()):
+            yield p + name, getattr(layer, name).data
+        br, = layer.branches
+        b = br.b
+        for name, (at, n) in br.cols.items():
+            yield m + name, layer.in_proj_weight.data[at:at + n]
+        yield m + "o", layer.o_proj_weight.data[:, :b.heads * b.vdim]
+        if b.kind == "attention":
+            yield m + "q.norm", br.q_norm.data
+            yield m + "k.norm", br.k_norm.data
+            yield m + "sink", br.sink.data
+        else:
+            for theirs, ours in (("a.b", "b_f"), ("w0", "b_e"), ("w2", "w2"), ("norm", "norm")):
+                yield m + theirs, getattr(br, ours).data
+        if layer.ff:
+            yield p + "mlp.up", layer.up_proj_weight.data[:layer.ff]
+            yield p + "mlp.up.b", layer.up_proj_bias.data[:layer.ff]
+            yield p + "mlp.down", layer.down_proj_weight.data[:, :layer.ff]
+            yield p + "mlp.down.b", layer.down_proj_bias.data
+            yield p + "mlp.act", layer.act_numbers.data
+        if layer.moe is not None:
+            x, e = layer.moe, layer.moe.spec
+            yield p + "mlp.router", x.router_weight.data[:e.outputs]
+            for j in range(e.experts):
+                yield p + f"mlp.e{j}.up", x.up_weight.data[j, :e.ff]
+                yield p + f"mlp.e{j}.down", x.down_weight.data[j, :, :e.ff]
+        if side:
+            yield p + "side.gate", layer.side_gate_weight.data[:side]
+            yield p + "side.proj", layer.side_proj_weight.data[:, :side]
+            yield p + "side.norm", layer.side_norm.data
+    yield "final.norm", model.norm.data
+
+
+_HYBRID_STATE = {"domavik": _domavik_state, "poralorn": _poralorn_state, "gumazen": _gumazen_state, "rizitar": _rizitar_state}
 
 
 def fill_hybrid_ranks(cfg: DecoderConfig, path: str) -> None:
@@ -390,8 +431,9 @@ def fill_hybrid_ranks(cfg: DecoderConfig, path: str) -> None:
     where = {k: h for h in handles for k in h.keys()}
     for i, layer in enumerate(cfg.hybrid.layers):
         for j, b in enumerate(layer.branches):
-            if b.kind == "gated_linear" and not b.rank:
-                name = f"l{i}.mix." + (("left.", "right.")[j] if len(layer.branches) > 1 else "") + "a1"
+            if b.kind in ("gated_linear", "general_delta") and not b.rank:
+                name = f"l{i}.mix." + (("left.", "right.")[j] if len(layer.branches) > 1 else "")
+                name += "a1" if b.kind == "gated_linear" else "w1"
                 if name not in where:
                     raise KeyError(f"{name} missing in {path}")
                 b.rank = int(where[name].get_slice(name).get_shape()[0])

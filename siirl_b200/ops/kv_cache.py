@@ -17,6 +17,11 @@ from . import lib as _lib
 BLOCK = 64
 
 
+def pool_blocks(tokens: int, pool: int) -> int:
+    """Cache blocks that hold the pooled entries (one per whole run of ``pool`` tokens) of a sequence."""
+    return (tokens // pool + BLOCK - 1) // BLOCK
+
+
 def kv_append(qkv: torch.Tensor, seq_ids: torch.Tensor, positions: torch.Tensor, block_table: torch.Tensor,
               cache_layer: torch.Tensor, n_heads: int, n_kv_heads: int, head_dim: int) -> None:
     """Write the k and v parts of every row of ``qkv`` ([T, (Hq+2Hkv)*D]) to ``cache_layer`` at

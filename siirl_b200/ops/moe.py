@@ -428,23 +428,25 @@ def route_topk(logits: torch.Tensor, top_k: int, norm_topk_prob: bool = True):
 # ---------------------------------------------------------------------------------------------
 # router with corrected, group-limited choice and identity experts; routed feed-forward of serving models
 # ---------------------------------------------------------------------------------------------
-def route_grouped(z: torch.Tensor, correction: torch.Tensor, experts: int, top: int, groups: int, keep: int, scale: float):
-    """Router logits ``z [S, T, >= E]`` (fp32 partial sums; ``E = correction.numel()`` outputs, those from ``experts`` on are
-    identity experts) -> ``(w [T, top], ids [T, top] int32, w_id [T])``.  Soft-max over all outputs; chosen by score plus
+def route_grouped(z: torch.Tensor, correction: Optional[torch.Tensor], experts: int, top: int, groups: int, keep: int,
+                  scale: float, outputs: int = 0, renormalize: bool = True):
+    """Router logits ``z [S, T, >= E]`` (fp32 partial sums; ``E = correction.numel()`` or ``outputs`` outputs, those from
+    ``experts`` on are identity experts) -> ``(w [T, top], ids [T, top] int32, w_id [T])``.  Soft-max over all outputs; chosen by score plus
     correction inside the ``keep`` groups (of ``groups`` equal groups of neighbours) with the largest best member; weights
-    are the scores of the chosen over their sum (+ 1e-20) times ``scale``.  An identity expert has id -1 and adds its
+    are the scores of the chosen, over their sum (+ 1e-20) when ``renormalize``, times ``scale``.  Without a correction the
+    scores alone choose.  An identity expert has id -1 and adds its
     weight to ``w_id``."""
-    E, T = correction.numel(), z.shape[1]
+    E, T = correction.numel() if correction is not None else outputs, z.shape[1]
     if E % groups or not 1 <= keep <= groups or top > keep * (E // groups) or not 1 <= experts <= E:
         raise ValueError(f"router: {top} of {E} outputs in {keep} of {groups} groups, {experts} experts")
     if not z.is_cuda:
         s = torch.softmax(z.float().sum(0)[:, :E], -1)
-        choice = (s + correction.float()).view(T, groups, E // groups)
+        choice = (s + correction.float() if correction is not None else s).view(T, groups, E // groups)
         best = choice.amax(-1).topk(keep, -1).indices
         hidden = torch.ones(T, groups, dtype=torch.bool).scatter_(1, best, False)
         ids = choice.masked_fill(hidden[:, :, None], float("-inf")).view(T, E).topk(top, -1).indices
         w = s.gather(1, ids)
-        w = w / (w.sum(-1, keepdim=True) + 1e-20) * scale
+        w = (w / (w.sum(-1, keepdim=True) + 1e-20) if renormalize else w) * scale
         ident = ids >= experts
         return w, torch.where(ident, torch.full_like(ids, -1), ids).to(torch.int32), (w * ident).sum(-1)
     assert z.dtype == torch.float32 and z.stride(2) == 1
@@ -453,29 +455,33 @@ def route_grouped(z: torch.Tensor, correction: torch.Tensor, experts: int, top: 
     w_id = torch.empty(T, dtype=torch.float32, device=z.device)
     _lib.check(_lib.get_lib().sb_moe_route_grouped(
         _lib.ptr(z), ctypes.c_longlong(z.stride(0)), z.shape[0], z.stride(1), _lib.ptr(correction),
-        int(correction.dtype == torch.float32), _lib.ptr(w), _lib.ptr(ids), _lib.ptr(w_id), T, E, experts, top, groups, keep,
-        ctypes.c_float(scale), _lib.stream()), "sb_moe_route_grouped")
+        int(correction is not None and correction.dtype == torch.float32), _lib.ptr(w), _lib.ptr(ids), _lib.ptr(w_id), T, E,
+        experts, top, groups, keep, ctypes.c_float(scale), int(renormalize), _lib.stream()), "sb_moe_route_grouped")
     return w, ids, w_id
 
 
-def routed_experts(x: torch.Tensor, ids: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, act: str):
-    """Gated experts on the rows each was chosen for (``ids [T, top]``, -1: nobody): ``gate_up [E, 2 I, W]``,
-    ``down [E, W, I]``.  Returns the experts' rows, sorted by expert, and the row of every (token, choice) pair (-1: none).
+def routed_experts(x: torch.Tensor, ids: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, act: str,
+                   gated: bool = True):
+    """Experts on the rows each was chosen for (``ids [T, top]``, -1: nobody): ``gate_up [E, 2 I, W]`` (not ``gated``:
+    ``[E, I, W]``), ``down [E, W, I]``.  Returns the experts' rows, sorted by expert, and the row of every (token, choice) pair (-1: none).
     One device, inference; rows of padding slots are undefined."""
-    from .rows import gated_act
+    from .rows import bias_act, gated_act
     E, W, I = down.shape
     T, k = ids.shape
     capacity = (T * k // BLOCK_ROWS + min(E, T * k)) * BLOCK_ROWS       # every expert ends in a partly filled block
     lay = build_layout(ids[None], E, 1, 0, capacity)
+
+    def activated(z):
+        return gated_act(z, act, lay.slot_src_row) if gated else bias_act(z[None], act, x.dtype, used=lay.slot_src_row)
     if not x.is_cuda:
         rows = x[lay.slot_src_row.long().clamp(min=0)]
-        return grouped_linear(gated_act(grouped_linear(rows, gate_up, lay), act), down, lay), lay.pair_slot
+        return grouped_linear(activated(grouped_linear(rows, gate_up, lay)), down, lay), lay.pair_slot
     if x.dtype == torch.bfloat16 and W % 8 == 0 and I % 8 == 0:
         rows = torch.empty(capacity, W, dtype=x.dtype, device=x.device)
         _lib.check(_lib.get_lib().sb_moe_gather_rows((ctypes.c_void_p * 1)(x.data_ptr()), 1, None, _lib.ptr(lay.slot_src_row),
                                                      None, _lib.ptr(rows), capacity, W, 1, _lib.stream()),
                    "sb_moe_gather_rows")
-        a = gated_act(grouped_linear(rows, gate_up, lay), act, lay.slot_src_row)
+        a = activated(grouped_linear(rows, gate_up, lay))
         return grouped_linear(a, down, lay), lay.pair_slot
 
     def product(a, weight, rows):       # any sizes, 32-bit: rows are fetched by the product itself
@@ -486,5 +492,5 @@ def routed_experts(x: torch.Tensor, ids: torch.Tensor, gate_up: torch.Tensor, do
             ll(weight.stride(1)), ll(out.stride(0)), _lib.ptr(lay.tile_group), _lib.ptr(rows), ll(weight.stride(0)),
             int(a.dtype == torch.float32), _lib.stream()), "sb_gemm_simt_grouped")
         return out
-    a = gated_act(product(x, gate_up, lay.slot_src_row), act, lay.slot_src_row)
+    a = activated(product(x, gate_up, lay.slot_src_row))
     return product(a, down, None), lay.pair_slot

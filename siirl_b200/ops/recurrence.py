@@ -2,18 +2,25 @@
 
     S_t = diag(a_t) S_(t-1) + w_t k_t v_t^T,    o_t = S_t^T q_t
 
-Two gate forms: ``"channel"`` (gated linear attention: ``a_t = sigmoid(W2 e_t + b)^(1 / tau)`` per key channel) and
+Three gate forms: ``"channel"`` (gated linear attention: ``a_t = sigmoid(W2 e_t + b)^(1 / tau)`` per key channel),
+``"delta"`` (generalized delta rule, below) and
 ``"head"`` (the stabilised matrix memory of xLSTM: exponential input gate, sigmoid forget gate, running maximum ``m`` and
 a normaliser that is kept as one more value column).  The output is RMS-normed per head, weighted, gated and scaled.
+
+Delta form, with the unit key ``u_t = k_t / sqrt(|k_t|^2 + 1e-6)``, decay ``a_t = exp(-e^(-1/2) sigmoid(W2 tanh(e_t) + b))``
+and removal rate ``f_t = sigmoid(f + b_f)`` per key channel:
+
+    S_t = diag(a_t) S_(t-1) - (f_t u_t) (u_t^T S_(t-1)) + k_t v_t^T,    o_t = S_t^T q_t
 
 State of a branch, all in 32-bit floats: ``S [slots, heads, vdim (+1), dim]`` and, for the head form, ``m [slots, heads]``.
 A portion that begins at position 0 starts from zero whatever its slot holds.
 
-CUDA tensors run ``csrc/recurrence.cu``: decoding and 32-bit models the token-by-token kernel, bf16 prompts the chunked
+CUDA tensors run ``csrc/recurrence.cu`` (delta form: ``csrc/delta_rule.cu``): decoding and 32-bit models the token-by-token kernel, bf16 prompts the chunked
 tensor-core kernels.  CPU tensors run the plain loop below."""
 from __future__ import annotations
 
 import ctypes
+import math
 from dataclasses import dataclass
 from typing import Dict, List, Optional, Sequence, Tuple
 
@@ -28,7 +35,7 @@ CHUNK = 16      # tokens per tile of the chunked kernels (kChunk in csrc/recurre
 @dataclass
 class RecurrenceSpec:
     """Sizes and constants of one branch; the offsets name its columns in the projected rows."""
-    gate: str                      # "channel" or "head"
+    gate: str                      # "channel", "head" or "delta"
     heads: int
     dim: int
     vdim: int
@@ -36,8 +43,8 @@ class RecurrenceSpec:
     k_off: int
     v_off: int
     g_off: int
-    e_off: int                     # "channel": low-rank row; "head": input-gate pre-activations
-    f_off: int = 0                 # "head": forget-gate pre-activations
+    e_off: int                     # "channel", "delta": low-rank row; "head": input-gate pre-activations
+    f_off: int = 0                 # "head": forget-gate pre-activations; "delta": those of the removal rates
     rank: int = 0
     tau: float = 1.0
     cap: float = 1.0
@@ -49,6 +56,10 @@ class RecurrenceSpec:
     @property
     def rows(self) -> int:
         return self.vdim + (1 if self.gate == "head" else 0)
+
+    @property
+    def q_scale(self) -> float:
+        return 1.0 if self.gate == "delta" else self.dim ** -0.5
 
     def state_shapes(self) -> Dict[str, tuple]:
         out = {"S": (self.heads, self.rows, self.dim)}
@@ -81,9 +92,10 @@ class PortionPlan:
 
     def __init__(self, lens: Sequence[int], starts: Sequence[int], slots: Sequence[int], device):
         self.lens, self.starts, self.slots = list(lens), list(starts), list(slots)
-        row0, chunk_row, chunk_len, at = [], [], [], 0
+        row0, chunk_row, chunk_len, chunk0, at = [], [], [], [], 0
         for n in self.lens:
             row0.append(at)
+            chunk0.append(len(chunk_row))
             for c in range(0, n, CHUNK):
                 chunk_row.append(at + c)
                 chunk_len.append(min(CHUNK, n - c))
@@ -92,9 +104,10 @@ class PortionPlan:
         self.device = device
         self._segments: Dict[int, Tuple[torch.Tensor, int]] = {}
         # one copy to the device: the pieces are views
-        parts = [row0, self.lens, self.slots, self.starts, chunk_row, chunk_len]
+        parts = [row0, self.lens, self.slots, self.starts, chunk_row, chunk_len, chunk0]
         flat = torch.tensor([v for p in parts for v in p], dtype=torch.int32).to(device)
-        self.row0, self.nrow, self.slot, self.pos0, self.chunk_row, self.chunk_len = flat.split([len(p) for p in parts])
+        (self.row0, self.nrow, self.slot, self.pos0, self.chunk_row, self.chunk_len,
+         self.chunk0) = flat.split([len(p) for p in parts])
 
     def segments(self, blocks: int) -> Tuple[torch.Tensor, int]:
         """Runs of chunks that work in parallel, about ``blocks`` of them in all, equal within a sequence:
@@ -120,16 +133,16 @@ class PortionPlan:
 
 def _params(spec: RecurrenceSpec, x, weights, state, out, out_off) -> _Params:
     assert x.stride(1) == 1 and out.stride(1) == 1 and state["S"].dtype == torch.float32
-    head = spec.gate == "head"
+    kinds = {"channel": 0, "head": 1, "delta": 2}
     addr = lambda t: None if t is None else t.data_ptr()  # noqa: E731
     for w in weights.values():
         assert w.dtype == x.dtype and w.is_contiguous()
     return _Params(
         x=x.data_ptr(), row_stride=x.stride(0), q_off=spec.q_off, k_off=spec.k_off, v_off=spec.v_off, g_off=spec.g_off,
-        e_off=spec.e_off, f_off=spec.f_off, kind=1 if head else 0, rank=spec.rank,
+        e_off=spec.e_off, f_off=spec.f_off, kind=kinds[spec.gate], rank=spec.rank,
         norm_per_head=int(spec.norm_per_head), gate_act=1 if spec.gate_act == "sigmoid" else 0,
         w2=addr(weights.get("w2")), b_e=addr(weights["b_e"]), b_f=addr(weights.get("b_f")),
-        norm_w=addr(weights["norm"]), inv_tau=1.0 / spec.tau, cap=spec.cap, q_scale=spec.dim ** -0.5, eps=spec.eps,
+        norm_w=addr(weights["norm"]), inv_tau=1.0 / spec.tau, cap=spec.cap, q_scale=spec.q_scale, eps=spec.eps,
         out_scale=spec.out_scale, S=state["S"].data_ptr(), m=addr(state.get("m")), out=out.data_ptr(),
         out_stride=out.stride(0), out_off=out_off, H=spec.heads, dk=spec.dim, dv=spec.vdim)
 
@@ -147,7 +160,18 @@ def recurrence_prefill(spec: RecurrenceSpec, x: torch.Tensor, weights: Dict[str,
     L = _lib.get_lib()
     p = _params(spec, x, weights, state, out, out_off)
     ref = ctypes.byref(p)
-    if x.dtype == torch.bfloat16 and not stepwise:
+    if x.dtype == torch.bfloat16 and not stepwise and spec.gate == "delta":
+        fn = L._cdll.sb_delta_workspace
+        fn.restype = ctypes.c_longlong
+        nbytes = int(fn(ref, plan.n_chunks))
+        if nbytes >= 0:
+            ws = torch.empty(max(nbytes, 16), dtype=torch.uint8, device=x.device)
+            _lib.check(L.sb_delta_prefill(
+                ref, _lib.ptr(plan.row0), _lib.ptr(plan.nrow), _lib.ptr(plan.slot), _lib.ptr(plan.pos0), plan.n_seq,
+                _lib.ptr(plan.chunk_row), _lib.ptr(plan.chunk_len), _lib.ptr(plan.chunk0), plan.n_chunks, _lib.ptr(ws),
+                _lib.stream()), "sb_delta_prefill")
+            return
+    elif x.dtype == torch.bfloat16 and not stepwise:
         fn = L._cdll.sb_recurrence_workspace
         fn.restype = ctypes.c_longlong
         segs, n_seg = plan.segments(int(L._cdll.sb_recurrence_resident(ref)) // spec.heads)
@@ -161,7 +185,8 @@ def recurrence_prefill(spec: RecurrenceSpec, x: torch.Tensor, weights: Dict[str,
             # counted as two kernels (chunk preparation or gate scan, chunk scan): segment states come on top
             _lib.add_launches(2 if n_seg > plan.n_seq else 0)
             return
-    _lib.check(L.sb_recurrence_step(ref, _lib.ptr(plan.row0), _lib.ptr(plan.nrow), _lib.ptr(plan.slot),
+    step = L.sb_delta_step if spec.gate == "delta" else L.sb_recurrence_step
+    _lib.check(step(ref, _lib.ptr(plan.row0), _lib.ptr(plan.nrow), _lib.ptr(plan.slot),
                                     _lib.ptr(plan.pos0), plan.n_seq, int(x.dtype == torch.float32), _lib.stream()),
                "sb_recurrence_step")
 
@@ -176,7 +201,8 @@ def recurrence_decode(spec: RecurrenceSpec, x: torch.Tensor, weights: Dict[str, 
         return
     L = _lib.get_lib()
     p = _params(spec, x, weights, state, out, out_off)
-    _lib.check(L.sb_recurrence_step(ctypes.byref(p), None, None, _lib.ptr(slots), _lib.ptr(positions), x.shape[0],
+    step = L.sb_delta_step if spec.gate == "delta" else L.sb_recurrence_step
+    _lib.check(step(ctypes.byref(p), None, None, _lib.ptr(slots), _lib.ptr(positions), x.shape[0],
                                     int(x.dtype == torch.float32), _lib.stream()), "sb_recurrence_step")
 
 
@@ -190,7 +216,7 @@ def _run_cpu(spec: RecurrenceSpec, x, weights, state, rows: List[List[int]], slo
             continue
         r = x[idx].float()
         n = len(idx)
-        q = r[:, spec.q_off:spec.q_off + H * dk].reshape(n, H, dk) * dk ** -0.5
+        q = r[:, spec.q_off:spec.q_off + H * dk].reshape(n, H, dk) * spec.q_scale
         k = r[:, spec.k_off:spec.k_off + H * dk].reshape(n, H, dk)
         v = r[:, spec.v_off:spec.v_off + H * dv].reshape(n, H, dv)
         g = r[:, spec.g_off:spec.g_off + H * dv]
@@ -201,6 +227,15 @@ def _run_cpu(spec: RecurrenceSpec, x, weights, state, rows: List[List[int]], slo
             a = torch.exp(F.logsigmoid(z) / spec.tau).reshape(n, H, 1, dk)
             for t in range(n):
                 S = S * a[t] + v[t][:, :, None] * k[t][:, None, :]
+                o[t] = torch.einsum("hvd,hd->hv", S, q[t])
+        elif spec.gate == "delta":
+            z = torch.tanh(r[:, spec.e_off:spec.e_off + spec.rank]) @ weights["w2"].float().t() + weights["b_e"].float()
+            a = torch.exp(-math.exp(-0.5) * torch.sigmoid(z)).reshape(n, H, 1, dk)
+            f = torch.sigmoid(r[:, spec.f_off:spec.f_off + H * dk] + weights["b_f"].float()).reshape(n, H, dk)
+            u = k * torch.rsqrt(k.pow(2).sum(-1, keepdim=True) + 1e-6)
+            for t in range(n):
+                seen = torch.einsum("hvd,hd->hv", S, u[t])
+                S = S * a[t] - seen[:, :, None] * (f[t] * u[t])[:, None, :] + v[t][:, :, None] * k[t][:, None, :]
                 o[t] = torch.einsum("hvd,hd->hv", S, q[t])
         else:
             i = spec.cap * torch.tanh((r[:, spec.e_off:spec.e_off + H] + weights["b_e"].float()) / spec.cap)

@@ -1,6 +1,6 @@
 """Row operations of decoders with a 32-bit residual stream (``csrc/hybrid_ops.cu``): scaled embedding, residual add fused
-with the following norm, gated residual update of two sublayers, entry of a layer loop's pass, activations, soft-capped
-logits.  Inference only; CPU tensors use the plain statements."""
+with the following norm (and with the norm of what is added), gated residual update of two sublayers, entry of a layer
+loop's pass, activations, soft-capped logits.  Inference only; CPU tensors use the plain statements."""
 from __future__ import annotations
 
 import ctypes
@@ -12,10 +12,14 @@ import torch.nn.functional as F
 
 from . import lib as _lib
 
-ACT = {"silu": 0, "gelu_tanh": 1, "gelu": 2, "relu2": 3}
+ACT = {"silu": 0, "gelu_tanh": 1, "gelu": 2, "relu2": 3, "xielu": 4}
 
 
-def _act(z: torch.Tensor, act: str) -> torch.Tensor:
+def _act(z: torch.Tensor, act: str, numbers: Optional[torch.Tensor] = None) -> torch.Tensor:
+    if act == "xielu":
+        p, q = F.softplus(numbers.float())
+        low = z.clamp(max=0.0)
+        return torch.where(z > 0, p * z * z, (0.5 + q) * (torch.expm1(low) - low)) + 0.5 * z
     if act == "relu2":
         return F.relu(z).square()
     return F.silu(z) if act == "silu" else F.gelu(z, approximate="tanh" if act == "gelu_tanh" else "none")
@@ -97,6 +101,41 @@ def partial_act(x: torch.Tensor, act: str, gated: bool = False) -> torch.Tensor:
         return out
     assert S == 1
     return gated_act(x[0], act) if gated else scaled_act(x[0], act)
+
+
+def bias_act(x: torch.Tensor, act: str, dtype: torch.dtype, bias: Optional[torch.Tensor] = None,
+             numbers: Optional[torch.Tensor] = None, used: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``act(sum of x [S, T, I] + bias)`` in ``dtype``, ``x`` as :func:`siirl_b200.ops.dense.linear_partial` returns it.
+    ``numbers``: the two learned numbers of ``"xielu"`` (for ``z > 0``: ``softplus(p) z^2 + z / 2``, else
+    ``(1/2 + softplus(q)) (e^z - 1 - z) + z / 2``).  Rows with a negative entry in ``used`` may be left unwritten."""
+    S, T, I = x.shape
+    assert (act == "xielu") == (numbers is not None)
+    if not x.is_cuda:
+        z = x.float().sum(0)
+        return _act(z + bias.float() if bias is not None else z, act, numbers).to(dtype)
+    assert x.is_contiguous() and (x.dtype == torch.float32 or (S == 1 and x.dtype == dtype))
+    out = torch.empty(T, I, dtype=dtype, device=x.device)
+    _lib.check(_lib.get_lib().sb_bias_act(
+        _lib.ptr(x), ctypes.c_longlong(T * I), S, _f32(x), _lib.ptr(bias), _lib.ptr(numbers), _lib.ptr(out),
+        ctypes.c_longlong(T), I, ACT[act], _lib.ptr(used), int(dtype == torch.float32), _lib.stream()), "sb_bias_act")
+    return out
+
+
+def token_gate(z: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, column: int, width: int,
+               dtype: torch.dtype) -> torch.Tensor:
+    """``gelu_tanh(sum of z [S, T, >= width]) * table[ids, column : column + width]``, padded columns zero."""
+    S, T, I = z.shape
+    if not z.is_cuda:
+        e = F.embedding(ids, table)[:, column:column + width].float()
+        return F.pad(_act(z.float().sum(0)[:, :width], "gelu_tanh") * e, (0, I - width)).to(dtype)
+    assert z.is_contiguous() and (z.dtype == torch.float32 or (S == 1 and z.dtype == dtype)) and table.dtype == dtype
+    assert ids.dtype == torch.int64 and ids.is_contiguous() and table.is_contiguous() and column + width <= table.shape[1]
+    out = torch.empty(T, I, dtype=dtype, device=z.device)
+    _lib.check(_lib.get_lib().sb_token_gate(
+        _lib.ptr(z), ctypes.c_longlong(T * I), S, _f32(z), _lib.ptr(ids), _lib.ptr(table),
+        ctypes.c_longlong(table.shape[1]), table.shape[0], column, width, _lib.ptr(out), T, I, int(dtype == torch.float32),
+        _lib.stream()), "sb_token_gate")
+    return out
 
 
 @dataclass
@@ -265,6 +304,69 @@ def hyper_rows(h: torch.Tensor, norm_w: torch.Tensor, norm_b: torch.Tensor, eps:
             assert r.x_id.is_contiguous() and r.x_id.dtype == out.dtype
             p.w_id, p.x_id = r.w_id.data_ptr(), r.x_id.data_ptr()
     _lib.check(_lib.get_lib().sb_hyper_rows(ctypes.byref(p), int(out.dtype == torch.float32), _lib.stream()), "sb_hyper_rows")
+    return out
+
+
+class _PostNorm(ctypes.Structure):
+    """Mirror of ``PostNormParams`` in csrc/post_norm_rows.cu."""
+    _fields_ = [("h", ctypes.c_void_p), ("rows", ctypes.c_int), ("W", ctypes.c_int), ("vocab", ctypes.c_int),
+                ("top", ctypes.c_int), ("ids", ctypes.c_void_p), ("table", ctypes.c_void_p), ("scale", ctypes.c_float),
+                ("eps", ctypes.c_float), ("y", ctypes.c_void_p), ("slab", ctypes.c_longlong), ("slabs", ctypes.c_int),
+                ("y_f32", ctypes.c_int), ("bias", ctypes.c_void_p), ("ys", ctypes.c_void_p), ("pair_slot", ctypes.c_void_p),
+                ("pair_w", ctypes.c_void_p), ("post", ctypes.c_void_p), ("norm_w", ctypes.c_void_p),
+                ("out", ctypes.c_void_p)]
+
+
+assert ctypes.sizeof(_PostNorm) == 128
+
+
+def post_norm_rows(h: torch.Tensor, weight: Optional[torch.Tensor], eps: float, dtype: torch.dtype, *,
+                   result: Optional[SublayerSum] = None, post: Optional[torch.Tensor] = None,
+                   ids: Optional[torch.Tensor] = None, table: Optional[torch.Tensor] = None,
+                   scale: float = 1.0) -> torch.Tensor:
+    """One step between two sublayers of a decoder with a norm behind each, ``h [T, W]`` fp32 in place:
+    ``h = table[ids] * scale`` (``ids`` given) or ``h += y / rms(y) * post`` with ``y`` the sum that ``result`` stands for;
+    returns ``h / rms(h) * weight`` in ``dtype``, or ``h`` itself in ``dtype`` (``weight = None``)."""
+    T, W = h.shape
+    assert h.dtype == torch.float32 and h.is_contiguous() and (ids is None) != (result is None)
+    r = result
+    assert r is None or r.x_id is None
+    if not h.is_cuda:
+        if ids is not None:
+            h.copy_(F.embedding(ids, table).float() * scale)
+        else:
+            y = torch.zeros(T, W)
+            if r.y is not None:
+                y = y + r.y.float().sum(0)
+            if r.bias is not None:
+                y = y + r.bias.float()
+            if r.ys is not None:
+                slot = r.pair_slot.reshape(T, -1).long()
+                for j in range(r.pair_w.shape[1]):
+                    y = y + torch.where((slot[:, j] >= 0)[:, None],
+                                        r.pair_w[:, j, None] * r.ys[slot[:, j].clamp(min=0)].float(), torch.zeros(()))
+            h += y * torch.rsqrt(y.square().mean(-1, keepdim=True) + eps) * post.float()
+        x = h if weight is None else h * torch.rsqrt(h.square().mean(-1, keepdim=True) + eps) * weight.float()
+        return x.to(dtype) if x is not h or dtype != torch.float32 else x.clone()
+    out = torch.empty(T, W, dtype=dtype, device=h.device)
+    ptr = lambda t: t.data_ptr() if t is not None else None  # noqa: E731
+    p = _PostNorm(h=h.data_ptr(), rows=T, W=W, scale=scale, eps=eps, post=ptr(post), norm_w=ptr(weight), out=out.data_ptr())
+    for w in (weight, post, table, r.bias if r is not None else None):
+        assert w is None or (w.dtype == dtype and w.is_contiguous())
+    if ids is not None:
+        assert ids.dtype == torch.int64 and ids.is_contiguous()
+        p.ids, p.table, p.vocab = ids.data_ptr(), table.data_ptr(), table.shape[0]
+    else:
+        p.bias = ptr(r.bias)
+        if r.y is not None:
+            assert r.y.is_contiguous() and r.y.shape[1:] == (T, W)
+            p.y, p.slab, p.slabs, p.y_f32 = r.y.data_ptr(), T * W, r.y.shape[0], _f32(r.y)
+            assert p.y_f32 or (p.slabs == 1 and r.y.dtype == dtype)
+        if r.ys is not None:
+            assert r.ys.is_contiguous() and r.ys.dtype == dtype and r.pair_w.dtype == torch.float32
+            p.ys, p.pair_slot, p.pair_w, p.top = r.ys.data_ptr(), ptr(r.pair_slot), ptr(r.pair_w), r.pair_w.shape[1]
+    _lib.check(_lib.get_lib().sb_post_norm_rows(ctypes.byref(p), int(dtype == torch.float32), _lib.stream()),
+               "sb_post_norm_rows")
     return out
 
 
