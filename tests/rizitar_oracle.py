@@ -209,3 +209,57 @@ def forward(cfg, weights, tokens, layers_out=None):
         if layers_out is not None:
             layers_out.append(x)
     return rms(x, eps) * weights["final.norm"] @ weights["embed"].t()
+
+
+# ---- random checkpoints ----------------------------------------------------------------------------------------------------
+def tensor_shapes(cfg):
+    """Names and shapes of the checkpoint of a config (``rank`` of a layer: low-rank width of its decay)."""
+    w, n = cfg["width"], cfg["token_side"]["dim"]
+    out = {"embed": (cfg["vocab"], w), "side.embed": (cfg["vocab"], n * len(cfg["layers"])), "final.norm": (w,)}
+    for i, c in enumerate(cfg["layers"]):
+        p, m, f = f"l{i}.", c["mixer"], c["mlp"]
+        out.update({p + k: (w,) for k in (("norm1", "norm1b", "norm2", "norm2b") if f else ("norm1", "norm1b"))})
+        out.update({p + "side.gate": (n, w), p + "side.proj": (w, n), p + "side.norm": (w,)})
+        hd = m["heads"] * m["dim"]
+        out[p + "mix.o"] = (w, hd)
+        if c["type"] == "attention":
+            out.update({p + "mix.q": (hd, w), p + "mix.k": (m["kv_heads"] * m["dim"], w), p + "mix.q.norm": (m["dim"],),
+                        p + "mix.k.norm": (m["dim"],), p + "mix.sink": (m["heads"],)})
+        else:
+            out.update({p + "mix." + k: (hd, w) for k in ("r", "k", "v", "g", "a")})
+            out.update({p + "mix.a.b": (hd,), p + "mix.w0": (hd,), p + "mix.norm": (hd,), p + "mix.w1": (c["rank"], w),
+                        p + "mix.w2": (hd, c["rank"])})
+        if f and f["kind"] == "dense":
+            out.update({p + "mlp.up": (f["ff"], w), p + "mlp.up.b": (f["ff"],), p + "mlp.down": (w, f["ff"]),
+                        p + "mlp.down.b": (w,), p + "mlp.act": (2,)})
+        elif f:
+            out[p + "mlp.router"] = (f["router"]["experts"], w)
+            for e in range(f["router"]["experts"]):
+                out.update({p + f"mlp.e{e}.up": (f["expert"]["ff"], w), p + f"mlp.e{e}.down": (w, f["expert"]["ff"])})
+    return out
+
+
+def random_checkpoint(cfg, seed=0):
+    g = torch.Generator().manual_seed(seed)
+    W = {}
+    for name, shape in tensor_shapes(cfg).items():
+        t = torch.randn(*shape, generator=g)
+        last = name.split(".")[-1]
+        if last.startswith("norm"):
+            t = 1.0 + 0.3 * t
+        elif last == "sink":
+            t = 1.5 + t
+        elif last in ("b", "w0"):
+            pass
+        elif name == "embed":
+            t = 1.5 * t * shape[-1] ** -0.5
+        elif last == "embed":
+            t = 1.5 * t
+        elif last == "act":
+            t = 0.7 * t
+        elif last == "router":
+            t = t * 2.0 * shape[-1] ** -0.5
+        elif len(shape) > 1:
+            t = t * shape[-1] ** -0.5
+        W[name] = t.bfloat16()
+    return W
