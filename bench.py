@@ -59,7 +59,7 @@ def parse_args():
     ap.add_argument("--workload", default="grpo", choices=["grpo", "serve"],
                     help="serve: prefill and decode throughput of a hybrid decoder beside the closest decoder of equal size "
                          "(1 GPU; benchmarks/hybrid_serving.py)")
-    ap.add_argument("--design", default="domavik", choices=["domavik", "poralorn", "gumazen"], help="hybrid decoder of --workload serve")
+    ap.add_argument("--design", default="domavik", choices=["domavik", "poralorn", "gumazen", "rizitar"], help="hybrid decoder of --workload serve")
     ap.add_argument("--budget-s", type=float, default=600.0,
                     help="wall-clock budget of the whole run, from process start; --steps/--warmup are upper bounds")
     ap.add_argument("--model", default="qwen2.5-7b")

@@ -1,11 +1,11 @@
-"""Serving throughput of a hybrid decoder (Domavik, Poralorn, Gumazen) beside the closest decoder of equal size, and its kernels
+"""Serving throughput of a hybrid decoder (Domavik, Poralorn, Gumazen, Rizitar) beside the closest decoder of equal size, and its kernels
 beside the like kernels of that model.
 
-    python bench.py --workload serve [--design poralorn|gumazen]             # end to end, a few sizes
-    python -m siirl_b200.benchmarks.hybrid_serving [--design poralorn|gumazen] --kernels
+    python bench.py --workload serve [--design poralorn|gumazen|rizitar]             # end to end, a few sizes
+    python -m siirl_b200.benchmarks.hybrid_serving [--design poralorn|gumazen|rizitar] --kernels
 
 End to end: random weights, the rollout engine's own prefill pass and CUDA-graph decode rounds, CUDA events on the
-launching stream.  Weights and caches are larger than L2 in every case.  Kernels: each alone, L2 flushed between
+launching stream.  Weights and caches are larger than L2 in every case.  Kernels: each alone as a CUDA graph, L2 flushed between
 iterations, against the measured copy bandwidth and GEMM rate (MEASURED_PEAKS.json, else the figures below)."""
 from __future__ import annotations
 
@@ -29,6 +29,8 @@ SIZES = {     # design -> size: preset, layers, (prompts, tokens) of a prefill p
                  "7b": ("poralorn-7b", 8, [(8, 1024), (1, 8192)], [(32, 2048), (256, 1024)])},
     "gumazen": {"a1b": ("gumazen-a1b", 12, [(8, 1024), (1, 8192)], [(32, 2048), (256, 1024)]),
                 "a3b": ("gumazen-a3b", 12, [(8, 1024), (1, 8192)], [(32, 2048), (256, 1024)])},
+    "rizitar": {"a1b": ("rizitar-a1b", 18, [(8, 1024), (1, 8192)], [(32, 2048), (256, 1024)]),
+                "a3b": ("rizitar-a3b", 18, [(8, 1024), (1, 8192)], [(32, 2048), (256, 1024)])},
 }
 
 
@@ -45,15 +47,18 @@ def peaks() -> Dict[str, float]:
 def closest(cfg: DecoderConfig) -> DecoderConfig:
     """The uniform decoder of the same width, feed-forward, number of layer runs, vocabulary and attention heads (seven
     query heads, or six, per key-value head where the design shares one latent between all); with experts where the design
-    has them: as many, as wide, as many per token, and a shared one."""
+    has them: as many, as many per token, as wide (two thirds where the design's experts have no gate: equal parameters), and
+    a shared one."""
     b = cfg.hybrid.attention[0]
     kv = b.kv_heads or b.heads // (7 if b.heads % 7 == 0 else 6)
     moe = next((x.moe for x in cfg.hybrid.layers if x.moe is not None), None)
     if moe is not None:
+        wide = moe.ff if moe.gated else moe.ff * 2 // 3
         return DecoderConfig(model_type="qwen2_moe", vocab_size=cfg.vocab_size, hidden_size=cfg.hidden_size,
                              intermediate_size=cfg.intermediate_size * 2 // 3 // 64 * 64, num_layers=len(cfg.hybrid.runs()),
                              num_heads=b.heads, num_kv_heads=kv, head_dim=b.dim, rope_theta=1e6, eos_token_id=2,
-                             num_experts=moe.experts, num_experts_per_tok=moe.top, moe_intermediate_size=moe.ff,
+                             num_experts=moe.experts, num_experts_per_tok=moe.top, moe_intermediate_size=wide,
+                             tie_word_embeddings=cfg.tie_word_embeddings,
                              shared_expert_intermediate_size=moe.shared_ff, first_k_dense_replace=1)
     return DecoderConfig(model_type="qwen2", vocab_size=cfg.vocab_size, hidden_size=cfg.hidden_size,
                          intermediate_size=cfg.intermediate_size, num_layers=len(cfg.hybrid.runs()), num_heads=b.heads,
@@ -193,10 +198,23 @@ class _Bench:
     def add(self, name, fn, flops=0.0, nbytes=0.0):
         if self.only and self.only not in name:
             return
-        ms = _events(fn, 3, self.iters, self.flush)
+        ms = _events(self.captured(fn), 3, self.iters, self.flush)
         ideal = max(flops / (self.pk["tflops"] * 1e9), nbytes / (self.pk["gbs"] * 1e6))
         self.rows.append({"kernel": name, "us": round(ms * 1e3, 1), "roofline_us": round(ideal * 1e3, 1),
                           "of_roofline": round(ideal / ms, 3)})
+
+    @staticmethod
+    def captured(fn):
+        """The launches of ``fn`` as a CUDA graph: what the host does between them (tens of microseconds) is left out."""
+        side = torch.cuda.Stream()
+        side.wait_stream(torch.cuda.current_stream())
+        with torch.cuda.stream(side):
+            fn()
+        torch.cuda.current_stream().wait_stream(side)
+        graph = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(graph):
+            fn()
+        return graph.replay
 
     def result(self):
         torch.cuda.synchronize()
@@ -210,7 +228,8 @@ def _rnd(*s):
 
 def kernels(design: str = "domavik", only: str = "", iters: int = 20) -> dict:
     b = _Bench(only, iters)
-    {"poralorn": _kernels_poralorn, "gumazen": _kernels_gumazen, "domavik": _kernels_domavik}[design](b)
+    {"poralorn": _kernels_poralorn, "gumazen": _kernels_gumazen, "rizitar": _kernels_rizitar,
+     "domavik": _kernels_domavik}[design](b)
     return b.result()
 
 
@@ -396,6 +415,140 @@ def _kernels_gumazen(b: _Bench) -> None:
         up = rnd(T, 2 * I)
         add(f"uniform: swiglu {T}x{I}", lambda: dense.swiglu(up), nbytes=T * I * 6)
         add(f"gumazen: squared relu {T}x{I}", lambda: R.scaled_act(up[:, :I], "relu2"), nbytes=T * I * 4)
+
+
+def _kernels_rizitar(b: _Bench) -> None:
+    """Windowed attention with pooled runs (32 heads of width 128, 4 key-value heads), the delta rule with 32 heads of width 64
+    beside the channel recurrence of the same size, the routed feed-forward with 120 plain experts, and the row operations."""
+    from ..models.decoder import _Init
+    from ..models.hybrid import HybridBranch
+    from ..models.moe import moe_forward
+    from ..ops import dense, kv_cache
+    from ..ops import moe as M
+    from ..ops import rows as R
+    from ..ops.attention import SeqInfo, attention_packed
+    from ..ops.recurrence import PortionPlan, RecurrenceSpec, empty_state, recurrence_decode, recurrence_prefill
+    from ..ops.window_attention import QueryTiles, WindowSpec, window_attention
+    dev, add, rnd = torch.device("cuda"), b.add, _rnd
+    base = get_config("rizitar-a3b")
+    W, H, G, D = base.hidden_size, 32, 4, 128
+    gen = _Init(0, "cuda")
+    kinds = [x.branches[0] for x in base.hybrid.layers]
+    att = HybridBranch(next(m for m in kinds if m.kind == "attention"), base, 0, 0, torch.bfloat16, "cuda", gen)
+    rule = HybridBranch(next(m for m in kinds if m.kind == "general_delta"), base, 0, 0, torch.bfloat16, "cuda", gen)
+    m, spec = att.b, att.spec
+    pr = copy.copy(att.prepare)
+    for k in ("q_norm", "k_norm", "sink"):
+        setattr(pr, k, getattr(att, k).detach())
+
+    def seen(i):
+        return min(i + 1, m.window) + max(0, i + 1 - m.window) // m.pool
+
+    for n, L in ((8, 1024), (1, 8192)):
+        T, nb, npool = n * L, L // 64, kv_cache.pool_blocks(L, m.pool)
+        x, xp = rnd(T, (H + 2 * G) * D), rnd(T, att.in_end)
+        info = SeqInfo([L] * n, device=dev)
+        flops = n * 4 * D * H * L * (L + 1) / 2
+        add(f"uniform: fmha_fwd {n}x{L}", lambda: attention_packed(x, info, H, G, D), flops)
+        order = torch.randperm(n * (nb + npool), device=dev).to(torch.int32)
+        table, pool_table = order[:n * nb].view(n, nb), order[n * nb:].view(n, npool).contiguous()
+        cache = torch.zeros(n * (nb + npool), G * 64 * 2 * D, dtype=torch.bfloat16, device=dev)
+        out = torch.empty(T, H * D, dtype=torch.bfloat16, device=dev)
+        ids = torch.repeat_interleave(torch.arange(n, dtype=torch.int32), L).to(dev)
+        pos = torch.arange(L, dtype=torch.int32).repeat(n).to(dev)
+        tiles = QueryTiles([L] * n, [0] * n, list(range(n)), dev)
+        tabs = dense.rope_tables(D, L, 1e6, device=dev)
+        add(f"uniform: rotation + append {n}x{L}",
+            lambda: kv_cache.rope_kv_append(x, pos, *tabs, None, ids, pos, table, cache[:n * nb].view(n * nb, 2, G, 64, D), H, G, D),
+            nbytes=T * ((H + G) * D * 2 + (H + 2 * G) * D * 2))
+        add(f"rizitar: norms, rotation, append, pooling {n}x{L}", lambda: pr.run(spec, xp, ids, pos, table, cache, pool_table),
+            nbytes=T * (H + G) * D * 2 + T * (H + 2 * G) * D * 2 * (1 + 1 / m.pool))
+        add(f"rizitar: attention window {m.window} pool {m.pool} {n}x{L}, with norms, rotation, append, pooling",
+            lambda: window_attention(spec, xp, ids, pos, table, cache, out, 0, tiles=tiles, prepare=pr, pool_table=pool_table),
+            n * 4 * D * H * sum(map(seen, range(L))))
+        plain = WindowSpec(H, G, D, D, 0, H * D, (H + G) * D, D ** -0.5, m.window)
+        add(f"domavik: window attention window {m.window} {n}x{L}, with append",
+            lambda: window_attention(plain, x, ids, pos, table, cache, out, 0, tiles=tiles),
+            n * 4 * D * H * sum(min(i + 1, m.window) for i in range(L)))
+    for B, ctx in ((32, 2048), (256, 1024), (32, 16384)):
+        nb, npool = (ctx + 63) // 64, kv_cache.pool_blocks(ctx, m.pool)
+        order = torch.randperm(B * (nb + npool), device=dev).to(torch.int32)
+        table, pool_table = order[:B * nb].view(B, nb), order[B * nb:].view(B, npool).contiguous()
+        lens = torch.full((B,), ctx, dtype=torch.int32, device=dev)
+        flat = torch.zeros(B * (nb + npool), G * 64 * 2 * D, dtype=torch.bfloat16, device=dev)
+        q, kvc = rnd(B, (H + 2 * G) * D), flat[:B * nb].view(B * nb, 2, G, 64, D)
+        place = torch.randperm(B * nb, device=dev).to(torch.int32).view(B, nb)
+        add(f"uniform: decode attention {B}x{ctx}", lambda: kv_cache.decode_attention(q, kvc, lens, place, H, G, D),
+            nbytes=B * ctx * 2 * G * D * 2)
+        out = torch.empty(B, H * D, dtype=torch.bfloat16, device=dev)
+        ids, pos = torch.arange(B, dtype=torch.int32, device=dev), lens - 1
+        xp = rnd(B, att.in_end)
+        add(f"rizitar: norms, rotation, append, pooling {B} at {ctx}",
+            lambda: pr.run(spec, xp, ids, pos, table, flat, pool_table, single=True),
+            nbytes=B * (H + 2 * G) * D * 4 + B * m.pool * 2 * G * D * 2)
+        add(f"rizitar: decode attention {B}x{ctx} window {m.window} pool {m.pool}, with norms, rotation, append, pooling",
+            lambda: window_attention(spec, xp, ids, pos, table, flat, out, 0, seq_lens=lens, prepare=pr, pool_table=pool_table),
+            nbytes=B * seen(ctx - 1) * 2 * G * D * 2)
+        plain = WindowSpec(H, G, D, D, 0, H * D, (H + G) * D, D ** -0.5, m.window)
+        add(f"domavik: window decode {B}x{ctx} window {m.window}, with append",
+            lambda: window_attention(plain, q, ids, pos, table, flat, out, 0, seq_lens=lens),
+            nbytes=B * min(ctx, m.window) * 2 * G * D * 2)
+    d, h, spec = rule.b.dim, rule.b.heads, rule.spec
+    hd = h * d
+    chan = RecurrenceSpec("channel", h, d, d, 0, hd, 2 * hd, 3 * hd, 4 * hd, 0, 16, 16.0, 15.0, 1e-5, 1.0)
+    for name, sp, wts, width in (
+            ("rizitar: delta rule", spec, rule.weights(), rule.in_end),
+            ("domavik: channel recurrence", chan, {"norm": rnd(d), "w2": rnd(hd, 16), "b_e": rnd(hd)}, 4 * hd + 16)):
+        for n, L in ((8, 1024), (1, 8192)):
+            x, out = rnd(n * L, width), torch.empty(n * L, hd, dtype=torch.bfloat16, device=dev)
+            st, plan = empty_state(sp, n, dev), PortionPlan([L] * n, [0] * n, list(range(n)), dev)
+            add(f"{name} {n}x{L} ({h} heads of {d})", lambda: recurrence_prefill(sp, x, wts, st, plan, out, 0),
+                nbytes=n * L * (width + hd) * 2 + n * h * d * d * 4)
+        for B in (32, 256):
+            x, out = rnd(B, width), torch.empty(B, hd, dtype=torch.bfloat16, device=dev)
+            st = empty_state(sp, B, dev)
+            slots, pos = torch.arange(B, dtype=torch.int32, device=dev), torch.full((B,), 9, dtype=torch.int32, device=dev)
+            add(f"{name} step {B} ({h} heads of {d})", lambda: recurrence_decode(sp, x, wts, st, slots, pos, out, 0),
+                nbytes=B * h * d * d * 8 + B * (width + hd) * 2)
+    e = next(x.moe for x in base.hybrid.layers if x.moe is not None)
+    wide, local, one = e.ff * 2 // 3, M.ExpertParallel(), rnd(W)
+    up, dn = rnd(e.experts, e.ff, W) * 0.04, rnd(e.experts, W, e.ff) * 0.04
+    gu, gd, router = rnd(e.experts, 2 * wide, W) * 0.04, rnd(e.experts, W, wide) * 0.04, rnd(e.experts, W)
+    side, numbers = base.hybrid.token_side, torch.tensor([0.5, 0.3], device=dev).bfloat16()
+    table = rnd(base.vocab_size, 4 * side)
+    for T in (32, 256, 8192):
+        x, z = rnd(T, W), torch.randn(1, T, e.experts, device=dev)
+        used = e.experts * (1 - (1 - e.top / e.experts) ** T)
+        flops, nbytes = T * e.top * 4.0 * W * e.ff, used * 4 * W * e.ff + T * W * 4
+        add(f"uniform: router {T}", lambda: M.route_topk(z[0], e.top, False), nbytes=T * e.experts * 4)
+        add(f"rizitar: router {T}", lambda: M.route_grouped(z, None, e.experts, e.top, 1, 1, 1.0, outputs=e.experts,
+                                                            renormalize=False), nbytes=T * e.experts * 4)
+        wt, ids = M.route_topk(z[0], e.top, False)
+        add(f"uniform: routed feed-forward {T} (dispatch, gated experts, combine)",
+            lambda: moe_forward(x, router, gu, gd, e.top, routed=(wt, ids)), flops, nbytes)
+        i32 = ids.to(torch.int32)
+        add(f"rizitar: routed feed-forward {T} (dispatch, plain experts)",
+            lambda: M.routed_experts(x, i32, up, dn, "relu2", gated=False), flops, nbytes)
+        h32, y, d16, res = torch.randn(T, W, device=dev), rnd(1, T, W), rnd(T, W), rnd(T, W)
+        add(f"uniform: residual + RMS norm {T}x{W} (bf16 stream)", lambda: dense.rmsnorm(d16, one, 1e-6, residual=res),
+            nbytes=T * W * 8)
+        add(f"rizitar: norm, residual, norm {T}x{W} (fp32 stream)",
+            lambda: R.post_norm_rows(h32, one, 1e-5, torch.bfloat16, post=one, result=R.SublayerSum(y)), nbytes=T * W * 12)
+        ys, slots = M.routed_experts(x, i32, up, dn, "relu2", gated=False)
+        add(f"uniform: combine {T}x{W}", lambda: local.combine(ys, None, slots, wt, T, e.top), nbytes=T * W * 2 * (e.top + 1))
+        add(f"rizitar: combine, norm, residual, norm {T}x{W}",
+            lambda: R.post_norm_rows(h32, one, 1e-5, torch.bfloat16, post=one,
+                                     result=R.SublayerSum(ys=ys, pair_slot=slots, pair_w=wt)), nbytes=T * W * (10 + 2 * e.top))
+        tok, zs = torch.randint(0, base.vocab_size, (T,), device=dev), rnd(1, T, side)
+        add(f"uniform: swiglu {T}x{side}", lambda: dense.swiglu(torch.cat([zs[0], zs[0]], 1)), nbytes=T * side * 6)
+        add(f"rizitar: token gate {T}x{side}", lambda: R.token_gate(zs, tok, table, side, side, torch.bfloat16),
+            nbytes=T * side * 6)
+        I = base.intermediate_size
+        a, bias = rnd(1, T, I), rnd(I)
+        pair = rnd(T, 2 * I)
+        add(f"uniform: swiglu {T}x{I}", lambda: dense.swiglu(pair), nbytes=T * I * 6)
+        add(f"rizitar: bias + xIELU {T}x{I}", lambda: R.bias_act(a, "xielu", torch.bfloat16, bias=bias, numbers=numbers),
+            nbytes=T * I * 4)
 
 
 def _kernels_domavik(b: _Bench) -> None:

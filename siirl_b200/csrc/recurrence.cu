@@ -444,17 +444,6 @@ struct ScanSmem {
   }
 };
 
-struct Segments {
-  const int* seq;       // [n] sequence of the segment
-  const int* chunk0;    // [n] its first chunk
-  const int* row;       // [n] its first row
-  const int* tokens;    // [n] its tokens
-  const int* flags;     // [n] bit 0: first of its sequence, bit 1: last
-  const int* seq_seg0;  // [n_seq + 1]
-  float* S;             // [n, H, rows, dk] local states, then start states
-  float* decay;         // [n, H, dkp]
-};
-
 // Warp w of the CTA owns value columns 16 w .. 16 w + 15 (rows of the fragments) and all key channels (NK steps of 16).
 // Iteration c multiplies chunk c and finishes (norm, gate, store) chunk c - 1: one block barrier per chunk.
 //

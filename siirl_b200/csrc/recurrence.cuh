@@ -51,6 +51,18 @@ __host__ __device__ inline int pad_dk(int dk) { return dk <= 64 ? (dk + 15) / 16
 __host__ __device__ inline int tile_row(int dkp) { return dkp + 8; }        // bf16 elements per row of a q / k tile
 constexpr int kARow = 24;                                                    // and of the score matrix
 
+// runs of consecutive chunks of one sequence
+struct Segments {
+  const int* seq;       // [n] sequence of the segment
+  const int* chunk0;    // [n] its first chunk
+  const int* row;       // [n] its first row
+  const int* tokens;    // [n] its tokens
+  const int* flags;     // [n] bit 0: first of its sequence, bit 1: last
+  const int* seq_seg0;  // [n_seq + 1]
+  float* S;             // [n, H, rows, dk] local states, then start states
+  float* decay;         // [n, H, dkp] (kGateDelta: [n, H, dk, dk], what a start state is multiplied by)
+};
+
 // x and y as two bf16 terms each: x = hi + lo to 16 mantissa bits
 __device__ __forceinline__ void split_pair(float x, float y, uint32_t& hi, uint32_t& lo) {
   const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);

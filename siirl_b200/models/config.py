@@ -1045,14 +1045,15 @@ def _gumazen(n_layers: int, width: int, ff: int, vocab: int, heads: int, kv_head
 
 def _rizitar(n_layers: int, width: int, ff: int, vocab: int, att: dict, delta: dict, moe: ExpertSpec, side: int,
              rot_base: float = 1e6, **kw) -> DecoderConfig:
-    """Rizitar layers in turn: two delta rules, then attention; the feed-forwards alternate between dense and routed."""
+    """Rizitar layers in turn: two delta rules, then attention; the first layer has a dense feed-forward, the others are
+    routed."""
     dim = att["dim"]
     base = dict(kind="attention", vdim=dim, scale=dim ** -0.5, bias_exp=0.0, qk_norm="head_weights", sink_weight=True,
                 key_values=True, rot_dims=dim, rot_base=rot_base,
                 rot_scaling={"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0})
     layers = [HybridLayer([MixerBranch(**base, **att) if i % 3 == 2 else
                            MixerBranch(kind="general_delta", vdim=delta["dim"], **delta)],
-                          ff=0 if i % 2 else ff, moe=moe if i % 2 else None) for i in range(n_layers)]
+                          ff=0 if i else ff, moe=moe if i else None) for i in range(n_layers)]
     spec = HybridSpec(layers=layers, embed_scale=width ** 0.5, norm="rms_norm", act="xielu", arrangement="sandwich",
                       token_side=side, ff_bias=True, hf_naming="rizitar")
     return DecoderConfig.for_hybrid(spec, vocab_size=vocab, hidden_size=width, rms_norm_eps=1e-5, model_type="rizitar",
@@ -1068,9 +1069,9 @@ PRESETS: Dict[str, DecoderConfig] = {
                              dict(heads=3, dim=24, rank=8), _plain_experts(6, 40, 2), side=16),
     # layer sizes of decoders with about 1 / 3 billion active parameters (benchmark shapes, random weights)
     "rizitar-a1b": _rizitar(18, 1536, 8960, 152064, dict(heads=12, kv_heads=2, dim=128, window=1024, pool=16),
-                            dict(heads=24, dim=64, rank=64), _plain_experts(64, 1024, 6), side=128),
+                            dict(heads=24, dim=64, rank=64), _plain_experts(56, 1152, 6), side=128),
     "rizitar-a3b": _rizitar(18, 2048, 11264, 152064, dict(heads=32, kv_heads=4, dim=128, window=1024, pool=16),
-                            dict(heads=32, dim=64, rank=64), _plain_experts(128, 1536, 8), side=256),
+                            dict(heads=32, dim=64, rank=64), _plain_experts(120, 1536, 8), side=256),
     "tiny-gumazen": _gumazen(3, 128, 192, 1024, heads=4, kv_heads=2, dim=32, vdim=24, window=70, rot_dims=16,
                              moe=ExpertSpec(experts=6, ff=40, top=3, groups=2, keep=1, identity=2, scale=1.5, shared_ff=56),
                              loop=LayerLoop(1, 3, 2)),

@@ -15,8 +15,8 @@ and removal rate ``f_t = sigmoid(f + b_f)`` per key channel:
 State of a branch, all in 32-bit floats: ``S [slots, heads, vdim (+1), dim]`` and, for the head form, ``m [slots, heads]``.
 A portion that begins at position 0 starts from zero whatever its slot holds.
 
-CUDA tensors run ``csrc/recurrence.cu`` (delta form: ``csrc/delta_rule.cu``): decoding and 32-bit models the token-by-token kernel, bf16 prompts the chunked
-tensor-core kernels.  CPU tensors run the plain loop below."""
+CUDA tensors run ``csrc/recurrence.cu`` (delta form: ``csrc/delta_rule.cu``): decoding and 32-bit models the token-by-token
+kernel, bf16 prompts the chunked tensor-core kernels.  CPU tensors run the plain loop below."""
 from __future__ import annotations
 
 import ctypes
@@ -92,10 +92,9 @@ class PortionPlan:
 
     def __init__(self, lens: Sequence[int], starts: Sequence[int], slots: Sequence[int], device):
         self.lens, self.starts, self.slots = list(lens), list(starts), list(slots)
-        row0, chunk_row, chunk_len, chunk0, at = [], [], [], [], 0
+        row0, chunk_row, chunk_len, at = [], [], [], 0
         for n in self.lens:
             row0.append(at)
-            chunk0.append(len(chunk_row))
             for c in range(0, n, CHUNK):
                 chunk_row.append(at + c)
                 chunk_len.append(min(CHUNK, n - c))
@@ -104,10 +103,9 @@ class PortionPlan:
         self.device = device
         self._segments: Dict[int, Tuple[torch.Tensor, int]] = {}
         # one copy to the device: the pieces are views
-        parts = [row0, self.lens, self.slots, self.starts, chunk_row, chunk_len, chunk0]
+        parts = [row0, self.lens, self.slots, self.starts, chunk_row, chunk_len]
         flat = torch.tensor([v for p in parts for v in p], dtype=torch.int32).to(device)
-        (self.row0, self.nrow, self.slot, self.pos0, self.chunk_row, self.chunk_len,
-         self.chunk0) = flat.split([len(p) for p in parts])
+        self.row0, self.nrow, self.slot, self.pos0, self.chunk_row, self.chunk_len = flat.split([len(p) for p in parts])
 
     def segments(self, blocks: int) -> Tuple[torch.Tensor, int]:
         """Runs of chunks that work in parallel, about ``blocks`` of them in all, equal within a sequence:
@@ -149,10 +147,11 @@ def _params(spec: RecurrenceSpec, x, weights, state, out, out_off) -> _Params:
 
 def recurrence_prefill(spec: RecurrenceSpec, x: torch.Tensor, weights: Dict[str, torch.Tensor],
                        state: Dict[str, torch.Tensor], plan: PortionPlan, out: torch.Tensor, out_off: int,
-                       stepwise: bool = False) -> None:
+                       stepwise: bool = False, segments: Optional[int] = None) -> None:
     """Run packed portions through the recurrence: rows ``x [T, width]``, results in ``out[:, out_off: ...]``, states
     read from and left in the portions' slots.  ``weights``: ``norm`` and ``w2``/``b_e`` (channel form) or ``b_e``/``b_f``
-    (head form).  ``stepwise`` forces the token-by-token kernel."""
+    (head form).  ``stepwise`` forces the token-by-token kernel; ``segments`` (delta form): about that many segments run in
+    parallel."""
     if not x.is_cuda:
         rows = [list(range(r, r + n)) for r, n in zip(plan.row0_cpu, plan.lens)]
         _run_cpu(spec, x, weights, state, rows, plan.slots, plan.starts, out, out_off)
@@ -163,13 +162,18 @@ def recurrence_prefill(spec: RecurrenceSpec, x: torch.Tensor, weights: Dict[str,
     if x.dtype == torch.bfloat16 and not stepwise and spec.gate == "delta":
         fn = L._cdll.sb_delta_workspace
         fn.restype = ctypes.c_longlong
-        nbytes = int(fn(ref, plan.n_chunks))
+        blocks = int(L._cdll.sb_delta_resident(ref)) // spec.heads if segments is None else segments
+        segs, n_seg = plan.segments(blocks)
+        if segments is None and n_seg < 3 * plan.n_seq:     # a segment costs two passes over its chunks
+            segs, n_seg = plan.segments(plan.n_seq)
+        nbytes = int(fn(ref, plan.n_chunks, n_seg, x.shape[0]))
         if nbytes >= 0:
             ws = torch.empty(max(nbytes, 16), dtype=torch.uint8, device=x.device)
             _lib.check(L.sb_delta_prefill(
-                ref, _lib.ptr(plan.row0), _lib.ptr(plan.nrow), _lib.ptr(plan.slot), _lib.ptr(plan.pos0), plan.n_seq,
-                _lib.ptr(plan.chunk_row), _lib.ptr(plan.chunk_len), _lib.ptr(plan.chunk0), plan.n_chunks, _lib.ptr(ws),
-                _lib.stream()), "sb_delta_prefill")
+                ref, _lib.ptr(plan.slot), _lib.ptr(plan.pos0), plan.n_seq, _lib.ptr(plan.chunk_row),
+                _lib.ptr(plan.chunk_len), plan.n_chunks, _lib.ptr(segs), n_seg, x.shape[0], _lib.ptr(ws), _lib.stream()),
+                "sb_delta_prefill")
+            _lib.add_launches(2 if n_seg > plan.n_seq else 0)
             return
     elif x.dtype == torch.bfloat16 and not stepwise:
         fn = L._cdll.sb_recurrence_workspace

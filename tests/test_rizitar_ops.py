@@ -381,11 +381,12 @@ def dirty(spec, slots, device):
     return state
 
 
-def scan(spec, w, xs, state, slots, starts, stepwise=False):
+def scan(spec, w, xs, state, slots, starts, stepwise=False, segments=None):
     dev, lens = xs[0].device, [x.shape[0] for x in xs]
     x = torch.cat(xs)
     out = torch.full((x.shape[0], 16 + (spec.heads * spec.vdim + 7) // 8 * 8), 9.0, dtype=x.dtype, device=dev)
-    recurrence_prefill(spec, x, w, state, PortionPlan(lens, starts, slots, dev), out, 16, stepwise=stepwise)
+    recurrence_prefill(spec, x, w, state, PortionPlan(lens, starts, slots, dev), out, 16, stepwise=stepwise,
+                       segments=segments)
     assert (out[:, :16] == 9).all()
     return out[:, 16:16 + spec.heads * spec.vdim].split(lens)
 
@@ -472,6 +473,28 @@ def test_delta_rule_of_unequal_sequences_in_one_batch(name, device, dtype):
         want, last = c.want()
         close(o, want[s:], dtype, f32=2e-4)
         close(state["S"][slot], last, dtype, f32=1e-4, bf16=1e-3)
+
+
+@pytest.mark.parametrize("device,dtype", WHERE)
+@pytest.mark.parametrize("name", ["small", "narrow", "middle", "uneven", "usual", "wide", "widest"])
+def test_segments_of_the_delta_rule_that_run_in_parallel(name, device, dtype):
+    """Long portions cut into segments, beside one of a single segment; from zero and from a state."""
+    lens, starts, slots = [470, 3, 200], [30, 0, 0], [2, 0, 1]
+    cases = [Delta(name, s + n, "same_key" if i else "keep", seed=i) for i, (n, s) in enumerate(zip(lens, starts))]
+    spec, w, _ = cases[0].branch(dtype, device)
+    for c in cases[1:]:
+        c.w2, c.w0, c.ab, c.norm = (getattr(cases[0], k) for k in ("w2", "w0", "ab", "norm"))
+    xs = [c.branch(dtype, device)[2] for c in cases]
+    for segments in (4, 9, 40):
+        state = dirty(spec, 4, device)
+        scan(spec, w, [xs[0][:30]], state, [2], [0])
+        got = scan(spec, w, [x[s:] for x, s in zip(xs, starts)], state, slots, starts, segments=segments)
+        finish(device)
+        for o, c, s, slot in zip(got, cases, starts, slots):
+            want, last = c.want()
+            close(o, want[s:], dtype, f"{segments}", f32=2e-3, bf16=2e-2)
+            close(state["S"][slot], last, dtype, f"{segments} state", f32=2e-4, bf16=2e-3)
+        assert (state["S"][3] == 11).all()
 
 
 @pytest.mark.parametrize("device,dtype", WHERE)
