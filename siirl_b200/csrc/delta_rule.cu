@@ -123,8 +123,10 @@ __host__ __device__ inline int delta_step_floats(int dk, int dv, int rank) {
 }
 
 // dk = dv <= 32 N, a multiple of four.  Eight lanes hold a state row (a value column's key channels), four rows per warp and pass.
+// Everything a token needs is asked for at once, before the first barrier: a decoding step waits for memory twice, for its slot
+// and for the rest.
 template <typename T, int N>
-__global__ void __launch_bounds__(kStepThreads)
+__global__ void __launch_bounds__(kStepThreads, N <= 2 ? 4 : 2)
 delta_step_regs_kernel(RecParams p, const int* __restrict__ row0, const int* __restrict__ nrow,
                        const int* __restrict__ slots, const int* __restrict__ pos0) {
   extern __shared__ __align__(16) float sm[];
@@ -153,12 +155,88 @@ delta_step_regs_kernel(RecParams p, const int* __restrict__ row0, const int* __r
       if (!fresh && row + 32 * i < p.dv && d0 + 32 * c < p.dk)
         load_vec<float, 4>(gs + (size_t)(row + 32 * i) * p.dk + d0 + 32 * c, st[i][c]);
     }
+  // four lanes share a channel's product with the low-rank row: channels tid / 4 and, for wide heads, + 64
+  constexpr int CN = (N + 1) / 2;
+  const int part = tid & 3;
+  const bool vec = sizeof(T) == 2 && p.rank % 8 == 0 && ((uintptr_t)p.w2 & 15) == 0;
+  float b_e[CN], b_f[CN];
+  uint4 w_pre[CN][2];      // this lane's first sixteen weights
+#pragma unroll
+  for (int c = 0; c < CN; ++c) {
+    const int d = (tid >> 2) + 64 * c;
+    b_e[c] = b_f[c] = 0.f;
+    w_pre[c][0] = w_pre[c][1] = make_uint4(0, 0, 0, 0);
+    if (d >= p.dk) continue;
+    b_e[c] = to_float(reinterpret_cast<const T*>(p.b_e)[h * p.dk + d]);
+    b_f[c] = to_float(reinterpret_cast<const T*>(p.b_f)[h * p.dk + d]);
+    if constexpr (sizeof(T) == 2) {
+#pragma unroll
+      for (int k = 0; k < 2; ++k)
+        if (vec && part * 8 + 32 * k < p.rank)
+          w_pre[c][k] = *reinterpret_cast<const uint4*>(reinterpret_cast<const T*>(p.w2) + (size_t)(h * p.dk + d) * p.rank + part * 8 + 32 * k);
+    }
+  }
+  const float nw = tid < p.dv ? to_float(reinterpret_cast<const T*>(p.norm_w)[p.norm_per_head ? h * p.dv + tid : tid]) : 0.f;
   for (int t = 0; t < n; ++t) {
     const T* xr = reinterpret_cast<const T*>(p.x) + (size_t)(r0 + t) * p.row_stride;
-    delta_token<T>(p, xr, h, sq, sk, su, sb_, sd, se, red);
-    float seen[N];
+    const float k_in = tid < p.dk ? to_float(xr[p.k_off + h * p.dk + tid]) : 0.f;
+    const float q_in = tid < p.dk ? to_float(xr[p.q_off + h * p.dk + tid]) : 0.f;
+    const float g_in = tid < p.dv ? to_float(xr[p.g_off + h * p.dv + tid]) : 0.f;
+    float a_in[CN], v[N], o[N], seen[N];
 #pragma unroll
-    for (int i = 0; i < N; ++i) seen[i] = 0.f;
+    for (int c = 0; c < CN; ++c) {
+      const int d = (tid >> 2) + 64 * c;
+      a_in[c] = d < p.dk ? to_float(xr[p.f_off + h * p.dk + d]) : 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      v[i] = row + 32 * i < p.dv ? to_float(xr[p.v_off + h * p.dv + row + 32 * i]) : 0.f;
+      o[i] = seen[i] = 0.f;
+    }
+    for (int r = tid; r < p.rank; r += kStepThreads) se[r] = tanhf(to_float(xr[p.e_off + r]));
+    if (tid < p.dk) {
+      sk[tid] = k_in;
+      sq[tid] = q_in;
+    }
+    float ss = warp_sum(k_in * k_in);
+    if (lane == 0) red[warp] = ss;
+    __syncthreads();
+    float tot = 0.f;
+#pragma unroll
+    for (int i = 0; i < kStepThreads / 32; ++i) tot += red[i];
+    const float inv = 1.f / sqrtf(tot + 1e-6f);
+#pragma unroll
+    for (int c = 0; c < CN; ++c) {
+      const int d = (tid >> 2) + 64 * c;
+      float z = 0.f;
+      if (d < p.dk) {
+        const T* w = reinterpret_cast<const T*>(p.w2) + (size_t)(h * p.dk + d) * p.rank;
+        if constexpr (sizeof(T) == 2) {
+          if (vec) {
+            for (int r = part * 8, k = 0; r < p.rank; r += 32, ++k) {
+              float x[8];
+              if (k == 0) load_vec<T, 8>(reinterpret_cast<const T*>(&w_pre[c][0]), x);
+              else if (k == 1) load_vec<T, 8>(reinterpret_cast<const T*>(&w_pre[c][1]), x);
+              else load_vec<T, 8>(w + r, x);
+              const float4 e0 = *reinterpret_cast<const float4*>(se + r), e1 = *reinterpret_cast<const float4*>(se + r + 4);
+              z = fmaf(x[0], e0.x, fmaf(x[1], e0.y, fmaf(x[2], e0.z, fmaf(x[3], e0.w, z))));
+              z = fmaf(x[4], e1.x, fmaf(x[5], e1.y, fmaf(x[6], e1.z, fmaf(x[7], e1.w, z))));
+            }
+          }
+        }
+        if (!vec)
+          for (int r = part; r < p.rank; r += 4) z = fmaf(to_float(w[r]), se[r], z);
+      }
+      z += __shfl_xor_sync(0xffffffffu, z, 1);
+      z += __shfl_xor_sync(0xffffffffu, z, 2);
+      if (d < p.dk && part == 0) {
+        sd[d] = expf(-kDecayRate / (1.f + expf(-(z + b_e[c]))));
+        const float u = sk[d] * inv;
+        su[d] = u;
+        sb_[d] = u / (1.f + expf(-(a_in[c] + b_f[c])));
+      }
+    }
+    __syncthreads();
 #pragma unroll
     for (int c = 0; c < N; ++c) {
       if (d0 + 32 * c >= p.dk) break;
@@ -174,12 +252,6 @@ delta_step_regs_kernel(RecParams p, const int* __restrict__ row0, const int* __r
       seen[i] += __shfl_xor_sync(0xffffffffu, seen[i], 4);
       seen[i] += __shfl_xor_sync(0xffffffffu, seen[i], 2);
       seen[i] += __shfl_xor_sync(0xffffffffu, seen[i], 1);
-    }
-    float v[N], o[N];
-#pragma unroll
-    for (int i = 0; i < N; ++i) {
-      v[i] = row + 32 * i < p.dv ? to_float(xr[p.v_off + h * p.dv + row + 32 * i]) : 0.f;
-      o[i] = 0.f;
     }
 #pragma unroll
     for (int c = 0; c < N; ++c) {
@@ -198,14 +270,27 @@ delta_step_regs_kernel(RecParams p, const int* __restrict__ row0, const int* __r
           o[i] = fmaf(x, q[j], o[i]);
         }
     }
+    ss = 0.f;
 #pragma unroll
     for (int i = 0; i < N; ++i) {
       o[i] += __shfl_xor_sync(0xffffffffu, o[i], 4);
       o[i] += __shfl_xor_sync(0xffffffffu, o[i], 2);
       o[i] += __shfl_xor_sync(0xffffffffu, o[i], 1);
-      if ((lane & 7) == 0 && row + 32 * i < p.dv) so[row + 32 * i] = o[i] * p.q_scale;
+      o[i] *= p.q_scale;
+      if ((lane & 7) == 0 && row + 32 * i < p.dv) {
+        so[row + 32 * i] = o[i];
+        ss = fmaf(o[i], o[i], ss);
+      }
     }
-    delta_finish<T>(p, xr, out + (size_t)(r0 + t) * p.out_stride, h, so, red + 8);
+    ss = warp_sum(ss);
+    if (lane == 0) red[8 + warp] = ss;
+    __syncthreads();
+    tot = 0.f;
+#pragma unroll
+    for (int i = 0; i < kStepThreads / 32; ++i) tot += red[8 + i];
+    const float rstd = 1.f / sqrtf(tot / (float)p.dv + p.eps);
+    if (tid < p.dv)
+      out[(size_t)(r0 + t) * p.out_stride + tid] = from_float<T>(so[tid] * rstd * nw * gate_value(g_in, p.gate_act) * p.out_scale);
   }
 #pragma unroll
   for (int i = 0; i < N; ++i)
@@ -283,8 +368,8 @@ struct DeltaPrepSmem {      // byte offsets
     ub = (cum + kChunk * (dkp + 1) * 4 + 15) / 16 * 16;              // [16][16] fp32
     small = ub + kChunk * kChunk * 4;                                // rk, rb, uk, inverse: [16][24], hi and lo
     e = small + 8 * kChunk * kARow * 2;                              // low-rank rows, hi and lo [16][rankp + 8]
-    inv = e + 2 * kChunk * (rankp + 8) * 2;                          // [16] 1 / |k|
-    total = inv + kChunk * 4;
+    inv = e + 2 * kChunk * (rankp + 8) * 2;                          // [16][dkp / 8] squares of the keys
+    total = inv + kChunk * (dkp / 8) * 4;
   }
 };
 
@@ -366,7 +451,7 @@ delta_prepare_kernel(RecParams p, const int* __restrict__ chunk_row, const int* 
   B16 *m_rk = reinterpret_cast<B16*>(smem + L.small), *m_rb = m_rk + 2 * mat, *m_uk = m_rk + 4 * mat, *m_inv = m_rk + 6 * mat;
   B16* s_e = reinterpret_cast<B16*>(smem + L.e);
   const int e_part = kChunk * (rankp + 8);
-  float* s_inv = reinterpret_cast<float*>(smem + L.inv);
+  float* s_sq = reinterpret_cast<float*>(smem + L.inv);
   const int h = blockIdx.x, c = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int row = chunk_row[c], len = chunk_len[c];
   const B16* x = reinterpret_cast<const B16*>(p.x) + (size_t)row * p.row_stride;
@@ -374,6 +459,21 @@ delta_prepare_kernel(RecParams p, const int* __restrict__ chunk_row, const int* 
   const B16* w0 = reinterpret_cast<const B16*>(p.b_e) + h * p.dk;
   const B16* ab = reinterpret_cast<const B16*>(p.b_f) + h * p.dk;
 
+  // a thread's vectors of eight channels of r, k, a: under way while the decays are made
+  constexpr int per = dkp / 8, items = (kChunk * per + kDeltaThreads - 1) / kDeltaThreads;
+  uint4 raw[items][3];
+#pragma unroll
+  for (int it = 0; it < items; ++it) {
+    const int i = tid + it * kDeltaThreads, t = i / per, d = i % per * 8;
+#pragma unroll
+    for (int m = 0; m < 3; ++m) raw[it][m] = make_uint4(0, 0, 0, 0);
+    if (t < len && d < p.dk) {
+      const B16* xr = x + (size_t)t * p.row_stride + h * p.dk + d;
+      raw[it][0] = *reinterpret_cast<const uint4*>(xr + p.k_off);
+      raw[it][1] = *reinterpret_cast<const uint4*>(xr + p.q_off);
+      raw[it][2] = *reinterpret_cast<const uint4*>(xr + p.f_off);
+    }
+  }
   {      // low-rank rows; eight threads per token
     const int t = tid >> 3;
     const B16* src = lowrank + (size_t)(row + t) * 2 * rankp;
@@ -383,23 +483,6 @@ delta_prepare_kernel(RecParams p, const int* __restrict__ chunk_row, const int* 
       else *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
     }
     copy_commit();
-    // lengths of the keys
-    float ss = 0.f;
-    if (t < len) {
-      const B16* k = x + (size_t)t * p.row_stride + p.k_off + h * p.dk;
-#pragma unroll
-      for (int d0 = 0; d0 < dkp; d0 += 64) {
-        const int d = d0 + (tid & 7) * 8;
-        float v[8] = {};
-        if (d < p.dk) load_vec<B16, 8>(k + d, v);
-#pragma unroll
-        for (int j = 0; j < 8; ++j) ss = fmaf(v[j], v[j], ss);
-      }
-    }
-    ss += __shfl_xor_sync(0xffffffffu, ss, 4);
-    ss += __shfl_xor_sync(0xffffffffu, ss, 2);
-    ss += __shfl_xor_sync(0xffffffffu, ss, 1);
-    if ((tid & 7) == 0) s_inv[t] = rsqrtf(ss + 1e-6f);
     copy_wait<0>();
   }
   __syncthreads();
@@ -413,6 +496,7 @@ delta_prepare_kernel(RecParams p, const int* __restrict__ chunk_row, const int* 
     float z[4] = {}, z2[4] = {};
     const int ch = 8 * j + g;      // the channel whose weights this lane brings
     const B16* w = w2 + (size_t)(ch < p.dk ? ch : 0) * p.rank + q2;
+#pragma unroll 4
     for (int k0 = 0; k0 < rankp; k0 += 16, w += 16) {
       uint32_t a[4], b[2] = {0, 0};
       if (whole) {
@@ -438,6 +522,15 @@ delta_prepare_kernel(RecParams p, const int* __restrict__ chunk_row, const int* 
       cum[t * ld + d + (i & 1)] = t < len && d < p.dk ? delta_log2_decay(z[i] + z2[i] + (i & 1 ? b1 : b0)) : 0.f;
     }
   }
+#pragma unroll
+  for (int it = 0; it < items; ++it) {
+    const int i = tid + it * kDeltaThreads;
+    float k[8], ss = 0.f;
+    load_vec<B16, 8>(reinterpret_cast<const B16*>(&raw[it][0]), k);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) ss = fmaf(k[j], k[j], ss);
+    if (i < kChunk * per) s_sq[i] = ss;
+  }
   __syncthreads();
   for (int d = tid; d < dkp; d += kDeltaThreads) {
     float acc = 0.f;
@@ -450,18 +543,18 @@ delta_prepare_kernel(RecParams p, const int* __restrict__ chunk_row, const int* 
   }
   __syncthreads();
   // r~, u~, k~, b~ relative to the decay through token 7
-#pragma unroll 1
-  for (int i = tid; i < kChunk * (dkp / 8); i += kDeltaThreads) {
-    const int t = i / (dkp / 8), d = i % (dkp / 8) * 8;
-    float r[8] = {}, k[8] = {}, a[8] = {}, bias[8] = {};
-    if (t < len && d < p.dk) {
-      const B16* xr = x + (size_t)t * p.row_stride + h * p.dk + d;
-      load_vec<B16, 8>(xr + p.q_off, r);
-      load_vec<B16, 8>(xr + p.k_off, k);
-      load_vec<B16, 8>(xr + p.f_off, a);
-      load_vec<B16, 8>(ab + d, bias);
-    }
-    const float inv = s_inv[t];
+#pragma unroll
+  for (int it = 0; it < items; ++it) {
+    const int i = tid + it * kDeltaThreads, t = i / per, d = i % per * 8;
+    if (kChunk * per % kDeltaThreads && i >= kChunk * per) break;
+    float r[8], k[8], a[8], bias[8] = {}, ss = 0.f;
+    load_vec<B16, 8>(reinterpret_cast<const B16*>(&raw[it][0]), k);
+    load_vec<B16, 8>(reinterpret_cast<const B16*>(&raw[it][1]), r);
+    load_vec<B16, 8>(reinterpret_cast<const B16*>(&raw[it][2]), a);
+    if (d < p.dk) load_vec<B16, 8>(ab + d, bias);
+#pragma unroll
+    for (int j = 0; j < per; ++j) ss += s_sq[t * per + j];
+    const float inv = rsqrtf(ss + 1e-6f);
     uint32_t out[8][4];
 #pragma unroll
     for (int j = 0; j < 8; j += 2) {

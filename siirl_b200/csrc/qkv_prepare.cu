@@ -88,8 +88,25 @@ __device__ __forceinline__ T* prepare_block(const PrepareParams& p, int t, int& 
   return reinterpret_cast<T*>(p.cache) + (size_t)blk * p.block_elems;
 }
 
-// output gates of row t and the angles' cosines and sines
+// Cosine and sine of a + lo.  Results that are rounded to 16 bits: a leaves its whole turns (2 pi as two floats, the first
+// product exact in the fused multiply-add), the rest takes the special-function units (absolute error below 2^-21).
 template <typename T>
+__device__ __forceinline__ void turn_of(float a, float lo, float& c, float& s) {
+  if constexpr (sizeof(T) == 2) {
+    const float k = rintf(a * 0.15915494309189535f);
+    const float r = fmaf(k, 1.7484556000744487e-07f, fmaf(k, -6.2831854820251465f, a)) + lo;
+    s = __sinf(r);
+    c = __cosf(r);
+  } else {
+    float s0, c0;
+    sincosf(a, &s0, &c0);
+    c = fmaf(-s0, lo, c0);
+    s = fmaf(c0, lo, s0);
+  }
+}
+
+// output gates of row t and the angles' cosines and sines.  PLANES: groups of eight angles as two planes of four
+template <typename T, bool PLANES>
 __device__ __forceinline__ void prepare_gates(const PrepareParams& p, int t, int pos, float* s_cos, float* s_sin) {
   if (p.g_off >= 0) {
     for (int h = threadIdx.x; h < p.Hq; h += blockDim.x) {
@@ -101,9 +118,10 @@ __device__ __forceinline__ void prepare_gates(const PrepareParams& p, int t, int
   for (int i = threadIdx.x; i < p.half; i += blockDim.x) {
     const float n = (float)pos, a = n * p.freq[2 * i], lo = fmaf(n, p.freq[2 * i], -a) + n * p.freq[2 * i + 1];
     float s, c;
-    sincosf(a, &s, &c);
-    s_cos[i] = fmaf(-s, lo, c) * p.rot_mag;
-    s_sin[i] = fmaf(c, lo, s) * p.rot_mag;
+    turn_of<T>(a, lo, c, s);
+    const int at = PLANES ? (i & 4 ? p.half / 2 : 0) + (i >> 3) * 4 + (i & 3) : i;
+    s_cos[at] = c * p.rot_mag;
+    s_sin[at] = s * p.rot_mag;
   }
 }
 
@@ -147,13 +165,21 @@ __device__ __forceinline__ void pool_run(const PrepareParams& p, int slot, int p
 }
 
 constexpr int kPoolThreads = 128;
+// rows of a block: about one run ends among them
+static int pool_rows(int pool) { return pool < 16 ? 16 : (pool < kPoolThreads ? pool : kPoolThreads); }
 
 template <typename T, int V>
-__global__ void __launch_bounds__(kPoolThreads) kv_pool_kernel(const __grid_constant__ PrepareParams p) {
-  for (int t = blockIdx.x; t < p.T; t += gridDim.x) {
+__global__ void __launch_bounds__(kPoolThreads) kv_pool_kernel(const __grid_constant__ PrepareParams p, int rows) {
+  __shared__ int s_row[kPoolThreads], s_n;
+  if (threadIdx.x == 0) s_n = 0;
+  __syncthreads();
+  const int t = blockIdx.x * rows + threadIdx.x;
+  if ((int)threadIdx.x < rows && t < p.T) {
     const int slot = p.seq_ids[t], pos = p.positions[t];
-    if (slot >= 0 && pos >= 0 && (pos + 1) % p.pool == 0) pool_run<T, V>(p, slot, pos);
+    if (slot >= 0 && pos >= 0 && (pos + 1) % p.pool == 0) s_row[atomicAdd(&s_n, 1)] = t;
   }
+  __syncthreads();
+  for (int i = 0; i < s_n; ++i) pool_run<T, V>(p, p.seq_ids[s_row[i]], p.positions[s_row[i]]);
 }
 
 // blocks behind the `row_blocks` of the rows: the table of biases by distance
@@ -177,6 +203,17 @@ struct Unit {
   __device__ __forceinline__ void get(float (&x)[8]) const { load_vec<T, 8>(reinterpret_cast<const T*>(r), x); }
 };
 
+// eight floats as two planes of four: a warp's accesses fall on all banks evenly
+__device__ __forceinline__ void store_planes(float* p, int plane, const float (&x)[8]) {
+  *reinterpret_cast<float4*>(p) = make_float4(x[0], x[1], x[2], x[3]);
+  *reinterpret_cast<float4*>(p + plane) = make_float4(x[4], x[5], x[6], x[7]);
+}
+__device__ __forceinline__ void load_planes(const float* p, int plane, float (&x)[8]) {
+  const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + plane);
+  x[0] = a.x; x[1] = a.y; x[2] = a.z; x[3] = a.w;
+  x[4] = b.x; x[5] = b.y; x[6] = b.z; x[7] = b.w;
+}
+
 // dk, dv and the rotated half are multiples of eight; a thread has U units of eight columns, the same in every row.  F32: the
 // projection comes as 32-bit partial sums.
 template <typename T, int U, bool F32>
@@ -187,6 +224,8 @@ __global__ void __launch_bounds__(512, U == 2 && !F32 ? 2 : 1) qkv_prepare_units
   const int nq = p.Hq * p.dk / 8, nk = p.Hkv * p.dk / 8, nv = p.Hkv * p.dv / 8, per = p.dk / 8;      // units
   // two buffers: [nq + nk][8] weighted values (the norm's factor still to come), cosines, sines, sums of squares (norm 2)
   const int x_len = p.half ? 8 * (nq + nk) : 0, buf_len = (x_len + 2 * p.half + (p.norm >= 2 ? nq + nk : 0) + 7) / 8 * 8;
+  const int plane = 4 * (nq + nk);
+  const float inv_dk = 1.f / (float)p.dk;
   __shared__ float red[2][2][16];
   // heads whose units are a power of two lie in aligned lanes of one warp: their sums need no shared memory
   const bool in_warp = per <= 32 && (per & (per - 1)) == 0;
@@ -212,6 +251,16 @@ __global__ void __launch_bounds__(512, U == 2 && !F32 ? 2 : 1) qkv_prepare_units
       const int e = 8 * (i - nq - nk), head = e / p.dv;
       col[u] = p.v_off + e;
       off[u] = p.Hkv * kPrepBlk * p.dk + head * kPrepBlk * p.dv + e - head * p.dv;
+    }
+  }
+  Unit<T> weight[U];                  // of norms 1 and 3
+  if (p.norm == 1 || p.norm == 3) {
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int i = tid + u * blockDim.x;
+      if (i >= nq + nk) continue;
+      weight[u].load(reinterpret_cast<const T*>(i < nq ? p.q_norm : p.k_norm) +
+                     (p.norm == 3 ? 8 * (i % per) : 8 * (i < nq ? i : i - nq)));
     }
   }
   using X = typename std::conditional<F32, float, T>::type;
@@ -260,7 +309,7 @@ __global__ void __launch_bounds__(512, U == 2 && !F32 ? 2 : 1) qkv_prepare_units
           for (int k = 0; k < 8; ++k) v[u][k] += y[k];
         }
     }
-    prepare_gates<T>(p, t, pos, s_cos, s_sin);
+    prepare_gates<T, true>(p, t, pos, s_cos, s_sin);
     float ssq = 0.f, ssk = 0.f, own[U];      // own: squares of a unit's values before weights
 #pragma unroll
     for (int u = 0; u < U; ++u) {
@@ -285,12 +334,11 @@ __global__ void __launch_bounds__(512, U == 2 && !F32 ? 2 : 1) qkv_prepare_units
       if (p.norm >= 2 && !in_warp) s_part[i] = ss;
       if (p.norm == 1 || p.norm == 3) {
         float w[8];
-        const T* wp = reinterpret_cast<const T*>(i < nq ? p.q_norm : p.k_norm);
-        load_vec<T, 8>(wp + (p.norm == 3 ? 8 * (i % per) : 8 * (i < nq ? i : i - nq)), w);
+        weight[u].get(w);
 #pragma unroll
         for (int k = 0; k < 8; ++k) v[u][k] *= w[k];
       }
-      if (turn[u] >= 0) store_vec<float, 8>(s_x + 8 * i, v[u]);
+      if (turn[u] >= 0) store_planes(s_x + 4 * i, plane, v[u]);
     }
     if (p.norm == 1) {
       ssq = warp_sum(ssq);
@@ -308,8 +356,8 @@ __global__ void __launch_bounds__(512, U == 2 && !F32 ? 2 : 1) qkv_prepare_units
         ssq += red[buf][0][w];
         ssk += red[buf][1][w];
       }
-      fq = 1.f / sqrtf(ssq / (float)(8 * nq) + p.eps);
-      fk = 1.f / sqrtf(ssk / (float)(8 * nk) + p.eps);
+      fq = rsqrtf(ssq / (float)(8 * nq) + p.eps);
+      fk = rsqrtf(ssk / (float)(8 * nk) + p.eps);
     }
 #pragma unroll
     for (int u = 0; u < U; ++u) {
@@ -319,26 +367,30 @@ __global__ void __launch_bounds__(512, U == 2 && !F32 ? 2 : 1) qkv_prepare_units
         float ss = 0.f;
         if (in_warp) {
           ss = own[u];
-          for (int o = per >> 1; o; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+#pragma unroll
+          for (int o = 16; o; o >>= 1)
+            if (o < per) ss += __shfl_xor_sync(0xffffffffu, ss, o);
         } else if (i < nq + nk) {
           const int h = i / per;
           for (int k = 0; k < per; ++k) ss += s_part[h * per + k];
         }
-        f = 1.f / sqrtf(ss / (float)p.dk + p.eps);
+        f = rsqrtf(fmaf(ss, inv_dk, p.eps));
       }
       if (i >= nq + nk) continue;
       if (turn[u] >= 0) {
         const bool first = turn[u] < 1 << 16;
-        const int r = turn[u] & 0xffff;
+        const int r = (turn[u] & 0xffff) >> 1;
         float y[8], c[8], sn[8];
-        load_vec<float, 8>(s_x + 8 * i + (first ? p.half : -p.half), y);
-        load_vec<float, 8>(s_cos + r, c);
-        load_vec<float, 8>(s_sin + r, sn);
+        load_planes(s_x + 4 * i + (first ? p.half : -p.half) / 2, plane, y);
+        load_planes(s_cos + r, p.half / 2, c);
+        load_planes(s_sin + r, p.half / 2, sn);
+        const float fy = first ? -f : f;
 #pragma unroll
-        for (int k = 0; k < 8; ++k) v[u][k] = fmaf(v[u][k], c[k], (first ? -y[k] : y[k]) * sn[k]);
+        for (int k = 0; k < 8; ++k) v[u][k] = fmaf(v[u][k] * f, c[k], y[k] * fy * sn[k]);
+      } else {
+#pragma unroll
+        for (int k = 0; k < 8; ++k) v[u][k] *= f;
       }
-#pragma unroll
-      for (int k = 0; k < 8; ++k) v[u][k] *= f;
       if (i < nq) store_vec<T, 8>(reinterpret_cast<T*>(p.q_out) + (size_t)t * p.q_stride + off[u], v[u]);
       else if (crow) store_vec<T, 8>(crow + off[u] + place * p.dk, v[u]);
     }
@@ -392,7 +444,7 @@ __global__ void __launch_bounds__(kPrepThreads) qkv_prepare_kernel(const __grid_
     if (crow)
       store_vec<T, V>(crow + (size_t)p.Hkv * kPrepBlk * p.dk + ((size_t)head * kPrepBlk + place) * p.dv + (e - head * p.dv), v);
   }
-  prepare_gates<T>(p, t, pos, s_cos, s_sin);
+  prepare_gates<T, false>(p, t, pos, s_cos, s_sin);
   float fq = 1.f, fk = 1.f;
   if (p.norm == 1) {
     ssq = warp_sum(ssq);
@@ -542,13 +594,13 @@ extern "C" int sb_kv_pool(const void* params, int f32, cudaStream_t stream) {
   if (p.pool < 1 || !p.pool_table || p.pool_blocks < 1 || p.Hkv < 1 || p.dk < 1 || p.dv < 1) return -3;
   const int V = f32 ? 4 : 8;
   const bool vec = p.dk % V == 0 && p.dv % V == 0 && p.block_elems % V == 0;
-  const int most = num_sms() * 16, grid = p.T < most ? p.T : most;
+  const int rows = pool_rows(p.pool), grid = (p.T + rows - 1) / rows;
   if (f32) {
-    if (vec) kv_pool_kernel<float, 4><<<grid, kPoolThreads, 0, stream>>>(p);
-    else kv_pool_kernel<float, 1><<<grid, kPoolThreads, 0, stream>>>(p);
+    if (vec) kv_pool_kernel<float, 4><<<grid, kPoolThreads, 0, stream>>>(p, rows);
+    else kv_pool_kernel<float, 1><<<grid, kPoolThreads, 0, stream>>>(p, rows);
   } else {
-    if (vec) kv_pool_kernel<__nv_bfloat16, 8><<<grid, kPoolThreads, 0, stream>>>(p);
-    else kv_pool_kernel<__nv_bfloat16, 1><<<grid, kPoolThreads, 0, stream>>>(p);
+    if (vec) kv_pool_kernel<__nv_bfloat16, 8><<<grid, kPoolThreads, 0, stream>>>(p, rows);
+    else kv_pool_kernel<__nv_bfloat16, 1><<<grid, kPoolThreads, 0, stream>>>(p, rows);
   }
   return (int)cudaGetLastError();
 }
