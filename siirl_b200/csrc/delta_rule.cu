@@ -954,35 +954,61 @@ delta_scan_kernel(RecParams p, Segments sg, const int* __restrict__ slots, const
 }
 
 // Start states of the segments of sequences that have several, in place of the states from zero: S <- S F + local, one segment
-// after the other.  A block has four rows (value columns), a thread one row's channels d, d + 64, ..
-constexpr int kChainRows = 4;
+// after the other; the next matrix is copied while one is used.  A block has sixteen rows (value columns), a thread four of them
+// and the channels d, d + 64, ..
+constexpr int kChainRows = 16, kChainThreads = 256;
+__host__ __device__ inline int chain_smem(int dk) { return (2 * dk * dk + 2 * kChainRows * dk) * 4; }
 
-__global__ void __launch_bounds__(256) delta_chain_kernel(RecParams p, Segments sg, const int* __restrict__ slots,
-                                                          const int* __restrict__ pos0) {
-  extern __shared__ __align__(16) float sm[];      // [2][4][dk] states
-  const int h = blockIdx.y, s = blockIdx.z, tid = threadIdx.x, d0 = tid & 63, v = blockIdx.x * kChainRows + (tid >> 6);
-  const int slot = slots[s], g0 = sg.seq_seg0[s], g1 = sg.seq_seg0[s + 1];
+__global__ void __launch_bounds__(kChainThreads) delta_chain_kernel(RecParams p, Segments sg, const int* __restrict__ slots,
+                                                                    const int* __restrict__ pos0) {
+  extern __shared__ __align__(16) float sm[];
+  const int h = blockIdx.y, s = blockIdx.z, tid = threadIdx.x, d0 = tid & 63, grp = tid >> 6;
+  const int slot = slots[s], g0 = sg.seq_seg0[s], g1 = sg.seq_seg0[s + 1], dk = p.dk;
   if (slot < 0 || g1 - g0 < 2) return;
-  const size_t mat = (size_t)p.dk * p.dk, at = (size_t)v * p.dk;
-  float* cur = sm + (tid >> 6) * p.dk;
-  const int other = kChainRows * p.dk;
-  for (int d = d0; d < p.dk; d += 64)
-    cur[d] = pos0[s] == 0 || v >= p.dv ? 0.f : p.S[((size_t)slot * p.H + h) * p.dv * p.dk + at + d];
-  __syncthreads();
-  for (int g = g0; g < g1; ++g) {
-    float* local = sg.S + ((size_t)g * p.H + h) * p.dv * p.dk + at;
-    const float* F = sg.decay + ((size_t)g * p.H + h) * mat;
-    const float* now = cur + ((g - g0) & 1 ? other : 0);
-    float* next = cur + ((g - g0) & 1 ? 0 : other);
-    for (int d = d0; d < p.dk; d += 64) {
-      float acc = g + 1 < g1 && v < p.dv ? local[d] : 0.f;
-      if (v < p.dv) local[d] = now[d];
-      if (g + 1 < g1)
-#pragma unroll 16
-        for (int j = 0; j < p.dk; ++j) acc = fmaf(now[j], F[(size_t)j * p.dk + d], acc);
-      next[d] = acc;
+  const int mat = dk * dk, v0 = blockIdx.x * kChainRows;
+  float* state = sm + 2 * mat;      // [2][16][dk]
+  auto copy = [&](int g) {          // the last segment's matrix is not needed
+    if (g + 1 < g1) {
+      const float* F = sg.decay + ((size_t)g * p.H + h) * mat;
+      for (int i = tid * 4; i < mat; i += kChainThreads * 4) copy16(sm + ((g - g0) & 1) * mat + i, F + i);
     }
-    __syncthreads();
+    copy_commit();
+  };
+  copy(g0);
+  for (int i = tid; i < kChainRows * dk; i += kChainThreads) {
+    const int v = v0 + i / dk;
+    state[i] = pos0[s] == 0 || v >= p.dv ? 0.f : p.S[((size_t)slot * p.H + h) * p.dv * dk + (size_t)v0 * dk + i];
+  }
+  for (int g = g0; g < g1; ++g) {
+    copy_wait<0>();
+    __syncthreads();                // this matrix and this state are there, the other buffers have been read
+    if (g + 1 < g1) copy(g + 1);
+    const float* F = sm + ((g - g0) & 1) * mat;
+    const float* now = state + (((g - g0) & 1) * kChainRows + grp * 4) * dk;
+    float* next = state + ((((g - g0) & 1) ^ 1) * kChainRows + grp * 4) * dk;
+    float* local = sg.S + ((size_t)g * p.H + h) * p.dv * dk + (size_t)(v0 + grp * 4) * dk;
+    const int rows = min(4, p.dv - v0 - grp * 4);
+    for (int d = d0; d < dk; d += 64) {
+      float acc[4];
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        acc[k] = g + 1 < g1 && k < rows ? local[k * dk + d] : 0.f;
+        if (k < rows) local[k * dk + d] = now[k * dk + d];
+      }
+      if (g + 1 < g1) {
+#pragma unroll 4
+        for (int j = 0; j < dk; j += 4) {
+          float4 n[4];
+#pragma unroll
+          for (int k = 0; k < 4; ++k) n[k] = *reinterpret_cast<const float4*>(now + k * dk + j);
+          const float f[4] = {F[j * dk + d], F[(j + 1) * dk + d], F[(j + 2) * dk + d], F[(j + 3) * dk + d]};
+#pragma unroll
+          for (int k = 0; k < 4; ++k) acc[k] = fmaf(n[k].x, f[0], fmaf(n[k].y, f[1], fmaf(n[k].z, f[2], fmaf(n[k].w, f[3], acc[k]))));
+        }
+      }
+#pragma unroll
+      for (int k = 0; k < 4; ++k) next[k * dk + d] = acc[k];
+    }
   }
 }
 
@@ -1021,7 +1047,9 @@ static int launch_delta(const RecParams& p, const Segments& sg, int n_seg, const
   if (n_seg > n_seq) {
     delta_scan_kernel<NK, false><<<dim3(p.H, n_seg), dvp * 2 + NK * 32, ssm, stream>>>(p, sg, slots, pos0, tiles);
     if ((e = cudaGetLastError()) != cudaSuccess) return (int)e;
-    delta_chain_kernel<<<dim3((p.dv + kChainRows - 1) / kChainRows, p.H, n_seq), 256, 2 * kChainRows * p.dk * 4, stream>>>(
+    static int chain_configured = 0;
+    if ((r = delta_configure(delta_chain_kernel, chain_smem(p.dk), chain_configured))) return r;
+    delta_chain_kernel<<<dim3((p.dv + kChainRows - 1) / kChainRows, p.H, n_seq), kChainThreads, chain_smem(p.dk), stream>>>(
         p, sg, slots, pos0);
     if ((e = cudaGetLastError()) != cudaSuccess) return (int)e;
   }

@@ -64,6 +64,9 @@ MODELS = {
     # attention only: blocks leave the windows, pooled entries stay; a pool wider than its window and than a page
     "windows": dict(vocab=96, width=40, eps=1e-2, scale=0.5, side=8, layers=[
         att(4, 2, 16, moe(6, 8, 4), window=33, pool=7), att(2, 2, 8, None, window=20, pool=70, dims=4)]),
+    # short pools: several blocks of pooled entries, full ones shared by the samples of a prompt
+    "short": dict(vocab=64, width=32, eps=1e-5, scale=2.0, side=8, layers=[
+        att(2, 1, 16, dense(24), window=9, pool=2), delta(2, 8, None, rank=4), att(2, 2, 16, None, window=30, pool=3)]),
     # recurrences only, wide and narrow heads
     "deltas": dict(vocab=64, width=96, eps=1e-3, scale=9.8, side=24, layers=[
         delta(1, 128, dense(48), rank=24), delta(5, 8, moe(33, 24, 5), rank=3), delta(2, 48, None, rank=32)]),
@@ -345,19 +348,19 @@ def greedy_is_consistent(cfg, W, prompt, new, logprobs, dtype):
 
 
 @pytest.mark.parametrize("device,dtype", WHERE)
-@pytest.mark.parametrize("name", ["mixed", "windows"])
+@pytest.mark.parametrize("name", ["mixed", "windows", "short"])
 def test_greedy_generation_through_the_scheduler(name, device, dtype, tmp_path):
     """More sequences than slots, two samples per prompt (which share full blocks of tokens and of pooled entries), chunked
     prompts: greedy tokens are the plain forward's."""
     path, cfg, W = make(tmp_path, name)
     model = load_engine(path, dtype, 640, device=device).model
-    lens = (5, 64, 130, 1, 77) if device == "cpu" and name == "mixed" else (5, 64, 130, 1, 77, 470)
+    lens = (5, 64, 130, 1, 77) if device == "cpu" and name == "mixed" else (5, 64, 130, 1, 77, 390)
     prompts = [tokens_of(cfg, n, 40 + n) for n in lens]
     sp = SamplingParams(n=2, temperature=0.0, max_new_tokens=12, ignore_eos=True)
     runs = []
     for kw in (dict(max_num_seqs=16), dict(max_num_seqs=4, enable_chunked_prefill=True, max_num_batched_tokens=33),
                dict(max_num_seqs=8, use_cuda_graph=False)):
-        eng = RolloutEngine(model, max_model_len=512, num_blocks=64, sync_interval=4, **kw)
+        eng = RolloutEngine(model, max_model_len=512, num_blocks=80, sync_interval=4, **kw)
         assert not eng.enable_prefix_caching
         outs = eng.generate(prompts, sp)
         assert len(outs) == 2 * len(prompts)

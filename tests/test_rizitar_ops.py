@@ -536,7 +536,8 @@ def test_router_without_correction(E, top, device, dtype):
 
 
 @pytest.mark.parametrize("device,dtype", WHERE)
-@pytest.mark.parametrize("T,W,I", [(1, 64, 24), (5, 72, 40), (300, 128, 64), (97, 51, 13), (33, 40, 20)])
+@pytest.mark.parametrize("T,W,I", [(1, 64, 24), (5, 72, 40), (300, 128, 64), (97, 51, 13), (33, 40, 20),
+                                   (1050, 72, 16)])
 def test_plain_experts_and_their_normed_sum(T, W, I, device, dtype):
     """Rows reach their experts and come back weighted, and the sum is normed before it enters the stream."""
     E, top, pad = 6, 3, (I + 7) // 8 * 8
@@ -566,7 +567,7 @@ def test_plain_experts_and_their_normed_sum(T, W, I, device, dtype):
 # ---- rows -------------------------------------------------------------------------------------------------------------------
 @pytest.mark.parametrize("device,dtype", WHERE)
 @pytest.mark.parametrize("W,T", [(64, 7), (40, 3), (1024, 5), (1536, 4), (2056, 300), (96, 1300), (51, 4), (4096, 3), (4104, 2),
-                                 (5000, 2)])
+                                 (5000, 2), (1000, 1025), (1536, 1024), (2048, 1026)])
 def test_rows_between_two_norms(W, T, device, dtype):
     g = torch.Generator().manual_seed(W)
     rnd = lambda *s: rounded(torch.randn(*s, generator=g))  # noqa: E731
