@@ -226,7 +226,7 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
             break;
           }
           int blk;
-          if (WIN && p.pool > 0 && t0 + t < sinks) blk = t0 + t < p.pool_blocks ? p.pool_table[(size_t)b * p.pool_blocks + t0 + t] : -1;
+          if (MODE == 1 && p.pool > 0 && t0 + t < sinks) blk = t0 + t < p.pool_blocks ? p.pool_table[(size_t)b * p.pool_blocks + t0 + t] : -1;
           else blk = blocks[!WIN || t0 + t < sinks ? t0 + t : w0 + t0 + t - sinks];
           if (WIN && blk < 0) blk = 0;      // never among the visible blocks of a well-formed table
           uint8_t* sk = sKV + stage * 2 * L::kKBytes;
@@ -328,8 +328,8 @@ fmha_decode_split_kernel(const __grid_constant__ CUtensorMap map_cache, const __
       int sinks = 0, w0 = 0, vis = 0;
       if constexpr (WIN) visible_tiles(ctx, p.window, p.keep_first, p.pool, sinks, w0, vis);
       // tile t holds pooled entries (numbers first_pos(t) ..) of which the first `pool_n` are visible
-      const int pool_n = WIN ? pooled_entries(ctx - 1, p.window, p.pool) : 0;
-      auto pooled = [&](int t) { return WIN && p.pool > 0 && t0 + t < sinks; };
+      const int pool_n = MODE == 1 ? pooled_entries(ctx - 1, p.window, p.pool) : 0;
+      auto pooled = [&](int t) { return MODE == 1 && p.pool > 0 && t0 + t < sinks; };
       auto first_pos = [&](int t) { return (!WIN || t0 + t < sinks ? t0 + t : w0 + t0 + t - sinks) * kSBlk; };
       // some key of the tile at kv0 is not visible / the key at `col` is not
       auto need_mask = [&](int t, int kv0) {
@@ -769,7 +769,7 @@ extern "C" int sb_attn_window_decode_chunks(const void* params) {
   if (p.dk % 8 || p.dv % 8 || p.dk > 128 || p.dv > 128 || p.Hq % p.Hkv || p.Hq / p.Hkv > 32 || p.row_stride % 8 ||
       p.q_off % 8 || p.out_stride % 8 || p.out_off % 8 || p.block_elems % 8 || p.kv_mode != kPaged || p.gain || p.gate ||
       (p.rel && (p.rel_n < 1 || p.bias_exp > 0.f)) ||
-      (p.pool > 0 && (p.window <= 0 || !p.pool_table || p.pool_blocks < 1 || p.keep_first || p.rel || p.bias_exp > 0.f)))
+      (p.pool > 0 && (p.window <= 0 || !p.pool_table || p.pool_blocks < 1 || p.keep_first || p.rel || p.softcap > 0.f || p.bias_exp > 0.f)))
     return -1;
   int tiles = p.max_blocks;
   if (p.pool > 0) {

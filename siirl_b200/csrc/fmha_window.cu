@@ -9,7 +9,7 @@
 //   window_prefill_kernel   bf16, dk and dv multiples of 8 up to 256: 128 query rows of one head per CTA, S = Q K^T and
 //                           O += P V on tcgen05 with accumulators in TMEM; one cache block is one K/V tile, fetched by
 //                           TMA straight from the paged cache (columns past dk / dv are filled with zeros)
-//                           (two forms: linear bias; soft cap and a bias table by distance)
+//                           (two forms: linear bias or pooled runs; soft cap and a bias table by distance)
 //   window_simt_kernel      any sizes, bf16 or fp32, one CTA per (row, head): the 32-bit path, and odd widths
 #include "common.cuh"
 #include "launchers.h"
@@ -213,7 +213,8 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
   win_blocks(q0, q0 + nrows - 1, p.window, p.keep_first, p.pool, sinks, w0, n_tiles);
   const bool packed = p.kv_mode == kPackedRows;
   const int* bt = p.block_table + (size_t)(packed ? 0 : slot) * p.max_blocks;
-  const int* pt = p.pool > 0 ? p.pool_table + (size_t)slot * p.pool_blocks : nullptr;
+  const bool pool = !TABLE && p.pool > 0;
+  const int* pt = pool ? p.pool_table + (size_t)slot * p.pool_blocks : nullptr;
   auto block_of = [&](int j) { return j < sinks ? j : w0 + j - sinks; };
 
   if (tid == 0) {
@@ -393,7 +394,7 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       }
       // every row of the tile sees every key of the block when the block lies behind q0 and, with a window, inside the
       // last row's window or among the kept tokens
-      if (p.pool > 0 && j < sinks) {      // entries kv0 .. of the pooled runs
+      if (pool && j < sinks) {      // entries kv0 .. of the pooled runs
         if (kv0 + kWBlk > pool_q0) {
 #pragma unroll
           for (int i = 0; i < kWBlk; ++i)
@@ -585,6 +586,7 @@ extern "C" int sb_attn_window_prefill(const void* params, const int* tile_row, c
   }
   const WinSmem L((p.dk + 63) / 64, (p.dv + 63) / 64);
   const bool table = p.softcap > 0.f || p.rel;
+  if (table && p.pool > 0) return -2;
   auto kernel = table ? window_prefill_kernel<true> : window_prefill_kernel<false>;
   static int configured[2] = {0, 0};
   if (configured[table] < L.total) {
