@@ -512,7 +512,8 @@ using namespace sb;
 
 // pooled runs: a window to be before, blocks to lie in, nothing that is defined by the distance of a key
 static bool pool_valid(const WinParams& p) {
-  return p.pool <= 0 || (p.window > 0 && p.pool_table && p.pool_blocks > 0 && p.kv_mode == kPaged && p.keep_first == 0 && !p.rel && !(p.bias_exp > 0.f));
+  return p.pool <= 0 || (p.window > 0 && p.pool_table && p.pool_blocks > 0 && p.kv_mode == kPaged && p.keep_first == 0 && !p.rel && !(p.bias_exp > 0.f) &&
+                         !(p.softcap > 0.f));
 }
 
 static int win_grid(long long total) {
@@ -586,7 +587,6 @@ extern "C" int sb_attn_window_prefill(const void* params, const int* tile_row, c
   }
   const WinSmem L((p.dk + 63) / 64, (p.dv + 63) / 64);
   const bool table = p.softcap > 0.f || p.rel;
-  if (table && p.pool > 0) return -2;
   auto kernel = table ? window_prefill_kernel<true> : window_prefill_kernel<false>;
   static int configured[2] = {0, 0};
   if (configured[table] < L.total) {

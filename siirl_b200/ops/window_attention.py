@@ -284,6 +284,8 @@ def window_attention(spec: WindowSpec, x: torch.Tensor, seq_ids: torch.Tensor, p
     general kernel."""
     if spec.pool and (spec.window < 1 or prepare is None or pool_table is None):
         raise ValueError("pooled blocks: a window, blocks to keep them in and a prepare step that makes them")
+    if spec.pool and (spec.softcap or spec.keep_first or spec.bias_exp or prepare.rel is not None):
+        raise ValueError("pooled blocks: no kept first tokens, biases by distance or soft-capped scores")
     if not x.is_cuda:
         gate = None
         if prepare is not None:
@@ -309,7 +311,7 @@ def window_attention(spec: WindowSpec, x: torch.Tensor, seq_ids: torch.Tensor, p
     status = _lib.ptr(_lib.status_word(x.device))
     aligned = spec.dim % 8 == 0 and spec.vdim % 8 == 0 and x.stride(0) % 8 == 0 and out.stride(0) % 8 == 0 and \
         spec.q_off % 8 == 0 and out_off % 8 == 0
-    if not f32 and not simt and aligned and not (spec.pool and spec.softcap):
+    if not f32 and not simt and aligned:
         if tiles is not None and max(spec.dim, spec.vdim) <= 256:
             _lib.check(L.sb_attn_window_prefill(ref, _lib.ptr(tiles.row), _lib.ptr(tiles.rows), _lib.ptr(tiles.pos),
                                                 _lib.ptr(tiles.slot), tiles.n, status, _lib.stream()),

@@ -317,8 +317,9 @@ def test_pooled_runs_need_a_window_and_blocks():
     for kw in (dict(prepare=pr), dict(pool_table=pages.pool_table)):
         with pytest.raises(ValueError):
             window_attention(spec, *args, **kw)
-    with pytest.raises(ValueError):
-        window_attention(replace(spec, window=0), *args, prepare=pr, pool_table=pages.pool_table)
+    for bad in (dict(window=0), dict(softcap=9.0), dict(keep_first=2), dict(bias_exp=8.0)):
+        with pytest.raises(ValueError):
+            window_attention(replace(spec, **bad), *args, prepare=pr, pool_table=pages.pool_table)
 
 
 # ---- generalized delta rule -------------------------------------------------------------------------------------------------
