@@ -56,7 +56,7 @@ MODELS = {
     "mixed": dict(vocab=203, width=72, eps=1e-4, scale=3.7, side=10, layers=[
         delta(3, 24, moe(7, 24, 3), rank=5),
         att(6, 3, 24, dense(104), window=21, pool=5, dims=16, scaling=(5.0, 4.0, 60, 0.5)),
-        att(4, 2, 32, None, window=40, pool=16, dims=32), delta(2, 16, dense(40), rank=16)]),
+        att(4, 2, 32, None, window=45, pool=14, dims=32), delta(2, 16, dense(40), rank=16)]),
     # sizes that are equal, constants that are one
     "ones": dict(vocab=128, width=64, eps=1e-5, scale=1.0, side=64, layers=[
         att(1, 1, 64, moe(1, 64, 1), window=1, pool=1, dims=64, scale=1.0, scaling=(1.0, 1.0, 64, 1.0)),
@@ -329,7 +329,7 @@ def test_long_decoding(name, device, dtype, tmp_path):
     check(torch.cat(got), O.forward(cfg, W, toks), dtype, "", cfg)
     seq = rp.live["x"]
     if name != "deltas":
-        span, pool = {"mixed": (40, 5), "windows": (70, 7)}[name]
+        span, pool = {"mixed": (45, 5), "windows": (70, 7)}[name]
         assert len([b for b in seq.blocks if b >= 0]) <= (span + 62) // 64 + 1
         assert len(seq.pool_blocks) == (n // pool + 63) // 64 and all(b >= 0 for b in seq.pool_blocks)
     rp.end(["x"])

@@ -68,7 +68,7 @@ ATT = {
     "plain": dict(size=(6, 2, 32), window=37, pool=5, rot=dict(dims=16, base=5e3, scaling=YARN)),
     "wide": dict(size=(4, 1, 128), window=70, pool=16, rot=dict(dims=32, base=1e5, scaling=YARN)),
     "whole_head": dict(size=(8, 8, 64), window=20, pool=8, rot=dict(dims=64, base=1e6)),
-    "middle": dict(size=(3, 3, 96), window=33, pool=7, rot=dict(dims=96, base=5e4, scaling=YARN)),
+    "middle": dict(size=(3, 3, 80), window=33, pool=7, rot=dict(dims=80, base=3e4, scaling=YARN)),
     "page": dict(size=(4, 2, 64), window=64, pool=64, rot=dict(dims=16, base=1e4)),
     "pool_over_window": dict(size=(4, 2, 40), window=10, pool=70, rot=dict(dims=8, base=1e4)),
     "one": dict(size=(2, 2, 32), window=1, pool=1, rot=dict(dims=32, base=1e4)),
